@@ -1,9 +1,11 @@
 """In-tree build of the native code.
 
-Two artefacts are produced next to the Python sources so they travel with the tree:
+These artefacts are produced next to the Python sources so they travel with the tree:
 
 * ``triune_b200/_C.so``            torch extension with every sm_100a kernel (nvcc, ``-gencode
                                    arch=compute_100a,code=sm_100a``) and its bindings;
+* ``triune_b200/_S.so``            the serving subset of it (GEMM family and heterogeneous-layer kernels), built on its own
+                                   where a process only serves such a model (``build_serving``, ``ensure_serving``);
 * ``triune_b200/libtriune_core.so`` C-ABI engine library (arena, CUDA-graph lifecycle, pinned staging ring,
                                    CPU fast paths) loadable through ``ctypes`` or from other languages.
 
@@ -24,6 +26,7 @@ PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 OBJ = CSRC / "_obj"
 EXT_SO = PKG / "_C.so"
+SERVING_SO = PKG / "_S.so"
 CORE_SO = PKG / "libtriune_core.so"
 NOALLOC_SO = PKG / "libtriune_noalloc.so"
 
@@ -70,15 +73,13 @@ def _run(cmd, verbose):
     return r
 
 
-def build_extension(force: bool = False, verbose: bool = False, ptxas_info: bool = False) -> Path:
+def _build_module(so: Path, sources, force: bool, verbose: bool, ptxas_info: bool) -> Path:
+    """Compile ``sources`` that are out of date and link them into the torch extension ``so``."""
     cuda = _cuda_home()
     nvcc = str(Path(cuda, "bin", "nvcc"))
     inc, defs, torch_lib = _torch_flags()
     OBJ.mkdir(parents=True, exist_ok=True)
     hdr_m = _newest_header_mtime()
-    sources = sorted(p for p in CSRC.rglob("*.cu") if "engine" not in p.parts and p.name != "gla_noalloc.cu") + sorted(
-        p for p in CSRC.rglob("*.cpp") if "engine" not in p.parts
-    )
     jobs = []
     objs = []
     for src in sources:
@@ -88,10 +89,12 @@ def build_extension(force: bool = False, verbose: bool = False, ptxas_info: bool
         if not stale:
             continue
         if src.suffix == ".cu":
+            # the heterogeneous-layer kernels keep the accurate functions: large angles, chained exponentials, 32-bit models
+            fast = [] if "hybrid" in src.parts else ["--use_fast_math"]
             cmd = (
                 [nvcc, "-c", str(src), "-o", str(obj)]
                 + NVCC_ARCH
-                + ["-lineinfo", "-O3", "-std=c++17", "--expt-relaxed-constexpr", "--use_fast_math"]
+                + ["-lineinfo", "-O3", "-std=c++17", "--expt-relaxed-constexpr"] + fast
                 + ["-Xcompiler", "-fPIC", f"-I{cuda}/include", f"-I{CSRC}"]
             )
             if ptxas_info:
@@ -105,22 +108,51 @@ def build_extension(force: bool = False, verbose: bool = False, ptxas_info: bool
             )
         jobs.append(cmd)
     if jobs:
-        with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
+        with ThreadPoolExecutor(max_workers=min(os.cpu_count() or 8, 16, len(jobs))) as ex:
             results = list(ex.map(lambda c: _run(c, verbose), jobs))
         if ptxas_info:
             for r in results:
                 if r.stderr.strip():
                     print(r.stderr)
-    need_link = force or jobs or not EXT_SO.exists() or any(o.stat().st_mtime > EXT_SO.stat().st_mtime for o in objs)
+    need_link = force or jobs or not so.exists() or any(o.stat().st_mtime > so.stat().st_mtime for o in objs)
     if need_link:
+        part = so.with_name(f"{so.name}.{os.getpid()}")
         cmd = (
-            ["g++", "-shared", "-o", str(EXT_SO)]
+            ["g++", "-shared", "-o", str(part)]
             + [str(o) for o in objs]
             + [f"-L{torch_lib}", "-lc10", "-ltorch", "-ltorch_cpu", "-ltorch_python", "-lc10_cuda", "-ltorch_cuda"]
             + [f"-L{cuda}/lib64", "-lcudart", f"-Wl,-rpath,{torch_lib}", f"-Wl,-rpath,{cuda}/lib64"]
         )
         _run(cmd, verbose)
-    return EXT_SO
+        os.replace(part, so)
+    return so
+
+
+def build_extension(force: bool = False, verbose: bool = False, ptxas_info: bool = False) -> Path:
+    sources = sorted(p for p in CSRC.rglob("*.cu") if "engine" not in p.parts and p.name != "gla_noalloc.cu") + sorted(
+        p for p in CSRC.rglob("*.cpp") if "engine" not in p.parts and p.name != "serving_module.cpp"
+    )
+    return _build_module(EXT_SO, sources, force, verbose, ptxas_info)
+
+
+def build_serving(force: bool = False, verbose: bool = False, ptxas_info: bool = False) -> Path:
+    """Only the kernels a heterogeneous-layer model is served with."""
+    sources = sorted(p for d in ("gemm", "hybrid") for p in (CSRC / d).iterdir() if p.suffix in (".cu", ".cpp"))
+    return _build_module(SERVING_SO, sources + [CSRC / "serving_module.cpp"], force, verbose, ptxas_info)
+
+
+def ensure_serving(verbose: bool = False) -> None:
+    """Make the serving kernels importable: nothing to do where the full extension or the subset is built, otherwise
+    compile the subset (one process at a time; the others wait for it)."""
+    if EXT_SO.exists() or SERVING_SO.exists():
+        return
+    import fcntl
+
+    OBJ.mkdir(parents=True, exist_ok=True)
+    with open(OBJ / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if not SERVING_SO.exists():
+            build_serving(verbose=verbose)
 
 
 def build_core(force: bool = False, verbose: bool = False) -> Path:

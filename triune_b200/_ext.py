@@ -33,6 +33,24 @@ def ext():
     return m
 
 
+@lru_cache(maxsize=1)
+def _load_serving():
+    try:
+        return importlib.import_module("triune_b200._S")
+    except ImportError as e:
+        return e
+
+
+def serving():
+    """The module with the GEMM family and the heterogeneous-layer kernels: the full extension, or the serving subset
+    where only that was built."""
+    m = _load()
+    if not isinstance(m, Exception):
+        return m
+    s = _load_serving()
+    return ext() if isinstance(s, Exception) else s
+
+
 def ext_available() -> bool:
     return not isinstance(_load(), Exception)
 
@@ -43,7 +61,7 @@ def use_kernels(*tensors) -> bool:
         return False
     if not tensors or not all(t is None or t.is_cuda for t in tensors):
         return False
-    ext()  # raises loudly if a CUDA tensor arrives and the extension is missing
+    serving()  # raises loudly if a CUDA tensor arrives and no extension is built
     return True
 
 

@@ -91,6 +91,12 @@ def cmd_infer(a) -> int:
     return 0
 
 
+def cmd_trace(a) -> int:
+    from .serve.trace import main as trace_main
+
+    return trace_main(args=a)
+
+
 def cmd_scan(a) -> int:
     from .runtime.model_scanner import scan_models
 
@@ -641,6 +647,12 @@ def build_parser() -> argparse.ArgumentParser:
     s.add_argument("--raw", action="store_true", help="do not wrap the prompt in the chat template")
     s.add_argument("--json", action="store_true")
     s.set_defaults(fn=cmd_infer)
+
+    from .serve.trace import add_arguments as trace_arguments
+
+    s = sub.add_parser("trace", help="replay a trace of token portions and write logits (bin/trace_run)")
+    trace_arguments(s)
+    s.set_defaults(fn=cmd_trace)
 
     s = sub.add_parser("scan", help="find models on this machine (checkpoints, HF caches, GGUF, Ollama, adapters)")
     s.add_argument("paths", nargs="*")

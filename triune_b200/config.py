@@ -18,7 +18,7 @@ import json
 import math
 import threading
 from dataclasses import asdict, dataclass, field, fields
-from typing import Any, Dict, Optional, Tuple
+from typing import Any, Dict, List, Optional, Tuple
 
 # ----------------------------------------------------------------------------
 # Behavioural constants (defaults of the reference, triune/model/config.py)
@@ -100,9 +100,9 @@ def is_checkpoint_recomputing() -> bool:
 
 @dataclass
 class ModelConfig:
-    """Architecture of a TriuneTransformer (MoE, multi-exit) or a dense UniversalTransformer."""
+    """Architecture of a TriuneTransformer (MoE, multi-exit), a dense UniversalTransformer or a HybridTransformer."""
 
-    family: str = "triune"  # "triune" (multi-exit MoE) or "universal" (dense)
+    family: str = "triune"  # "triune" (multi-exit MoE), "universal" (dense) or "hybrid" (layers that differ)
     vocab_size: int = VOCAB_SIZE
     hidden_dim: int = HIDDEN_DIM
     num_layers: int = NUM_LAYERS
@@ -131,6 +131,11 @@ class ModelConfig:
     use_fp8: bool = False
     use_fp4: bool = False
     tie_embeddings: bool = True
+    # family "hybrid": one entry per layer, {"mixers": [{"kind": "attention" | "mamba2" | "delta", sizes ...}, ...],
+    # "ff": hidden width or None, "act": its activation}; see models/hybrid_mixers.py for the sizes of each kind
+    layers: Optional[List[Dict[str, Any]]] = None
+    norm: str = "rms"  # family "hybrid": "rms" | "layer" (with a weight, without a bias)
+    norm_eps: float = EPS
 
     def resolved_expert_hidden(self) -> int:
         return int(self.expert_hidden) if self.expert_hidden else EXPERT_HIDDEN_MULTIPLIER * self.hidden_dim
@@ -138,7 +143,40 @@ class ModelConfig:
     def resolved_dense_hidden(self) -> int:
         return int(self.dense_hidden) if self.dense_hidden else DENSE_HIDDEN_MULTIPLIER * self.hidden_dim
 
+    def _validate_hybrid(self) -> "ModelConfig":
+        if not self.layers or self.num_layers != len(self.layers):
+            raise ValueError("a hybrid model lists its layers, num_layers of them")
+        if self.norm not in ("rms", "layer") or not self.norm_eps > 0:
+            raise ValueError(f"unknown norm {self.norm!r} or eps {self.norm_eps}")
+        if self.vocab_size < 1 or self.hidden_dim < 1:
+            raise ValueError("vocab_size and hidden_dim must be >= 1")
+        for i, layer in enumerate(self.layers):
+            if not layer.get("mixers"):
+                raise ValueError(f"layer {i} has no mixer")
+            if layer.get("act", "silu") not in ("relu", "silu", "gelu_tanh"):
+                raise ValueError(f"layer {i}: unknown activation {layer['act']!r}")
+            for m in layer["mixers"]:
+                kind = m.get("kind")
+                need = {"attention": ("heads", "kv_heads", "dim", "vdim", "scale"), "delta": ("heads", "kv_heads", "dim", "vdim", "conv"),
+                        "mamba2": ("heads", "vdim", "state", "groups", "conv", "norm_groups")}.get(kind)
+                if need is None:
+                    raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+                for k in need:
+                    if not m.get(k, 0) > 0:
+                        raise ValueError(f"layer {i}: {kind} needs a positive {k!r}")
+                groups = m["groups"] if kind == "mamba2" else m["kv_heads"]
+                if m["heads"] % groups:
+                    raise ValueError(f"layer {i}: heads ({m['heads']}) must be a multiple of {groups}")
+                if kind == "mamba2" and (m["heads"] * m["vdim"]) % m["norm_groups"]:
+                    raise ValueError(f"layer {i}: norm_groups must divide heads * vdim")
+                rot = m.get("rot_dims", 0)
+                if kind == "attention" and (rot % 2 or not 0 <= rot <= m["dim"]):
+                    raise ValueError(f"layer {i}: rot_dims must be even and at most dim")
+        return self
+
     def validate(self) -> "ModelConfig":
+        if self.family == "hybrid":
+            return self._validate_hybrid()
         if self.hidden_dim != self.num_heads * self.head_dim:
             raise ValueError(
                 f"hidden_dim ({self.hidden_dim}) must equal num_heads * head_dim ({self.num_heads * self.head_dim})"
@@ -186,6 +224,21 @@ class ModelConfig:
         hd = self.num_heads * self.head_dim
         attn = 4 * d * hd + hd * d
         norms = 2 * d
+        if self.family == "hybrid":
+            total = 2 * v * d + d
+            for layer in self.layers:
+                total += d + (3 * d * layer["ff"] + d if layer.get("ff") else 0)
+                for m in layer["mixers"]:
+                    h, e = m["heads"], m["vdim"]
+                    if m["kind"] == "attention":
+                        total += d * (h * m["dim"] + m["kv_heads"] * (m["dim"] + e) + h * e) + 2 * m["dim"] + h
+                    elif m["kind"] == "mamba2":
+                        u = h * e + 2 * m["groups"] * m["state"]
+                        total += d * (2 * h * e + u - h * e + h + h * e) + u * (m["conv"] + 1) + 3 * h + h * e
+                    else:
+                        u = 2 * m["kv_heads"] * m["dim"] + h * e
+                        total += d * (u + 2 * h * e + 2 * h) + u * m["conv"] + 2 * h + e
+            return total, total
         if self.family == "universal":
             ff = self.resolved_dense_hidden()
             ffn = (3 if self.ffn == "swiglu" else 2) * d * ff

@@ -1,0 +1,147 @@
+// Softmax attention with per-head query / key norm, partial interleaved rotation and a sink: preparation of queries,
+// keys and values, and an fp32 CUDA-core attention kernel for every head size (fp32 models, and bf16 head sizes that
+// the tensor-core kernel does not take).
+#include "hybrid.cuh"
+
+namespace tb {
+namespace {
+
+// block: one token of one sequence, four warps over the heads of q, k and v
+template <class T>
+__global__ void attn_prep_kernel(const AttnPrepArgs p) {
+  extern __shared__ float sm[];  // cos [rot/2], sin [rot/2], then one head row per warp
+  const int half = p.rot_dims / 2;
+  float *cs = sm, *sn = sm + half;
+  const int t = blockIdx.x, b = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  float* row = sm + 2 * half + warp * p.D;
+  const long long pos = pos_of(p.pos) + t;
+  if (pos < 0 || pos >= p.cap) return;  // outside the cache: skipped, the host reserves before every call
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    rotation(pos, p.freqs[i], &s, &c);
+    cs[i] = c;
+    sn[i] = s;
+  }
+  __syncthreads();
+  const T* pr = (const T*)p.proj + ((long long)b * p.T + t) * p.ld;
+  for (int hh = warp; hh < p.H + p.G; hh += nw) {
+    const bool isq = hh < p.H;
+    const int h = isq ? hh : hh - p.H;
+    const T* src = pr + (isq ? p.col_q : p.col_k) + h * p.D;
+    T* dst = isq ? (T*)p.q + (((long long)b * p.H + h) * p.T + t) * p.pitch_k
+                 : (T*)p.kc + (((long long)b * p.G + h) * p.cap + pos) * p.pitch_k;
+    const float* w = isq ? p.q_w : p.k_w;
+    float ss = 0.f;
+    for (int d = lane; d < p.D; d += 32) {
+      const float v = ldf(src + d);
+      row[d] = v;
+      ss += v * v;
+    }
+    ss = warp_sum(ss);
+    const float r = w != nullptr ? 1.f / sqrtf(ss / p.D + p.eps) : 1.f;
+    __syncwarp();
+    for (int d = lane; d < p.pitch_k; d += 32) {
+      float v = 0.f;
+      if (d < p.D) {
+        v = row[d] * r * (w != nullptr ? w[d] : 1.f);
+        if (d < p.rot_dims) {
+          const int o = d ^ 1, i = d >> 1;
+          const float other = row[o] * r * (w != nullptr ? w[o] : 1.f);
+          v = (d & 1) ? v * cs[i] + other * sn[i] : v * cs[i] - other * sn[i];
+        }
+      }
+      stf(dst + d, v);
+    }
+    __syncwarp();
+  }
+  for (int i = threadIdx.x; i < p.G * p.pitch_v; i += blockDim.x) {
+    const int g = i / p.pitch_v, e = i % p.pitch_v;
+    stf((T*)p.vc + (((long long)b * p.G + g) * p.cap + pos) * p.pitch_v + e, e < p.E ? ldf(pr + p.col_v + g * p.E + e) : 0.f);
+  }
+}
+
+constexpr int AS_Q = 8, AS_K = 32;
+
+// block: AS_Q consecutive queries of one head, a warp each; keys and values in tiles of 32
+template <class T>
+__global__ void attn_simple_kernel(const AttnArgs p) {
+  extern __shared__ float sm[];
+  const int dp = p.D + 1;
+  float *sk = sm, *sv = sk + AS_K * dp, *sq = sv + AS_K * p.E;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.y, b = blockIdx.z, t = blockIdx.x * AS_Q + warp, g = h / (p.H / p.G);
+  const long long p0 = pos_of(p.pos);
+  const bool live = t < p.T;
+  const long long qpos = p0 + t;
+  const long long kend = min(p0 + min((blockIdx.x + 1) * AS_Q, p.T), (long long)p.cap);  // keys any query of the block sees
+  const T* Q = (const T*)p.q + (((long long)b * p.H + h) * p.T + t) * p.pitch_k;
+  const T *K = (const T*)p.kc + ((long long)b * p.G + g) * p.cap * p.pitch_k, *V = (const T*)p.vc + ((long long)b * p.G + g) * p.cap * p.pitch_v;
+  float* q = sq + warp * p.D;
+  if (live)
+    for (int d = lane; d < p.D; d += 32) q[d] = ldf(Q + d);
+  float m = p.sink != nullptr ? p.sink[h] : -INFINITY, l = p.sink != nullptr ? 1.f : 0.f;
+  float acc[8];  // value dimensions up to 256
+#pragma unroll
+  for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+  for (long long k0 = 0; k0 < kend; k0 += AS_K) {
+    const int n = (int)min((long long)AS_K, kend - k0);
+    __syncthreads();
+    for (int i = threadIdx.x; i < n * p.D; i += blockDim.x) sk[(i / p.D) * dp + i % p.D] = ldf(K + (k0 + i / p.D) * p.pitch_k + i % p.D);
+    for (int i = threadIdx.x; i < n * p.E; i += blockDim.x) sv[i] = ldf(V + (k0 + i / p.E) * p.pitch_v + i % p.E);
+    __syncthreads();
+    if (!live || k0 > qpos) continue;
+    float s = -INFINITY;
+    if (lane < n && k0 + lane <= qpos) {
+      float a = 0.f;
+      for (int d = 0; d < p.D; ++d) a += q[d] * sk[lane * dp + d];
+      s = a * p.scale;
+    }
+    const float mn = fmaxf(m, warp_max(s));
+    const float corr = expf(m - mn), e = expf(s - mn);
+    l = l * corr + warp_sum(e);
+    m = mn;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) acc[i] *= corr;
+    for (int j = 0; j < n; ++j) {
+      const float w = __shfl_sync(0xffffffffu, e, j);
+#pragma unroll
+      for (int i = 0; i < 8; ++i)
+        if (lane + 32 * i < p.E) acc[i] += w * sv[j * p.E + lane + 32 * i];
+    }
+  }
+  if (live) {
+    T* o = (T*)p.out + ((long long)b * p.T + t) * p.ldo + h * p.E;
+    const float r = p.out_scale / l;
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+      if (lane + 32 * i < p.E) stf(o + lane + 32 * i, acc[i] * r);
+  }
+}
+
+}  // namespace
+
+void launch_attn_prep(const AttnPrepArgs& a, cudaStream_t s) {
+  if (a.B <= 0 || a.T <= 0) return;
+  const size_t sm = (size_t)(a.rot_dims / 2 * 2 + 4 * a.D) * 4;
+  dim3 grid(a.T, a.B);
+  if (a.f32) attn_prep_kernel<float><<<grid, 128, sm, s>>>(a);
+  else attn_prep_kernel<__nv_bfloat16><<<grid, 128, sm, s>>>(a);
+  check_launch("attn_prep");
+}
+
+void launch_attn_simple(const AttnArgs& a, cudaStream_t s) {
+  if (a.B <= 0 || a.T <= 0) return;
+  if (a.E > 256) throw std::runtime_error("attention: value dimensions up to 256");
+  const size_t sm = (size_t)(AS_K * (a.D + 1) + AS_K * a.E + AS_Q * a.D) * 4;
+  if (sm > 200 * 1024) throw std::runtime_error("attention: head dimension too large");
+  dim3 grid((a.T + AS_Q - 1) / AS_Q, a.H, a.B);
+  auto go = [&](auto* kern) {
+    if (sm > 47 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
+    kern<<<grid, AS_Q * 32, sm, s>>>(a);
+  };
+  if (a.f32) go(attn_simple_kernel<float>);
+  else go(attn_simple_kernel<__nv_bfloat16>);
+  check_launch("attn_simple");
+}
+
+}  // namespace tb

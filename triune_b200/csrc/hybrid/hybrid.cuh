@@ -1,0 +1,233 @@
+// Kernels of the heterogeneous-layer family: models whose layers mix softmax attention (per-head query / key norm,
+// partial rotation, a sink in the softmax), gated delta rule and Mamba-2 mixers, with a 32-bit residual stream.
+//
+// Every kernel exists for bf16 and for fp32 compute tensors (`f32` flag of the launchers). Sequence rows are laid out
+// [B * T, ld]; `pos` is the position of the first of the T tokens, given by value or, when `pos_ptr` is not null, in
+// device memory (graph-replayed decoding). Norms, positions, scores, softmax, decays and recurrent states are fp32 in
+// both. These translation units are compiled without fast-math: angles reach thousands of radians and the decay
+// chain is an exponential of an exponential.
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include <stdexcept>
+#include <string>
+
+namespace tb {
+
+enum HybridNorm : int { HN_LAYER = 0, HN_RMS = 1 };
+enum HybridAct : int { HA_RELU = 0, HA_SILU = 1, HA_GELU_TANH = 2, HA_IDENTITY = 3 };
+enum GateOrder : int { GO_GATE_THEN_NORM = 0, GO_NORM_THEN_GATE = 1 };
+enum RecurrentKind : int { RK_MAMBA2 = 0, RK_DELTA = 1 };
+
+struct Pos {
+  long long host;
+  const long long* dev;
+};
+
+// ---- rows ------------------------------------------------------------------------------------------------------
+// out[row] = table[ids[row]] as fp32; ids outside [0, V) give zero rows.
+void launch_embed_rows(const void* table, bool f32, const long long* ids, float* out, int rows, int W, int V,
+                       cudaStream_t s);
+// y = norm(x) * w over fp32 rows.
+void launch_norm_rows(const float* x, const float* w, void* y, bool f32, int rows, int W, float eps, int kind,
+                      cudaStream_t s);
+// out = act(gate) * up, gate at column 0 and up at column F of gu.
+void launch_glu_rows(const void* gu, long long ld, void* out, long long ldo, bool f32, int rows, int F, int act,
+                     cudaStream_t s);
+// Gated norm of a mixer's output y [rows, inner] with gate rows: parts of inner / groups elements are divided by their
+// own root mean square. w has inner entries (w_period = inner) or one part's entries repeated (w_period = part).
+void launch_gated_norm(const void* y, long long ldy, const void* gate, long long ldg, const float* w, int w_period,
+                       void* out, long long ldo, bool f32, int rows, int inner, int groups, float eps, int order,
+                       float scale, cudaStream_t s);
+
+// ---- causal convolution ----------------------------------------------------------------------------------------
+// u [B*T, ldu] (C channels), w [C, taps] fp32, bias [C] or null, silu. The state is a ring [B, taps, C] (fp32): slot
+// p % taps holds the input of position p. ring_out receives the ring after the last token; it must not alias ring_in.
+void launch_causal_conv(const void* u, long long ldu, const float* w, const float* bias, const float* ring_in,
+                        float* ring_out, void* out, long long ldo, bool f32, int B, int T, int C, int taps, Pos pos,
+                        cudaStream_t s);
+
+// ---- recurrences -----------------------------------------------------------------------------------------------
+//   delta:   k, q unit vectors (q also times Dk^-1/2), g = exp(-exp(A_log) softplus(a + dt_bias)), beta = sigmoid(b)
+//            u = beta (v - g S^T k)
+//   mamba2:  dt = softplus(a + dt_bias), g = exp(-exp(A_log) dt), u = dt v
+//   S <- g S + k u^T,  out = S^T q (+ D v)      (S: Dk x Dv fp32 per head)
+struct RecurrentArgs {
+  const void *q, *k, *v;             // [B*T, ld*]: head groups of Dk (q, k: KG groups), heads of Dv (v)
+  long long ldq, ldk, ldv;
+  const void *a, *b;                 // [B*T, ld]: one column per head (b: delta only)
+  long long lda, ldb;
+  const float *A_log, *dt_bias, *D;  // [H] (D: mamba2 only)
+  float* state;                      // [B, H, Dk, Dv], updated in place
+  void* out;                         // [B*T, ldo], heads of Dv
+  long long ldo;
+  int B, T, H, KG, Dk, Dv;
+  int kind;
+  float unit_eps;                    // under the root of the unit norm (delta)
+  bool f32;
+};
+void launch_recurrent(const RecurrentArgs& a, cudaStream_t s);
+
+// ---- softmax attention -----------------------------------------------------------------------------------------
+// Query / key head norm + rotation; appends k and v to the cache [B, G, cap, pitch*] at positions pos .. pos+T-1 and
+// writes q [B, H, T, pitch_k].
+struct AttnPrepArgs {
+  const void* proj;  // [B*T, ld]: q at col_q (H*D), k at col_k (G*D), v at col_v (G*E)
+  long long ld;
+  int col_q, col_k, col_v;
+  const float *q_w, *k_w;  // [D] or null (no norm)
+  float eps;
+  int rot_dims;
+  const double* freqs;  // [rot_dims / 2], radians per position
+  void *q, *kc, *vc;
+  int B, T, H, G, D, E, cap, pitch_k, pitch_v;
+  Pos pos;
+  bool f32;
+};
+void launch_attn_prep(const AttnPrepArgs& a, cudaStream_t s);
+
+struct AttnArgs {
+  const void *q, *kc, *vc;  // as written by attn_prep
+  const float* sink;        // [H] or null
+  void* out;                // [B*T, ldo], heads of E
+  long long ldo;
+  int B, T, H, G, D, E, cap, pitch_k, pitch_v;
+  float scale, out_scale;
+  Pos pos;
+  bool f32;
+};
+void launch_attn_simple(const AttnArgs& a, cudaStream_t s);
+
+// ---- decoding (one token per sequence, B <= 8) ------------------------------------------------------------------
+// y[b, n] (+)= sum_k W[n, k] in[b, k] with the input formed in the kernel's prologue from one or two segments:
+// plain fp32 rows, norm(x) * w, or the gated norm of a mixer output. Everything but W is fp32.
+struct GemvSegment {
+  const float* x;     // [B, ld]
+  long long ld;
+  int n;              // entries of this segment
+  int kind;           // 0 plain, 1 norm over the n entries, 2 gated norm
+  int norm_kind;      // kind 1: HN_*; kind 2: GO_*
+  const float* w;     // norm weight
+  int w_period;
+  const float* gate;  // kind 2: [B, ldg]
+  long long ldg;
+  int groups;
+  float eps, scale;
+};
+struct GemvArgs {
+  GemvSegment seg[2];
+  int nseg;
+  const void* W;  // [N, ldw] bf16 or fp32
+  long long ldw;
+  bool f32;
+  float* y;       // [B, ldy]
+  long long ldy;
+  int B, N, K;    // K = sum of the segments' entries
+  int epilogue;   // 0 store, 1 add, 2 act(row n) * row n + N (W has 2 N rows)
+  int act;
+};
+void launch_gemv(const GemvArgs& a, cudaStream_t s);
+
+// One step of a mixer: any of a recurrence (short convolution, unit norms and scalars, state update) and an attention
+// (head norm, rotation, cache append, split-key softmax and its combination), as blocks of one launch.
+struct StepRecurrent {
+  const float* proj;  // [B, ld]: conv channels at col_u, a at col_a, b at col_b
+  long long ld;
+  int col_u, col_a, col_b;
+  int off_q, off_k, off_v;         // inside the conv channels
+  const float *conv_w, *conv_b;    // [C, taps], [C] or null
+  float* ring;                     // [B, taps, C], slot pos % taps is written
+  int C, taps;
+  const float *A_log, *dt_bias, *D;
+  float* state;
+  float* out;                      // [B, ldo]
+  long long ldo;
+  int H, KG, Dk, Dv, kind;
+  float unit_eps;
+};
+struct StepAttention {
+  const float* proj;
+  long long ld;
+  int col_q, col_k, col_v;
+  const float *q_w, *k_w;
+  float eps;
+  int rot_dims;
+  const double* freqs;
+  const float* sink;
+  void *kc, *vc;
+  bool cache_f32;
+  int cap, pitch_k, pitch_v;
+  float* part;      // [B, H, splits, E + 2]
+  int* counters;    // [B * G * head chunks], zero between calls
+  int splits;
+  float* out;       // [B, ldo]
+  long long ldo;
+  int H, G, D, E;
+  float scale, out_scale;
+};
+struct StepArgs {
+  StepRecurrent rec;
+  StepAttention att;
+  bool has_rec, has_att;
+  int B;
+  Pos pos;
+};
+int step_head_chunk(int heads_per_group);  // query heads one attention block serves
+void launch_mixer_step(const StepArgs& a, cudaStream_t s);
+
+// ---- device helpers --------------------------------------------------------------------------------------------
+#ifdef __CUDACC__
+__device__ __forceinline__ float ldf(const float* p) { return *p; }
+__device__ __forceinline__ float ldf(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void stf(float* p, float v) { *p = v; }
+__device__ __forceinline__ void stf(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ long long pos_of(const Pos& p) { return p.dev != nullptr ? *p.dev : p.host; }
+__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float act_f(float x, int act) {
+  if (act == HA_RELU) return fmaxf(x, 0.f);
+  if (act == HA_SILU) return silu_f(x);
+  if (act == HA_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+  return x;
+}
+// sine and cosine of pos * f radians; the turn count is removed in double so that far positions lose nothing
+__device__ __forceinline__ void rotation(long long pos, double f, float* s, float* c) {
+  const double a = (double)pos * f;
+  sincosf((float)(a - 6.283185307179586 * rint(a * 0.15915494309189535)), s, c);
+}
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+__device__ __forceinline__ float warp_max(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
+  return v;
+}
+// Sum over a block of up to 32 warps; every thread receives it. `red` holds 33 floats.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;
+  __syncthreads();
+  if (l == 0) red[w] = v;
+  __syncthreads();
+  if (w == 0) {
+    float t = l < nw ? red[l] : 0.f;
+    t = warp_sum(t);
+    if (l == 0) red[32] = t;
+  }
+  __syncthreads();
+  return red[32];
+}
+#endif
+
+inline void check_launch(const char* what) {
+  cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) throw std::runtime_error(std::string(what) + " launch failed: " + cudaGetErrorString(e));
+}
+
+}  // namespace tb

@@ -1,0 +1,154 @@
+// Row kernels: embedding rows, layer / RMS norm of the fp32 residual stream, gated activations, gated norms.
+#include "hybrid.cuh"
+
+namespace tb {
+namespace {
+
+template <class T>
+__global__ void embed_rows_kernel(const T* __restrict__ table, const long long* __restrict__ ids, float* __restrict__ out,
+                                  int W, int V) {
+  const long long row = blockIdx.x;
+  const long long id = ids[row];
+  const bool ok = id >= 0 && id < V;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) out[row * W + i] = ok ? ldf(table + id * W + i) : 0.f;
+}
+
+template <class T>
+__global__ void norm_rows_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __restrict__ y, int W,
+                                 float eps, int kind) {
+  extern __shared__ float sx[];
+  __shared__ float red[33];
+  const float* xr = x + (long long)blockIdx.x * W;
+  T* yr = y + (long long)blockIdx.x * W;
+  float mean = 0.f;
+  if ((W & 3) == 0) {
+    float s = 0.f;
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(xr + i);
+      *reinterpret_cast<float4*>(sx + i) = v;
+      s += (v.x + v.y) + (v.z + v.w);
+    }
+    if (kind == HN_LAYER) mean = block_sum(s, red) / W;
+    float q = 0.f;
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {  // each thread re-reads only what it wrote
+      const float4 v = *reinterpret_cast<const float4*>(sx + i);
+      const float a = v.x - mean, b = v.y - mean, c = v.z - mean, d = v.w - mean;
+      q += (a * a + b * b) + (c * c + d * d);
+    }
+    const float r = 1.f / sqrtf(block_sum(q, red) / W + eps);
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(sx + i);
+      const float4 g = *reinterpret_cast<const float4*>(w + i);
+      const float o0 = (v.x - mean) * r * g.x, o1 = (v.y - mean) * r * g.y, o2 = (v.z - mean) * r * g.z,
+                  o3 = (v.w - mean) * r * g.w;
+      if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(yr + i) = make_float4(o0, o1, o2, o3);
+      } else {
+        __nv_bfloat162 p0 = __floats2bfloat162_rn(o0, o1), p1 = __floats2bfloat162_rn(o2, o3);
+        uint2 u;
+        u.x = *reinterpret_cast<uint32_t*>(&p0);
+        u.y = *reinterpret_cast<uint32_t*>(&p1);
+        *reinterpret_cast<uint2*>(yr + i) = u;
+      }
+    }
+  } else {
+    float s = 0.f;
+    for (int i = threadIdx.x; i < W; i += blockDim.x) {
+      sx[i] = xr[i];
+      s += sx[i];
+    }
+    if (kind == HN_LAYER) mean = block_sum(s, red) / W;
+    float q = 0.f;
+    for (int i = threadIdx.x; i < W; i += blockDim.x) q += (sx[i] - mean) * (sx[i] - mean);
+    const float r = 1.f / sqrtf(block_sum(q, red) / W + eps);
+    for (int i = threadIdx.x; i < W; i += blockDim.x) stf(yr + i, (sx[i] - mean) * r * w[i]);
+  }
+}
+
+template <class T>
+__global__ void glu_rows_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, long long ldo, int F,
+                                long long n, int act) {
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const long long row = i / F, c = i % F;
+    stf(out + row * ldo + c, act_f(ldf(gu + row * ld + c), act) * ldf(gu + row * ld + F + c));
+  }
+}
+
+// one warp per (row, part)
+template <class T>
+__global__ void gated_norm_kernel(const T* __restrict__ y, long long ldy, const T* __restrict__ gate, long long ldg,
+                                  const float* __restrict__ w, int w_period, T* __restrict__ out, long long ldo,
+                                  long long parts_total, int groups, int part, float eps, int order, float scale) {
+  const long long id = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (id >= parts_total) return;
+  const int lane = threadIdx.x & 31;
+  const long long row = id / groups;
+  const int c0 = (int)(id % groups) * part;
+  const T *yr = y + row * ldy + c0, *gr = gate + row * ldg + c0;
+  const float* wr = w + c0 % w_period;
+  T* orow = out + row * ldo + c0;
+  float q = 0.f;
+  for (int i = lane; i < part; i += 32) {
+    float v = ldf(yr + i);
+    if (order == GO_GATE_THEN_NORM) v *= silu_f(ldf(gr + i));
+    q += v * v;
+  }
+  const float r = scale / sqrtf(warp_sum(q) / part + eps);
+  for (int i = lane; i < part; i += 32) {
+    const float v = ldf(yr + i) * silu_f(ldf(gr + i));
+    stf(orow + i, v * r * wr[i]);
+  }
+}
+
+}  // namespace
+
+void launch_embed_rows(const void* table, bool f32, const long long* ids, float* out, int rows, int W, int V,
+                       cudaStream_t s) {
+  if (rows <= 0) return;
+  const int th = W >= 256 ? 256 : 64;
+  if (f32) embed_rows_kernel<<<rows, th, 0, s>>>((const float*)table, ids, out, W, V);
+  else embed_rows_kernel<<<rows, th, 0, s>>>((const __nv_bfloat16*)table, ids, out, W, V);
+  check_launch("embed_rows");
+}
+
+void launch_norm_rows(const float* x, const float* w, void* y, bool f32, int rows, int W, float eps, int kind,
+                      cudaStream_t s) {
+  if (rows <= 0) return;
+  const size_t sm = (size_t)W * 4;
+  if (sm > 160 * 1024) throw std::runtime_error("norm_rows: rows of at most 40960 elements");
+  const int th = W >= 2048 ? 256 : 128;
+  auto run = [&](auto* kern, auto* out) {
+    if (sm > 47 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
+    kern<<<rows, th, sm, s>>>(x, w, out, W, eps, kind);
+  };
+  if (f32) run(norm_rows_kernel<float>, (float*)y);
+  else run(norm_rows_kernel<__nv_bfloat16>, (__nv_bfloat16*)y);
+  check_launch("norm_rows");
+}
+
+void launch_glu_rows(const void* gu, long long ld, void* out, long long ldo, bool f32, int rows, int F, int act,
+                     cudaStream_t s) {
+  const long long n = (long long)rows * F;
+  if (n <= 0) return;
+  const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+  if (f32) glu_rows_kernel<<<blocks, 256, 0, s>>>((const float*)gu, ld, (float*)out, ldo, F, n, act);
+  else glu_rows_kernel<<<blocks, 256, 0, s>>>((const __nv_bfloat16*)gu, ld, (__nv_bfloat16*)out, ldo, F, n, act);
+  check_launch("glu_rows");
+}
+
+void launch_gated_norm(const void* y, long long ldy, const void* gate, long long ldg, const float* w, int w_period,
+                       void* out, long long ldo, bool f32, int rows, int inner, int groups, float eps, int order,
+                       float scale, cudaStream_t s) {
+  if (rows <= 0) return;
+  const long long parts = (long long)rows * groups;
+  const int blocks = (int)((parts + 3) / 4);
+  if (f32)
+    gated_norm_kernel<<<blocks, 128, 0, s>>>((const float*)y, ldy, (const float*)gate, ldg, w, w_period, (float*)out, ldo,
+                                             parts, groups, inner / groups, eps, order, scale);
+  else
+    gated_norm_kernel<<<blocks, 128, 0, s>>>((const __nv_bfloat16*)y, ldy, (const __nv_bfloat16*)gate, ldg, w, w_period,
+                                             (__nv_bfloat16*)out, ldo, parts, groups, inner / groups, eps, order, scale);
+  check_launch("gated_norm");
+}
+
+}  // namespace tb

@@ -1,0 +1,498 @@
+// Decoding: one token per sequence. A layer is a handful of launches that each read their weights or state once:
+// a matrix-vector product whose prologue forms its input (norm of the residual, gated norm of a mixer's output) and
+// whose epilogue adds into the residual or applies the gated activation, and one launch for the mixer itself.
+#include "../common/ptx.cuh"
+#include "hybrid.cuh"
+
+namespace tb {
+namespace {
+
+constexpr int GV_WARPS = 8;
+
+__device__ void gemv_segment(const GemvSegment& g, int b, float* dst, float* red) {
+  const float* x = g.x + (long long)b * g.ld;
+  const int tid = threadIdx.x, nt = blockDim.x;
+  if (g.kind == 0) {
+    for (int i = tid; i < g.n; i += nt) dst[i] = x[i] * g.scale;
+  } else if (g.kind == 1) {
+    float s = 0.f, mean = 0.f;
+    for (int i = tid; i < g.n; i += nt) {
+      dst[i] = x[i];
+      s += dst[i];
+    }
+    if (g.norm_kind == HN_LAYER) mean = block_sum(s, red) / g.n;
+    float q = 0.f;
+    for (int i = tid; i < g.n; i += nt) q += (dst[i] - mean) * (dst[i] - mean);
+    const float r = g.scale / sqrtf(block_sum(q, red) / g.n + g.eps);
+    for (int i = tid; i < g.n; i += nt) dst[i] = (dst[i] - mean) * r * g.w[i];
+  } else {
+    const float* gt = g.gate + (long long)b * g.ldg;
+    const int part = g.n / g.groups, warp = tid >> 5, lane = tid & 31;
+    for (int p = warp; p < g.groups; p += nt >> 5) {
+      float q = 0.f;
+      for (int i = lane; i < part; i += 32) {
+        const int c = p * part + i;
+        const float z = silu_f(gt[c]), v = x[c];
+        const float in = g.norm_kind == GO_GATE_THEN_NORM ? v * z : v;
+        q += in * in;
+        dst[c] = v * z * g.w[c % g.w_period];
+      }
+      const float r = g.scale / sqrtf(warp_sum(q) / part + g.eps);
+      for (int i = lane; i < part; i += 32) dst[p * part + i] *= r;
+    }
+  }
+}
+
+template <class T>
+__device__ __forceinline__ void load_vec(const T* p, float (&f)[16 / sizeof(T)]) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  if constexpr (sizeof(T) == 4) {
+    f[0] = __uint_as_float(u.x); f[1] = __uint_as_float(u.y); f[2] = __uint_as_float(u.z); f[3] = __uint_as_float(u.w);
+  } else {
+    const uint32_t a[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      f[2 * i] = __uint_as_float(a[i] << 16);
+      f[2 * i + 1] = __uint_as_float(a[i] & 0xffff0000u);
+    }
+  }
+}
+
+// A warp works on two rows at a time (for the gated epilogue: a gate row and its up row).
+template <class T, int NB>
+__global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const GemvArgs p) {
+  extern __shared__ __align__(16) float sx[];  // [NB][KP]
+  __shared__ float red[33];
+  constexpr int VEC = 16 / sizeof(T), STEP = 32 * VEC;
+  const int KP = (p.K + 3) & ~3;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int b = 0; b < p.B; ++b) {
+    int off = 0;
+    for (int i = 0; i < p.nseg; ++i) {
+      gemv_segment(p.seg[i], b, sx + b * KP + off, red);
+      off += p.seg[i].n;
+    }
+  }
+  __syncthreads();
+  const bool glu = p.epilogue == 2;
+  const int pairs = glu ? p.N : (p.N + 1) / 2;
+  const bool vec = p.K % VEC == 0 && p.ldw % VEC == 0 && (reinterpret_cast<uintptr_t>(p.W) & 15) == 0;
+  for (int pr = blockIdx.x * GV_WARPS + warp; pr < pairs; pr += gridDim.x * GV_WARPS) {
+    const int r0 = glu ? pr : 2 * pr, r1 = glu ? pr + p.N : 2 * pr + 1;
+    const bool two = glu || r1 < p.N;
+    const T *w0 = (const T*)p.W + (long long)r0 * p.ldw, *w1 = (const T*)p.W + (long long)(two ? r1 : r0) * p.ldw;
+    float a0[NB], a1[NB];
+#pragma unroll
+    for (int b = 0; b < NB; ++b) a0[b] = a1[b] = 0.f;
+    if (vec) {
+#pragma unroll 4
+      for (int k = lane * VEC; k < p.K; k += STEP) {
+        float f0[VEC], f1[VEC];
+        load_vec(w0 + k, f0);
+        load_vec(w1 + k, f1);
+#pragma unroll
+        for (int b = 0; b < NB; ++b) {
+          if (b < p.B) {
+#pragma unroll
+            for (int i = 0; i < VEC; i += 4) {
+              const float4 x = *reinterpret_cast<const float4*>(sx + b * KP + k + i);
+              a0[b] += f0[i] * x.x + f0[i + 1] * x.y + f0[i + 2] * x.z + f0[i + 3] * x.w;
+              a1[b] += f1[i] * x.x + f1[i + 1] * x.y + f1[i + 2] * x.z + f1[i + 3] * x.w;
+            }
+          }
+        }
+      }
+    } else {
+      for (int k = lane; k < p.K; k += 32) {
+        const float f0 = ldf(w0 + k), f1 = ldf(w1 + k);
+#pragma unroll
+        for (int b = 0; b < NB; ++b)
+          if (b < p.B) {
+            a0[b] += f0 * sx[b * KP + k];
+            a1[b] += f1 * sx[b * KP + k];
+          }
+      }
+    }
+#pragma unroll
+    for (int b = 0; b < NB; ++b) {
+      if (b >= p.B) break;
+      const float s0 = warp_sum(a0[b]), s1 = warp_sum(a1[b]);
+      if (lane == 0) {
+        float* y = p.y + (long long)b * p.ldy;
+        if (glu) y[r0] = act_f(s0, p.act) * s1;
+        else if (p.epilogue == 1) {
+          y[r0] += s0;
+          if (two) y[r1] += s1;
+        } else {
+          y[r0] = s0;
+          if (two) y[r1] = s1;
+        }
+      }
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ recurrent step
+constexpr int ST_COLS = 16, ST_THREADS = 128;
+
+__device__ float conv_step(const StepRecurrent& p, int b, int c, long long pos, bool write) {
+  const float cur = p.proj[(long long)b * p.ld + p.col_u + c];
+  float* ring = p.ring + (long long)b * p.taps * p.C + c;
+  float acc = p.conv_b != nullptr ? p.conv_b[c] : 0.f;
+  const float* w = p.conv_w + (long long)c * p.taps;
+  for (int j = 0; j < p.taps - 1; ++j) {
+    const long long q = pos - (p.taps - 1) + j;
+    if (q >= 0) acc += w[j] * ring[(q % p.taps) * p.C];
+  }
+  acc += w[p.taps - 1] * cur;
+  // the slot of this position last held position pos - taps, which no tap reads any more
+  if (write) ring[(pos % p.taps) * p.C] = cur;
+  return silu_f(acc);
+}
+
+__device__ void recurrent_step(const StepRecurrent& p, int block, long long pos, float* sm) {
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, sub = lane & 7;
+  const int slices = (p.Dv + ST_COLS - 1) / ST_COLS;
+  const int slice = block % slices, bh = block / slices, h = bh % p.H, b = bh / p.H;
+  const int rep = p.H / p.KG, kh = h / rep;
+  const int DP = (p.Dk + 31) & ~31;
+  float *sk = sm, *sq = sk + DP, *sv = sq + DP, *red = sv + ST_COLS;
+  const bool owner = slice == 0 && h % rep == 0;
+  float kk = 0.f, qq = 0.f, kq = 0.f;
+  for (int d = tid; d < DP; d += ST_THREADS) {
+    const float kv = d < p.Dk ? conv_step(p, b, p.off_k + kh * p.Dk + d, pos, owner) : 0.f;
+    const float qv = d < p.Dk ? conv_step(p, b, p.off_q + kh * p.Dk + d, pos, owner) : 0.f;
+    sk[d] = kv;
+    sq[d] = qv;
+    kk += kv * kv;
+    qq += qv * qv;
+    kq += kv * qv;
+  }
+  if (tid < ST_COLS) {
+    const int c = slice * ST_COLS + tid;
+    sv[tid] = c < p.Dv ? conv_step(p, b, p.off_v + h * p.Dv + c, pos, true) : 0.f;
+  }
+  kq = block_sum(kq, red);
+  float rk = 1.f, rq = 1.f;
+  if (p.kind == RK_DELTA) {
+    rk = 1.f / sqrtf(block_sum(kk, red) + p.unit_eps);
+    rq = 1.f / (sqrtf(block_sum(qq, red) + p.unit_eps) * sqrtf((float)p.Dk));
+  }
+  const float* pr = p.proj + (long long)b * p.ld;
+  const float dt = softplus_f(pr[p.col_a + h] + p.dt_bias[h]);
+  const float g = expf(-expf(p.A_log[h]) * dt);
+  const int cl = warp * 4 + (lane >> 3), col = slice * ST_COLS + cl;
+  const bool live = col < p.Dv;
+  float* st = p.state + (long long)bh * p.Dk * p.Dv;
+  float ak = 0.f, aq = 0.f;
+  const float v = sv[cl];
+  float S[32];
+  if (live) {
+#pragma unroll
+    for (int r = 0; r < 32; ++r) {
+      const int d = r * 8 + sub;
+      if (d < p.Dk) {
+        S[r] = st[(long long)d * p.Dv + col];
+        ak += sk[d] * S[r];
+        aq += sq[d] * S[r];
+      }
+    }
+  }
+#pragma unroll
+  for (int o = 4; o > 0; o >>= 1) {
+    ak += __shfl_xor_sync(0xffffffffu, ak, o);
+    aq += __shfl_xor_sync(0xffffffffu, aq, o);
+  }
+  const float u = p.kind == RK_DELTA ? sigmoid_f(pr[p.col_b + h]) * (v - g * rk * ak) : dt * v;
+  if (live) {
+#pragma unroll
+    for (int r = 0; r < 32; ++r) {
+      const int d = r * 8 + sub;
+      if (d < p.Dk) st[(long long)d * p.Dv + col] = g * S[r] + sk[d] * rk * u;
+    }
+    if (sub == 0)
+      p.out[(long long)b * p.ldo + h * p.Dv + col] =
+          g * rq * aq + kq * rk * rq * u + (p.kind == RK_MAMBA2 ? p.D[h] * v : 0.f);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ attention step
+constexpr int AT_KEYS = 256;  // keys whose scores are in shared memory at a time
+
+// Head norm and rotation of one projected head row by a warp; dst fp32 [D].
+__device__ void head_row(const float* src, const float* w, float eps, int D, int rot, const float* cs, const float* sn,
+                         float* dst, int padded) {
+  const int lane = threadIdx.x & 31;
+  float ss = 0.f;
+  for (int d = lane; d < D; d += 32) ss += src[d] * src[d];
+  ss = warp_sum(ss);
+  const float r = w != nullptr ? 1.f / sqrtf(ss / D + eps) : 1.f;
+  for (int d = lane; d < D; d += 32) {
+    float v = src[d] * r * (w != nullptr ? w[d] : 1.f);
+    if (d < rot) {
+      const int o = d ^ 1, i = d >> 1;
+      const float x = src[o] * r * (w != nullptr ? w[o] : 1.f);
+      v = (d & 1) ? v * cs[i] + x * sn[i] : v * cs[i] - x * sn[i];
+    }
+    dst[d] = v;
+  }
+  for (int d = D + lane; d < padded; d += 32) dst[d] = 0.f;
+}
+
+// Keys of split `s` of `splits` over n keys: whole multiples of 32, at least 64 keys per split.
+__device__ __forceinline__ void split_range(int n, int splits, int s, int* k0, int* k1) {
+  int per = (n + splits - 1) / splits;
+  per = max(64, (per + 31) & ~31);
+  *k0 = min(n, s * per);
+  *k1 = min(n, *k0 + per);
+}
+
+template <class T, int RM>
+__device__ void attention_step(const StepAttention& p, int block, long long pos, float* sm) {
+  constexpr int VEC = 16 / sizeof(T);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int rep = p.H / p.G, chunks = (rep + RM - 1) / RM;
+  const int split = block % p.splits, bgc = block / p.splits, hc = bgc % chunks, bg = bgc / chunks, g = bg % p.G, b = bg / p.G;
+  const int h0 = g * rep + hc * RM, nh = min(RM, rep - hc * RM);
+  const int DP = (p.D + 7) & ~7, half = p.rot_dims / 2;
+  float *sq = sm, *sp = sq + RM * DP, *cs = sp + RM * AT_KEYS, *sn = cs + half, *sk = sn + half, *ml = sk + DP, *sacc = ml + 2 * RM;
+  int* flag = reinterpret_cast<int*>(sacc);
+  if (pos < 0 || pos >= p.cap) return;  // the host reserves the cache before every step
+  int k0, k1;
+  split_range((int)pos + 1, p.splits, split, &k0, &k1);
+  T *K = (T*)p.kc + (long long)bg * p.cap * p.pitch_k, *V = (T*)p.vc + (long long)bg * p.cap * p.pitch_v;
+  float* part = p.part + (((long long)b * p.H + h0) * p.splits + split) * (p.E + 2);
+  const long long hstride = (long long)p.splits * (p.E + 2);
+  const float* pr = p.proj + (long long)b * p.ld;
+
+  if (k0 < k1) {
+    for (int i = tid; i < half; i += ST_THREADS) rotation(pos, p.freqs[i], sn + i, cs + i);
+    __syncthreads();
+    for (int r = warp; r < nh; r += 4) head_row(pr + p.col_q + (h0 + r) * p.D, p.q_w, p.eps, p.D, p.rot_dims, cs, sn, sq + r * DP, DP);
+    const bool has_new = (int)pos < k1;
+    if (has_new) {
+      // several head chunks of a group write the same values: the readers below only need their own block's copy
+      if (warp == 3) head_row(pr + p.col_k + g * p.D, p.k_w, p.eps, p.D, p.rot_dims, cs, sn, sk, DP);
+      for (int i = tid; i < p.pitch_v; i += ST_THREADS) stf(V + pos * p.pitch_v + i, i < p.E ? pr[p.col_v + g * p.E + i] : 0.f);
+      __syncthreads();
+      for (int i = tid; i < p.pitch_k; i += ST_THREADS) stf(K + pos * p.pitch_k + i, i < p.D ? sk[i] : 0.f);
+    }
+    if (tid < RM) {
+      ml[2 * tid] = -INFINITY;
+      ml[2 * tid + 1] = 0.f;
+    }
+    __syncthreads();
+    // value accumulation: a thread owns two neighbouring value dimensions of a subset of the keys
+    const int PC = (p.E + 1) / 2, KS = max(1, ST_THREADS / PC);
+    float acc[RM][2];
+    const int pc = tid % PC, ks = tid / PC;       // PC <= 128: value dimensions up to 256
+    const bool vlive = ks < KS;
+#pragma unroll
+    for (int r = 0; r < RM; ++r) acc[r][0] = acc[r][1] = 0.f;
+    for (int kb = k0; kb < k1; kb += AT_KEYS) {
+      const int n = min(AT_KEYS, k1 - kb);
+      // scores: four lanes per key
+      for (int j = warp * 8 + (lane >> 2); j < ((n + 31) & ~31); j += 32) {
+        float s[RM];
+#pragma unroll
+        for (int r = 0; r < RM; ++r) s[r] = 0.f;
+        if (j < n) {
+          const T* kr = K + (long long)(kb + j) * p.pitch_k;
+          for (int d = (lane & 3) * VEC; d < DP; d += 4 * VEC) {
+            float f[VEC];
+            load_vec(kr + d, f);  // rows are padded with zeros to a multiple of 16 bytes
+#pragma unroll
+            for (int r = 0; r < RM; ++r)
+              if (r < nh) {
+#pragma unroll
+                for (int i = 0; i < VEC; i += 4) {
+                  const float4 x = *reinterpret_cast<const float4*>(sq + r * DP + d + i);
+                  s[r] += f[i] * x.x + f[i + 1] * x.y + f[i + 2] * x.z + f[i + 3] * x.w;
+                }
+              }
+          }
+        }
+#pragma unroll
+        for (int r = 0; r < RM; ++r) {
+          s[r] += __shfl_xor_sync(0xffffffffu, s[r], 1);
+          s[r] += __shfl_xor_sync(0xffffffffu, s[r], 2);
+          if ((lane & 3) == 0 && j < n && r < nh) sp[r * AT_KEYS + j] = s[r] * p.scale;
+        }
+      }
+      __syncthreads();
+      // softmax of the tile: a warp per head; the running maximum's correction goes through sk
+      for (int r = warp; r < nh; r += 4) {
+        float m = -INFINITY;
+        for (int j = lane; j < n; j += 32) m = fmaxf(m, sp[r * AT_KEYS + j]);
+        m = fmaxf(warp_max(m), ml[2 * r]);
+        float l = 0.f;
+        for (int j = lane; j < n; j += 32) {
+          const float e = expf(sp[r * AT_KEYS + j] - m);
+          sp[r * AT_KEYS + j] = e;
+          l += e;
+        }
+        l = warp_sum(l);
+        if (lane == 0) {
+          const float corr = expf(ml[2 * r] - m);
+          ml[2 * r + 1] = ml[2 * r + 1] * corr + l;
+          ml[2 * r] = m;
+          sacc[1 + r] = corr;
+        }
+      }
+      __syncthreads();
+      if (vlive) {
+#pragma unroll
+        for (int r = 0; r < RM; ++r)
+          if (r < nh) {
+            acc[r][0] *= sacc[1 + r];
+            acc[r][1] *= sacc[1 + r];
+          }
+        const int e0 = 2 * pc;
+#pragma unroll 4
+        for (int j = ks; j < n; j += KS) {
+          float v0, v1;
+          const T* vr = V + (long long)(kb + j) * p.pitch_v + e0;  // pitch_v is even: the pair stays inside the row
+          if constexpr (sizeof(T) == 4) {
+            const float2 t = *reinterpret_cast<const float2*>(vr);
+            v0 = t.x; v1 = t.y;
+          } else {
+            const uint32_t t = *reinterpret_cast<const uint32_t*>(vr);
+            v0 = __uint_as_float(t << 16); v1 = __uint_as_float(t & 0xffff0000u);
+          }
+#pragma unroll
+          for (int r = 0; r < RM; ++r)
+            if (r < nh) {
+              const float w = sp[r * AT_KEYS + j];
+              acc[r][0] += w * v0;
+              acc[r][1] += w * v1;
+            }
+        }
+      }
+      __syncthreads();
+    }
+    // sum over the key subsets, one head at a time, through the score buffer
+    for (int r = 0; r < nh; ++r) {
+      if (vlive) {
+        sp[tid * 2] = acc[r][0];
+        sp[tid * 2 + 1] = acc[r][1];
+      }
+      __syncthreads();
+      for (int e = tid; e < p.E; e += ST_THREADS) {
+        float t = 0.f;
+        for (int q = 0; q < KS; ++q) t += sp[(q * PC + (e >> 1)) * 2 + (e & 1)];
+        part[r * hstride + 2 + e] = t;
+      }
+      if (tid == 0) {
+        part[r * hstride] = ml[2 * r];
+        part[r * hstride + 1] = ml[2 * r + 1];
+      }
+      __syncthreads();
+    }
+  } else {
+    if (tid < nh) {
+      part[tid * hstride] = -INFINITY;
+      part[tid * hstride + 1] = 0.f;
+    }
+  }
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) *flag = atomicAdd(p.counters + bgc, 1) == p.splits - 1 ? 1 : 0;
+  __syncthreads();
+  if (*flag == 0) return;
+  __threadfence();
+  if (tid == 0) p.counters[bgc] = 0;
+  const float* base = p.part + ((long long)b * p.H + h0) * p.splits * (p.E + 2);
+  for (int r = 0; r < nh; ++r) {
+    const float* ph = base + r * hstride;
+    const float sink = p.sink != nullptr ? p.sink[h0 + r] : -INFINITY;
+    float m = sink;
+    for (int s = 0; s < p.splits; ++s) m = fmaxf(m, __ldcg(ph + s * (p.E + 2)));
+    float l = p.sink != nullptr ? expf(sink - m) : 0.f;
+    for (int s = 0; s < p.splits; ++s) l += __ldcg(ph + s * (p.E + 2) + 1) * expf(__ldcg(ph + s * (p.E + 2)) - m);
+    for (int e = tid; e < p.E; e += ST_THREADS) {
+      float t = 0.f;
+      for (int s = 0; s < p.splits; ++s) {
+        const float c = expf(__ldcg(ph + s * (p.E + 2)) - m);
+        if (c > 0.f) t += c * __ldcg(ph + s * (p.E + 2) + 2 + e);
+      }
+      p.out[(long long)b * p.ldo + (h0 + r) * p.E + e] = t / l * p.out_scale;
+    }
+  }
+}
+
+template <class T, int RM>
+__global__ void __launch_bounds__(ST_THREADS) mixer_step_kernel(const StepArgs p, int att_blocks) {
+  extern __shared__ __align__(16) float sm[];
+  const long long pos = pos_of(p.pos);
+  if ((int)blockIdx.x < att_blocks) attention_step<T, RM>(p.att, blockIdx.x, pos, sm);
+  else recurrent_step(p.rec, blockIdx.x - att_blocks, pos, sm);
+}
+
+}  // namespace
+
+int step_head_chunk(int rep) { return rep <= 1 ? 1 : rep <= 2 ? 2 : rep <= 4 ? 4 : 8; }
+
+void launch_mixer_step(const StepArgs& a, cudaStream_t s) {
+  if (a.B <= 0) return;
+  int att = 0, rec = 0, rm = 1;
+  size_t sm = 0;
+  if (a.has_att) {
+    const StepAttention& p = a.att;
+    if (p.E > 256 || p.D > 512) throw std::runtime_error("mixer_step: head dimensions up to 512 / 256");
+    rm = step_head_chunk(p.H / p.G);
+    att = a.B * p.G * ((p.H / p.G + rm - 1) / rm) * p.splits;
+    const int dp = (p.D + 7) & ~7;
+    sm = (size_t)(rm * dp + rm * AT_KEYS + p.rot_dims + 4 + dp + 2 * rm + rm + 4) * 4;
+  }
+  if (a.has_rec) {
+    const StepRecurrent& p = a.rec;
+    if (p.Dk > 256) throw std::runtime_error("mixer_step: key dimensions up to 256");
+    rec = a.B * p.H * ((p.Dv + ST_COLS - 1) / ST_COLS);
+    const size_t need = (size_t)(2 * ((p.Dk + 31) & ~31) + ST_COLS + 40) * 4;
+    sm = need > sm ? need : sm;
+  }
+  if (att + rec == 0) return;
+  const bool f32 = a.has_att && a.att.cache_f32;
+  auto go = [&](auto* kern) { kern<<<att + rec, ST_THREADS, sm, s>>>(a, att); };
+  if (f32) {
+    if (rm == 1) go(mixer_step_kernel<float, 1>);
+    else if (rm == 2) go(mixer_step_kernel<float, 2>);
+    else if (rm == 4) go(mixer_step_kernel<float, 4>);
+    else go(mixer_step_kernel<float, 8>);
+  } else {
+    if (rm == 1) go(mixer_step_kernel<__nv_bfloat16, 1>);
+    else if (rm == 2) go(mixer_step_kernel<__nv_bfloat16, 2>);
+    else if (rm == 4) go(mixer_step_kernel<__nv_bfloat16, 4>);
+    else go(mixer_step_kernel<__nv_bfloat16, 8>);
+  }
+  check_launch("mixer_step");
+}
+
+void launch_gemv(const GemvArgs& a, cudaStream_t s) {
+  if (a.B <= 0 || a.N <= 0) return;
+  if (a.B > 8) throw std::runtime_error("gemv: at most 8 rows");
+  const size_t sm = (size_t)a.B * ((a.K + 3) & ~3) * 4;
+  if (sm > 200 * 1024) throw std::runtime_error("gemv: the input rows do not fit into shared memory");
+  const int pairs = a.epilogue == 2 ? a.N : (a.N + 1) / 2;
+  int blocks = (pairs + GV_WARPS - 1) / GV_WARPS;
+  const int per_sm = sm > 100 * 1024 ? 1 : sm > 50 * 1024 ? 2 : 4;
+  if (blocks > 148 * per_sm) blocks = 148 * per_sm;
+  auto go = [&](auto* kern) {
+    if (sm > 47 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
+    kern<<<blocks, GV_WARPS * 32, sm, s>>>(a);
+  };
+  if (a.f32) {
+    if (a.B == 1) go(gemv_kernel<float, 1>);
+    else if (a.B == 2) go(gemv_kernel<float, 2>);
+    else if (a.B <= 4) go(gemv_kernel<float, 4>);
+    else go(gemv_kernel<float, 8>);
+  } else {
+    if (a.B == 1) go(gemv_kernel<__nv_bfloat16, 1>);
+    else if (a.B == 2) go(gemv_kernel<__nv_bfloat16, 2>);
+    else if (a.B <= 4) go(gemv_kernel<__nv_bfloat16, 4>);
+    else go(gemv_kernel<__nv_bfloat16, 8>);
+  }
+  check_launch("gemv");
+}
+
+}  // namespace tb

@@ -22,6 +22,7 @@ import torch
 import torch.nn.functional as F
 
 from .config import ModelConfig
+from .models.layer_state import LayerState
 
 DEFAULT_STOPS = ("\nUser:", "\nSystem:", "User:", "Assistant:")
 
@@ -53,7 +54,7 @@ def infer_config_from_state_dict(sd: Dict[str, torch.Tensor]) -> ModelConfig:
 
 def load_checkpoint_model(path: str, device="cpu", dtype: Optional[torch.dtype] = None):
     """Load a ``.pt`` checkpoint (ours or the reference's) into a freshly built model. Returns (model, checkpoint)."""
-    from .models.transformer import TriuneTransformer
+    from .models.factory import build_model
     from .utils import place_model
 
     from .trainer.checkpoint import safe_torch_load
@@ -74,7 +75,7 @@ def load_checkpoint_model(path: str, device="cpu", dtype: Optional[torch.dtype] 
         cfg = infer_config_from_state_dict(sd)
     if cfg_dict and "top_k" in cfg_dict:
         cfg.top_k = int(cfg_dict["top_k"])
-    model = TriuneTransformer.from_config(cfg)
+    model = build_model(cfg)
     model.load_state_dict(sd, strict=False)
     place_model(model, device, dtype)
     model.eval()
@@ -82,12 +83,16 @@ def load_checkpoint_model(path: str, device="cpu", dtype: Optional[torch.dtype] 
 
 
 def load_model_for_inference(spec: str, device="cpu", dtype: Optional[torch.dtype] = None):
-    """``spec`` is a checkpoint path or a preset name (random-initialised)."""
+    """``spec`` is a checkpoint path, the folder of a registered architecture, or a preset name (random-initialised)."""
     import os
 
     from .models.factory import build_model
+    from .models.zoo import pretrained_class
     from .utils import place_model
 
+    cls = pretrained_class(spec)
+    if cls is not None:
+        return cls.from_pretrained(spec, device=device, dtype=dtype)
     if os.path.exists(spec):
         return load_checkpoint_model(spec, device, dtype)[0]
     model = build_model(spec)
@@ -110,6 +115,13 @@ def _apply_penalties(logits: torch.Tensor, history: torch.Tensor, repetition_pen
     return logits
 
 
+def advance(model, input_ids: torch.Tensor, cache: List[Any], decode_depth: Optional[int] = 2, **select):
+    """One step: the given tokens [B, T] after those the cache holds -> (logits, advanced cache). ``select`` picks the
+    rows of the logits (``last_token_only=True``, or ``positions=[...]`` where the model offers it). Every generation
+    path and the trace runner go through here."""
+    return model(input_ids, force_depth=decode_depth, cache=cache, **select)
+
+
 @torch.no_grad()
 def generate_tokens(model, input_ids: torch.Tensor, max_new_tokens: int = 64, temperature: float = 0.7, top_k: int = 50,
                     repetition_penalty: float = 1.1, count_penalty: float = 0.35, eos_token_id: Optional[int] = None,
@@ -126,8 +138,7 @@ def generate_tokens(model, input_ids: torch.Tensor, max_new_tokens: int = 64, te
         cache = model.init_cache(1)
     logits = None
     for s in range(0, input_ids.shape[1], prefill_chunk):
-        logits, cache = model(input_ids[:, s : s + prefill_chunk], force_depth=decode_depth, cache=cache,
-                              last_token_only=True)
+        logits, cache = advance(model, input_ids[:, s : s + prefill_chunk], cache, decode_depth, last_token_only=True)
     ttft = None
     history = input_ids[0]
     out: List[int] = []
@@ -154,8 +165,7 @@ def generate_tokens(model, input_ids: torch.Tensor, max_new_tokens: int = 64, te
             break
         if eos_token_id is not None and tok == eos_token_id:
             break
-        logits, cache = model(torch.tensor([[tok]], device=dev), force_depth=decode_depth, cache=cache,
-                              last_token_only=True)
+        logits, cache = advance(model, torch.tensor([[tok]], device=dev), cache, decode_depth, last_token_only=True)
     dt = max(1e-9, time.perf_counter() - t_dec)
     model.train(was)
     tele = {"ttft_s": ttft or 0.0, "decode_tok_s": len(out) / dt, "new_tokens": len(out),
@@ -347,6 +357,7 @@ class GraphedGreedyDecoder:
         self.step_idx = torch.zeros(1, dtype=torch.long, device=self.device)
         self.token = torch.zeros(batch_size, 1, dtype=torch.long, device=self.device)
         self.out: Optional[torch.Tensor] = None
+        self.host_pos = 0
 
     @torch.no_grad()
     def prefill(self, input_ids: torch.Tensor, prefill_chunk: int = 4096) -> torch.Tensor:
@@ -356,7 +367,7 @@ class GraphedGreedyDecoder:
         cache = m.init_cache(self.B)
         logits = None
         for s in range(0, input_ids.shape[1], prefill_chunk):
-            logits, cache = m(input_ids[:, s : s + prefill_chunk], force_depth=self.depth, cache=cache, last_token_only=True)
+            logits, cache = advance(m, input_ids[:, s : s + prefill_chunk], cache, self.depth, last_token_only=True)
         # make sure every rotary table covers the positions the graph will index
         for mod in m.modules():
             if hasattr(mod, "_build") and hasattr(mod, "head_dim") and hasattr(mod, "_cos"):
@@ -364,18 +375,21 @@ class GraphedGreedyDecoder:
         new_states = [c[0] if isinstance(c, tuple) else None for c in cache]
         if len(self.states) == len(new_states) and all((a is None) == (b is None) for a, b in zip(self.states, new_states)):
             for a, b in zip(self.states, new_states):
+                if isinstance(a, LayerState) and a.capacity is not None and a.reserve(b.capacity):
+                    self.graph = None  # the capture holds the old addresses
                 if a is not None:
                     a.copy_(b)
         else:
             self.states = [None if s is None else s.clone() for s in new_states]
             self.graph = None
         self.pos.fill_(input_ids.shape[1])
+        self.host_pos = input_ids.shape[1]
         self.token.copy_(logits[:, -1].argmax(-1, keepdim=True))
         return self.token.clone()
 
     def _step(self):
         cache = [(s, self.pos) if s is not None else (None, self.pos) for s in self.states]
-        logits, new_cache = self.model(self.token, force_depth=self.depth, cache=cache, last_token_only=True)
+        logits, new_cache = advance(self.model, self.token, cache, self.depth, last_token_only=True)
         for s, c in zip(self.states, new_cache):
             if s is not None and isinstance(c, tuple) and c[0] is not None:
                 s.copy_(c[0])
@@ -391,6 +405,10 @@ class GraphedGreedyDecoder:
             self.out = torch.zeros(self.B, max_new_tokens, dtype=torch.long, device=self.device)
             self.graph = None
         self.step_idx.zero_()
+        for s in self.states:  # key/value caches cannot grow inside a capture
+            if isinstance(s, LayerState) and s.reserve(self.host_pos + max_new_tokens + 4):
+                self.graph = None
+        self.host_pos += max_new_tokens
         if self.device.type != "cuda":
             for _ in range(max_new_tokens):
                 self._step()

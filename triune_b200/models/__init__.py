@@ -1,7 +1,10 @@
-"""Model families: multi-exit MoE ``TriuneTransformer`` and dense ``UniversalTransformer``."""
+"""Model families: multi-exit MoE ``TriuneTransformer``, dense ``UniversalTransformer`` and ``HybridTransformer`` with
+layers that differ (``Famalorn``)."""
 
 from .attention import HybridAttention, SoftmaxAttention, VectorisedGLA
 from .block import DenseFFN, TransformerBlock
+from .famalorn import Famalorn
+from .hybrid import HybridTransformer
 from .moe import MoE_FFN, RoutingResult
 from .norms import RMSNorm
 from .rotary import RotaryEmbedding
@@ -9,6 +12,6 @@ from .router import GumbelSoftmaxRouter
 from .transformer import TriuneTransformer
 
 __all__ = [
-    "HybridAttention", "SoftmaxAttention", "VectorisedGLA", "DenseFFN", "TransformerBlock", "MoE_FFN",
+    "Famalorn", "HybridTransformer", "HybridAttention", "SoftmaxAttention", "VectorisedGLA", "DenseFFN", "TransformerBlock", "MoE_FFN",
     "RoutingResult", "RMSNorm", "RotaryEmbedding", "GumbelSoftmaxRouter", "TriuneTransformer",
 ]

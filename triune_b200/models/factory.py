@@ -16,6 +16,10 @@ def build_model(cfg: Union[ModelConfig, str, Dict[str, Any]]):
         from .universal import UniversalTransformer
 
         return UniversalTransformer.from_config(cfg)
+    if cfg.family == "hybrid":
+        from .hybrid import HybridTransformer
+
+        return HybridTransformer.from_config(cfg)
     from .transformer import TriuneTransformer
 
     return TriuneTransformer.from_config(cfg)

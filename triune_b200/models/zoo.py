@@ -224,13 +224,29 @@ def _load_state(path: Path) -> Dict[str, Any]:
     return safe_torch_load(path)
 
 
+def pretrained_class(folder) -> Optional[Type[nn.Module]]:
+    """The registered class that loads a model folder: the one named by ``architecture`` in its ``config.json``."""
+    cfg = Path(str(folder)) / "config.json"
+    if not cfg.is_file():
+        return None
+    try:
+        name = json.loads(cfg.read_text(encoding="utf-8")).get("architecture")
+    except (ValueError, AttributeError):
+        return None
+    cls = MODEL_REGISTRY.get(str(name).lower())
+    return cls if cls is not None and hasattr(cls, "from_pretrained") else None
+
+
 def load_model(model_name_or_path, **kwargs: Any) -> nn.Module:
-    """Resolution order: ``.json`` config file, checkpoint file, registered architecture, canonical preset (or alias),
+    """Resolution order: folder of a registered architecture, ``.json`` config file, checkpoint file, registered architecture, canonical preset (or alias),
     ``models/configs/<name>.json`` next to the package, ``default``, then Hugging Face ``AutoModelForCausalLM``."""
     from .factory import build_model
 
     name = str(model_name_or_path).lower()
     path = Path(str(model_name_or_path))
+    cls = pretrained_class(path)
+    if cls is not None:
+        return cls.from_pretrained(path, **kwargs)
     if path.is_file() and path.suffix.lower() == ".json":
         return build_model(build_config({**json.loads(path.read_text(encoding="utf-8")), **kwargs}))
     if path.is_file():

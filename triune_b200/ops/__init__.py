@@ -111,7 +111,7 @@ def gemm(
         assert dgelu_aux is None and not gelu and not accumulate and out_dtype == torch.bfloat16
         flags |= GF_ADDAUX
         aux_in = add_aux
-    _ext.ext().tc_gemm(
+    _ext.serving().tc_gemm(
         a, b, out, a_mn, b_mn, mode, flags, float(alpha), bias, aux_in, aux_out, row_scale, tile_group,
         group_offsets, None, float(beta), k_runs,
     )
@@ -297,7 +297,7 @@ class _SwiGLUMLPFn(torch.autograd.Function):
         train = any(ctx.needs_input_grad)  # (grad mode is off inside forward: ask the context, not torch)
         h = torch.empty(M, H, device=x.device, dtype=x.dtype)
         gu = torch.empty(M, 2 * H, device=x.device, dtype=x.dtype) if train else None
-        _ext.ext().tc_gemm_swiglu(x2, w13, h, gu)
+        _ext.serving().tc_gemm_swiglu(x2, w13, h, gu)
         _tick()
         y = gemm(h, w2)
         if train:
@@ -312,7 +312,7 @@ class _SwiGLUMLPFn(torch.autograd.Function):
         if not _tma_ok(dy2):
             dy2 = dy2.contiguous()
         dgu = torch.empty_like(gu)
-        _ext.ext().tc_gemm_dswiglu(dy2, w2, True, gu, dgu)   # d(hidden) = dy @ w2, w2 stored [d, H] = [K, N]
+        _ext.serving().tc_gemm_dswiglu(dy2, w2, True, gu, dgu)   # d(hidden) = dy @ w2, w2 stored [d, H] = [K, N]
         _tick()
         dw2 = _accumulate_weight_grad(w2, dy2, h)
         dx = gemm(dgu, w13, b_mn=True).view(ctx.in_shape) if ctx.needs_input_grad[0] else None

@@ -20,6 +20,8 @@ from typing import Any, Dict, List, Optional, Tuple
 
 import torch
 
+from ..models.layer_state import LayerState
+
 
 class _Entry:
     __slots__ = ("flat", "layout", "depth", "last_active", "on_device")
@@ -33,11 +35,34 @@ class _Entry:
         return self.flat.numel() * self.flat.element_size() if self.flat is not None else 0
 
 
+def _as_words(t: torch.Tensor) -> torch.Tensor:
+    """A flat tensor's bytes as fp32 words, padded with zeros to a whole number of words."""
+    b = t.contiguous().view(torch.uint8)
+    if b.numel() % 4:
+        b = torch.cat((b, b.new_zeros(4 - b.numel() % 4)))
+    return b.view(torch.float32)
+
+
+def _from_words(words: torch.Tensor, shape, dtype) -> torch.Tensor:
+    n = 1
+    for s in shape:
+        n *= s
+    size = n * torch.empty(0, dtype=dtype).element_size()
+    return words.clone().view(torch.uint8)[:size].clone().view(dtype)
+
+
 def _pack(cache: List[Any]):
     """-> (flat tensor or None, layout). layout[i] = (shape or None, numel, offset value, dtype, passthrough item)."""
     tensors, layout = [], []
     for item in cache:
         state, off = (item if isinstance(item, tuple) else (None, 0)) if not torch.is_tensor(item) else (item, 0)
+        if isinstance(state, LayerState):
+            # several tensors of their own dtypes: kept bit for bit, reinterpreted as fp32 words
+            flats, inner = state.pack(int(off))
+            words = [_as_words(f) for f in flats]
+            layout.append(("state", inner, [w.numel() for w in words], off))
+            tensors += words
+            continue
         if item is not None and not isinstance(item, tuple) and not torch.is_tensor(item):
             layout.append(("raw", item))
         elif torch.is_tensor(state):
@@ -56,6 +81,13 @@ def _unpack(flat: Optional[torch.Tensor], layout) -> List[Any]:
             out.append(rec[1])
         elif rec[0] == "none":
             out.append((None, rec[1]))
+        elif rec[0] == "state":
+            _, inner, sizes, off = rec
+            flats = []
+            for (_, shape, dt, _), n in zip(inner, sizes):
+                flats.append(_from_words(flat[pos : pos + n], shape, dt))
+                pos += n
+            out.append((LayerState.unpack(flats, inner), off))
         else:
             _, shape, n, off, dt = rec
             out.append((flat[pos : pos + n].view(shape).to(dt), off))
