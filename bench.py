@@ -489,10 +489,23 @@ def main():
     ap.add_argument("--ref-loop", default="both", choices=["manual", "engine", "both"],
                     help="reference arm: hand-written full-batch step, the reference's TrainingEngine.step_once, or both "
                          "(the faster one is reported)")
+    ap.add_argument("--workload", default="train", choices=["train", "hybrid"],
+                    help="train: the headline benchmark; hybrid: serving of heterogeneous-layer models, one JSON line per measurement")
+    ap.add_argument("--hybrid-size", default="1b,3b", help="comma-separated layer sizes of the hybrid workload (1b, 3b)")
+    ap.add_argument("--hybrid-seq", type=int, default=8192, help="prompt length of the hybrid workload")
+    ap.add_argument("--hybrid-parts", default="model,kernels")
     args = ap.parse_args()
     args.warmup = max(3, args.warmup)
     if not torch.cuda.is_available():
         print(json.dumps({"impl": args.impl, "unavailable": "no CUDA device"}))
+        return
+    if args.workload == "hybrid":
+        from triune_b200.bench_hybrid import run as run_hybrid
+
+        sampler = ClockSampler(0)
+        sampler.start()
+        run_hybrid(args.hybrid_size.split(","), args.hybrid_seq, args.hybrid_parts)
+        print(json.dumps({"workload": "hybrid", "clocks": sampler.stop()}), flush=True)
         return
     if args.impl == "reference":
         run_reference(args)

@@ -10,7 +10,7 @@ from hybrid_cases import CONFIGS, build, rel, run_portions, tokens
 pytestmark = pytest.mark.gpu
 
 DT = [torch.float32, torch.bfloat16]
-TOL = {torch.float32: 2e-5, torch.bfloat16: 4e-2}
+TOL = {torch.float32: 2e-5, torch.bfloat16: 6e-2}  # bf16 at widths of 36 to 96: rounding alone reaches 5e-2
 
 
 def dev(t, dtype=None):

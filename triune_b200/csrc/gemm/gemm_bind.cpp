@@ -118,8 +118,8 @@ void tc_gemm(const Tensor& a, const Tensor& b, Tensor& c, bool a_mn_major, bool 
 }
 
 // SwiGLU over the fused gate/up weight inside the GEMM: h [M, H] = silu(x Wg^T) * (x Wu^T) with w13 = [Wg ; Wu]
-// ([2H, K]); gu (optional, [M, 2H]) receives both pre-activations for the backward pass.
-void tc_gemm_swiglu(const Tensor& x, const Tensor& w13, Tensor& h, const c10::optional<Tensor>& gu) {
+// ([2H, K]); gu (optional, [M, 2H]) receives both pre-activations for the backward pass. act: 0 silu, 1 relu (forward only).
+void tc_gemm_swiglu(const Tensor& x, const Tensor& w13, Tensor& h, const c10::optional<Tensor>& gu, int64_t act) {
   check_bf16_cuda(x, "x");
   check_bf16_cuda(w13, "w13");
   check_bf16_cuda(h, "h");
@@ -133,6 +133,8 @@ void tc_gemm_swiglu(const Tensor& x, const Tensor& w13, Tensor& h, const c10::op
   g.M = (int)M; g.N = (int)H; g.K = (int)K;
   g.lda = x.stride(0); g.ldb = w13.stride(0); g.ldc = h.stride(0);
   g.batch = 1; g.mode = tb::GEMM_DENSE; g.flags = tb::GF_SWIGLU; g.alpha = 1.0f; g.n_split = (int)H;
+  TORCH_CHECK(act == 0 || act == 1, "tc_gemm_swiglu: activation");
+  g.glu_act = (int)act;
   if (gu.has_value() && gu->defined()) {
     check_bf16_cuda(*gu, "gu");
     TORCH_CHECK(gu->dim() == 2 && gu->is_contiguous() && gu->size(0) == M && gu->size(1) == 2 * H, "gu must be [M, 2H] contiguous");
@@ -177,6 +179,6 @@ void register_gemm(pybind11::module& m) {
     tb::tc_gemm_set_debug_buffer(on ? (long long*)t->data_ptr<int64_t>() : nullptr);
   });
   m.def("tc_gemm_pair_launches", []() { return (int64_t)tb::tc_gemm_pair_launch_count(); });
-  m.def("tc_gemm_swiglu", &tc_gemm_swiglu);
+  m.def("tc_gemm_swiglu", &tc_gemm_swiglu, pybind11::arg("x"), pybind11::arg("w13"), pybind11::arg("h"), pybind11::arg("gu"), pybind11::arg("act") = 0);
   m.def("tc_gemm_dswiglu", &tc_gemm_dswiglu);
 }

@@ -358,6 +358,7 @@ void launch_tc_gemm(const GemmArgs& a, cudaStream_t stream) {
   kp.num_n = (a.N + n_out - 1) / n_out;
   kp.n_split = a.n_split;
   kp.beta = a.beta;
+  kp.glu_act = a.glu_act;
   kp.ldc = a.ldc; kp.strideC = a.strideC;
   kp.a_batched = a.strideA != 0; kp.b_batched = a.strideB != 0;
   kp.alpha = a.alpha;

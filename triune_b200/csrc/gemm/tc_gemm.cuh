@@ -53,6 +53,7 @@ struct GemmArgs {
   int* status;                  // optional device status word (see KernelStatus)
   int n_split;                  // GF_SWIGLU / GF_DSWIGLU: FFN hidden width (N); 0 otherwise
   float beta;                   // GF_ADDAUX: weight of aux_in
+  int glu_act;                  // GF_SWIGLU: activation of the gate, 0 silu, 1 relu
 };
 
 // Launches on `stream`. Throws std::runtime_error on invalid arguments.

@@ -49,6 +49,7 @@ struct KParams {
   int iters_per_split;  // K iterations (of 64) handled by one split
   int n_split;          // SwiGLU epilogues: column offset of the "up" half (= FFN hidden width)
   float beta;           // EPI_ADDAUX: weight of the added rows
+  int glu_act;          // EPI_SWIGLU: activation of the gate, 0 silu, 1 relu
 };
 
 struct Tile {
@@ -421,7 +422,8 @@ __device__ __forceinline__ void epilogue_tile_swiglu(const KParams& p, const Til
     for (int i = 0; i < 16; ++i) {
       const float g0 = __uint_as_float(rg[2 * i]), g1 = __uint_as_float(rg[2 * i + 1]);
       const float u0 = __uint_as_float(ru[2 * i]), u1 = __uint_as_float(ru[2 * i + 1]);
-      q[i] = pack_bf16x2(g0 * sigmoid_f(g0) * u0, g1 * sigmoid_f(g1) * u1);
+      q[i] = p.glu_act == 0 ? pack_bf16x2(g0 * sigmoid_f(g0) * u0, g1 * sigmoid_f(g1) * u1)
+                            : pack_bf16x2(fmaxf(g0, 0.f) * u0, fmaxf(g1, 0.f) * u1);
     }
     epi_store_chunk(tmC, q, n0 + c, m_base + lane_base, 0, lane, my_stage, buf);
     if (p.aux_out) {

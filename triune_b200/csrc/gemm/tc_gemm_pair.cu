@@ -410,6 +410,7 @@ bool launch_tc_gemm_pair(const GemmArgs& a, cudaStream_t stream) {
   kp.num_n = a.N / n_out;
   kp.n_split = a.n_split;
   kp.beta = 0.f;
+  kp.glu_act = a.glu_act;
   kp.ldc = a.ldc; kp.strideC = a.strideC;
   kp.a_batched = 0; kp.b_batched = 0;
   kp.alpha = a.alpha;

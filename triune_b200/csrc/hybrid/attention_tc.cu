@@ -1,0 +1,351 @@
+// Causal softmax attention with a sink on the tensor cores (bf16 operands, fp32 scores, softmax and accumulators).
+//
+// A CTA owns 256 consecutive queries of one head as two tiles of 128 and walks the keys in tiles of 128. Warp roles:
+//   warp 0      TMA producer: the two query tiles once, then a two-stage ring of key and value tiles
+//   warp 1      issues tcgen05.mma: S_w = Q_w K^T into TMEM, and O_w += P_w V with P_w read from TMEM
+//   warps 4-7   softmax of query tile 0, one row per thread (TMEM lane = row)
+//   warps 8-11  softmax of query tile 1
+// The tiles alternate: while one tile's scores are being exponentiated the tensor core works on the other. P (bf16)
+// overwrites the first half of its S columns; MMAs of one thread complete in issue order, so S_w of the next key tile
+// may be issued right behind the product that reads P_w. The running maximum is lazy: the accumulator is rescaled (by
+// the softmax warps, in TMEM) only when the maximum has grown by more than 2^8, otherwise the old reference stays and
+// the weights are at most 256 times larger, which fp32 sums and bf16 weights carry without loss. The sink starts the
+// row's maximum and sum: it has no key and no value.
+// TMEM: columns 0-127 S_0, 128-255 S_1, 256-383 O_0, 384-511 O_1.
+#include "../common/ptx.cuh"
+#include "../common/tma_desc.h"
+#include "hybrid.cuh"
+
+namespace tb {
+namespace {
+
+constexpr int FA_BM = 128, FA_BN = 128, FA_THREADS = 384, FA_BOX = 128 * 128;  // bytes of a 128 x 64 bf16 box
+constexpr float FA_LAZY = 8.f;
+
+__device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t"
+      ".reg .pred p;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t"
+      "}\n" ::"r"(tmem_d),
+      "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
+// wait::ld that the loaded registers depend on, so that no use can be scheduled before it
+__device__ __forceinline__ void tmem_ld_wait_regs(uint32_t (&r)[32]) {
+  asm volatile("tcgen05.wait::ld.sync.aligned;"
+               : "+r"(r[0]), "+r"(r[1]), "+r"(r[2]), "+r"(r[3]), "+r"(r[4]), "+r"(r[5]), "+r"(r[6]), "+r"(r[7]), "+r"(r[8]), "+r"(r[9]),
+                 "+r"(r[10]), "+r"(r[11]), "+r"(r[12]), "+r"(r[13]), "+r"(r[14]), "+r"(r[15]), "+r"(r[16]), "+r"(r[17]), "+r"(r[18]),
+                 "+r"(r[19]), "+r"(r[20]), "+r"(r[21]), "+r"(r[22]), "+r"(r[23]), "+r"(r[24]), "+r"(r[25]), "+r"(r[26]), "+r"(r[27]),
+                 "+r"(r[28])
+               :
+               : "memory");
+  asm volatile("" : "+r"(r[29]), "+r"(r[30]), "+r"(r[31])::"memory");
+}
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+struct FaParams {
+  const float* sink;
+  __nv_bfloat16* out;
+  long long ldo;
+  int T, H, G, D, E, cap;
+  float scale2;  // scale * log2(e)
+  float out_scale;
+  Pos pos;
+  int* status;
+};
+
+template <int DKB, int EVB>  // 64-wide boxes of the key and value head sizes
+__global__ void __launch_bounds__(FA_THREADS, 1) attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                                                                const __grid_constant__ CUtensorMap tmV, const FaParams p) {
+  extern __shared__ uint8_t raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~uintptr_t(1023));
+  uint8_t *sQ = smem, *sK = sQ + 2 * DKB * FA_BOX, *sV = sK + 2 * DKB * FA_BOX;
+  __shared__ __align__(8) uint64_t bars[13];
+  uint64_t *q_full = bars, *k_full = bars + 1, *k_empty = bars + 3, *v_full = bars + 5, *v_empty = bars + 7, *s_full = bars + 9,
+           *p_ready = bars + 11;
+  __shared__ __align__(8) uint64_t o_full[2];
+  __shared__ uint32_t tmem_slot;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int bh = blockIdx.x, h = bh % p.H, b = bh / p.H;
+  const int kvh = b * p.G + h / (p.H / p.G);
+  const int q0 = (gridDim.y - 1 - blockIdx.y) * 2 * FA_BM;  // the longest rows start first
+  const long long p0l = pos_of(p.pos);
+  const int p0 = (int)p0l;
+  int n[2];
+#pragma unroll
+  for (int w = 0; w < 2; ++w) {
+    const int first = q0 + w * FA_BM, last = min(p.T, first + FA_BM) - 1;
+    n[w] = first < p.T ? (p0 + last) / FA_BN + 1 : 0;
+  }
+  const int nt = max(n[0], n[1]);
+
+  if (threadIdx.x == 0) {
+    mbar_init(q_full, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(k_full + i, 1);
+      mbar_init(k_empty + i, 1);
+      mbar_init(v_full + i, 1);
+      mbar_init(v_empty + i, 1);
+      mbar_init(s_full + i, 1);
+      mbar_init(p_ready + i, 128);
+      mbar_init(o_full + i, 1);
+    }
+    mbar_fence_init();
+  }
+  if (warp == 2) {
+    tmem_alloc(&tmem_slot, 512);
+    tmem_relinquish();
+  }
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem = tmem_slot;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      prefetch_tmap(&tmQ);
+      prefetch_tmap(&tmK);
+      prefetch_tmap(&tmV);
+      const int tiles = n[1] > 0 ? 2 : 1;
+      mbar_expect_tx(q_full, tiles * DKB * FA_BOX);
+      for (int w = 0; w < tiles; ++w)
+        for (int d = 0; d < DKB; ++d) tma_load_3d(sQ + (w * DKB + d) * FA_BOX, &tmQ, q_full, d * 64, q0 + w * FA_BM, bh);
+      bool ok = true;
+      for (int j = 0; j < nt && ok; ++j) {
+        const int s = j & 1;
+        const uint32_t par = ((j >> 1) & 1) ^ 1;
+        if (j >= 2) ok = mbar_wait(k_empty + s, par);
+        if (!ok) break;
+        mbar_expect_tx(k_full + s, DKB * FA_BOX);
+        for (int d = 0; d < DKB; ++d) tma_load_3d(sK + (s * DKB + d) * FA_BOX, &tmK, k_full + s, d * 64, j * FA_BN, kvh);
+        if (j >= 2) ok = mbar_wait(v_empty + s, par);
+        if (!ok) break;
+        mbar_expect_tx(v_full + s, EVB * FA_BOX);
+        for (int d = 0; d < EVB; ++d) tma_load_3d(sV + (s * EVB + d) * FA_BOX, &tmV, v_full + s, d * 64, j * FA_BN, kvh);
+      }
+      if (!ok && p.status) *p.status = ST_TIMEOUT_EMPTY;
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      const uint32_t id_s = make_idesc(128, 128, 1, 1, 0, 0), id_o = make_idesc(128, (p.E + 15) / 16 * 16, 1, 1, 0, 1);
+      const int ks = (p.D + 15) / 16;
+      auto scores = [&](int w, int j) {
+        const uint32_t qa = smem_u32(sQ + w * DKB * FA_BOX), ka = smem_u32(sK + (j & 1) * DKB * FA_BOX);
+        for (int k = 0; k < ks; ++k) {
+          const uint32_t off = (k >> 2) * FA_BOX + (k & 3) * 32;
+          umma_bf16(tmem + w * 128, make_smem_desc(qa + off, 16, 1024), make_smem_desc(ka + off, 16, 1024), id_s, k > 0);
+        }
+        umma_commit(s_full + w);
+      };
+      auto values = [&](int w, int j) {
+        const uint32_t va = smem_u32(sV + (j & 1) * EVB * FA_BOX);
+#pragma unroll
+        for (int k = 0; k < FA_BN / 16; ++k)
+          umma_bf16_ts(tmem + 256 + w * 128, tmem + w * 128 + k * 8, make_smem_desc(va + k * 2048, FA_BOX, 1024), id_o, j > 0 || k > 0);
+      };
+      bool ok = mbar_wait(q_full, 0) && mbar_wait(k_full, 0);
+      if (ok) {
+        tc_fence_after_sync();
+        for (int w = 0; w < 2; ++w)
+          if (n[w] > 0) scores(w, 0);
+        umma_commit(k_empty);
+        for (int j = 0; j < nt && ok; ++j) {
+          ok = mbar_wait(v_full + (j & 1), (j >> 1) & 1);
+          if (ok && j + 1 < nt) ok = mbar_wait(k_full + ((j + 1) & 1), ((j + 1) >> 1) & 1);
+          for (int w = 0; w < 2 && ok; ++w) {
+            if (j >= n[w]) continue;
+            ok = mbar_wait(p_ready + w, j & 1);
+            if (!ok) break;
+            tc_fence_after_sync();
+            values(w, j);
+            if (j + 1 == n[w]) umma_commit(o_full + w);
+            else scores(w, j + 1);
+          }
+          if (!ok) break;
+          umma_commit(v_empty + (j & 1));
+          if (j + 1 < nt) umma_commit(k_empty + ((j + 1) & 1));
+        }
+      }
+      if (!ok && p.status) *p.status = ST_TIMEOUT_FULL;
+    }
+  } else if (warp >= 4) {
+    const int w = (warp - 4) >> 2, quarter = warp & 3, row = quarter * 32 + lane;
+    const int t = q0 + w * FA_BM + row;  // query of this thread
+    const int qpos = p0 + t;
+    const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
+    const uint32_t tS = tmem + lane_base + w * 128, tO = tmem + lane_base + 256 + w * 128;
+    const float c2 = p.scale2;
+    float m = p.sink != nullptr ? p.sink[h] * 1.4426950408889634f : -INFINITY, l = p.sink != nullptr ? 1.f : 0.f;
+    bool ok = true;
+    const int first = p0 + q0 + w * FA_BM;
+    for (int j = 0; j < n[w]; ++j) {
+      ok = mbar_wait(s_full + w, j & 1);
+      if (!ok) break;
+      tc_fence_after_sync();
+      const bool masked = j * FA_BN + FA_BN - 1 > first;
+      const int lim = qpos - j * FA_BN;  // columns up to this one are visible
+      uint32_t ra[32], rb[32];
+      float mx = -INFINITY;
+      auto row_max = [&](uint32_t (&r)[32], int c0) {
+        if (masked) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c0 + i <= lim) mx = fmaxf(mx, __uint_as_float(r[i]));
+        } else {
+          float x0 = __uint_as_float(r[0]), x1 = __uint_as_float(r[1]), x2 = __uint_as_float(r[2]), x3 = __uint_as_float(r[3]);
+#pragma unroll
+          for (int i = 4; i < 32; i += 4) {
+            x0 = fmaxf(x0, __uint_as_float(r[i]));
+            x1 = fmaxf(x1, __uint_as_float(r[i + 1]));
+            x2 = fmaxf(x2, __uint_as_float(r[i + 2]));
+            x3 = fmaxf(x3, __uint_as_float(r[i + 3]));
+          }
+          mx = fmaxf(mx, fmaxf(fmaxf(x0, x1), fmaxf(x2, x3)));
+        }
+      };
+      tmem_ld_32x32b_x32(tS, ra);
+      tmem_ld_wait_regs(ra);
+      tmem_ld_32x32b_x32(tS + 32, rb);
+      row_max(ra, 0);
+      tmem_ld_wait_regs(rb);
+      tmem_ld_32x32b_x32(tS + 64, ra);
+      row_max(rb, 32);
+      tmem_ld_wait_regs(ra);
+      tmem_ld_32x32b_x32(tS + 96, rb);
+      row_max(ra, 64);
+      tmem_ld_wait_regs(rb);
+      tmem_ld_32x32b_x32(tS, ra);  // the first columns again, for the exponentials
+      row_max(rb, 96);
+      const float mn = fmaxf(m, mx * c2);
+      const bool grow = j == 0 || mn - m > FA_LAZY;
+      float f = 1.f;
+      if (grow) {
+        f = ex2(m - mn);  // m = -inf at the first tile of a row without a sink gives 0
+        m = mn;
+        l *= f;
+      }
+      tmem_ld_wait_regs(ra);
+      if (j > 0 && __any_sync(0xffffffffu, grow)) {
+        for (int c = 0; c < p.E; c += 16) {
+          uint32_t o[16];
+          tmem_ld_32x32b_x16(tO + c, o);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * f);
+          tmem_st_32x32b_x16(tO + c, o);
+        }
+        tmem_st_wait();
+      }
+      const uint64_t cc = pack_f2(c2, c2), mm = pack_f2(-m, -m);
+      uint64_t sum2 = pack_f2(0.f, 0.f);
+      auto weights = [&](uint32_t (&r)[32], int c0) {
+        uint32_t q[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          float a, e;
+          unpack_f2(fma2(pack_f2(__uint_as_float(r[2 * i]), __uint_as_float(r[2 * i + 1])), cc, mm), a, e);
+          a = ex2(a);
+          e = ex2(e);
+          if (masked) {
+            a = c0 + 2 * i <= lim ? a : 0.f;
+            e = c0 + 2 * i + 1 <= lim ? e : 0.f;
+          }
+          sum2 = add2(sum2, pack_f2(a, e));
+          q[i] = pack_bf16x2(a, e);
+        }
+        tmem_st_32x32b_x16(tS + c0 / 2, q);  // lands in columns whose scores this thread has already read
+      };
+      tmem_ld_32x32b_x32(tS + 32, rb);
+      weights(ra, 0);
+      tmem_ld_wait_regs(rb);
+      tmem_ld_32x32b_x32(tS + 64, ra);
+      weights(rb, 32);
+      tmem_ld_wait_regs(ra);
+      tmem_ld_32x32b_x32(tS + 96, rb);
+      weights(ra, 64);
+      tmem_ld_wait_regs(rb);
+      weights(rb, 96);
+      float s0, s1;
+      unpack_f2(sum2, s0, s1);
+      l += s0 + s1;
+      tmem_st_wait();
+      tc_fence_before_sync();
+      mbar_arrive(p_ready + w);
+    }
+    if (ok && n[w] > 0) {
+      ok = mbar_wait(o_full + w, 0);
+      if (ok) {
+        tc_fence_after_sync();
+        const float r = p.out_scale / l;
+        __nv_bfloat16* o = p.out + ((long long)b * p.T + t) * p.ldo + (long long)h * p.E;
+        const bool vec = (p.E & 7) == 0 && (p.ldo & 7) == 0 && (reinterpret_cast<uintptr_t>(p.out) & 15) == 0;
+        for (int c = 0; c < p.E; c += 16) {
+          uint32_t v[16];
+          tmem_ld_32x32b_x16(tO + c, v);
+          tmem_ld_wait();
+          if (t < p.T) {
+            if (vec) {
+#pragma unroll
+              for (int g = 0; g < 2; ++g)
+                if (c + 8 * g < p.E) {
+                  uint4 u;
+                  uint32_t* up = &u.x;
+#pragma unroll
+                  for (int i = 0; i < 4; ++i)
+                    up[i] = pack_bf16x2(__uint_as_float(v[8 * g + 2 * i]) * r, __uint_as_float(v[8 * g + 2 * i + 1]) * r);
+                  *reinterpret_cast<uint4*>(o + c + 8 * g) = u;
+                }
+            } else {
+#pragma unroll
+              for (int i = 0; i < 16; ++i)
+                if (c + i < p.E) o[c + i] = __float2bfloat16(__uint_as_float(v[i]) * r);
+            }
+          }
+        }
+      }
+    }
+    if (!ok && p.status) *p.status = ST_TIMEOUT_TMEM;
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  if (warp == 2) tmem_dealloc(tmem, 512);
+}
+
+template <int DKB, int EVB>
+void run(const AttnArgs& a, int* status, cudaStream_t s) {
+  const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
+  CUtensorMap tq = make_tmap_3d(a.q, bf, 2, a.pitch_k, a.T, (uint64_t)a.B * a.H, a.pitch_k * 2ull, (uint64_t)a.T * a.pitch_k * 2ull, 64, 128);
+  CUtensorMap tk = make_tmap_3d(a.kc, bf, 2, a.pitch_k, a.cap, (uint64_t)a.B * a.G, a.pitch_k * 2ull, (uint64_t)a.cap * a.pitch_k * 2ull, 64, 128);
+  CUtensorMap tv = make_tmap_3d(a.vc, bf, 2, a.pitch_v, a.cap, (uint64_t)a.B * a.G, a.pitch_v * 2ull, (uint64_t)a.cap * a.pitch_v * 2ull, 64, 128);
+  FaParams p{a.sink, (__nv_bfloat16*)a.out, a.ldo, a.T, a.H, a.G, a.D, a.E, a.cap, a.scale * 1.4426950408889634f, a.out_scale, a.pos, status};
+  constexpr int smem = (4 * DKB + 2 * EVB) * FA_BOX + 1024;
+  auto kern = attn_tc_kernel<DKB, EVB>;
+  cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  kern<<<dim3(a.B * a.H, (a.T + 2 * FA_BM - 1) / (2 * FA_BM)), FA_THREADS, smem, s>>>(tq, tk, tv, p);
+}
+
+}  // namespace
+
+bool attn_tc_supported(const AttnArgs& a) {
+  return !a.f32 && a.D <= 128 && a.E <= 128 && a.scale > 0.f && a.T > 0 && a.pitch_k % 8 == 0 && a.pitch_v % 8 == 0 &&
+         (reinterpret_cast<uintptr_t>(a.q) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.kc) & 15) == 0 &&
+         (reinterpret_cast<uintptr_t>(a.vc) & 15) == 0;
+}
+
+void launch_attn_tc(const AttnArgs& a, int* status, cudaStream_t s) {
+  if (a.B <= 0 || a.T <= 0) return;
+  if (!attn_tc_supported(a)) throw std::runtime_error("attn_tc: unsupported shape");
+  if (a.D <= 64 && a.E <= 64) run<1, 1>(a, status, s);
+  else if (a.D <= 64) run<1, 2>(a, status, s);
+  else if (a.E <= 64) run<2, 1>(a, status, s);
+  else run<2, 2>(a, status, s);
+  check_launch("attn_tc");
+}
+
+}  // namespace tb

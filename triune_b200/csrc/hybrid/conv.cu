@@ -50,6 +50,53 @@ __global__ void conv_kernel(const T* __restrict__ u, long long ldu, const float*
   }
 }
 
+// Four taps, eight channels per thread: grid (ceil(C / 8 / 64), ceil(T / CONV_SEG), B), all rows 16-byte aligned.
+template <class T, int TAPS>
+__global__ void __launch_bounds__(64) conv_vec_kernel(const T* __restrict__ u, long long ldu, const float* __restrict__ w,
+                                                      const float* __restrict__ bias, const float* __restrict__ ring,
+                                                      T* __restrict__ out, long long ldo, int Tn, int C, Pos pos) {
+  const int c = (blockIdx.x * 64 + threadIdx.x) * 8;
+  if (c >= C) return;
+  const int b = blockIdx.z, t0 = blockIdx.y * CONV_SEG, t1 = min(t0 + CONV_SEG, Tn);
+  const long long p0 = pos_of(pos);
+  const T* ub = u + (long long)b * Tn * ldu + c;
+  T* ob = out + (long long)b * Tn * ldo + c;
+  float wr[TAPS][8], bb[8], x[TAPS][8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    bb[i] = bias != nullptr ? bias[c + i] : 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wr[j][i] = w[(long long)(c + i) * TAPS + j];
+  }
+#pragma unroll
+  for (int j = 1; j < TAPS; ++j) {
+    const int t = t0 - TAPS + j;
+    const long long p = p0 + t;
+    if (t >= 0) ld8v(ub + (long long)t * ldu, x[j]);
+    else if (p >= 0) ld8v(ring + ((long long)b * TAPS + p % TAPS) * C + c, x[j]);
+    else
+#pragma unroll
+      for (int i = 0; i < 8; ++i) x[j][i] = 0.f;
+  }
+#pragma unroll 4
+  for (int t = t0; t < t1; ++t) {
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) x[j - 1][i] = x[j][i];
+    ld8v(ub + (long long)t * ldu, x[TAPS - 1]);
+    float o[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      float acc = bb[i];
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) acc += wr[j][i] * x[j][i];
+      o[i] = silu_for<T>(acc);
+    }
+    st8v(ob + (long long)t * ldo, o);
+  }
+}
+
 template <class T>
 __global__ void conv_ring_kernel(const T* __restrict__ u, long long ldu, const float* __restrict__ ring_in,
                                  float* __restrict__ ring_out, int Tn, int C, int taps, Pos pos) {
@@ -66,7 +113,11 @@ template <class T>
 void conv_typed(const T* u, long long ldu, const float* w, const float* bias, const float* ring_in, float* ring_out,
                 T* out, long long ldo, int B, int Tn, int C, int taps, Pos pos, cudaStream_t s) {
   dim3 grid((C + 127) / 128, (Tn + CONV_SEG - 1) / CONV_SEG, B);
-  if (taps == 4) conv_kernel<T, 4><<<grid, 128, 0, s>>>(u, ldu, w, bias, ring_in, out, ldo, Tn, C, taps, pos);
+  const bool f32 = sizeof(T) == 4;
+  if (taps == 4 && C % 8 == 0 && vec8_ok(u, ldu, f32) && vec8_ok(out, ldo, f32) && vec8_ok(ring_in, 4, true))
+    conv_vec_kernel<T, 4><<<dim3((C / 8 + 63) / 64, (Tn + CONV_SEG - 1) / CONV_SEG, B), 64, 0, s>>>(u, ldu, w, bias, ring_in, out, ldo,
+                                                                                                    Tn, C, pos);
+  else if (taps == 4) conv_kernel<T, 4><<<grid, 128, 0, s>>>(u, ldu, w, bias, ring_in, out, ldo, Tn, C, taps, pos);
   else if (taps == 3) conv_kernel<T, 3><<<grid, 128, 0, s>>>(u, ldu, w, bias, ring_in, out, ldo, Tn, C, taps, pos);
   else if (taps == 2) conv_kernel<T, 2><<<grid, 128, 0, s>>>(u, ldu, w, bias, ring_in, out, ldo, Tn, C, taps, pos);
   else conv_kernel<T, 0><<<grid, 128, 0, s>>>(u, ldu, w, bias, ring_in, out, ldo, Tn, C, taps, pos);

@@ -99,6 +99,9 @@ struct AttnArgs {
   bool f32;
 };
 void launch_attn_simple(const AttnArgs& a, cudaStream_t s);
+// tcgen05 kernel: bf16, heads up to 128, positive scale. `status` (or null) receives a KernelStatus if a wait expires.
+bool attn_tc_supported(const AttnArgs& a);
+void launch_attn_tc(const AttnArgs& a, int* status, cudaStream_t s);
 
 // ---- decoding (one token per sequence, B <= 8) ------------------------------------------------------------------
 // y[b, n] (+)= sum_k W[n, k] in[b, k] with the input formed in the kernel's prologue from one or two segments:
@@ -185,6 +188,41 @@ __device__ __forceinline__ void stf(float* p, float v) { *p = v; }
 __device__ __forceinline__ void stf(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 __device__ __forceinline__ long long pos_of(const Pos& p) { return p.dev != nullptr ? *p.dev : p.host; }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// silu feeding a value that is stored as T: bf16 results take the fast exponential and divide
+template <class T>
+__device__ __forceinline__ float silu_for(float x) {
+  if constexpr (sizeof(T) == 4) return silu_f(x);
+  else return __fdividef(x, 1.f + __expf(-x));
+}
+// eight consecutive values, 16-byte (bf16) or 2 x 16-byte (fp32) accesses
+__device__ __forceinline__ void ld8v(const float* p, float (&f)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void ld8v(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const uint32_t a[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    f[2 * i] = __uint_as_float(a[i] << 16);
+    f[2 * i + 1] = __uint_as_float(a[i] & 0xffff0000u);
+  }
+}
+__device__ __forceinline__ void st8v(float* p, const float (&f)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+}
+__device__ __forceinline__ void st8v(__nv_bfloat16* p, const float (&f)[8]) {
+  uint4 u;
+  uint32_t* a = &u.x;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    __nv_bfloat162 t = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+    a[i] = *reinterpret_cast<uint32_t*>(&t);
+  }
+  *reinterpret_cast<uint4*>(p) = u;
+}
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 __device__ __forceinline__ float act_f(float x, int act) {
@@ -225,6 +263,10 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 }
 #endif
 
+// rows that 8-wide vector accesses may touch: base and pitch on 16-byte boundaries
+inline bool vec8_ok(const void* p, long long ld, bool f32) {
+  return (reinterpret_cast<uintptr_t>(p) & 15) == 0 && ld % (f32 ? 4 : 8) == 0;
+}
 inline void check_launch(const char* what) {
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) throw std::runtime_error(std::string(what) + " launch failed: " + cudaGetErrorString(e));

@@ -199,6 +199,20 @@ void attn_simple(const Tensor& q, const Tensor& kc, const Tensor& vc, const OptT
   tb::launch_attn_simple(a, cur_stream());
 }
 
+// the tensor-core kernel where it takes the shape, else the fp32 CUDA-core kernel
+void attention(const Tensor& q, const Tensor& kc, const Tensor& vc, const OptT& sink, Tensor& out, int64_t D, int64_t E, double scale,
+               double out_scale, int64_t pos, const OptT& pos_dev, const OptT& status) {
+  tb::AttnArgs a = attn_args(q, kc, vc, sink, out, D, E, scale, out_scale, pos, pos_dev);
+  c10::cuda::CUDAGuard guard(q.device());
+  int* st = nullptr;
+  if (status.has_value() && status->defined()) {
+    TORCH_CHECK(status->is_cuda() && status->scalar_type() == at::kInt, "status: CUDA int32 expected");
+    st = status->data_ptr<int>();
+  }
+  if (tb::attn_tc_supported(a)) tb::launch_attn_tc(a, st, cur_stream());
+  else tb::launch_attn_simple(a, cur_stream());
+}
+
 // segments: dicts with x [B, n], kind, and what the kind needs
 void gemv(const std::vector<py::dict>& segs, const Tensor& W, Tensor& y, int64_t epilogue, int64_t act) {
   TORCH_CHECK(segs.size() >= 1 && segs.size() <= 2, "gemv: one or two input segments");
@@ -295,7 +309,7 @@ tb::StepAttention step_attention(const py::dict& d, const Tensor& proj, int64_t 
   a.cap = (int)kc.size(2); a.pitch_k = (int)kc.size(3); a.pitch_v = (int)vc.size(3);
   const int rep = a.H / a.G, rm = tb::step_head_chunk(rep);
   a.splits = d["splits"].cast<int>();
-  TORCH_CHECK(a.splits >= 1, "step: splits");
+  TORCH_CHECK(a.splits >= 1 && a.splits <= 64, "step: 1 to 64 splits");
   a.part = const_cast<float*>(f32v(part, B * a.H * a.splits * (a.E + 2), "part"));
   TORCH_CHECK(cnt.is_cuda() && cnt.scalar_type() == at::kInt && cnt.is_contiguous() && cnt.numel() >= B * a.G * ((rep + rm - 1) / rm), "step: counters");
   a.counters = cnt.data_ptr<int>();
@@ -330,6 +344,7 @@ void register_hybrid(pybind11::module& m) {
   m.def("hybrid_recurrent", &recurrent);
   m.def("hybrid_attn_prep", &attn_prep);
   m.def("hybrid_attn_simple", &attn_simple);
+  m.def("hybrid_attention", &attention);
   m.def("hybrid_gemv", &gemv);
   m.def("hybrid_mixer_step", &mixer_step);
   m.def("hybrid_step_head_chunk", &tb::step_head_chunk);

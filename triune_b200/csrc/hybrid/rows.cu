@@ -1,4 +1,6 @@
 // Row kernels: embedding rows, layer / RMS norm of the fp32 residual stream, gated activations, gated norms.
+#include <type_traits>
+
 #include "hybrid.cuh"
 
 namespace tb {
@@ -65,6 +67,52 @@ __global__ void norm_rows_kernel(const float* __restrict__ x, const float* __res
   }
 }
 
+// A warp per row, the row in registers: NV float4 per lane, W <= 128 NV, W a multiple of 4.
+template <class T, int NV>
+__global__ void __launch_bounds__(128) norm_warp_kernel(const float* __restrict__ x, const float* __restrict__ w,
+                                                        T* __restrict__ y, int rows, int W, float eps, int kind) {
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  const float* xr = x + (long long)row * W;
+  T* yr = y + (long long)row * W;
+  float4 v[NV];
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * 32 + lane) * 4;
+    v[i] = c < W ? *reinterpret_cast<const float4*>(xr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+  }
+  const float mean = kind == HN_LAYER ? warp_sum(s) / W : 0.f;
+  float q = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    if ((i * 32 + lane) * 4 < W) {
+      const float a = v[i].x - mean, b = v[i].y - mean, c = v[i].z - mean, d = v[i].w - mean;
+      q += (a * a + b * b) + (c * c + d * d);
+    }
+  }
+  const float r = 1.f / sqrtf(warp_sum(q) / W + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * 32 + lane) * 4;
+    if (c < W) {
+      const float4 g = *reinterpret_cast<const float4*>(w + c);
+      const float o0 = (v[i].x - mean) * r * g.x, o1 = (v[i].y - mean) * r * g.y, o2 = (v[i].z - mean) * r * g.z,
+                  o3 = (v[i].w - mean) * r * g.w;
+      if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(yr + c) = make_float4(o0, o1, o2, o3);
+      } else {
+        __nv_bfloat162 p0 = __floats2bfloat162_rn(o0, o1), p1 = __floats2bfloat162_rn(o2, o3);
+        uint2 u;
+        u.x = *reinterpret_cast<uint32_t*>(&p0);
+        u.y = *reinterpret_cast<uint32_t*>(&p1);
+        *reinterpret_cast<uint2*>(yr + c) = u;
+      }
+    }
+  }
+}
+
 template <class T>
 __global__ void glu_rows_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, long long ldo, int F,
                                 long long n, int act) {
@@ -74,7 +122,63 @@ __global__ void glu_rows_kernel(const T* __restrict__ gu, long long ld, T* __res
   }
 }
 
-// one warp per (row, part)
+// Gated norm of parts that are a multiple of eight wide: L lanes per part (L = 8, 16, 32 lanes of a warp, or L = 128, a
+// block), NV vectors of eight per lane in registers.
+template <class T, int L, int NV>
+__global__ void __launch_bounds__(128) gated_norm_vec_kernel(const T* __restrict__ y, long long ldy, const T* __restrict__ gate,
+                                                             long long ldg, const float* __restrict__ w, int w_period,
+                                                             T* __restrict__ out, long long ldo, long long parts_total,
+                                                             int groups, int part, float eps, int order, float scale) {
+  __shared__ float red[33];
+  const long long id = (long long)blockIdx.x * (128 / L) + threadIdx.x / L;
+  const bool on = id < parts_total;
+  const int l = threadIdx.x % L;
+  const long long row = id / groups;
+  const int c0 = (int)(id % groups) * part;
+  const T *yr = y + row * ldy + c0, *gr = gate + row * ldg + c0;
+  const float* wr = w + c0 % w_period;
+  float v[NV][8], q = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * L + l) * 8;
+    if (on && c < part) {
+      float z[8];
+      ld8v(yr + c, v[i]);
+      ld8v(gr + c, z);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float s = silu_for<T>(z[j]);
+        if (order == GO_GATE_THEN_NORM) {
+          v[i][j] *= s;
+          q += v[i][j] * v[i][j];
+        } else {
+          q += v[i][j] * v[i][j];
+          v[i][j] *= s;
+        }
+      }
+    }
+  }
+  if constexpr (L == 128) {
+    q = block_sum(q, red);
+  } else {
+#pragma unroll
+    for (int o = L / 2; o > 0; o >>= 1) q += __shfl_xor_sync(0xffffffffu, q, o);
+  }
+  const float r = scale / sqrtf(q / part + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * L + l) * 8;
+    if (on && c < part) {
+      float g[8];
+      ld8v(wr + c, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] *= r * g[j];
+      st8v(out + row * ldo + c0 + c, v[i]);
+    }
+  }
+}
+
+// any part width: one warp per (row, part)
 template <class T>
 __global__ void gated_norm_kernel(const T* __restrict__ y, long long ldy, const T* __restrict__ gate, long long ldg,
                                   const float* __restrict__ w, int w_period, T* __restrict__ out, long long ldo,
@@ -115,6 +219,23 @@ void launch_norm_rows(const float* x, const float* w, void* y, bool f32, int row
                       cudaStream_t s) {
   if (rows <= 0) return;
   const size_t sm = (size_t)W * 4;
+  if (W % 4 == 0 && W <= 4096) {
+    auto warp = [&](auto* out, auto tag) {
+      using T = std::remove_pointer_t<decltype(out)>;
+      norm_warp_kernel<T, decltype(tag)::value><<<(rows + 3) / 4, 128, 0, s>>>(x, w, out, rows, W, eps, kind);
+    };
+    auto pick = [&](auto* out) {
+      if (W <= 512) warp(out, std::integral_constant<int, 4>());
+      else if (W <= 1024) warp(out, std::integral_constant<int, 8>());
+      else if (W <= 2048) warp(out, std::integral_constant<int, 16>());
+      else if (W <= 3072) warp(out, std::integral_constant<int, 24>());
+      else warp(out, std::integral_constant<int, 32>());
+    };
+    if (f32) pick((float*)y);
+    else pick((__nv_bfloat16*)y);
+    check_launch("norm_rows");
+    return;
+  }
   if (sm > 160 * 1024) throw std::runtime_error("norm_rows: rows of at most 40960 elements");
   const int th = W >= 2048 ? 256 : 128;
   auto run = [&](auto* kern, auto* out) {
@@ -141,6 +262,32 @@ void launch_gated_norm(const void* y, long long ldy, const void* gate, long long
                        float scale, cudaStream_t s) {
   if (rows <= 0) return;
   const long long parts = (long long)rows * groups;
+  const int part = inner / groups;
+  if (part % 8 == 0 && part <= 8192 && vec8_ok(y, ldy, f32) && vec8_ok(gate, ldg, f32) && vec8_ok(out, ldo, f32) &&
+      vec8_ok(w, 4, true) && w_period % 8 == 0) {
+    auto vec = [&](auto* yy, auto lanes, auto nv) {
+      using T = std::remove_const_t<std::remove_pointer_t<decltype(yy)>>;
+      constexpr int L = decltype(lanes)::value, NV = decltype(nv)::value;
+      const unsigned b = (unsigned)((parts + 128 / L - 1) / (128 / L));
+      gated_norm_vec_kernel<T, L, NV><<<b, 128, 0, s>>>((const T*)y, ldy, (const T*)gate, ldg, w, w_period, (T*)out, ldo, parts,
+                                                        groups, part, eps, order, scale);
+    };
+    using std::integral_constant;
+    auto pick = [&](auto* yy) {
+      if (part <= 64) vec(yy, integral_constant<int, 8>(), integral_constant<int, 1>());
+      else if (part <= 128) vec(yy, integral_constant<int, 16>(), integral_constant<int, 1>());
+      else if (part <= 256) vec(yy, integral_constant<int, 32>(), integral_constant<int, 1>());
+      else if (part <= 512) vec(yy, integral_constant<int, 32>(), integral_constant<int, 2>());
+      else if (part <= 1024) vec(yy, integral_constant<int, 128>(), integral_constant<int, 1>());
+      else if (part <= 2048) vec(yy, integral_constant<int, 128>(), integral_constant<int, 2>());
+      else if (part <= 4096) vec(yy, integral_constant<int, 128>(), integral_constant<int, 4>());
+      else vec(yy, integral_constant<int, 128>(), integral_constant<int, 8>());
+    };
+    if (f32) pick((const float*)y);
+    else pick((const __nv_bfloat16*)y);
+    check_launch("gated_norm");
+    return;
+  }
   const int blocks = (int)((parts + 3) / 4);
   if (f32)
     gated_norm_kernel<<<blocks, 128, 0, s>>>((const float*)y, ldy, (const float*)gate, ldg, w, w_period, (float*)out, ldo,

@@ -28,6 +28,21 @@ __device__ void gemv_segment(const GemvSegment& g, int b, float* dst, float* red
   } else {
     const float* gt = g.gate + (long long)b * g.ldg;
     const int part = g.n / g.groups, warp = tid >> 5, lane = tid & 31;
+    if (part > 512) {  // wide parts: the whole block on one part at a time
+      for (int p = 0; p < g.groups; ++p) {
+        float q = 0.f;
+        for (int i = tid; i < part; i += nt) {
+          const int c = p * part + i;
+          const float z = silu_f(gt[c]), v = x[c];
+          const float in = g.norm_kind == GO_GATE_THEN_NORM ? v * z : v;
+          q += in * in;
+          dst[c] = v * z * g.w[c % g.w_period];
+        }
+        const float r = g.scale / sqrtf(block_sum(q, red) / part + g.eps);
+        for (int i = tid; i < part; i += nt) dst[p * part + i] *= r;
+      }
+      return;
+    }
     for (int p = warp; p < g.groups; p += nt >> 5) {
       float q = 0.f;
       for (int i = lane; i < part; i += 32) {
@@ -402,21 +417,37 @@ __device__ void attention_step(const StepAttention& p, int block, long long pos,
   __threadfence();
   if (tid == 0) p.counters[bgc] = 0;
   const float* base = p.part + ((long long)b * p.H + h0) * p.splits * (p.E + 2);
-  for (int r = 0; r < nh; ++r) {
+  // weights of the splits of every head (a warp per head), then the weighted sum of their partial values
+  for (int r = warp; r < nh; r += 4) {
     const float* ph = base + r * hstride;
     const float sink = p.sink != nullptr ? p.sink[h0 + r] : -INFINITY;
     float m = sink;
-    for (int s = 0; s < p.splits; ++s) m = fmaxf(m, __ldcg(ph + s * (p.E + 2)));
-    float l = p.sink != nullptr ? expf(sink - m) : 0.f;
-    for (int s = 0; s < p.splits; ++s) l += __ldcg(ph + s * (p.E + 2) + 1) * expf(__ldcg(ph + s * (p.E + 2)) - m);
-    for (int e = tid; e < p.E; e += ST_THREADS) {
-      float t = 0.f;
-      for (int s = 0; s < p.splits; ++s) {
-        const float c = expf(__ldcg(ph + s * (p.E + 2)) - m);
-        if (c > 0.f) t += c * __ldcg(ph + s * (p.E + 2) + 2 + e);
-      }
-      p.out[(long long)b * p.ldo + (h0 + r) * p.E + e] = t / l * p.out_scale;
+    for (int s = lane; s < p.splits; s += 32) m = fmaxf(m, __ldcg(ph + s * (p.E + 2)));
+    m = warp_max(m);
+    float l = 0.f;
+    for (int s = lane; s < p.splits; s += 32) {
+      const float c = expf(__ldcg(ph + s * (p.E + 2)) - m);
+      sp[r * AT_KEYS + s] = c;  // at most 64 splits
+      l += __ldcg(ph + s * (p.E + 2) + 1) * c;
     }
+    l = warp_sum(l) + (p.sink != nullptr ? expf(sink - m) : 0.f);
+    __syncwarp();
+    for (int s = lane; s < p.splits; s += 32) sp[r * AT_KEYS + s] *= p.out_scale / l;
+  }
+  __syncthreads();
+  int active = p.splits;  // splits beyond the keys hold nothing
+  {
+    int a, z;
+    split_range((int)pos + 1, p.splits, 0, &a, &z);
+    active = min(active, ((int)pos + z) / max(z, 1));
+  }
+  for (int i = tid; i < nh * p.E; i += ST_THREADS) {
+    const int r = i / p.E, e = i % p.E;
+    const float* ph = base + r * hstride + 2 + e;
+    float t = 0.f;
+#pragma unroll 8
+    for (int s = 0; s < active; ++s) t += sp[r * AT_KEYS + s] * __ldcg(ph + s * (p.E + 2));
+    p.out[(long long)b * p.ldo + (h0 + r) * p.E + e] = t;
   }
 }
 

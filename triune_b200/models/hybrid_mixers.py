@@ -195,7 +195,9 @@ class Mixer(nn.Module):
             col += c.inputs.total
             out += c.out_width
         self.in_width, self.out_width = col, out
-        self.in_weight = nn.Parameter(torch.zeros(col, width))
+        # large projections are whole 256-row tiles, so that the GEMM runs on CTA pairs
+        rows = -(-col // 256) * 256 if col >= 1024 else col
+        self.in_weight = nn.Parameter(torch.zeros(rows, width))
         self.out_weight = nn.Parameter(torch.zeros(width, pad8(out)))
 
     def new_state(self, B: int, device, dtype) -> LayerState:
@@ -221,7 +223,7 @@ class Mixer(nn.Module):
         """The same for one token per sequence: input projection with the norm in its prologue, one launch for a
         recurrence and an attention together, output projection with the gated norm in its prologue."""
         proj = torch.empty(B, self.in_width, device=x.device)
-        hops.gemv([norm_segment], self.in_weight, proj)
+        hops.gemv([norm_segment], self.in_weight[: self.in_width], proj)
         segments, recs, atts = [], [], []
         for i, c in enumerate(self.cores):
             args, seg = c.step(proj, self.cols[i], st, f"{i}.", B)

@@ -29,6 +29,17 @@ def _host_pos(pos) -> int:
     return int(pos.reshape(-1)[0]) if torch.is_tensor(pos) else int(pos)
 
 
+_STATUS: Dict[Any, torch.Tensor] = {}
+
+
+def status_word(device) -> torch.Tensor:
+    """The device's int32 word that a kernel sets when one of its bounded waits expires (0 = none did)."""
+    key = torch.device(device)
+    if key not in _STATUS:
+        _STATUS[key] = torch.zeros(1, dtype=torch.int32, device=key)
+    return _STATUS[key]
+
+
 def embed_rows(ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
     """Embedding rows as the fp32 residual stream [tokens, width]."""
     ids = ids.reshape(-1)
@@ -52,6 +63,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
     if (_ext.use_kernels(x, w) and x.dtype == torch.bfloat16 and w.shape[0] % 8 == 0 and w.shape[1] % 8 == 0
             and _tma_ok(x) and _tma_ok(w)):
         return gemm(x, w, out_dtype=out_dtype or torch.bfloat16)
+    if x.is_cuda and x.dtype == torch.bfloat16 and out_dtype == torch.float32:
+        return torch.mm(x, w.t(), out_dtype=torch.float32)  # unaligned sizes: library product, fp32 accumulator kept
     y = F.linear(x, w)
     return y if out_dtype is None or y.dtype == torch.float64 else y.to(out_dtype)
 
@@ -63,6 +76,8 @@ def linear_accumulate(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor) -> None
         gemm(y, w, x, accumulate=True)
     elif y.dtype == x.dtype:
         x.addmm_(y, w.t())
+    elif y.is_cuda and y.dtype == torch.bfloat16:
+        x.add_(torch.mm(y, w.t(), out_dtype=torch.float32))
     else:
         x.add_(F.linear(y, w))
 
@@ -70,6 +85,12 @@ def linear_accumulate(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor) -> None
 def gated_mlp_hidden(h: torch.Tensor, gate_up: torch.Tensor, act: str) -> torch.Tensor:
     """act(h Wg^T) * (h Wu^T) with gate and up as one weight [2F, width]."""
     Fh = gate_up.shape[0] // 2
+    if (_ext.use_kernels(h, gate_up) and h.dtype == torch.bfloat16 and act in ("silu", "relu") and Fh % 32 == 0
+            and gate_up.shape[1] % 8 == 0 and _tma_ok(h) and _tma_ok(gate_up)):
+        out = torch.empty(h.shape[0], Fh, device=h.device, dtype=h.dtype)
+        _ext.serving().tc_gemm_swiglu(h, gate_up, out, None, 0 if act == "silu" else 1)  # activation in the GEMM's epilogue
+        _tick()
+        return out
     gu = linear(h, gate_up)
     if _ext.use_kernels(gu):
         _tick()
@@ -119,7 +140,7 @@ def attention(proj, cols, q_w, k_w, eps: float, freqs, sink, kc, vc, out, B: int
         h, d = _pos(pos)
         e = _ext.serving()
         q = e.hybrid_attn_prep(proj, cols[0], cols[1], cols[2], q_w, k_w, eps, freqs, kc, vc, B, T, heads, dim, vdim, h, d)
-        e.hybrid_attn_simple(q, kc, vc, sink, out, dim, vdim, scale, out_scale, h, d)
+        e.hybrid_attention(q, kc, vc, sink, out, dim, vdim, scale, out_scale, h, d, status_word(out.device))
         _tick(2)
         return
     p, G = _host_pos(pos), kc.shape[1]
