@@ -1,0 +1,621 @@
+// Chunk-parallel form of the matrix-state recurrences (Mamba-2 and gated delta rule) for prompts, bf16 inputs, with the
+// arithmetic of the recurrence kept at 32-bit grade.
+//
+// With b_i the running sum of the log decays inside a chunk of 64 tokens and S_0 the state before it:
+//   delta:   (I + L) U = R,  L_ij = beta_i e^{b_i-b_j} k_i.k_j (j < i),  R_i = beta_i (v_i - e^{b_i} S_0^T k_i)
+//   mamba2:  u_j = dt_j x_j
+//   out_i = e^{b_i} S_0^T q_i + sum_{j<=i} e^{b_i-b_j} (q_i.k_j) u_j,      S_64 = e^{b_64} S_0 + sum_j e^{b_64-b_j} k_j u_j^T
+//
+// Precision. Queries, keys and values are bf16 as stored (the unit-norm factors of the delta rule are applied as fp32
+// scalars to the products), so they enter the tensor core exactly. Every other operand (state, decayed scores, the
+// triangle's inverse, U) is fp32 and enters as the sum of two bf16 numbers; products of two such operands take three
+// MMAs. Accumulators, decays and the carried state are fp32.
+//
+// Two kernels. (1) Scores, parallel over chunks: q k^T per key group (mamba2), or per head the decayed q k^T and the
+// inverse of I + L (delta). They are written in the register order of the B operand they become, one 16-byte vector per
+// lane. (2) The walk: a block owns 16 * MT value columns of a head and walks the chunks; its four warps (per 16 columns)
+// split the tokens for the outputs and the key dimensions for the state, which stays in accumulator registers as
+// S^T [columns, Dk] and is handed between warps as bf16 pairs in shared memory. The products here are small, chained and
+// re-split between steps, so they run on mma.sync register fragments: the accumulator layout of one product is the
+// operand layout of the next, with no trip through TMEM or shared memory in between.
+#include "../common/ptx.cuh"
+#include "hybrid.cuh"
+
+namespace tb {
+namespace {
+
+constexpr int CL = 64;  // tokens per chunk
+
+__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p))
+               : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p))
+               : "memory");
+}
+__device__ __forceinline__ float lo_f(uint32_t x) { return __uint_as_float(x << 16); }
+__device__ __forceinline__ float hi_f(uint32_t x) { return __uint_as_float(x & 0xffff0000u); }
+// (a, b) as two bf16 pairs whose sum is the fp32 pair to 2^-17
+__device__ __forceinline__ void split2(float a, float b, uint32_t& h, uint32_t& l) {
+  h = pack_bf16x2(a, b);
+  l = pack_bf16x2(a - lo_f(h), b - hi_f(h));
+}
+// e^x for x <= 0
+__device__ __forceinline__ float exp_neg(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x * 1.4426950408889634f));
+  return y;
+}
+
+// Rows [t0, t0 + 64) x [0, D) of a bf16 matrix into shared memory [64][pitch]; rows past T and columns past D are zero.
+// `vec`: 16-byte asynchronous copies (D a multiple of 8, aligned rows), otherwise plain stores.
+template <int COLS, int PITCH>
+__device__ __forceinline__ void stage_rows(__nv_bfloat16* dst, const __nv_bfloat16* src, long long ld, int t0, int T, int D,
+                                           bool vec, int tid, int nt) {
+  if (vec) {
+    for (int i = tid; i < CL * (COLS / 8); i += nt) {
+      const int r = i / (COLS / 8), c = (i % (COLS / 8)) * 8;
+      __nv_bfloat16* d = dst + r * PITCH + c;
+      if (t0 + r < T && c < D)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(d)), "l"(src + (long long)(t0 + r) * ld + c) : "memory");
+      else
+        *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
+    }
+  } else {
+    for (int i = tid; i < CL * COLS; i += nt) {
+      const int r = i / COLS, c = i % COLS;
+      dst[r * PITCH + c] = t0 + r < T && c < D ? src[(long long)(t0 + r) * ld + c] : __float2bfloat16(0.f);
+    }
+  }
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_wait0() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+struct ScanParams {
+  RecurrentArgs a;
+  int nchunks;
+  bool vec_qk, vec_v;
+  uint4* frag0;   // mamba2: [B, KG, nchunks][8][4][32] fp32 scores; delta: [B, H, nchunks][8][4][32] decayed q k^T (hi, lo)
+  uint4* frag1;   // delta: the same of the inverse
+  float* unit;    // delta: [B, H, nchunks, 2, 64] 1 / |k| and Dk^-1/2 / |q|
+};
+
+// Log decay and gate of the 64 tokens of a chunk by one warp: lane i holds tokens 2 i and 2 i + 1. Tokens past T change
+// nothing (no decay, zero gate). gate: dt (mamba2) or beta (delta).
+__device__ __forceinline__ void chunk_scalars(const RecurrentArgs& p, float ra0, float ra1, float rb0, float rb1, float ea, float bias,
+                                              int t0, float* sb, float* sgate) {
+  const int lane = threadIdx.x & 31, t = t0 + 2 * lane;
+  const float d0 = t < p.T ? softplus_f(ra0 + bias) : 0.f, d1 = t + 1 < p.T ? softplus_f(ra1 + bias) : 0.f;
+  float x = -ea * (d0 + d1);
+  const float own = x;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float y = __shfl_up_sync(0xffffffffu, x, o);
+    if (lane >= o) x += y;
+  }
+  const float before = x - own;
+  sb[2 * lane] = before - ea * d0;
+  sb[2 * lane + 1] = x;
+  if (p.kind == RK_DELTA) {
+    sgate[2 * lane] = t < p.T ? sigmoid_f(rb0) : 0.f;
+    sgate[2 * lane + 1] = t + 1 < p.T ? sigmoid_f(rb1) : 0.f;
+  } else {
+    sgate[2 * lane] = d0;
+    sgate[2 * lane + 1] = d1;
+  }
+}
+__device__ __forceinline__ float load_or0(const __nv_bfloat16* p, long long ld, int t, int T) {
+  return t < T ? __bfloat162float(p[(long long)t * ld]) : 0.f;
+}
+
+// ------------------------------------------------------------------------------------------------ scores
+template <int KIND, int DK>
+__global__ void __launch_bounds__(128) chunk_scores_kernel(const ScanParams sp) {
+  constexpr int P = DK + 8;
+  extern __shared__ __align__(16) uint8_t raw[];
+  __nv_bfloat16 *sQ = reinterpret_cast<__nv_bfloat16*>(raw), *sK = sQ + CL * P;
+  const RecurrentArgs& p = sp.a;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int heads = KIND == RK_DELTA ? p.H : p.KG;
+  const int c = blockIdx.x % sp.nchunks, bh = blockIdx.x / sp.nchunks, h = bh % heads, b = bh / heads;
+  const int kh = KIND == RK_DELTA ? h / (p.H / p.KG) : h, t0 = c * CL;
+  const __nv_bfloat16 *Q = (const __nv_bfloat16*)p.q + (long long)b * p.rows * p.ldq + kh * p.Dk,
+                      *K = (const __nv_bfloat16*)p.k + (long long)b * p.rows * p.ldk + kh * p.Dk;
+  stage_rows<DK, P>(sQ, Q, p.ldq, t0, p.T, p.Dk, sp.vec_qk, tid, 128);
+  stage_rows<DK, P>(sK, K, p.ldk, t0, p.T, p.Dk, sp.vec_qk, tid, 128);
+  cp_commit();
+  __shared__ float sb[CL], sgate[CL], srk[CL], srq[CL];
+  if (KIND == RK_DELTA && warp == 0) {
+    const __nv_bfloat16 *A = (const __nv_bfloat16*)p.a + (long long)b * p.rows * p.lda + h, *Bt = (const __nv_bfloat16*)p.b + (long long)b * p.rows * p.ldb + h;
+    const int t = t0 + 2 * lane;
+    chunk_scalars(p, load_or0(A, p.lda, t, p.T), load_or0(A, p.lda, t + 1, p.T), load_or0(Bt, p.ldb, t, p.T), load_or0(Bt, p.ldb, t + 1, p.T),
+                  expf(p.A_log[h]), p.dt_bias[h], t0, sb, sgate);
+  }
+  cp_wait0();
+  __syncthreads();
+  if (KIND == RK_DELTA) {  // unit-norm factors: two threads per row
+    const int r = tid >> 1;
+    float kk = 0.f, qq = 0.f;
+    for (int d = (tid & 1) * 2; d < DK; d += 4) {
+      const uint32_t kv = *reinterpret_cast<const uint32_t*>(sK + r * P + d), qv = *reinterpret_cast<const uint32_t*>(sQ + r * P + d);
+      kk += lo_f(kv) * lo_f(kv) + hi_f(kv) * hi_f(kv);
+      qq += lo_f(qv) * lo_f(qv) + hi_f(qv) * hi_f(qv);
+    }
+    kk += __shfl_xor_sync(0xffffffffu, kk, 1);
+    qq += __shfl_xor_sync(0xffffffffu, qq, 1);
+    if ((tid & 1) == 0) {
+      srk[r] = 1.f / sqrtf(kk + p.unit_eps);
+      srq[r] = 1.f / (sqrtf(qq + p.unit_eps) * sqrtf((float)p.Dk));
+      float* un = sp.unit + ((long long)bh * sp.nchunks + c) * 2 * CL;
+      un[r] = srk[r];
+      un[CL + r] = srq[r];
+    }
+    __syncthreads();
+  }
+  // warp w: rows i of tile w against all columns j up to the diagonal. As a B operand row i is n, column j is k, and the
+  // accumulator of (A = K tile rows j, B = Q rows i) has rows j and columns i, so compute it transposed: A = rows i.
+  float* sL = reinterpret_cast<float*>(sK + CL * P);  // delta: L, then its inverse, [64][65]
+  uint32_t aq[4], ak[4], bk[4];
+  float gq[8][4], gk[8][4];
+#pragma unroll
+  for (int n = 0; n < 8; ++n)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) gq[n][i] = gk[n][i] = 0.f;
+#pragma unroll
+  for (int ks = 0; ks < DK / 16; ++ks) {
+    const int ar = warp * 16 + (lane & 15), ac = ks * 16 + (lane >> 4) * 8;
+    ldsm4(aq, sQ + ar * P + ac);
+    if (KIND == RK_DELTA) ldsm4(ak, sK + ar * P + ac);
+#pragma unroll
+    for (int nn = 0; nn < 4; ++nn) {  // 16 columns j at a time
+      if (nn > warp) break;
+      const int br = nn * 16 + (lane & 7) + ((lane >> 4) << 3), bc = ks * 16 + ((lane >> 3) & 1) * 8;
+      ldsm4(bk, sK + br * P + bc);
+      mma16816(gq[2 * nn], aq, bk[0], bk[1]);
+      mma16816(gq[2 * nn + 1], aq, bk[2], bk[3]);
+      if (KIND == RK_DELTA) {
+        mma16816(gk[2 * nn], ak, bk[0], bk[1]);
+        mma16816(gk[2 * nn + 1], ak, bk[2], bk[3]);
+      }
+    }
+  }
+  // accumulator [n][e]: row i = 16 warp + lane / 4 (+ 8 for e >= 2), column j = 8 n + 2 (lane % 4) + (e & 1).
+  // Fragment of row tile it (8 rows), column step kt (16): lane l holds (i = l / 4, j = 2 (l % 4) + {0, 1}) and j + 8: the
+  // rows of this lane are the same, so it owns whole fragments: row tile 2 warp from e = 0, 1 and 2 warp + 1 from e = 2, 3.
+  const long long base = ((long long)bh * sp.nchunks + c) * 8 * 4 * 32;
+  if constexpr (KIND == RK_MAMBA2) {
+#pragma unroll
+    for (int half = 0; half < 2; ++half)
+#pragma unroll
+      for (int kt = 0; kt < 4; ++kt) {
+        if (kt > warp) break;
+        uint4 v;
+        v.x = __float_as_uint(gq[2 * kt][2 * half]);
+        v.y = __float_as_uint(gq[2 * kt][2 * half + 1]);
+        v.z = __float_as_uint(gq[2 * kt + 1][2 * half]);
+        v.w = __float_as_uint(gq[2 * kt + 1][2 * half + 1]);
+        sp.frag0[base + ((2 * warp + half) * 4 + kt) * 32 + lane] = v;
+      }
+  } else {
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int i = 16 * warp + 8 * half + (lane >> 2);
+      const float bi = sb[i], si = srq[i], gi = sgate[i] * srk[i];
+#pragma unroll
+      for (int kt = 0; kt < 4; ++kt) {
+        if (kt > warp) break;
+        float pv[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int n = 2 * kt + (e >> 1), j = 8 * n + 2 * (lane & 3) + (e & 1);
+          const float dec = j <= i ? exp_neg(bi - sb[j]) * srk[j] : 0.f;
+          pv[e] = gq[n][2 * half + (e & 1)] * si * dec;
+          sL[i * 65 + j] = j < i ? gk[n][2 * half + (e & 1)] * gi * dec : 0.f;
+        }
+        uint4 v;
+        split2(pv[0], pv[1], v.x, v.z);
+        split2(pv[2], pv[3], v.y, v.w);
+        sp.frag0[base + ((2 * warp + half) * 4 + kt) * 32 + lane] = v;  // (hi b0, hi b1, lo b0, lo b1)
+      }
+    }
+    __syncthreads();
+    // inverse of I + L, a thread per column: T_ij = -sum_{j <= m < i} L_im T_mj, in 16-row blocks so that the running
+    // column sits in registers while L is read as broadcasts
+    float* sT = sL + CL * 65;
+    if (tid < CL) {
+      const int j = tid;
+      for (int i = 0; i < CL; ++i) sT[i * 65 + j] = i == j ? 1.f : 0.f;
+      for (int i0 = 0; i0 < CL; i0 += 16) {
+        float acc[16];
+#pragma unroll
+        for (int r = 0; r < 16; ++r) acc[r] = 0.f;
+        for (int m = 0; m < i0; ++m) {
+          const float t = sT[m * 65 + j];
+#pragma unroll
+          for (int r = 0; r < 16; ++r) acc[r] += sL[(i0 + r) * 65 + m] * t;
+        }
+        float col[16];
+#pragma unroll
+        for (int r = 0; r < 16; ++r) {
+          float s = acc[r];
+#pragma unroll
+          for (int m = 0; m < r; ++m) s += sL[(i0 + r) * 65 + i0 + m] * col[m];
+          col[r] = i0 + r == j ? 1.f : (i0 + r > j ? -s : 0.f);
+          sT[(i0 + r) * 65 + j] = col[r];
+        }
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int i = 16 * warp + 8 * half + (lane >> 2);
+      for (int kt = 0; kt <= warp; ++kt) {
+        const float* tr = sT + i * 65 + 16 * kt + 2 * (lane & 3);
+        uint4 v;
+        split2(tr[0], tr[1], v.x, v.z);
+        split2(tr[8], tr[9], v.y, v.w);
+        sp.frag1[base + ((2 * warp + half) * 4 + kt) * 32 + lane] = v;
+      }
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ walk
+template <int KIND, int DK, int MT>
+struct WalkSmem {
+  static constexpr int P = DK + 8, PV = 16 * MT + 8, PR = CL + 8;
+  __nv_bfloat16 q[2][CL * P], k[2][CL * P], v[2][CL * PV];
+  __nv_bfloat16 s[2][2][16 * MT * P];  // state buffer, hi / lo, [columns][Dk]
+  __nv_bfloat16 r[KIND == RK_DELTA ? 2 : 1][2][KIND == RK_DELTA ? 16 * MT * PR : 8];  // R and U, hi / lo, [columns][tokens]
+  __nv_bfloat16 o[CL * PV];
+  float b[2][CL], gate[2][CL], unit[2][2 * CL];
+};
+
+template <int KIND, int DK, int MT>
+__global__ void __launch_bounds__(128 * MT) chunk_walk_kernel(const ScanParams sp) {
+  using Sm = WalkSmem<KIND, DK, MT>;
+  constexpr int P = Sm::P, PV = Sm::PV, PR = Sm::PR, NT = 128 * MT, COLS = 16 * MT, KT = DK / 16, NU = DK / 32;
+  extern __shared__ __align__(16) uint8_t raw[];
+  Sm& sm = *reinterpret_cast<Sm*>(raw);
+  const RecurrentArgs& p = sp.a;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, mt = warp >> 2, wq = warp & 3;
+  const int slices = (p.Dv + COLS - 1) / COLS;
+  const int slice = blockIdx.x % slices, bh = blockIdx.x / slices, h = bh % p.H, b = bh / p.H;
+  const int kh = h / (p.H / p.KG), c0 = slice * COLS, ncol = min(COLS, p.Dv - c0);
+  const __nv_bfloat16 *Q = (const __nv_bfloat16*)p.q + (long long)b * p.rows * p.ldq + kh * p.Dk,
+                      *K = (const __nv_bfloat16*)p.k + (long long)b * p.rows * p.ldk + kh * p.Dk,
+                      *V = (const __nv_bfloat16*)p.v + (long long)b * p.rows * p.ldv + h * p.Dv + c0,
+                      *A = (const __nv_bfloat16*)p.a + (long long)b * p.rows * p.lda + h,
+                      *Bt = KIND == RK_DELTA ? (const __nv_bfloat16*)p.b + (long long)b * p.rows * p.ldb + h : A;
+  __nv_bfloat16* O = (__nv_bfloat16*)p.out + (long long)b * p.rows * p.ldo + h * p.Dv + c0;
+  const float ea = expf(p.A_log[h]), bias = p.dt_bias[h], Dh = KIND == RK_MAMBA2 ? p.D[h] : 0.f;
+  const long long fh = KIND == RK_DELTA ? bh : (long long)b * p.KG + kh;
+  const uint4 *f0 = sp.frag0 + fh * sp.nchunks * 1024, *f1 = KIND == RK_DELTA ? sp.frag1 + fh * sp.nchunks * 1024 : nullptr;
+  const float* unit = KIND == RK_DELTA ? sp.unit + (long long)bh * sp.nchunks * 2 * CL : nullptr;
+
+  auto stage = [&](int c) {
+    const int t0 = c * CL, u = c & 1;
+    stage_rows<DK, P>(sm.q[u], Q, p.ldq, t0, p.T, p.Dk, sp.vec_qk, tid, NT);
+    stage_rows<DK, P>(sm.k[u], K, p.ldk, t0, p.T, p.Dk, sp.vec_qk, tid, NT);
+    stage_rows<COLS, PV>(sm.v[u], V, p.ldv, t0, p.T, ncol, sp.vec_v, tid, NT);
+    if (KIND == RK_DELTA && tid < 2 * CL) sm.unit[u][tid] = unit[c * 2 * CL + tid];
+    cp_commit();
+  };
+  float ra0, ra1, rb0, rb1;
+  auto scalars_load = [&](int c) {
+    const int t = c * CL + 2 * lane;
+    ra0 = load_or0(A, p.lda, t, p.T);
+    ra1 = load_or0(A, p.lda, t + 1, p.T);
+    rb0 = KIND == RK_DELTA ? load_or0(Bt, p.ldb, t, p.T) : 0.f;
+    rb1 = KIND == RK_DELTA ? load_or0(Bt, p.ldb, t + 1, p.T) : 0.f;
+  };
+
+  // this warp's part of the state: columns 16 mt + {lane / 4, + 8}, key dimensions wq DK / 4 + 8 n + 2 (lane % 4) + {0, 1}
+  float S[NU][4];
+  float* st = p.state + (long long)bh * p.Dk * p.Dv;
+  const int col_lo = 16 * mt + (lane >> 2), d_lo = wq * (DK / 4) + 2 * (lane & 3);
+#pragma unroll
+  for (int n = 0; n < NU; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = d_lo + 8 * n + (e & 1), cc = col_lo + (e >> 1) * 8;
+      S[n][e] = d < p.Dk && cc < ncol ? st[(long long)d * p.Dv + c0 + cc] : 0.f;
+    }
+  auto publish = [&](int buf) {
+#pragma unroll
+    for (int n = 0; n < NU; ++n)
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        uint32_t hi, lo;
+        split2(S[n][2 * half], S[n][2 * half + 1], hi, lo);
+        const int at = (col_lo + 8 * half) * P + d_lo + 8 * n;
+        *reinterpret_cast<uint32_t*>(sm.s[buf][0] + at) = hi;
+        *reinterpret_cast<uint32_t*>(sm.s[buf][1] + at) = lo;
+      }
+  };
+  publish(0);
+  stage(0);
+  if (warp == 0) {
+    scalars_load(0);
+    chunk_scalars(p, ra0, ra1, rb0, rb1, ea, bias, 0, sm.b[0], sm.gate[0]);
+  }
+  const int a_row = 16 * mt + (lane & 15), a_col = (lane >> 4) * 8;            // ldmatrix addresses of an A operand
+  const int b_row = (lane & 7) + ((lane >> 4) << 3), b_col = ((lane >> 3) & 1) * 8;  // and of a B operand [n][k]
+  const int tok0 = 16 * wq;
+
+  for (int c = 0; c < sp.nchunks; ++c) {
+    const int u = c & 1, t0 = c * CL;
+    cp_wait0();
+    __syncthreads();  // tile c, the state before it and its scalars are in place; every warp has left chunk c - 1
+    const bool more = c + 1 < sp.nchunks;
+    if (more) stage(c + 1);
+    if (more && warp == 0) scalars_load(c + 1);
+    const float *sb = sm.b[u], *sg = sm.gate[u];
+    // score fragments of this warp's tokens (row tiles 2 wq, 2 wq + 1): issued early, used after the state products
+    uint4 fr[2][4];
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int kt = 0; kt < 4; ++kt)
+        if (kt <= wq) fr[nt][kt] = f0[(long long)c * 1024 + ((2 * wq + nt) * 4 + kt) * 32 + lane];
+    uint4 ft[2][4];
+    if constexpr (KIND == RK_DELTA) {
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int kt = 0; kt < 4; ++kt)
+          if (kt <= wq) ft[nt][kt] = f1[(long long)c * 1024 + ((2 * wq + nt) * 4 + kt) * 32 + lane];
+    }
+    // state products of this warp's 16 tokens: (S^T q) and, for the delta rule, (S^T k)
+    float oq[2][4], ok[2][4];
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) oq[nt][e] = ok[nt][e] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < KT; ++ks) {
+      uint32_t ah[4], al[4], bq[4];
+      ldsm4(ah, sm.s[u][0] + a_row * P + ks * 16 + a_col);
+      ldsm4(al, sm.s[u][1] + a_row * P + ks * 16 + a_col);
+      ldsm4(bq, sm.q[u] + (tok0 + b_row) * P + ks * 16 + b_col);
+      mma16816(oq[0], ah, bq[0], bq[1]);
+      mma16816(oq[1], ah, bq[2], bq[3]);
+      mma16816(oq[0], al, bq[0], bq[1]);
+      mma16816(oq[1], al, bq[2], bq[3]);
+      if constexpr (KIND == RK_DELTA) {
+        ldsm4(bq, sm.k[u] + (tok0 + b_row) * P + ks * 16 + b_col);
+        mma16816(ok[0], ah, bq[0], bq[1]);
+        mma16816(ok[1], ah, bq[2], bq[3]);
+        mma16816(ok[0], al, bq[0], bq[1]);
+        mma16816(ok[1], al, bq[2], bq[3]);
+      }
+    }
+    const float bl = sb[CL - 1];
+    if constexpr (KIND == RK_MAMBA2) {
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) oq[nt][e] *= exp_neg(sb[tok0 + 8 * nt + 2 * (lane & 3) + (e & 1)]);
+#pragma unroll
+      for (int kt = 0; kt < 4; ++kt) {
+        if (kt > wq) break;
+        uint32_t ax[4];
+        ldsm4t(ax, sm.v[u] + (kt * 16 + (lane & 7) + ((lane >> 4) << 3)) * PV + 16 * mt + ((lane >> 3) & 1) * 8);
+        const int j = kt * 16 + 2 * (lane & 3);
+        const float b0 = sb[j], b1 = sb[j + 1], b8 = sb[j + 8], b9 = sb[j + 9];
+        const float g0 = sg[j], g1 = sg[j + 1], g8 = sg[j + 8], g9 = sg[j + 9];
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          const int i = tok0 + 8 * nt + (lane >> 2);
+          const float bi = sb[i];
+          const float m0 = j <= i ? __uint_as_float(fr[nt][kt].x) * exp_neg(bi - b0) * g0 : 0.f;
+          const float m1 = j + 1 <= i ? __uint_as_float(fr[nt][kt].y) * exp_neg(bi - b1) * g1 : 0.f;
+          const float m8 = j + 8 <= i ? __uint_as_float(fr[nt][kt].z) * exp_neg(bi - b8) * g8 : 0.f;
+          const float m9 = j + 9 <= i ? __uint_as_float(fr[nt][kt].w) * exp_neg(bi - b9) * g9 : 0.f;
+          uint32_t h0, l0, h1, l1;
+          split2(m0, m1, h0, l0);
+          split2(m8, m9, h1, l1);
+          mma16816(oq[nt], ax, h0, h1);
+          mma16816(oq[nt], ax, l0, l1);
+        }
+      }
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = tok0 + 8 * nt + 2 * (lane & 3) + (e & 1);
+          oq[nt][e] += Dh * __bfloat162float(sm.v[u][i * PV + col_lo + (e >> 1) * 8]);
+        }
+    } else {
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = tok0 + 8 * nt + 2 * (lane & 3) + (e & 1);
+          oq[nt][e] *= exp_neg(sb[i]) * sm.unit[u][CL + i];
+        }
+      // R of this warp's tokens, as bf16 pairs for every warp of these columns
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          float r[2];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int i = tok0 + 8 * nt + 2 * (lane & 3) + e;
+            r[e] = sg[i] * (__bfloat162float(sm.v[u][i * PV + col_lo + 8 * half]) - exp_neg(sb[i]) * sm.unit[u][i] * ok[nt][2 * half + e]);
+          }
+          uint32_t hi, lo;
+          split2(r[0], r[1], hi, lo);
+          const int at = (col_lo + 8 * half) * PR + tok0 + 8 * nt + 2 * (lane & 3);
+          *reinterpret_cast<uint32_t*>(sm.r[0][0] + at) = hi;
+          *reinterpret_cast<uint32_t*>(sm.r[0][1] + at) = lo;
+        }
+      __syncthreads();
+      float uu[2][4];
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) uu[nt][e] = 0.f;
+#pragma unroll
+      for (int kt = 0; kt < 4; ++kt) {
+        if (kt > wq) break;
+        uint32_t ah[4], al[4];
+        ldsm4(ah, sm.r[0][0] + a_row * PR + kt * 16 + a_col);
+        ldsm4(al, sm.r[0][1] + a_row * PR + kt * 16 + a_col);
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          mma16816(uu[nt], ah, ft[nt][kt].x, ft[nt][kt].y);
+          mma16816(uu[nt], ah, ft[nt][kt].z, ft[nt][kt].w);
+          mma16816(uu[nt], al, ft[nt][kt].x, ft[nt][kt].y);
+        }
+      }
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          uint32_t hi, lo;
+          split2(uu[nt][2 * half], uu[nt][2 * half + 1], hi, lo);
+          const int at = (col_lo + 8 * half) * PR + tok0 + 8 * nt + 2 * (lane & 3);
+          *reinterpret_cast<uint32_t*>(sm.r[1 % (KIND == RK_DELTA ? 2 : 1)][0] + at) = hi;
+          *reinterpret_cast<uint32_t*>(sm.r[1 % (KIND == RK_DELTA ? 2 : 1)][1] + at) = lo;
+        }
+      __syncthreads();
+    }
+    // decay the state and add this chunk's keys: A = weighted values or U (columns x tokens), B = key rows
+    const float dl = exp_neg(bl);
+#pragma unroll
+    for (int n = 0; n < NU; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) S[n][e] *= dl;
+#pragma unroll
+    for (int kt = 0; kt < 4; ++kt) {
+      const int j = kt * 16 + 2 * (lane & 3);
+      uint32_t ah[4], al[4];
+      float w0 = exp_neg(bl - sb[j]), w1 = exp_neg(bl - sb[j + 1]), w8 = exp_neg(bl - sb[j + 8]), w9 = exp_neg(bl - sb[j + 9]);
+      if constexpr (KIND == RK_MAMBA2) {
+        uint32_t ax[4];
+        ldsm4t(ax, sm.v[u] + (kt * 16 + (lane & 7) + ((lane >> 4) << 3)) * PV + 16 * mt + ((lane >> 3) & 1) * 8);
+        w0 *= sg[j]; w1 *= sg[j + 1]; w8 *= sg[j + 8]; w9 *= sg[j + 9];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) split2(lo_f(ax[i]) * (i < 2 ? w0 : w8), hi_f(ax[i]) * (i < 2 ? w1 : w9), ah[i], al[i]);
+      } else {
+        uint32_t xh[4], xl[4];
+        ldsm4(xh, sm.r[KIND == RK_DELTA ? 1 : 0][0] + a_row * PR + kt * 16 + a_col);
+        ldsm4(xl, sm.r[KIND == RK_DELTA ? 1 : 0][1] + a_row * PR + kt * 16 + a_col);
+        if (kt <= wq) {
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt) {
+            mma16816(oq[nt], xh, fr[nt][kt].x, fr[nt][kt].y);
+            mma16816(oq[nt], xh, fr[nt][kt].z, fr[nt][kt].w);
+            mma16816(oq[nt], xl, fr[nt][kt].x, fr[nt][kt].y);
+          }
+        }
+        const float *su = sm.unit[u];
+        w0 *= su[j]; w1 *= su[j + 1]; w8 *= su[j + 8]; w9 *= su[j + 9];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          split2((lo_f(xh[i]) + lo_f(xl[i])) * (i < 2 ? w0 : w8), (hi_f(xh[i]) + hi_f(xl[i])) * (i < 2 ? w1 : w9), ah[i], al[i]);
+      }
+#pragma unroll
+      for (int n2 = 0; n2 < NU / 2; ++n2) {
+        uint32_t bk[4];  // key rows [token][d], transposed into B fragments of two 8-wide tiles
+        ldsm4t(bk, sm.k[u] + (kt * 16 + (lane & 15)) * P + wq * (DK / 4) + n2 * 16 + (lane >> 4) * 8);
+        mma16816(S[2 * n2], ah, bk[0], bk[1]);
+        mma16816(S[2 * n2 + 1], ah, bk[2], bk[3]);
+        mma16816(S[2 * n2], al, bk[0], bk[1]);
+        mma16816(S[2 * n2 + 1], al, bk[2], bk[3]);
+      }
+    }
+    publish(u ^ 1);
+    // outputs: transpose through shared memory (this warp's tokens and columns only), then 16-byte rows
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        sm.o[(tok0 + 8 * nt + 2 * (lane & 3) + (e & 1)) * PV + col_lo + (e >> 1) * 8] = __float2bfloat16(oq[nt][e]);
+    __syncwarp();
+    {
+      const int i = tok0 + (lane >> 1), cc = 16 * mt + (lane & 1) * 8, t = t0 + i;
+      if (t < p.T) {
+        const __nv_bfloat16* src = sm.o + i * PV + cc;
+        __nv_bfloat16* dst = O + (long long)t * p.ldo + cc;
+        if (sp.vec_v && cc + 8 <= ncol) *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src);
+        else
+          for (int e = 0; e < 8 && cc + e < ncol; ++e) dst[e] = src[e];
+      }
+    }
+    if (more && warp == 0) chunk_scalars(p, ra0, ra1, rb0, rb1, ea, bias, t0 + CL, sm.b[u ^ 1], sm.gate[u ^ 1]);
+  }
+#pragma unroll
+  for (int n = 0; n < NU; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = d_lo + 8 * n + (e & 1), cc = col_lo + (e >> 1) * 8;
+      if (d < p.Dk && cc < ncol) st[(long long)d * p.Dv + c0 + cc] = S[n][e];
+    }
+}
+
+template <int KIND, int DK, int MT>
+void run_walk(const ScanParams& sp, cudaStream_t s) {
+  const RecurrentArgs& a = sp.a;
+  auto kern = chunk_walk_kernel<KIND, DK, MT>;
+  constexpr int smem = (int)sizeof(WalkSmem<KIND, DK, MT>);
+  cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  kern<<<a.B * a.H * ((a.Dv + 16 * MT - 1) / (16 * MT)), 128 * MT, smem, s>>>(sp);
+}
+
+template <int KIND, int DK>
+void run_scan(const ScanParams& sp, cudaStream_t s) {
+  const RecurrentArgs& a = sp.a;
+  auto kern = chunk_scores_kernel<KIND, DK>;
+  constexpr int smem = 2 * CL * (DK + 8) * 2 + (KIND == RK_DELTA ? 2 * CL * 65 * 4 : 0);
+  cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  kern<<<a.B * (KIND == RK_DELTA ? a.H : a.KG) * sp.nchunks, 128, smem, s>>>(sp);
+  check_launch("chunk_scores");
+  // 32 columns per block halve the key / query traffic; 16 where the wider blocks would leave SMs without work
+  if (a.B * a.H * ((a.Dv + 31) / 32) >= 100) run_walk<KIND, DK, 2>(sp, s);
+  else run_walk<KIND, DK, 1>(sp, s);
+  check_launch("chunk_walk");
+}
+
+}  // namespace
+
+bool chunk_scan_supported(const RecurrentArgs& a) { return !a.f32 && a.Dk <= 128 && a.T >= 32; }
+
+long long chunk_scan_scratch(const RecurrentArgs& a) {
+  const long long n = (a.T + CL - 1) / CL;
+  return a.kind == RK_DELTA ? a.B * a.H * n * (2 * 16384 + 2 * CL * 4) : a.B * a.KG * n * 16384;
+}
+
+void launch_chunk_scan(const RecurrentArgs& a, void* scratch, cudaStream_t s) {
+  if (a.B <= 0 || a.T <= 0) return;
+  if (!chunk_scan_supported(a)) throw std::runtime_error("chunk_scan: unsupported shape");
+  ScanParams sp{};
+  sp.a = a;
+  sp.nchunks = (a.T + CL - 1) / CL;
+  sp.vec_qk = a.Dk % 8 == 0 && vec8_ok(a.q, a.ldq, false) && vec8_ok(a.k, a.ldk, false);
+  sp.vec_v = a.Dv % 8 == 0 && vec8_ok(a.v, a.ldv, false) && vec8_ok(a.out, a.ldo, false);
+  sp.frag0 = (uint4*)scratch;
+  if (a.kind == RK_DELTA) {
+    sp.frag1 = sp.frag0 + (long long)a.B * a.H * sp.nchunks * 1024;
+    sp.unit = (float*)(sp.frag1 + (long long)a.B * a.H * sp.nchunks * 1024);
+    if (a.Dk <= 64) run_scan<RK_DELTA, 64>(sp, s);
+    else run_scan<RK_DELTA, 128>(sp, s);
+  } else {
+    if (a.Dk <= 64) run_scan<RK_MAMBA2, 64>(sp, s);
+    else run_scan<RK_MAMBA2, 128>(sp, s);
+  }
+}
+
+}  // namespace tb

@@ -64,11 +64,16 @@ struct RecurrentArgs {
   void* out;                         // [B*T, ldo], heads of Dv
   long long ldo;
   int B, T, H, KG, Dk, Dv;
+  long long rows;                    // rows between the sequences of a batch (T unless this is a part of longer ones)
   int kind;
   float unit_eps;                    // under the root of the unit norm (delta)
   bool f32;
 };
 void launch_recurrent(const RecurrentArgs& a, cudaStream_t s);
+// Chunk-parallel form for prompts (bf16, Dk <= 128); scratch of chunk_scan_scratch(a) bytes, 16-byte aligned.
+bool chunk_scan_supported(const RecurrentArgs& a);
+long long chunk_scan_scratch(const RecurrentArgs& a);
+void launch_chunk_scan(const RecurrentArgs& a, void* scratch, cudaStream_t s);
 
 // ---- softmax attention -----------------------------------------------------------------------------------------
 // Query / key head norm + rotation; appends k and v to the cache [B, G, cap, pitch*] at positions pos .. pos+T-1 and

@@ -125,17 +125,41 @@ void fill_recurrent(tb::RecurrentArgs& r, const Tensor& q, const Tensor& k, cons
   r.out = out.data_ptr();
   r.ldo = out.stride(0);
   r.B = (int)B; r.T = (int)T; r.H = (int)H; r.KG = (int)KG; r.Dk = (int)Dk; r.Dv = (int)Dv;
+  r.rows = T;
   r.kind = (int)kind;
   r.unit_eps = (float)unit_eps;
 }
 
 void recurrent(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& a, const OptT& b, const Tensor& A_log,
                const Tensor& dt_bias, const OptT& D, Tensor& state, Tensor& out, int64_t B, int64_t T, int64_t KG, int64_t kind,
-               double unit_eps) {
+               double unit_eps, bool chunked) {
   tb::RecurrentArgs r{};
   fill_recurrent(r, q, k, v, a, b, A_log, dt_bias, D, state, out, B, T, KG, kind, unit_eps);
   c10::cuda::CUDAGuard guard(q.device());
-  tb::launch_recurrent(r, cur_stream());
+  if (!chunked || !tb::chunk_scan_supported(r)) {
+    tb::launch_recurrent(r, cur_stream());
+    return;
+  }
+  // prompts longer than the scratch budget go in parts: the state carries over
+  constexpr int64_t budget = 768ll << 20;
+  tb::RecurrentArgs part = r;
+  part.T = 64;
+  const int64_t per = std::max<int64_t>(1, budget / std::max<int64_t>(1, tb::chunk_scan_scratch(part))) * 64;
+  Tensor scratch;
+  for (int64_t t = 0; t < T; t += per) {
+    part.T = (int)std::min(per, T - t);
+    auto at = [&](const void* p, int64_t ld) { return static_cast<const char*>(p) + t * ld * 2; };
+    part.q = at(r.q, r.ldq); part.k = at(r.k, r.ldk); part.v = at(r.v, r.ldv); part.a = at(r.a, r.lda);
+    if (r.b != nullptr) part.b = at(r.b, r.ldb);
+    part.out = const_cast<char*>(at(r.out, r.ldo));
+    if (!tb::chunk_scan_supported(part)) {  // a short rest
+      tb::launch_recurrent(part, cur_stream());
+      continue;
+    }
+    const int64_t need = tb::chunk_scan_scratch(part);
+    if (!scratch.defined() || scratch.numel() < need) scratch = torch::empty({need}, q.options().dtype(at::kByte));
+    tb::launch_chunk_scan(part, scratch.data_ptr(), cur_stream());
+  }
 }
 
 bool cache_of(const Tensor& c, int64_t B, int64_t G, int64_t d, const char* n) {
@@ -341,7 +365,9 @@ void register_hybrid(pybind11::module& m) {
   m.def("hybrid_glu_rows", &glu_rows);
   m.def("hybrid_gated_norm", &gated_norm);
   m.def("hybrid_causal_conv", &causal_conv);
-  m.def("hybrid_recurrent", &recurrent);
+  m.def("hybrid_recurrent", &recurrent, pybind11::arg("q"), pybind11::arg("k"), pybind11::arg("v"), pybind11::arg("a"), pybind11::arg("b"),
+        pybind11::arg("A_log"), pybind11::arg("dt_bias"), pybind11::arg("D"), pybind11::arg("state"), pybind11::arg("out"), pybind11::arg("B"),
+        pybind11::arg("T"), pybind11::arg("key_groups"), pybind11::arg("kind"), pybind11::arg("unit_eps"), pybind11::arg("chunked") = true);
   m.def("hybrid_attn_prep", &attn_prep);
   m.def("hybrid_attn_simple", &attn_simple);
   m.def("hybrid_attention", &attention);

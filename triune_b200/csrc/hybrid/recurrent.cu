@@ -33,11 +33,11 @@ __global__ void __launch_bounds__(RB_WARPS * 32) recurrent_kernel(const Recurren
     const int d = (r >> 2) * 32 + sub * 4 + (r & 3);
     S[r] = live && d < p.Dk ? st[(long long)d * p.Dv + col] : 0.f;
   }
-  const T *Q = (const T*)p.q + (long long)b * p.T * p.ldq + kh * p.Dk, *K = (const T*)p.k + (long long)b * p.T * p.ldk + kh * p.Dk;
-  const T* V = (const T*)p.v + (long long)b * p.T * p.ldv + h * p.Dv;
-  const T* A = (const T*)p.a + (long long)b * p.T * p.lda + h;
-  const T* Bt = p.kind == RK_DELTA ? (const T*)p.b + (long long)b * p.T * p.ldb + h : nullptr;
-  T* O = (T*)p.out + (long long)b * p.T * p.ldo + h * p.Dv;
+  const T *Q = (const T*)p.q + (long long)b * p.rows * p.ldq + kh * p.Dk, *K = (const T*)p.k + (long long)b * p.rows * p.ldk + kh * p.Dk;
+  const T* V = (const T*)p.v + (long long)b * p.rows * p.ldv + h * p.Dv;
+  const T* A = (const T*)p.a + (long long)b * p.rows * p.lda + h;
+  const T* Bt = p.kind == RK_DELTA ? (const T*)p.b + (long long)b * p.rows * p.ldb + h : nullptr;
+  T* O = (T*)p.out + (long long)b * p.rows * p.ldo + h * p.Dv;
   const float ea = expf(p.A_log[h]), bias = p.dt_bias[h], Dh = p.kind == RK_MAMBA2 ? p.D[h] : 0.f;
   const float qs = p.kind == RK_DELTA ? 1.f / sqrtf((float)p.Dk) : 1.f;
 
