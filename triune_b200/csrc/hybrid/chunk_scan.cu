@@ -13,9 +13,10 @@
 //
 // Two kernels. (1) Scores, parallel over chunks: q k^T per key group (mamba2), or per head the decayed q k^T and the
 // inverse of I + L (delta). They are written in the register order of the B operand they become, one 16-byte vector per
-// lane. (2) The walk: a block owns 16 * MT value columns of a head and walks the chunks; its four warps (per 16 columns)
-// split the tokens for the outputs and the key dimensions for the state, which stays in accumulator registers as
-// S^T [columns, Dk] and is handed between warps as bf16 pairs in shared memory. The products here are small, chained and
+// lane. (2) The walk: a block owns 16 value columns of a head and walks the chunks; its eight warps split the tokens for
+// the outputs and the key dimensions for the state, which stays in accumulator registers as S^T [columns, Dk] and is
+// handed between warps as bf16 pairs in shared memory. A walk is one long dependent chain, so what can be formed ahead of
+// it is: the per-token factors (decays, gates, unit norms) are written by the scores kernel or a small kernel before it. The products here are small, chained and
 // re-split between steps, so they run on mma.sync register fragments: the accumulator layout of one product is the
 // operand layout of the next, with no trip through TMEM or shared memory in between.
 #include "../common/ptx.cuh"
@@ -81,13 +82,18 @@ __device__ __forceinline__ void stage_rows(__nv_bfloat16* dst, const __nv_bfloat
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void cp_wait0() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 
+// Per-token factors of the walk, [B, H, nchunks][FACTORS][64] fp32 (b is the running log decay of the chunk):
+//   mamba2:  0 b   1 dt   2 dt e^{b_end - b}   3 e^{b_end} in entry 0
+//   delta:   0 beta   1 beta e^b / |k|   2 e^{b_end - b} / |k|   3 e^b Dk^-1/2 / |q|   4 e^{b_end} in entry 0
+constexpr int FACTORS = 5;
+
 struct ScanParams {
   RecurrentArgs a;
   int nchunks;
   bool vec_qk, vec_v;
   uint4* frag0;   // mamba2: [B, KG, nchunks][8][4][32] fp32 scores; delta: [B, H, nchunks][8][4][32] decayed q k^T (hi, lo)
   uint4* frag1;   // delta: the same of the inverse
-  float* unit;    // delta: [B, H, nchunks, 2, 64] 1 / |k| and Dk^-1/2 / |q|
+  float* fac;
 };
 
 // Log decay and gate of the 64 tokens of a chunk by one warp: lane i holds tokens 2 i and 2 i + 1. Tokens past T change
@@ -156,9 +162,12 @@ __global__ void __launch_bounds__(128) chunk_scores_kernel(const ScanParams sp) 
     if ((tid & 1) == 0) {
       srk[r] = 1.f / sqrtf(kk + p.unit_eps);
       srq[r] = 1.f / (sqrtf(qq + p.unit_eps) * sqrtf((float)p.Dk));
-      float* un = sp.unit + ((long long)bh * sp.nchunks + c) * 2 * CL;
-      un[r] = srk[r];
-      un[CL + r] = srq[r];
+      float* f = sp.fac + ((long long)bh * sp.nchunks + c) * FACTORS * CL;
+      f[r] = sgate[r];
+      f[CL + r] = sgate[r] * exp_neg(sb[r]) * srk[r];
+      f[2 * CL + r] = exp_neg(sb[CL - 1] - sb[r]) * srk[r];
+      f[3 * CL + r] = exp_neg(sb[r]) * srq[r];
+      f[4 * CL + r] = exp_neg(sb[CL - 1]);
     }
     __syncthreads();
   }
@@ -270,65 +279,84 @@ __global__ void __launch_bounds__(128) chunk_scores_kernel(const ScanParams sp) 
   }
 }
 
+// Factors of mamba2, a warp per (batch, head, chunk).
+__global__ void __launch_bounds__(128) chunk_factors_kernel(const ScanParams sp) {
+  __shared__ float sb[4][CL], sg[4][CL];
+  const RecurrentArgs& p = sp.a;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long id = (long long)blockIdx.x * 4 + warp;
+  if (id >= (long long)p.B * p.H * sp.nchunks) return;
+  const int c = (int)(id % sp.nchunks), bh = (int)(id / sp.nchunks), h = bh % p.H, b = bh / p.H, t = c * CL + 2 * lane;
+  const __nv_bfloat16* A = (const __nv_bfloat16*)p.a + (long long)b * p.rows * p.lda + h;
+  chunk_scalars(p, load_or0(A, p.lda, t, p.T), load_or0(A, p.lda, t + 1, p.T), 0.f, 0.f, expf(p.A_log[h]), p.dt_bias[h], c * CL, sb[warp], sg[warp]);
+  __syncwarp();
+  float* f = sp.fac + id * FACTORS * CL;
+  const float bl = sb[warp][CL - 1];
+#pragma unroll
+  for (int i = lane; i < CL; i += 32) {
+    f[i] = sb[warp][i];
+    f[CL + i] = sg[warp][i];
+    f[2 * CL + i] = sg[warp][i] * exp_neg(bl - sb[warp][i]);
+    f[3 * CL + i] = exp_neg(bl);
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ walk
-template <int KIND, int DK, int MT>
+constexpr int WW = 8, WCOLS = 16;  // warps and value columns of a block; a warp owns 8 tokens and DK / 8 key dimensions
+
+template <int KIND, int DK>
 struct WalkSmem {
-  static constexpr int P = DK + 8, PV = 16 * MT + 8, PR = CL + 8;
+  static constexpr int P = DK + 8, PV = WCOLS + 8, PR = CL + 8, NR = KIND == RK_DELTA ? 3 : 1;
   __nv_bfloat16 q[2][CL * P], k[2][CL * P], v[2][CL * PV];
-  __nv_bfloat16 s[2][2][16 * MT * P];  // state buffer, hi / lo, [columns][Dk]
-  __nv_bfloat16 r[KIND == RK_DELTA ? 2 : 1][2][KIND == RK_DELTA ? 16 * MT * PR : 8];  // R and U, hi / lo, [columns][tokens]
+  __nv_bfloat16 s[2][2][WCOLS * P];     // state buffer, hi / lo, [columns][Dk]
+  __nv_bfloat16 r[NR][2][WCOLS * PR];   // 0: weighted values or U of the state update; delta 1: R, 2: U; hi / lo, [columns][tokens]
   __nv_bfloat16 o[CL * PV];
-  float b[2][CL], gate[2][CL], unit[2][2 * CL];
+  float f[2][FACTORS * CL];
 };
 
-template <int KIND, int DK, int MT>
-__global__ void __launch_bounds__(128 * MT) chunk_walk_kernel(const ScanParams sp) {
-  using Sm = WalkSmem<KIND, DK, MT>;
-  constexpr int P = Sm::P, PV = Sm::PV, PR = Sm::PR, NT = 128 * MT, COLS = 16 * MT, KT = DK / 16, NU = DK / 32;
+__device__ __forceinline__ void ldsm2t(uint32_t& r0, uint32_t& r1, const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(smem_u32(p)) : "memory");
+}
+
+template <int KIND, int DK>
+__global__ void __launch_bounds__(32 * WW) chunk_walk_kernel(const ScanParams sp) {
+  using Sm = WalkSmem<KIND, DK>;
+  constexpr int P = Sm::P, PV = Sm::PV, PR = Sm::PR, NT = 32 * WW, KT = DK / 16, DW = DK / WW, NU = DW / 8;
   extern __shared__ __align__(16) uint8_t raw[];
   Sm& sm = *reinterpret_cast<Sm*>(raw);
   const RecurrentArgs& p = sp.a;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, mt = warp >> 2, wq = warp & 3;
-  const int slices = (p.Dv + COLS - 1) / COLS;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int slices = (p.Dv + WCOLS - 1) / WCOLS;
   const int slice = blockIdx.x % slices, bh = blockIdx.x / slices, h = bh % p.H, b = bh / p.H;
-  const int kh = h / (p.H / p.KG), c0 = slice * COLS, ncol = min(COLS, p.Dv - c0);
+  const int kh = h / (p.H / p.KG), c0 = slice * WCOLS, ncol = min(WCOLS, p.Dv - c0);
   const __nv_bfloat16 *Q = (const __nv_bfloat16*)p.q + (long long)b * p.rows * p.ldq + kh * p.Dk,
                       *K = (const __nv_bfloat16*)p.k + (long long)b * p.rows * p.ldk + kh * p.Dk,
-                      *V = (const __nv_bfloat16*)p.v + (long long)b * p.rows * p.ldv + h * p.Dv + c0,
-                      *A = (const __nv_bfloat16*)p.a + (long long)b * p.rows * p.lda + h,
-                      *Bt = KIND == RK_DELTA ? (const __nv_bfloat16*)p.b + (long long)b * p.rows * p.ldb + h : A;
+                      *V = (const __nv_bfloat16*)p.v + (long long)b * p.rows * p.ldv + h * p.Dv + c0;
   __nv_bfloat16* O = (__nv_bfloat16*)p.out + (long long)b * p.rows * p.ldo + h * p.Dv + c0;
-  const float ea = expf(p.A_log[h]), bias = p.dt_bias[h], Dh = KIND == RK_MAMBA2 ? p.D[h] : 0.f;
+  const float Dh = KIND == RK_MAMBA2 ? p.D[h] : 0.f;
   const long long fh = KIND == RK_DELTA ? bh : (long long)b * p.KG + kh;
   const uint4 *f0 = sp.frag0 + fh * sp.nchunks * 1024, *f1 = KIND == RK_DELTA ? sp.frag1 + fh * sp.nchunks * 1024 : nullptr;
-  const float* unit = KIND == RK_DELTA ? sp.unit + (long long)bh * sp.nchunks * 2 * CL : nullptr;
+  const float* fac = sp.fac + (long long)bh * sp.nchunks * FACTORS * CL;
 
   auto stage = [&](int c) {
     const int t0 = c * CL, u = c & 1;
     stage_rows<DK, P>(sm.q[u], Q, p.ldq, t0, p.T, p.Dk, sp.vec_qk, tid, NT);
     stage_rows<DK, P>(sm.k[u], K, p.ldk, t0, p.T, p.Dk, sp.vec_qk, tid, NT);
-    stage_rows<COLS, PV>(sm.v[u], V, p.ldv, t0, p.T, ncol, sp.vec_v, tid, NT);
-    if (KIND == RK_DELTA && tid < 2 * CL) sm.unit[u][tid] = unit[c * 2 * CL + tid];
+    stage_rows<WCOLS, PV>(sm.v[u], V, p.ldv, t0, p.T, ncol, sp.vec_v, tid, NT);
+    if (tid < FACTORS * CL / 4)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(sm.f[u] + tid * 4)), "l"(fac + (long long)c * FACTORS * CL + tid * 4) : "memory");
     cp_commit();
   };
-  float ra0, ra1, rb0, rb1;
-  auto scalars_load = [&](int c) {
-    const int t = c * CL + 2 * lane;
-    ra0 = load_or0(A, p.lda, t, p.T);
-    ra1 = load_or0(A, p.lda, t + 1, p.T);
-    rb0 = KIND == RK_DELTA ? load_or0(Bt, p.ldb, t, p.T) : 0.f;
-    rb1 = KIND == RK_DELTA ? load_or0(Bt, p.ldb, t + 1, p.T) : 0.f;
-  };
 
-  // this warp's part of the state: columns 16 mt + {lane / 4, + 8}, key dimensions wq DK / 4 + 8 n + 2 (lane % 4) + {0, 1}
+  // this warp's part of the state: columns lane / 4 and + 8, key dimensions warp DW + 8 n + 2 (lane % 4) + {0, 1}
   float S[NU][4];
   float* st = p.state + (long long)bh * p.Dk * p.Dv;
-  const int col_lo = 16 * mt + (lane >> 2), d_lo = wq * (DK / 4) + 2 * (lane & 3);
+  const int col = lane >> 2, pair = 2 * (lane & 3), d_lo = warp * DW + pair;
 #pragma unroll
   for (int n = 0; n < NU; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = d_lo + 8 * n + (e & 1), cc = col_lo + (e >> 1) * 8;
+      const int d = d_lo + 8 * n + (e & 1), cc = col + (e >> 1) * 8;
       S[n][e] = d < p.Dk && cc < ncol ? st[(long long)d * p.Dv + c0 + cc] : 0.f;
     }
   auto publish = [&](int buf) {
@@ -338,215 +366,198 @@ __global__ void __launch_bounds__(128 * MT) chunk_walk_kernel(const ScanParams s
       for (int half = 0; half < 2; ++half) {
         uint32_t hi, lo;
         split2(S[n][2 * half], S[n][2 * half + 1], hi, lo);
-        const int at = (col_lo + 8 * half) * P + d_lo + 8 * n;
+        const int at = (col + 8 * half) * P + d_lo + 8 * n;
         *reinterpret_cast<uint32_t*>(sm.s[buf][0] + at) = hi;
         *reinterpret_cast<uint32_t*>(sm.s[buf][1] + at) = lo;
       }
   };
   publish(0);
   stage(0);
-  if (warp == 0) {
-    scalars_load(0);
-    chunk_scalars(p, ra0, ra1, rb0, rb1, ea, bias, 0, sm.b[0], sm.gate[0]);
-  }
-  const int a_row = 16 * mt + (lane & 15), a_col = (lane >> 4) * 8;            // ldmatrix addresses of an A operand
-  const int b_row = (lane & 7) + ((lane >> 4) << 3), b_col = ((lane >> 3) & 1) * 8;  // and of a B operand [n][k]
-  const int tok0 = 16 * wq;
+  const int a_row = lane & 15, a_col = (lane >> 4) * 8;  // ldmatrix addresses of an A operand [column][k]
+  const int tok0 = 8 * warp, wt = warp >> 1;             // this warp's tokens; their 16-token tile
+  const int b_at = (tok0 + (lane & 7)) * P + (lane >> 3) * 8;  // B operand [token][k], two steps of 16 per load
+  // a value pair of this lane's tokens, columns col and col + 8, as bf16 pairs into r[which]
+  auto put = [&](int which, const float (&x)[4]) {
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      uint32_t hi, lo;
+      split2(x[2 * half], x[2 * half + 1], hi, lo);
+      const int at = (col + 8 * half) * PR + tok0 + pair;
+      *reinterpret_cast<uint32_t*>(sm.r[which][0] + at) = hi;
+      *reinterpret_cast<uint32_t*>(sm.r[which][1] + at) = lo;
+    }
+  };
 
   for (int c = 0; c < sp.nchunks; ++c) {
     const int u = c & 1, t0 = c * CL;
     cp_wait0();
-    __syncthreads();  // tile c, the state before it and its scalars are in place; every warp has left chunk c - 1
-    const bool more = c + 1 < sp.nchunks;
-    if (more) stage(c + 1);
-    if (more && warp == 0) scalars_load(c + 1);
-    const float *sb = sm.b[u], *sg = sm.gate[u];
-    // score fragments of this warp's tokens (row tiles 2 wq, 2 wq + 1): issued early, used after the state products
-    uint4 fr[2][4];
+    __syncthreads();  // tile c, its factors and the state before it are in place; every warp has left chunk c - 1
+    if (c + 1 < sp.nchunks) stage(c + 1);
+    const float* F = sm.f[u];
+    // score fragments of this warp's row tile: issued early, used after the state products
+    uint4 fr[4], ft[KIND == RK_DELTA ? 4 : 1];
 #pragma unroll
-    for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-      for (int kt = 0; kt < 4; ++kt)
-        if (kt <= wq) fr[nt][kt] = f0[(long long)c * 1024 + ((2 * wq + nt) * 4 + kt) * 32 + lane];
-    uint4 ft[2][4];
-    if constexpr (KIND == RK_DELTA) {
-#pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-        for (int kt = 0; kt < 4; ++kt)
-          if (kt <= wq) ft[nt][kt] = f1[(long long)c * 1024 + ((2 * wq + nt) * 4 + kt) * 32 + lane];
-    }
-    // state products of this warp's 16 tokens: (S^T q) and, for the delta rule, (S^T k)
-    float oq[2][4], ok[2][4];
-#pragma unroll
-    for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) oq[nt][e] = ok[nt][e] = 0.f;
-#pragma unroll
-    for (int ks = 0; ks < KT; ++ks) {
-      uint32_t ah[4], al[4], bq[4];
-      ldsm4(ah, sm.s[u][0] + a_row * P + ks * 16 + a_col);
-      ldsm4(al, sm.s[u][1] + a_row * P + ks * 16 + a_col);
-      ldsm4(bq, sm.q[u] + (tok0 + b_row) * P + ks * 16 + b_col);
-      mma16816(oq[0], ah, bq[0], bq[1]);
-      mma16816(oq[1], ah, bq[2], bq[3]);
-      mma16816(oq[0], al, bq[0], bq[1]);
-      mma16816(oq[1], al, bq[2], bq[3]);
-      if constexpr (KIND == RK_DELTA) {
-        ldsm4(bq, sm.k[u] + (tok0 + b_row) * P + ks * 16 + b_col);
-        mma16816(ok[0], ah, bq[0], bq[1]);
-        mma16816(ok[1], ah, bq[2], bq[3]);
-        mma16816(ok[0], al, bq[0], bq[1]);
-        mma16816(ok[1], al, bq[2], bq[3]);
+    for (int kt = 0; kt < 4; ++kt)
+      if (kt <= wt) {
+        fr[kt] = f0[(long long)c * 1024 + (warp * 4 + kt) * 32 + lane];
+        if constexpr (KIND == RK_DELTA) ft[kt] = f1[(long long)c * 1024 + (warp * 4 + kt) * 32 + lane];
       }
-    }
-    const float bl = sb[CL - 1];
+    float x[4];  // values of this lane's tokens: [column half][token of the pair]
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[e] = __bfloat162float(sm.v[u][(tok0 + pair + (e & 1)) * PV + col + (e >> 1) * 8]);
     if constexpr (KIND == RK_MAMBA2) {
+      const float w0 = F[2 * CL + tok0 + pair], w1 = F[2 * CL + tok0 + pair + 1];
+      const float xw[4] = {x[0] * w0, x[1] * w1, x[2] * w0, x[3] * w1};
+      put(0, xw);
+    }
+    // state products of this warp's tokens: S^T q and, for the delta rule, S^T k (hi and lo in separate accumulators)
+    float oq[4] = {0.f, 0.f, 0.f, 0.f}, oq2[4] = {0.f, 0.f, 0.f, 0.f}, ok[4] = {0.f, 0.f, 0.f, 0.f}, ok2[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
+    for (int ks = 0; ks < KT; ks += 2) {
+      uint32_t ah[2][4], al[2][4], bq[4], bk[4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) oq[nt][e] *= exp_neg(sb[tok0 + 8 * nt + 2 * (lane & 3) + (e & 1)]);
+      for (int i = 0; i < 2; ++i) {
+        ldsm4(ah[i], sm.s[u][0] + a_row * P + (ks + i) * 16 + a_col);
+        ldsm4(al[i], sm.s[u][1] + a_row * P + (ks + i) * 16 + a_col);
+      }
+      ldsm4(bq, sm.q[u] + b_at + ks * 16);
+      if constexpr (KIND == RK_DELTA) ldsm4(bk, sm.k[u] + b_at + ks * 16);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        mma16816(oq, ah[i], bq[2 * i], bq[2 * i + 1]);
+        mma16816(oq2, al[i], bq[2 * i], bq[2 * i + 1]);
+        if constexpr (KIND == RK_DELTA) {
+          mma16816(ok, ah[i], bk[2 * i], bk[2 * i + 1]);
+          mma16816(ok2, al[i], bk[2 * i], bk[2 * i + 1]);
+        }
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      oq[e] += oq2[e];
+      ok[e] += ok2[e];
+    }
+    if constexpr (KIND == RK_MAMBA2) {
+      // tokens before this 16-token tile: e^{b_i - b_j} = e^{b_i - b_ref} e^{b_ref - b_j} with the tile's first token as
+      // reference, both factors at most 1; the first is applied once to the whole sum
+      const float br = F[16 * wt], er = exp_neg(br);
+      float od[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) oq[e] *= er;
+      const int i = tok0 + col;  // as a B operand, the row of the scores is lane / 4
+      const float bi = F[i];
 #pragma unroll
       for (int kt = 0; kt < 4; ++kt) {
-        if (kt > wq) break;
+        if (kt > wt) break;
         uint32_t ax[4];
-        ldsm4t(ax, sm.v[u] + (kt * 16 + (lane & 7) + ((lane >> 4) << 3)) * PV + 16 * mt + ((lane >> 3) & 1) * 8);
-        const int j = kt * 16 + 2 * (lane & 3);
-        const float b0 = sb[j], b1 = sb[j + 1], b8 = sb[j + 8], b9 = sb[j + 9];
-        const float g0 = sg[j], g1 = sg[j + 1], g8 = sg[j + 8], g9 = sg[j + 9];
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          const int i = tok0 + 8 * nt + (lane >> 2);
-          const float bi = sb[i];
-          const float m0 = j <= i ? __uint_as_float(fr[nt][kt].x) * exp_neg(bi - b0) * g0 : 0.f;
-          const float m1 = j + 1 <= i ? __uint_as_float(fr[nt][kt].y) * exp_neg(bi - b1) * g1 : 0.f;
-          const float m8 = j + 8 <= i ? __uint_as_float(fr[nt][kt].z) * exp_neg(bi - b8) * g8 : 0.f;
-          const float m9 = j + 9 <= i ? __uint_as_float(fr[nt][kt].w) * exp_neg(bi - b9) * g9 : 0.f;
-          uint32_t h0, l0, h1, l1;
-          split2(m0, m1, h0, l0);
-          split2(m8, m9, h1, l1);
-          mma16816(oq[nt], ax, h0, h1);
-          mma16816(oq[nt], ax, l0, l1);
+        ldsm4t(ax, sm.v[u] + (kt * 16 + (lane & 7) + ((lane >> 4) << 3)) * PV + ((lane >> 3) & 1) * 8);
+        const int j = kt * 16 + pair;
+        const bool diag = kt == wt;
+        const float ref = diag ? bi : br;
+        const float2 b0 = *reinterpret_cast<const float2*>(F + j), b8 = *reinterpret_cast<const float2*>(F + j + 8);
+        const float2 g0 = *reinterpret_cast<const float2*>(F + CL + j), g8 = *reinterpret_cast<const float2*>(F + CL + j + 8);
+        float m0 = __uint_as_float(fr[kt].x) * g0.x * exp_neg(fminf(ref - b0.x, 0.f));
+        float m1 = __uint_as_float(fr[kt].y) * g0.y * exp_neg(fminf(ref - b0.y, 0.f));
+        float m8 = __uint_as_float(fr[kt].z) * g8.x * exp_neg(fminf(ref - b8.x, 0.f));
+        float m9 = __uint_as_float(fr[kt].w) * g8.y * exp_neg(fminf(ref - b8.y, 0.f));
+        if (diag) {
+          m0 = j <= i ? m0 : 0.f;
+          m1 = j + 1 <= i ? m1 : 0.f;
+          m8 = j + 8 <= i ? m8 : 0.f;
+          m9 = j + 9 <= i ? m9 : 0.f;
+        }
+        uint32_t h0, l0, h1, l1;
+        split2(m0, m1, h0, l0);
+        split2(m8, m9, h1, l1);
+        if (diag) {
+          mma16816(od, ax, h0, h1);
+          mma16816(od, ax, l0, l1);
+        } else {
+          mma16816(oq, ax, h0, h1);
+          mma16816(oq, ax, l0, l1);
         }
       }
+      const float e0 = exp_neg(F[tok0 + pair] - br), e1 = exp_neg(F[tok0 + pair + 1] - br);
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int i = tok0 + 8 * nt + 2 * (lane & 3) + (e & 1);
-          oq[nt][e] += Dh * __bfloat162float(sm.v[u][i * PV + col_lo + (e >> 1) * 8]);
-        }
+      for (int e = 0; e < 4; ++e) oq[e] = oq[e] * ((e & 1) ? e1 : e0) + od[e] + Dh * x[e];
+      __syncthreads();  // weighted values of every warp
     } else {
+      float r[4];
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int i = tok0 + 8 * nt + 2 * (lane & 3) + (e & 1);
-          oq[nt][e] *= exp_neg(sb[i]) * sm.unit[u][CL + i];
-        }
-      // R of this warp's tokens, as bf16 pairs for every warp of these columns
-#pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          float r[2];
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            const int i = tok0 + 8 * nt + 2 * (lane & 3) + e;
-            r[e] = sg[i] * (__bfloat162float(sm.v[u][i * PV + col_lo + 8 * half]) - exp_neg(sb[i]) * sm.unit[u][i] * ok[nt][2 * half + e]);
-          }
-          uint32_t hi, lo;
-          split2(r[0], r[1], hi, lo);
-          const int at = (col_lo + 8 * half) * PR + tok0 + 8 * nt + 2 * (lane & 3);
-          *reinterpret_cast<uint32_t*>(sm.r[0][0] + at) = hi;
-          *reinterpret_cast<uint32_t*>(sm.r[0][1] + at) = lo;
-        }
+      for (int e = 0; e < 4; ++e) {
+        const int i = tok0 + pair + (e & 1);
+        oq[e] *= F[3 * CL + i];
+        r[e] = F[i] * x[e] - F[CL + i] * ok[e];
+      }
+      put(1, r);
       __syncthreads();
-      float uu[2][4];
-#pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) uu[nt][e] = 0.f;
+      float uu[4] = {0.f, 0.f, 0.f, 0.f}, u2[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int kt = 0; kt < 4; ++kt) {
-        if (kt > wq) break;
+        if (kt > wt) break;
         uint32_t ah[4], al[4];
-        ldsm4(ah, sm.r[0][0] + a_row * PR + kt * 16 + a_col);
-        ldsm4(al, sm.r[0][1] + a_row * PR + kt * 16 + a_col);
-#pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          mma16816(uu[nt], ah, ft[nt][kt].x, ft[nt][kt].y);
-          mma16816(uu[nt], ah, ft[nt][kt].z, ft[nt][kt].w);
-          mma16816(uu[nt], al, ft[nt][kt].x, ft[nt][kt].y);
-        }
+        ldsm4(ah, sm.r[Sm::NR > 1 ? 1 : 0][0] + a_row * PR + kt * 16 + a_col);
+        ldsm4(al, sm.r[Sm::NR > 1 ? 1 : 0][1] + a_row * PR + kt * 16 + a_col);
+        mma16816(uu, ah, ft[kt].x, ft[kt].y);
+        mma16816(u2, ah, ft[kt].z, ft[kt].w);
+        mma16816(u2, al, ft[kt].x, ft[kt].y);
       }
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          uint32_t hi, lo;
-          split2(uu[nt][2 * half], uu[nt][2 * half + 1], hi, lo);
-          const int at = (col_lo + 8 * half) * PR + tok0 + 8 * nt + 2 * (lane & 3);
-          *reinterpret_cast<uint32_t*>(sm.r[1 % (KIND == RK_DELTA ? 2 : 1)][0] + at) = hi;
-          *reinterpret_cast<uint32_t*>(sm.r[1 % (KIND == RK_DELTA ? 2 : 1)][1] + at) = lo;
-        }
+      for (int e = 0; e < 4; ++e) uu[e] += u2[e];
+      put(Sm::NR > 2 ? 2 : 0, uu);
+      const float w0 = F[2 * CL + tok0 + pair], w1 = F[2 * CL + tok0 + pair + 1];
+      const float uw[4] = {uu[0] * w0, uu[1] * w1, uu[2] * w0, uu[3] * w1};
+      put(0, uw);
       __syncthreads();
     }
     // decay the state and add this chunk's keys: A = weighted values or U (columns x tokens), B = key rows
-    const float dl = exp_neg(bl);
+    const float dl = F[(KIND == RK_DELTA ? 4 : 3) * CL];
 #pragma unroll
     for (int n = 0; n < NU; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) S[n][e] *= dl;
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
-      const int j = kt * 16 + 2 * (lane & 3);
       uint32_t ah[4], al[4];
-      float w0 = exp_neg(bl - sb[j]), w1 = exp_neg(bl - sb[j + 1]), w8 = exp_neg(bl - sb[j + 8]), w9 = exp_neg(bl - sb[j + 9]);
-      if constexpr (KIND == RK_MAMBA2) {
-        uint32_t ax[4];
-        ldsm4t(ax, sm.v[u] + (kt * 16 + (lane & 7) + ((lane >> 4) << 3)) * PV + 16 * mt + ((lane >> 3) & 1) * 8);
-        w0 *= sg[j]; w1 *= sg[j + 1]; w8 *= sg[j + 8]; w9 *= sg[j + 9];
-#pragma unroll
-        for (int i = 0; i < 4; ++i) split2(lo_f(ax[i]) * (i < 2 ? w0 : w8), hi_f(ax[i]) * (i < 2 ? w1 : w9), ah[i], al[i]);
+      ldsm4(ah, sm.r[0][0] + a_row * PR + kt * 16 + a_col);
+      ldsm4(al, sm.r[0][1] + a_row * PR + kt * 16 + a_col);
+      const __nv_bfloat16* kr = sm.k[u] + (kt * 16 + (lane & 15)) * P + warp * DW;  // key rows, transposed into B fragments
+      if constexpr (NU == 2) {
+        uint32_t bk[4];
+        ldsm4t(bk, kr + (lane >> 4) * 8);
+        mma16816(S[0], ah, bk[0], bk[1]);
+        mma16816(S[1], ah, bk[2], bk[3]);
+        mma16816(S[0], al, bk[0], bk[1]);
+        mma16816(S[1], al, bk[2], bk[3]);
       } else {
-        uint32_t xh[4], xl[4];
-        ldsm4(xh, sm.r[KIND == RK_DELTA ? 1 : 0][0] + a_row * PR + kt * 16 + a_col);
-        ldsm4(xl, sm.r[KIND == RK_DELTA ? 1 : 0][1] + a_row * PR + kt * 16 + a_col);
-        if (kt <= wq) {
-#pragma unroll
-          for (int nt = 0; nt < 2; ++nt) {
-            mma16816(oq[nt], xh, fr[nt][kt].x, fr[nt][kt].y);
-            mma16816(oq[nt], xh, fr[nt][kt].z, fr[nt][kt].w);
-            mma16816(oq[nt], xl, fr[nt][kt].x, fr[nt][kt].y);
-          }
-        }
-        const float *su = sm.unit[u];
-        w0 *= su[j]; w1 *= su[j + 1]; w8 *= su[j + 8]; w9 *= su[j + 9];
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-          split2((lo_f(xh[i]) + lo_f(xl[i])) * (i < 2 ? w0 : w8), (hi_f(xh[i]) + hi_f(xl[i])) * (i < 2 ? w1 : w9), ah[i], al[i]);
-      }
-#pragma unroll
-      for (int n2 = 0; n2 < NU / 2; ++n2) {
-        uint32_t bk[4];  // key rows [token][d], transposed into B fragments of two 8-wide tiles
-        ldsm4t(bk, sm.k[u] + (kt * 16 + (lane & 15)) * P + wq * (DK / 4) + n2 * 16 + (lane >> 4) * 8);
-        mma16816(S[2 * n2], ah, bk[0], bk[1]);
-        mma16816(S[2 * n2 + 1], ah, bk[2], bk[3]);
-        mma16816(S[2 * n2], al, bk[0], bk[1]);
-        mma16816(S[2 * n2 + 1], al, bk[2], bk[3]);
+        uint32_t k0, k1;
+        ldsm2t(k0, k1, kr);
+        mma16816(S[0], ah, k0, k1);
+        mma16816(S[0], al, k0, k1);
       }
     }
     publish(u ^ 1);
-    // outputs: transpose through shared memory (this warp's tokens and columns only), then 16-byte rows
+    if constexpr (KIND == RK_DELTA) {
+      float o2[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-    for (int nt = 0; nt < 2; ++nt)
+      for (int kt = 0; kt < 4; ++kt) {
+        if (kt > wt) break;
+        uint32_t ah[4], al[4];
+        ldsm4(ah, sm.r[Sm::NR > 2 ? 2 : 0][0] + a_row * PR + kt * 16 + a_col);
+        ldsm4(al, sm.r[Sm::NR > 2 ? 2 : 0][1] + a_row * PR + kt * 16 + a_col);
+        mma16816(oq, ah, fr[kt].x, fr[kt].y);
+        mma16816(o2, ah, fr[kt].z, fr[kt].w);
+        mma16816(o2, al, fr[kt].x, fr[kt].y);
+      }
 #pragma unroll
-      for (int e = 0; e < 4; ++e)
-        sm.o[(tok0 + 8 * nt + 2 * (lane & 3) + (e & 1)) * PV + col_lo + (e >> 1) * 8] = __float2bfloat16(oq[nt][e]);
+      for (int e = 0; e < 4; ++e) oq[e] += o2[e];
+    }
+    // outputs: transpose through shared memory (this warp's tokens only), then 16-byte rows
+#pragma unroll
+    for (int e = 0; e < 4; ++e) sm.o[(tok0 + pair + (e & 1)) * PV + col + (e >> 1) * 8] = __float2bfloat16(oq[e]);
     __syncwarp();
-    {
-      const int i = tok0 + (lane >> 1), cc = 16 * mt + (lane & 1) * 8, t = t0 + i;
+    if (lane < 16) {
+      const int i = tok0 + (lane >> 1), cc = (lane & 1) * 8, t = t0 + i;
       if (t < p.T) {
         const __nv_bfloat16* src = sm.o + i * PV + cc;
         __nv_bfloat16* dst = O + (long long)t * p.ldo + cc;
@@ -555,24 +566,14 @@ __global__ void __launch_bounds__(128 * MT) chunk_walk_kernel(const ScanParams s
           for (int e = 0; e < 8 && cc + e < ncol; ++e) dst[e] = src[e];
       }
     }
-    if (more && warp == 0) chunk_scalars(p, ra0, ra1, rb0, rb1, ea, bias, t0 + CL, sm.b[u ^ 1], sm.gate[u ^ 1]);
   }
 #pragma unroll
   for (int n = 0; n < NU; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = d_lo + 8 * n + (e & 1), cc = col_lo + (e >> 1) * 8;
+      const int d = d_lo + 8 * n + (e & 1), cc = col + (e >> 1) * 8;
       if (d < p.Dk && cc < ncol) st[(long long)d * p.Dv + c0 + cc] = S[n][e];
     }
-}
-
-template <int KIND, int DK, int MT>
-void run_walk(const ScanParams& sp, cudaStream_t s) {
-  const RecurrentArgs& a = sp.a;
-  auto kern = chunk_walk_kernel<KIND, DK, MT>;
-  constexpr int smem = (int)sizeof(WalkSmem<KIND, DK, MT>);
-  cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  kern<<<a.B * a.H * ((a.Dv + 16 * MT - 1) / (16 * MT)), 128 * MT, smem, s>>>(sp);
 }
 
 template <int KIND, int DK>
@@ -583,9 +584,15 @@ void run_scan(const ScanParams& sp, cudaStream_t s) {
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   kern<<<a.B * (KIND == RK_DELTA ? a.H : a.KG) * sp.nchunks, 128, smem, s>>>(sp);
   check_launch("chunk_scores");
-  // 32 columns per block halve the key / query traffic; 16 where the wider blocks would leave SMs without work
-  if (a.B * a.H * ((a.Dv + 31) / 32) >= 100) run_walk<KIND, DK, 2>(sp, s);
-  else run_walk<KIND, DK, 1>(sp, s);
+  if (KIND == RK_MAMBA2) {
+    const long long n = (long long)a.B * a.H * sp.nchunks;
+    chunk_factors_kernel<<<(unsigned)((n + 3) / 4), 128, 0, s>>>(sp);
+    check_launch("chunk_factors");
+  }
+  auto walk = chunk_walk_kernel<KIND, DK>;
+  constexpr int wsm = (int)sizeof(WalkSmem<KIND, DK>);
+  cudaFuncSetAttribute(walk, cudaFuncAttributeMaxDynamicSharedMemorySize, wsm);
+  walk<<<a.B * a.H * ((a.Dv + WCOLS - 1) / WCOLS), 32 * WW, wsm, s>>>(sp);
   check_launch("chunk_walk");
 }
 
@@ -595,7 +602,7 @@ bool chunk_scan_supported(const RecurrentArgs& a) { return !a.f32 && a.Dk <= 128
 
 long long chunk_scan_scratch(const RecurrentArgs& a) {
   const long long n = (a.T + CL - 1) / CL;
-  return a.kind == RK_DELTA ? a.B * a.H * n * (2 * 16384 + 2 * CL * 4) : a.B * a.KG * n * 16384;
+  return (long long)a.B * n * (a.H * FACTORS * CL * 4ll + (a.kind == RK_DELTA ? a.H * 2 * 16384ll : a.KG * 16384ll));
 }
 
 void launch_chunk_scan(const RecurrentArgs& a, void* scratch, cudaStream_t s) {
@@ -609,10 +616,11 @@ void launch_chunk_scan(const RecurrentArgs& a, void* scratch, cudaStream_t s) {
   sp.frag0 = (uint4*)scratch;
   if (a.kind == RK_DELTA) {
     sp.frag1 = sp.frag0 + (long long)a.B * a.H * sp.nchunks * 1024;
-    sp.unit = (float*)(sp.frag1 + (long long)a.B * a.H * sp.nchunks * 1024);
+    sp.fac = (float*)(sp.frag1 + (long long)a.B * a.H * sp.nchunks * 1024);
     if (a.Dk <= 64) run_scan<RK_DELTA, 64>(sp, s);
     else run_scan<RK_DELTA, 128>(sp, s);
   } else {
+    sp.fac = (float*)(sp.frag0 + (long long)a.B * a.KG * sp.nchunks * 1024);
     if (a.Dk <= 64) run_scan<RK_MAMBA2, 64>(sp, s);
     else run_scan<RK_MAMBA2, 128>(sp, s);
   }

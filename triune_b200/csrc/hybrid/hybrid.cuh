@@ -167,7 +167,7 @@ struct StepAttention {
   void *kc, *vc;
   bool cache_f32;
   int cap, pitch_k, pitch_v;
-  float* part;      // [B, H, splits, E + 2]
+  float* part;      // [B, H, splits, step_part_stride(E)]
   int* counters;    // [B * G * head chunks], zero between calls
   int splits;
   float* out;       // [B, ldo]
@@ -182,6 +182,7 @@ struct StepArgs {
   int B;
   Pos pos;
 };
+int step_part_stride(int E);
 int step_head_chunk(int heads_per_group);  // query heads one attention block serves
 void launch_mixer_step(const StepArgs& a, cudaStream_t s);
 

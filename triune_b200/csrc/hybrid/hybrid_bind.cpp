@@ -334,7 +334,7 @@ tb::StepAttention step_attention(const py::dict& d, const Tensor& proj, int64_t 
   const int rep = a.H / a.G, rm = tb::step_head_chunk(rep);
   a.splits = d["splits"].cast<int>();
   TORCH_CHECK(a.splits >= 1 && a.splits <= 64, "step: 1 to 64 splits");
-  a.part = const_cast<float*>(f32v(part, B * a.H * a.splits * (a.E + 2), "part"));
+  a.part = const_cast<float*>(f32v(part, B * a.H * a.splits * tb::step_part_stride(a.E), "part"));
   TORCH_CHECK(cnt.is_cuda() && cnt.scalar_type() == at::kInt && cnt.is_contiguous() && cnt.numel() >= B * a.G * ((rep + rm - 1) / rm), "step: counters");
   a.counters = cnt.data_ptr<int>();
   TORCH_CHECK(rows_of(out, B, (int64_t)a.H * a.E, "out"), "step: fp32 output expected");
@@ -374,4 +374,5 @@ void register_hybrid(pybind11::module& m) {
   m.def("hybrid_gemv", &gemv);
   m.def("hybrid_mixer_step", &mixer_step);
   m.def("hybrid_step_head_chunk", &tb::step_head_chunk);
+  m.def("hybrid_step_part_stride", &tb::step_part_stride);
 }

@@ -59,8 +59,7 @@ __device__ void gemv_segment(const GemvSegment& g, int b, float* dst, float* red
 }
 
 template <class T>
-__device__ __forceinline__ void load_vec(const T* p, float (&f)[16 / sizeof(T)]) {
-  const uint4 u = *reinterpret_cast<const uint4*>(p);
+__device__ __forceinline__ void unpack_vec(const uint4& u, float (&f)[16 / sizeof(T)]) {
   if constexpr (sizeof(T) == 4) {
     f[0] = __uint_as_float(u.x); f[1] = __uint_as_float(u.y); f[2] = __uint_as_float(u.z); f[3] = __uint_as_float(u.w);
   } else {
@@ -73,14 +72,67 @@ __device__ __forceinline__ void load_vec(const T* p, float (&f)[16 / sizeof(T)])
   }
 }
 
+template <class T>
+__device__ __forceinline__ void load_vec(const T* p, float (&f)[16 / sizeof(T)]) {
+  unpack_vec<T>(*reinterpret_cast<const uint4*>(p), f);
+}
+
+// Programmatic dependent launch: the step's kernels follow one another closely, so each lets its successor start at once
+// and itself waits for its predecessor's results before it touches anything but weights.
+__device__ __forceinline__ void launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+__device__ __forceinline__ void wait_for_previous() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+
+template <class Args, class... Rest>
+void launch_chained(void (*kern)(Args, Rest...), int blocks, int threads, size_t smem, cudaStream_t s, const Args& a, Rest... rest) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(blocks);
+  cfg.blockDim = dim3(threads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = s;
+  cudaLaunchAttribute at[1];
+  at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  at[0].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = at;
+  cfg.numAttrs = 1;
+  cudaLaunchKernelEx(&cfg, kern, a, rest...);
+}
+
 // A warp works on two rows at a time (for the gated epilogue: a gate row and its up row).
 template <class T, int NB>
 __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const GemvArgs p) {
   extern __shared__ __align__(16) float sx[];  // [NB][KP]
   __shared__ float red[33];
-  constexpr int VEC = 16 / sizeof(T), STEP = 32 * VEC;
+  constexpr int VEC = 16 / sizeof(T), STEP = 32 * VEC, PRE = 4;
   const int KP = (p.K + 3) & ~3;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool glu = p.epilogue == 2;
+  const int pairs = glu ? p.N : (p.N + 1) / 2;
+  const bool vec = p.K % VEC == 0 && p.ldw % VEC == 0 && (reinterpret_cast<uintptr_t>(p.W) & 15) == 0;
+  auto rows = [&](int pr, const T*& w0, const T*& w1) {
+    const int r0 = glu ? pr : 2 * pr, r1 = glu ? pr + p.N : 2 * pr + 1;
+    w0 = (const T*)p.W + (long long)r0 * p.ldw;
+    w1 = glu || r1 < p.N ? (const T*)p.W + (long long)r1 * p.ldw : w0;
+  };
+  // The first weights of a pair of rows are fetched ahead: before the previous kernel has finished (weights do not
+  // depend on it) and before the prologue, then behind the sums of the pair before.
+  uint4 pre0[PRE], pre1[PRE];
+  auto fetch = [&](int pr) {
+    if (!vec || pr >= pairs) return;
+    const T *w0, *w1;
+    rows(pr, w0, w1);
+#pragma unroll
+    for (int i = 0; i < PRE; ++i) {
+      const int k = lane * VEC + i * STEP;
+      if (k < p.K) {
+        pre0[i] = *reinterpret_cast<const uint4*>(w0 + k);
+        pre1[i] = *reinterpret_cast<const uint4*>(w1 + k);
+      }
+    }
+  };
+  int pr = blockIdx.x * GV_WARPS + warp;
+  fetch(pr);
+  launch_dependents();
+  wait_for_previous();
   for (int b = 0; b < p.B; ++b) {
     int off = 0;
     for (int i = 0; i < p.nseg; ++i) {
@@ -89,33 +141,42 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const GemvArgs p) {
     }
   }
   __syncthreads();
-  const bool glu = p.epilogue == 2;
-  const int pairs = glu ? p.N : (p.N + 1) / 2;
-  const bool vec = p.K % VEC == 0 && p.ldw % VEC == 0 && (reinterpret_cast<uintptr_t>(p.W) & 15) == 0;
-  for (int pr = blockIdx.x * GV_WARPS + warp; pr < pairs; pr += gridDim.x * GV_WARPS) {
-    const int r0 = glu ? pr : 2 * pr, r1 = glu ? pr + p.N : 2 * pr + 1;
-    const bool two = glu || r1 < p.N;
-    const T *w0 = (const T*)p.W + (long long)r0 * p.ldw, *w1 = (const T*)p.W + (long long)(two ? r1 : r0) * p.ldw;
+  while (pr < pairs) {
+    const T *w0, *w1;
+    rows(pr, w0, w1);
     float a0[NB], a1[NB];
 #pragma unroll
     for (int b = 0; b < NB; ++b) a0[b] = a1[b] = 0.f;
+    auto dot = [&](const float (&f0)[VEC], const float (&f1)[VEC], int k) {
+#pragma unroll
+      for (int b = 0; b < NB; ++b) {
+        if (b < p.B) {
+#pragma unroll
+          for (int i = 0; i < VEC; i += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(sx + b * KP + k + i);
+            a0[b] += f0[i] * x.x + f0[i + 1] * x.y + f0[i + 2] * x.z + f0[i + 3] * x.w;
+            a1[b] += f1[i] * x.x + f1[i + 1] * x.y + f1[i + 2] * x.z + f1[i + 3] * x.w;
+          }
+        }
+      }
+    };
     if (vec) {
+#pragma unroll
+      for (int i = 0; i < PRE; ++i) {
+        const int k = lane * VEC + i * STEP;
+        if (k < p.K) {
+          float f0[VEC], f1[VEC];
+          unpack_vec<T>(pre0[i], f0);
+          unpack_vec<T>(pre1[i], f1);
+          dot(f0, f1, k);
+        }
+      }
 #pragma unroll 4
-      for (int k = lane * VEC; k < p.K; k += STEP) {
+      for (int k = lane * VEC + PRE * STEP; k < p.K; k += STEP) {
         float f0[VEC], f1[VEC];
         load_vec(w0 + k, f0);
         load_vec(w1 + k, f1);
-#pragma unroll
-        for (int b = 0; b < NB; ++b) {
-          if (b < p.B) {
-#pragma unroll
-            for (int i = 0; i < VEC; i += 4) {
-              const float4 x = *reinterpret_cast<const float4*>(sx + b * KP + k + i);
-              a0[b] += f0[i] * x.x + f0[i + 1] * x.y + f0[i + 2] * x.z + f0[i + 3] * x.w;
-              a1[b] += f1[i] * x.x + f1[i + 1] * x.y + f1[i + 2] * x.z + f1[i + 3] * x.w;
-            }
-          }
-        }
+        dot(f0, f1, k);
       }
     } else {
       for (int k = lane; k < p.K; k += 32) {
@@ -128,6 +189,10 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const GemvArgs p) {
           }
       }
     }
+    const int next = pr + gridDim.x * GV_WARPS;
+    fetch(next);
+    const int r0 = glu ? pr : 2 * pr, r1 = 2 * pr + 1;
+    const bool two = r1 < p.N;
 #pragma unroll
     for (int b = 0; b < NB; ++b) {
       if (b >= p.B) break;
@@ -144,6 +209,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const GemvArgs p) {
         }
       }
     }
+    pr = next;
   }
 }
 
@@ -254,6 +320,9 @@ __device__ void head_row(const float* src, const float* w, float eps, int D, int
   for (int d = D + lane; d < padded; d += 32) dst[d] = 0.f;
 }
 
+// Floats of one partial result: maximum, sum, two of padding, the values padded to whole quads.
+__host__ __device__ constexpr int part_stride(int E) { return ((E + 3) & ~3) + 4; }
+
 // Keys of split `s` of `splits` over n keys: whole multiples of 32, at least 64 keys per split.
 __device__ __forceinline__ void split_range(int n, int splits, int s, int* k0, int* k1) {
   int per = (n + splits - 1) / splits;
@@ -270,14 +339,16 @@ __device__ void attention_step(const StepAttention& p, int block, long long pos,
   const int split = block % p.splits, bgc = block / p.splits, hc = bgc % chunks, bg = bgc / chunks, g = bg % p.G, b = bg / p.G;
   const int h0 = g * rep + hc * RM, nh = min(RM, rep - hc * RM);
   const int DP = (p.D + 7) & ~7, half = p.rot_dims / 2;
-  float *sq = sm, *sp = sq + RM * DP, *cs = sp + RM * AT_KEYS, *sn = cs + half, *sk = sn + half, *ml = sk + DP, *sacc = ml + 2 * RM;
+  const int ES = part_stride(p.E);
+  float *sq = sm, *sp = sq + RM * DP, *sred = sp + RM * AT_KEYS, *cs = sred + ST_THREADS * 8, *sn = cs + half, *sk = sn + half,
+        *ml = sk + DP, *sacc = ml + 2 * RM;
   int* flag = reinterpret_cast<int*>(sacc);
   if (pos < 0 || pos >= p.cap) return;  // the host reserves the cache before every step
   int k0, k1;
   split_range((int)pos + 1, p.splits, split, &k0, &k1);
   T *K = (T*)p.kc + (long long)bg * p.cap * p.pitch_k, *V = (T*)p.vc + (long long)bg * p.cap * p.pitch_v;
-  float* part = p.part + (((long long)b * p.H + h0) * p.splits + split) * (p.E + 2);
-  const long long hstride = (long long)p.splits * (p.E + 2);
+  float* part = p.part + (((long long)b * p.H + h0) * p.splits + split) * ES;
+  const long long hstride = (long long)p.splits * ES;
   const float* pr = p.proj + (long long)b * p.ld;
 
   if (k0 < k1) {
@@ -297,42 +368,49 @@ __device__ void attention_step(const StepAttention& p, int block, long long pos,
       ml[2 * tid + 1] = 0.f;
     }
     __syncthreads();
-    // value accumulation: a thread owns two neighbouring value dimensions of a subset of the keys
-    const int PC = (p.E + 1) / 2, KS = max(1, ST_THREADS / PC);
-    float acc[RM][2];
-    const int pc = tid % PC, ks = tid / PC;       // PC <= 128: value dimensions up to 256
+    // value accumulation: a thread owns eight neighbouring value dimensions of a subset of the keys
+    const int PC = (p.E + 7) / 8, KS = ST_THREADS / PC;  // value dimensions up to 256: PC <= 32
+    float acc[RM][8];
+    const int pc = tid % PC, ks = tid / PC;
     const bool vlive = ks < KS;
 #pragma unroll
-    for (int r = 0; r < RM; ++r) acc[r][0] = acc[r][1] = 0.f;
+    for (int r = 0; r < RM; ++r)
+#pragma unroll
+      for (int i = 0; i < 8; ++i) acc[r][i] = 0.f;
     for (int kb = k0; kb < k1; kb += AT_KEYS) {
       const int n = min(AT_KEYS, k1 - kb);
-      // scores: four lanes per key
-      for (int j = warp * 8 + (lane >> 2); j < ((n + 31) & ~31); j += 32) {
-        float s[RM];
+      // scores: four lanes per key, two keys at a time
+      for (int j = warp * 8 + (lane >> 2); j < ((n + 31) & ~31); j += 64) {
+        float s[2][RM];
 #pragma unroll
-        for (int r = 0; r < RM; ++r) s[r] = 0.f;
-        if (j < n) {
-          const T* kr = K + (long long)(kb + j) * p.pitch_k;
-          for (int d = (lane & 3) * VEC; d < DP; d += 4 * VEC) {
-            float f[VEC];
-            load_vec(kr + d, f);  // rows are padded with zeros to a multiple of 16 bytes
+        for (int r = 0; r < RM; ++r) s[0][r] = s[1][r] = 0.f;
+        // keys past the tile repeat its last one; their scores are not kept
+        const T *ka = K + (long long)(kb + min(j, n - 1)) * p.pitch_k, *kc = K + (long long)(kb + min(j + 32, n - 1)) * p.pitch_k;
+#pragma unroll 4
+        for (int d = (lane & 3) * VEC; d < DP; d += 4 * VEC) {
+          float fa[VEC], fc[VEC];
+          load_vec(ka + d, fa);  // rows are padded with zeros to a multiple of 16 bytes
+          load_vec(kc + d, fc);
 #pragma unroll
-            for (int r = 0; r < RM; ++r)
-              if (r < nh) {
+          for (int r = 0; r < RM; ++r)
+            if (r < nh) {
 #pragma unroll
-                for (int i = 0; i < VEC; i += 4) {
-                  const float4 x = *reinterpret_cast<const float4*>(sq + r * DP + d + i);
-                  s[r] += f[i] * x.x + f[i + 1] * x.y + f[i + 2] * x.z + f[i + 3] * x.w;
-                }
+              for (int i = 0; i < VEC; i += 4) {
+                const float4 x = *reinterpret_cast<const float4*>(sq + r * DP + d + i);
+                s[0][r] += fa[i] * x.x + fa[i + 1] * x.y + fa[i + 2] * x.z + fa[i + 3] * x.w;
+                s[1][r] += fc[i] * x.x + fc[i + 1] * x.y + fc[i + 2] * x.z + fc[i + 3] * x.w;
               }
-          }
+            }
         }
 #pragma unroll
-        for (int r = 0; r < RM; ++r) {
-          s[r] += __shfl_xor_sync(0xffffffffu, s[r], 1);
-          s[r] += __shfl_xor_sync(0xffffffffu, s[r], 2);
-          if ((lane & 3) == 0 && j < n && r < nh) sp[r * AT_KEYS + j] = s[r] * p.scale;
-        }
+        for (int g2 = 0; g2 < 2; ++g2)
+#pragma unroll
+          for (int r = 0; r < RM; ++r) {
+            float t = s[g2][r];
+            t += __shfl_xor_sync(0xffffffffu, t, 1);
+            t += __shfl_xor_sync(0xffffffffu, t, 2);
+            if ((lane & 3) == 0 && j + 32 * g2 < n && r < nh) sp[r * AT_KEYS + j + 32 * g2] = t * p.scale;
+          }
       }
       __syncthreads();
       // softmax of the tile: a warp per head; the running maximum's correction goes through sk
@@ -359,49 +437,44 @@ __device__ void attention_step(const StepAttention& p, int block, long long pos,
 #pragma unroll
         for (int r = 0; r < RM; ++r)
           if (r < nh) {
-            acc[r][0] *= sacc[1 + r];
-            acc[r][1] *= sacc[1 + r];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) acc[r][i] *= sacc[1 + r];
           }
-        const int e0 = 2 * pc;
 #pragma unroll 4
         for (int j = ks; j < n; j += KS) {
-          float v0, v1;
-          const T* vr = V + (long long)(kb + j) * p.pitch_v + e0;  // pitch_v is even: the pair stays inside the row
-          if constexpr (sizeof(T) == 4) {
-            const float2 t = *reinterpret_cast<const float2*>(vr);
-            v0 = t.x; v1 = t.y;
-          } else {
-            const uint32_t t = *reinterpret_cast<const uint32_t*>(vr);
-            v0 = __uint_as_float(t << 16); v1 = __uint_as_float(t & 0xffff0000u);
-          }
+          float v[8];
+          ld8v(V + (long long)(kb + j) * p.pitch_v + 8 * pc, v);  // value rows are padded to a multiple of eight
 #pragma unroll
           for (int r = 0; r < RM; ++r)
             if (r < nh) {
               const float w = sp[r * AT_KEYS + j];
-              acc[r][0] += w * v0;
-              acc[r][1] += w * v1;
+#pragma unroll
+              for (int i = 0; i < 8; ++i) acc[r][i] += w * v[i];
             }
         }
       }
       __syncthreads();
     }
-    // sum over the key subsets, one head at a time, through the score buffer
-    for (int r = 0; r < nh; ++r) {
-      if (vlive) {
-        sp[tid * 2] = acc[r][0];
-        sp[tid * 2 + 1] = acc[r][1];
+    // sum over the key subsets, one head at a time
+#pragma unroll
+    for (int r = 0; r < RM; ++r) {
+      if (r < nh) {
+        if (vlive) {
+#pragma unroll
+          for (int i = 0; i < 8; ++i) sred[tid * 8 + i] = acc[r][i];
+        }
+        __syncthreads();
+        for (int e = tid; e < p.E; e += ST_THREADS) {
+          float t = 0.f;
+          for (int q = 0; q < KS; ++q) t += sred[(q * PC + (e >> 3)) * 8 + (e & 7)];
+          part[r * hstride + 4 + e] = t;
+        }
+        if (tid == 0) {
+          part[r * hstride] = ml[2 * r];
+          part[r * hstride + 1] = ml[2 * r + 1];
+        }
+        __syncthreads();
       }
-      __syncthreads();
-      for (int e = tid; e < p.E; e += ST_THREADS) {
-        float t = 0.f;
-        for (int q = 0; q < KS; ++q) t += sp[(q * PC + (e >> 1)) * 2 + (e & 1)];
-        part[r * hstride + 2 + e] = t;
-      }
-      if (tid == 0) {
-        part[r * hstride] = ml[2 * r];
-        part[r * hstride + 1] = ml[2 * r + 1];
-      }
-      __syncthreads();
     }
   } else {
     if (tid < nh) {
@@ -416,19 +489,19 @@ __device__ void attention_step(const StepAttention& p, int block, long long pos,
   if (*flag == 0) return;
   __threadfence();
   if (tid == 0) p.counters[bgc] = 0;
-  const float* base = p.part + ((long long)b * p.H + h0) * p.splits * (p.E + 2);
+  const float* base = p.part + ((long long)b * p.H + h0) * p.splits * ES;
   // weights of the splits of every head (a warp per head), then the weighted sum of their partial values
   for (int r = warp; r < nh; r += 4) {
     const float* ph = base + r * hstride;
     const float sink = p.sink != nullptr ? p.sink[h0 + r] : -INFINITY;
     float m = sink;
-    for (int s = lane; s < p.splits; s += 32) m = fmaxf(m, __ldcg(ph + s * (p.E + 2)));
+    for (int s = lane; s < p.splits; s += 32) m = fmaxf(m, __ldcg(ph + s * ES));
     m = warp_max(m);
     float l = 0.f;
     for (int s = lane; s < p.splits; s += 32) {
-      const float c = expf(__ldcg(ph + s * (p.E + 2)) - m);
+      const float c = expf(__ldcg(ph + s * ES) - m);
       sp[r * AT_KEYS + s] = c;  // at most 64 splits
-      l += __ldcg(ph + s * (p.E + 2) + 1) * c;
+      l += __ldcg(ph + s * ES + 1) * c;
     }
     l = warp_sum(l) + (p.sink != nullptr ? expf(sink - m) : 0.f);
     __syncwarp();
@@ -441,19 +514,30 @@ __device__ void attention_step(const StepAttention& p, int block, long long pos,
     split_range((int)pos + 1, p.splits, 0, &a, &z);
     active = min(active, ((int)pos + z) / max(z, 1));
   }
-  for (int i = tid; i < nh * p.E; i += ST_THREADS) {
-    const int r = i / p.E, e = i % p.E;
-    const float* ph = base + r * hstride + 2 + e;
-    float t = 0.f;
-#pragma unroll 8
-    for (int s = 0; s < active; ++s) t += sp[r * AT_KEYS + s] * __ldcg(ph + s * (p.E + 2));
-    p.out[(long long)b * p.ldo + (h0 + r) * p.E + e] = t;
+  const int quads = (p.E + 3) / 4;  // partial rows are padded to whole quads
+  for (int i = tid; i < nh * quads; i += ST_THREADS) {
+    const int r = i / quads, e = (i % quads) * 4;
+    const float* ph = base + r * hstride + 4 + e;
+    float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 16
+    for (int s = 0; s < active; ++s) {
+      const float c = sp[r * AT_KEYS + s];
+      const float4 v = __ldcg(reinterpret_cast<const float4*>(ph + s * ES));
+      t.x += c * v.x; t.y += c * v.y; t.z += c * v.z; t.w += c * v.w;
+    }
+    float* o = p.out + (long long)b * p.ldo + (h0 + r) * p.E + e;
+    o[0] = t.x;
+    if (e + 1 < p.E) o[1] = t.y;
+    if (e + 2 < p.E) o[2] = t.z;
+    if (e + 3 < p.E) o[3] = t.w;
   }
 }
 
 template <class T, int RM>
 __global__ void __launch_bounds__(ST_THREADS) mixer_step_kernel(const StepArgs p, int att_blocks) {
   extern __shared__ __align__(16) float sm[];
+  launch_dependents();
+  wait_for_previous();
   const long long pos = pos_of(p.pos);
   if ((int)blockIdx.x < att_blocks) attention_step<T, RM>(p.att, blockIdx.x, pos, sm);
   else recurrent_step(p.rec, blockIdx.x - att_blocks, pos, sm);
@@ -461,6 +545,7 @@ __global__ void __launch_bounds__(ST_THREADS) mixer_step_kernel(const StepArgs p
 
 }  // namespace
 
+int step_part_stride(int E) { return part_stride(E); }
 int step_head_chunk(int rep) { return rep <= 1 ? 1 : rep <= 2 ? 2 : rep <= 4 ? 4 : 8; }
 
 void launch_mixer_step(const StepArgs& a, cudaStream_t s) {
@@ -473,7 +558,7 @@ void launch_mixer_step(const StepArgs& a, cudaStream_t s) {
     rm = step_head_chunk(p.H / p.G);
     att = a.B * p.G * ((p.H / p.G + rm - 1) / rm) * p.splits;
     const int dp = (p.D + 7) & ~7;
-    sm = (size_t)(rm * dp + rm * AT_KEYS + p.rot_dims + 4 + dp + 2 * rm + rm + 4) * 4;
+    sm = (size_t)(rm * dp + rm * AT_KEYS + ST_THREADS * 8 + p.rot_dims + 4 + dp + 2 * rm + rm + 4) * 4;
   }
   if (a.has_rec) {
     const StepRecurrent& p = a.rec;
@@ -484,7 +569,7 @@ void launch_mixer_step(const StepArgs& a, cudaStream_t s) {
   }
   if (att + rec == 0) return;
   const bool f32 = a.has_att && a.att.cache_f32;
-  auto go = [&](auto* kern) { kern<<<att + rec, ST_THREADS, sm, s>>>(a, att); };
+  auto go = [&](auto* kern) { launch_chained(kern, att + rec, ST_THREADS, sm, s, a, att); };
   if (f32) {
     if (rm == 1) go(mixer_step_kernel<float, 1>);
     else if (rm == 2) go(mixer_step_kernel<float, 2>);
@@ -510,7 +595,7 @@ void launch_gemv(const GemvArgs& a, cudaStream_t s) {
   if (blocks > 148 * per_sm) blocks = 148 * per_sm;
   auto go = [&](auto* kern) {
     if (sm > 47 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
-    kern<<<blocks, GV_WARPS * 32, sm, s>>>(a);
+    launch_chained(kern, blocks, GV_WARPS * 32, sm, s, a);
   };
   if (a.f32) {
     if (a.B == 1) go(gemv_kernel<float, 1>);

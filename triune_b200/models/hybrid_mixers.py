@@ -97,7 +97,7 @@ class AttentionCore(Core):
         splits = max(1, min(64, 2 * 148 // groups))
         s = st.scratch
         if pre + "part" not in s or s[pre + "part"].shape[:2] != (B, self.heads):
-            s[pre + "part"] = torch.empty(B, self.heads, splits, self.vdim + 2, device=proj.device)
+            s[pre + "part"] = torch.empty(B, self.heads, splits, hops.step_part_stride(self.vdim), device=proj.device)
             s[pre + "counters"] = torch.zeros(groups, dtype=torch.int32, device=proj.device)
         out = torch.empty(B, self.out_width, device=proj.device)
         at = self.inputs.at

@@ -190,5 +190,9 @@ def mixer_step(proj: torch.Tensor, recurrent: Optional[Dict[str, Any]], attentio
     _tick()
 
 
+def step_part_stride(vdim: int) -> int:
+    return _ext.serving().hybrid_step_part_stride(vdim)
+
+
 def step_head_chunk(heads_per_group: int) -> int:
     return _ext.serving().hybrid_step_head_chunk(heads_per_group)
