@@ -13,9 +13,9 @@
 //
 // Two kernels. (1) Scores, parallel over chunks: q k^T per key group (mamba2), or per head the decayed q k^T and the
 // inverse of I + L (delta). They are written in the register order of the B operand they become, one 16-byte vector per
-// lane. (2) The walk: a block owns 16 value columns of a head and walks the chunks; its eight warps split the tokens for
+// lane. (2) The walk. Delta rule: a block owns 16 value columns of a head and walks the chunks; its eight warps split the tokens for
 // the outputs and the key dimensions for the state, which stays in accumulator registers as S^T [columns, Dk] and is
-// handed between warps as bf16 pairs in shared memory. A walk is one long dependent chain, so what can be formed ahead of
+// handed between warps as bf16 pairs in shared memory; Mamba-2: see below. A walk is one long dependent chain, so what can be formed ahead of
 // it is: the per-token factors (decays, gates, unit norms) are written by the scores kernel or a small kernel before it. The products here are small, chained and
 // re-split between steps, so they run on mma.sync register fragments: the accumulator layout of one product is the
 // operand layout of the next, with no trip through TMEM or shared memory in between.
@@ -301,15 +301,15 @@ __global__ void __launch_bounds__(128) chunk_factors_kernel(const ScanParams sp)
   }
 }
 
-// ------------------------------------------------------------------------------------------------ walk
+// ------------------------------------------------------------------------------------------------ delta rule: walk
 constexpr int WW = 8, WCOLS = 16;  // warps and value columns of a block; a warp owns 8 tokens and DK / 8 key dimensions
 
-template <int KIND, int DK>
+template <int DK>
 struct WalkSmem {
-  static constexpr int P = DK + 8, PV = WCOLS + 8, PR = CL + 8, NR = KIND == RK_DELTA ? 3 : 1;
+  static constexpr int P = DK + 8, PV = WCOLS + 8, PR = CL + 8;
   __nv_bfloat16 q[2][CL * P], k[2][CL * P], v[2][CL * PV];
   __nv_bfloat16 s[2][2][WCOLS * P];     // state buffer, hi / lo, [columns][Dk]
-  __nv_bfloat16 r[NR][2][WCOLS * PR];   // 0: weighted values or U of the state update; delta 1: R, 2: U; hi / lo, [columns][tokens]
+  __nv_bfloat16 r[3][2][WCOLS * PR];   // 0: weighted U of the state update, 1: R, 2: U; hi / lo, [columns][tokens]
   __nv_bfloat16 o[CL * PV];
   float f[2][FACTORS * CL];
 };
@@ -318,9 +318,9 @@ __device__ __forceinline__ void ldsm2t(uint32_t& r0, uint32_t& r1, const void* p
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(smem_u32(p)) : "memory");
 }
 
-template <int KIND, int DK>
-__global__ void __launch_bounds__(32 * WW) chunk_walk_kernel(const ScanParams sp) {
-  using Sm = WalkSmem<KIND, DK>;
+template <int DK>
+__global__ void __launch_bounds__(32 * WW) delta_walk_kernel(const ScanParams sp) {
+  using Sm = WalkSmem<DK>;
   constexpr int P = Sm::P, PV = Sm::PV, PR = Sm::PR, NT = 32 * WW, KT = DK / 16, DW = DK / WW, NU = DW / 8;
   extern __shared__ __align__(16) uint8_t raw[];
   Sm& sm = *reinterpret_cast<Sm*>(raw);
@@ -333,9 +333,7 @@ __global__ void __launch_bounds__(32 * WW) chunk_walk_kernel(const ScanParams sp
                       *K = (const __nv_bfloat16*)p.k + (long long)b * p.rows * p.ldk + kh * p.Dk,
                       *V = (const __nv_bfloat16*)p.v + (long long)b * p.rows * p.ldv + h * p.Dv + c0;
   __nv_bfloat16* O = (__nv_bfloat16*)p.out + (long long)b * p.rows * p.ldo + h * p.Dv + c0;
-  const float Dh = KIND == RK_MAMBA2 ? p.D[h] : 0.f;
-  const long long fh = KIND == RK_DELTA ? bh : (long long)b * p.KG + kh;
-  const uint4 *f0 = sp.frag0 + fh * sp.nchunks * 1024, *f1 = KIND == RK_DELTA ? sp.frag1 + fh * sp.nchunks * 1024 : nullptr;
+  const uint4 *f0 = sp.frag0 + (long long)bh * sp.nchunks * 1024, *f1 = sp.frag1 + (long long)bh * sp.nchunks * 1024;
   const float* fac = sp.fac + (long long)bh * sp.nchunks * FACTORS * CL;
 
   auto stage = [&](int c) {
@@ -395,22 +393,17 @@ __global__ void __launch_bounds__(32 * WW) chunk_walk_kernel(const ScanParams sp
     if (c + 1 < sp.nchunks) stage(c + 1);
     const float* F = sm.f[u];
     // score fragments of this warp's row tile: issued early, used after the state products
-    uint4 fr[4], ft[KIND == RK_DELTA ? 4 : 1];
+    uint4 fr[4], ft[4];
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt)
       if (kt <= wt) {
         fr[kt] = f0[(long long)c * 1024 + (warp * 4 + kt) * 32 + lane];
-        if constexpr (KIND == RK_DELTA) ft[kt] = f1[(long long)c * 1024 + (warp * 4 + kt) * 32 + lane];
+        ft[kt] = f1[(long long)c * 1024 + (warp * 4 + kt) * 32 + lane];
       }
     float x[4];  // values of this lane's tokens: [column half][token of the pair]
 #pragma unroll
     for (int e = 0; e < 4; ++e) x[e] = __bfloat162float(sm.v[u][(tok0 + pair + (e & 1)) * PV + col + (e >> 1) * 8]);
-    if constexpr (KIND == RK_MAMBA2) {
-      const float w0 = F[2 * CL + tok0 + pair], w1 = F[2 * CL + tok0 + pair + 1];
-      const float xw[4] = {x[0] * w0, x[1] * w1, x[2] * w0, x[3] * w1};
-      put(0, xw);
-    }
-    // state products of this warp's tokens: S^T q and, for the delta rule, S^T k (hi and lo in separate accumulators)
+    // state products of this warp's tokens: S^T q and S^T k (hi and lo in separate accumulators)
     float oq[4] = {0.f, 0.f, 0.f, 0.f}, oq2[4] = {0.f, 0.f, 0.f, 0.f}, ok[4] = {0.f, 0.f, 0.f, 0.f}, ok2[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
     for (int ks = 0; ks < KT; ks += 2) {
@@ -421,12 +414,12 @@ __global__ void __launch_bounds__(32 * WW) chunk_walk_kernel(const ScanParams sp
         ldsm4(al[i], sm.s[u][1] + a_row * P + (ks + i) * 16 + a_col);
       }
       ldsm4(bq, sm.q[u] + b_at + ks * 16);
-      if constexpr (KIND == RK_DELTA) ldsm4(bk, sm.k[u] + b_at + ks * 16);
+      ldsm4(bk, sm.k[u] + b_at + ks * 16);
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         mma16816(oq, ah[i], bq[2 * i], bq[2 * i + 1]);
         mma16816(oq2, al[i], bq[2 * i], bq[2 * i + 1]);
-        if constexpr (KIND == RK_DELTA) {
+        {
           mma16816(ok, ah[i], bk[2 * i], bk[2 * i + 1]);
           mma16816(ok2, al[i], bk[2 * i], bk[2 * i + 1]);
         }
@@ -437,51 +430,7 @@ __global__ void __launch_bounds__(32 * WW) chunk_walk_kernel(const ScanParams sp
       oq[e] += oq2[e];
       ok[e] += ok2[e];
     }
-    if constexpr (KIND == RK_MAMBA2) {
-      // tokens before this 16-token tile: e^{b_i - b_j} = e^{b_i - b_ref} e^{b_ref - b_j} with the tile's first token as
-      // reference, both factors at most 1; the first is applied once to the whole sum
-      const float br = F[16 * wt], er = exp_neg(br);
-      float od[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-      for (int e = 0; e < 4; ++e) oq[e] *= er;
-      const int i = tok0 + col;  // as a B operand, the row of the scores is lane / 4
-      const float bi = F[i];
-#pragma unroll
-      for (int kt = 0; kt < 4; ++kt) {
-        if (kt > wt) break;
-        uint32_t ax[4];
-        ldsm4t(ax, sm.v[u] + (kt * 16 + (lane & 7) + ((lane >> 4) << 3)) * PV + ((lane >> 3) & 1) * 8);
-        const int j = kt * 16 + pair;
-        const bool diag = kt == wt;
-        const float ref = diag ? bi : br;
-        const float2 b0 = *reinterpret_cast<const float2*>(F + j), b8 = *reinterpret_cast<const float2*>(F + j + 8);
-        const float2 g0 = *reinterpret_cast<const float2*>(F + CL + j), g8 = *reinterpret_cast<const float2*>(F + CL + j + 8);
-        float m0 = __uint_as_float(fr[kt].x) * g0.x * exp_neg(fminf(ref - b0.x, 0.f));
-        float m1 = __uint_as_float(fr[kt].y) * g0.y * exp_neg(fminf(ref - b0.y, 0.f));
-        float m8 = __uint_as_float(fr[kt].z) * g8.x * exp_neg(fminf(ref - b8.x, 0.f));
-        float m9 = __uint_as_float(fr[kt].w) * g8.y * exp_neg(fminf(ref - b8.y, 0.f));
-        if (diag) {
-          m0 = j <= i ? m0 : 0.f;
-          m1 = j + 1 <= i ? m1 : 0.f;
-          m8 = j + 8 <= i ? m8 : 0.f;
-          m9 = j + 9 <= i ? m9 : 0.f;
-        }
-        uint32_t h0, l0, h1, l1;
-        split2(m0, m1, h0, l0);
-        split2(m8, m9, h1, l1);
-        if (diag) {
-          mma16816(od, ax, h0, h1);
-          mma16816(od, ax, l0, l1);
-        } else {
-          mma16816(oq, ax, h0, h1);
-          mma16816(oq, ax, l0, l1);
-        }
-      }
-      const float e0 = exp_neg(F[tok0 + pair] - br), e1 = exp_neg(F[tok0 + pair + 1] - br);
-#pragma unroll
-      for (int e = 0; e < 4; ++e) oq[e] = oq[e] * ((e & 1) ? e1 : e0) + od[e] + Dh * x[e];
-      __syncthreads();  // weighted values of every warp
-    } else {
+    {
       float r[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
@@ -496,22 +445,22 @@ __global__ void __launch_bounds__(32 * WW) chunk_walk_kernel(const ScanParams sp
       for (int kt = 0; kt < 4; ++kt) {
         if (kt > wt) break;
         uint32_t ah[4], al[4];
-        ldsm4(ah, sm.r[Sm::NR > 1 ? 1 : 0][0] + a_row * PR + kt * 16 + a_col);
-        ldsm4(al, sm.r[Sm::NR > 1 ? 1 : 0][1] + a_row * PR + kt * 16 + a_col);
+        ldsm4(ah, sm.r[1][0] + a_row * PR + kt * 16 + a_col);
+        ldsm4(al, sm.r[1][1] + a_row * PR + kt * 16 + a_col);
         mma16816(uu, ah, ft[kt].x, ft[kt].y);
         mma16816(u2, ah, ft[kt].z, ft[kt].w);
         mma16816(u2, al, ft[kt].x, ft[kt].y);
       }
 #pragma unroll
       for (int e = 0; e < 4; ++e) uu[e] += u2[e];
-      put(Sm::NR > 2 ? 2 : 0, uu);
+      put(2, uu);
       const float w0 = F[2 * CL + tok0 + pair], w1 = F[2 * CL + tok0 + pair + 1];
       const float uw[4] = {uu[0] * w0, uu[1] * w1, uu[2] * w0, uu[3] * w1};
       put(0, uw);
       __syncthreads();
     }
-    // decay the state and add this chunk's keys: A = weighted values or U (columns x tokens), B = key rows
-    const float dl = F[(KIND == RK_DELTA ? 4 : 3) * CL];
+    // decay the state and add this chunk's keys: A = weighted U (columns x tokens), B = key rows
+    const float dl = F[4 * CL];
 #pragma unroll
     for (int n = 0; n < NU; ++n)
 #pragma unroll
@@ -537,14 +486,14 @@ __global__ void __launch_bounds__(32 * WW) chunk_walk_kernel(const ScanParams sp
       }
     }
     publish(u ^ 1);
-    if constexpr (KIND == RK_DELTA) {
+    {
       float o2[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int kt = 0; kt < 4; ++kt) {
         if (kt > wt) break;
         uint32_t ah[4], al[4];
-        ldsm4(ah, sm.r[Sm::NR > 2 ? 2 : 0][0] + a_row * PR + kt * 16 + a_col);
-        ldsm4(al, sm.r[Sm::NR > 2 ? 2 : 0][1] + a_row * PR + kt * 16 + a_col);
+        ldsm4(ah, sm.r[2][0] + a_row * PR + kt * 16 + a_col);
+        ldsm4(al, sm.r[2][1] + a_row * PR + kt * 16 + a_col);
         mma16816(oq, ah, fr[kt].x, fr[kt].y);
         mma16816(o2, ah, fr[kt].z, fr[kt].w);
         mma16816(o2, al, fr[kt].x, fr[kt].y);
@@ -576,24 +525,332 @@ __global__ void __launch_bounds__(32 * WW) chunk_walk_kernel(const ScanParams sp
     }
 }
 
+// ------------------------------------------------------------------------------------------------ Mamba-2
+// The state's transition is a scalar per head, so a sequence is cut into segments that are walked independently: one pass
+// leaves every segment's own contribution to its end state, a small scan turns these into the state before every segment,
+// and the second pass walks the segments again for the outputs. A block owns 64 value columns of a head (two halves of
+// four warps); as output tiles [tokens, columns] the decayed scores are the A operand, formed in registers once for 32
+// columns, and values, weighted values and the state [Dk, columns] are B operands.
+constexpr int SW = 8, SC = 64;  // warps, value columns
+
+template <int DK, bool OUT>
+struct SsdSmem {
+  static constexpr int P = DK + 8, PC = SC + 8;
+  __nv_bfloat16 k[CL * P], x[CL * PC], w[2][CL * PC];
+  __nv_bfloat16 q[OUT ? CL * P : 8], s[2][OUT ? DK * PC : 8];
+  float f[4 * CL];
+};
+
+template <int DK, bool OUT>
+__global__ void __launch_bounds__(32 * SW, 2) ssd_kernel(const ScanParams sp, float* seg_state, int seg_chunks, int nseg) {
+  using Sm = SsdSmem<DK, OUT>;
+  constexpr int P = Sm::P, PC = Sm::PC, NT = 32 * SW, KT = DK / 16, MU = DK / 64;  // MU: 16-row tiles of this warp's key dimensions
+  extern __shared__ __align__(16) uint8_t raw[];
+  Sm& sm = *reinterpret_cast<Sm*>(raw);
+  const RecurrentArgs& p = sp.a;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wt = warp & 3, wc = (warp >> 2) * 32;
+  const int slices = (p.Dv + SC - 1) / SC;
+  const int slice = blockIdx.x % slices, bh = blockIdx.x / slices, h = bh % p.H, b = bh / p.H, seg = blockIdx.y;
+  const int kh = h / (p.H / p.KG), c0 = slice * SC, ncol = min(SC, p.Dv - c0);
+  const __nv_bfloat16 *Q = (const __nv_bfloat16*)p.q + (long long)b * p.rows * p.ldq + kh * p.Dk,
+                      *K = (const __nv_bfloat16*)p.k + (long long)b * p.rows * p.ldk + kh * p.Dk,
+                      *V = (const __nv_bfloat16*)p.v + (long long)b * p.rows * p.ldv + h * p.Dv + c0;
+  __nv_bfloat16* O = (__nv_bfloat16*)p.out + (long long)b * p.rows * p.ldo + h * p.Dv + c0;
+  const float Dh = p.D[h];
+  const float4* f0 = reinterpret_cast<const float4*>(sp.frag0) + ((long long)b * p.KG + kh) * sp.nchunks * 1024;
+  const float* fac = sp.fac + (long long)bh * sp.nchunks * FACTORS * CL;
+  const int first = seg * seg_chunks, last = min(first + seg_chunks, sp.nchunks);
+
+  // accumulators of this warp's part of the state: key dimensions wt DK / 4 + 16 m + {lane / 4, + 8}, columns
+  // wc + 8 n + 2 (lane % 4) + {0, 1}
+  const int rl = lane >> 2, pair = 2 * (lane & 3), d0 = wt * (DK / 4);
+  float S[MU][4][4];
+  const long long plane = (long long)p.Dk * p.Dv;
+  float* mine = nseg > 1 ? seg_state + ((long long)seg * p.B * p.H + bh) * plane : p.state + (long long)bh * plane;
+#pragma unroll
+  for (int m = 0; m < MU; ++m)
+#pragma unroll
+    for (int n = 0; n < 4; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = d0 + 16 * m + rl + (e >> 1) * 8, cc = wc + 8 * n + pair + (e & 1);
+        S[m][n][e] = OUT && d < p.Dk && cc < ncol ? mine[(long long)d * p.Dv + c0 + cc] : 0.f;
+      }
+  auto publish = [&]() {
+#pragma unroll
+    for (int m = 0; m < MU; ++m)
+#pragma unroll
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          uint32_t hi, lo;
+          split2(S[m][n][2 * half], S[m][n][2 * half + 1], hi, lo);
+          const int at = (d0 + 16 * m + rl + 8 * half) * PC + wc + 8 * n + pair;
+          *reinterpret_cast<uint32_t*>(sm.s[0] + at) = hi;
+          *reinterpret_cast<uint32_t*>(sm.s[1] + at) = lo;
+        }
+  };
+  auto stage_kx = [&](int c) {
+    stage_rows<DK, P>(sm.k, K, p.ldk, c * CL, p.T, p.Dk, sp.vec_qk, tid, NT);
+    stage_rows<SC, PC>(sm.x, V, p.ldv, c * CL, p.T, ncol, sp.vec_v, tid, NT);
+    if (tid < CL)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(sm.f + tid * 4)), "l"(fac + (long long)c * FACTORS * CL + tid * 4) : "memory");
+  };
+  auto stage_q = [&](int c) {
+    if constexpr (OUT) stage_rows<DK, P>(sm.q, Q, p.ldq, c * CL, p.T, p.Dk, sp.vec_qk, tid, NT);
+  };
+  if (first < last) {
+    stage_q(first);
+    stage_kx(first);
+    cp_commit();
+  }
+  if constexpr (OUT) publish();
+  const int nt_row = (lane & 7) + ((lane >> 4) << 3), nt_col = ((lane >> 3) & 1) * 8;  // transposed A: stored [k][row]
+  const int tr_row = lane & 15, tr_col = (lane >> 4) * 8;                              // A [row][k]; transposed B: stored [k][n]
+
+  for (int c = first; c < last; ++c) {
+    const int t0 = c * CL;
+    float4 fr[2][OUT ? 4 : 1];
+    if constexpr (OUT) {
+#pragma unroll
+      for (int kt = 0; kt < 4; ++kt)
+        if (kt <= wt)
+#pragma unroll
+          for (int i = 0; i < 2; ++i) fr[i][kt] = f0[(long long)c * 1024 + ((2 * wt + i) * 4 + kt) * 32 + lane];
+    }
+    cp_wait0();
+    __syncthreads();  // the chunk's tiles and the state before it
+    const float* F = sm.f;
+    {  // weighted values of 16 tokens x 32 columns: a lane has 16 columns of one token
+      const int t = 16 * wt + (lane >> 1), at = t * PC + wc + (lane & 1) * 16;
+      const float w = F[2 * CL + t];
+#pragma unroll
+      for (int g = 0; g < 2; ++g) {
+        const uint4 v = *reinterpret_cast<const uint4*>(sm.x + at + 8 * g);
+        uint4 hi, lo;
+        split2(lo_f(v.x) * w, hi_f(v.x) * w, hi.x, lo.x);
+        split2(lo_f(v.y) * w, hi_f(v.y) * w, hi.y, lo.y);
+        split2(lo_f(v.z) * w, hi_f(v.z) * w, hi.z, lo.z);
+        split2(lo_f(v.w) * w, hi_f(v.w) * w, hi.w, lo.w);
+        *reinterpret_cast<uint4*>(sm.w[0] + at + 8 * g) = hi;
+        *reinterpret_cast<uint4*>(sm.w[1] + at + 8 * g) = lo;
+      }
+    }
+    if constexpr (OUT) {
+      float o[4][4];
+#pragma unroll
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[n][e] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < KT; ++ks) {
+        uint32_t aq[4];
+        ldsm4(aq, sm.q + (16 * wt + tr_row) * P + ks * 16 + tr_col);
+#pragma unroll
+        for (int n2 = 0; n2 < 2; ++n2) {
+          uint32_t bh4[4], bl4[4];
+          const int at = (ks * 16 + tr_row) * PC + wc + n2 * 16 + tr_col;
+          ldsm4t(bh4, sm.s[0] + at);
+          ldsm4t(bl4, sm.s[1] + at);
+          mma16816(o[2 * n2], aq, bh4[0], bh4[1]);
+          mma16816(o[2 * n2 + 1], aq, bh4[2], bh4[3]);
+          mma16816(o[2 * n2], aq, bl4[0], bl4[1]);
+          mma16816(o[2 * n2 + 1], aq, bl4[2], bl4[3]);
+        }
+      }
+      // e^{b_i - b_j} = e^{b_i - b_ref} e^{b_ref - b_j} for tokens j before this tile, the tile's first token as reference:
+      // both factors are at most 1, and the first is applied once to the whole sum; within the tile, pair by pair
+      const float br = F[16 * wt], er = exp_neg(br), bi0 = F[16 * wt + rl], bi1 = F[16 * wt + rl + 8];
+#pragma unroll
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[n][e] *= er;
+#pragma unroll
+      for (int kt = 0; kt < 4; ++kt) {
+        if (kt > wt) break;
+        const int j = kt * 16 + pair;
+        const float2 b0 = *reinterpret_cast<const float2*>(F + j), b8 = *reinterpret_cast<const float2*>(F + j + 8);
+        const float2 g0 = *reinterpret_cast<const float2*>(F + CL + j), g8 = *reinterpret_cast<const float2*>(F + CL + j + 8);
+        uint32_t ah[4], al[4];
+        if (kt < wt) {
+          const float w0 = g0.x * exp_neg(br - b0.x), w1 = g0.y * exp_neg(br - b0.y), w8 = g8.x * exp_neg(br - b8.x), w9 = g8.y * exp_neg(br - b8.y);
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            split2(fr[i][kt].x * w0, fr[i][kt].y * w1, ah[i], al[i]);
+            split2(fr[i][kt].z * w8, fr[i][kt].w * w9, ah[2 + i], al[2 + i]);
+          }
+        } else {
+          const float s0 = exp_neg(bi0 - br), s1 = exp_neg(bi1 - br);
+#pragma unroll
+          for (int n = 0; n < 4; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[n][e] *= e < 2 ? s0 : s1;
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            const int row = 16 * wt + rl + 8 * i;
+            const float bi = i == 0 ? bi0 : bi1;
+            const float m0 = j <= row ? fr[i][kt].x * g0.x * exp_neg(bi - b0.x) : 0.f, m1 = j + 1 <= row ? fr[i][kt].y * g0.y * exp_neg(bi - b0.y) : 0.f;
+            const float m8 = j + 8 <= row ? fr[i][kt].z * g8.x * exp_neg(bi - b8.x) : 0.f, m9 = j + 9 <= row ? fr[i][kt].w * g8.y * exp_neg(bi - b8.y) : 0.f;
+            split2(m0, m1, ah[i], al[i]);
+            split2(m8, m9, ah[2 + i], al[2 + i]);
+          }
+        }
+#pragma unroll
+        for (int n2 = 0; n2 < 2; ++n2) {
+          uint32_t bx[4];
+          ldsm4t(bx, sm.x + (kt * 16 + tr_row) * PC + wc + n2 * 16 + tr_col);
+          mma16816(o[2 * n2], ah, bx[0], bx[1]);
+          mma16816(o[2 * n2 + 1], ah, bx[2], bx[3]);
+          mma16816(o[2 * n2], al, bx[0], bx[1]);
+          mma16816(o[2 * n2 + 1], al, bx[2], bx[3]);
+        }
+      }
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int i = 16 * wt + rl + 8 * half, t = t0 + i;
+        if (t < p.T) {
+          __nv_bfloat16* dst = O + (long long)t * p.ldo;
+#pragma unroll
+          for (int n = 0; n < 4; ++n) {
+            const int cc = wc + 8 * n + pair;
+            const uint32_t xv = *reinterpret_cast<const uint32_t*>(sm.x + i * PC + cc);
+            const uint32_t y = pack_bf16x2(o[n][2 * half] + Dh * lo_f(xv), o[n][2 * half + 1] + Dh * hi_f(xv));
+            if (sp.vec_v && cc < ncol) *reinterpret_cast<uint32_t*>(dst + cc) = y;
+            else {
+              if (cc < ncol) dst[cc] = __float2bfloat16(lo_f(y));
+              if (cc + 1 < ncol) dst[cc + 1] = __float2bfloat16(hi_f(y));
+            }
+          }
+        }
+      }
+    }
+    __syncthreads();  // every warp's weighted values are there; queries and the published state have been read
+    const bool more = c + 1 < last;
+    if (more) stage_q(c + 1);
+    const float dl = F[3 * CL];
+#pragma unroll
+    for (int m = 0; m < MU; ++m)
+#pragma unroll
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[m][n][e] *= dl;
+#pragma unroll
+    for (int kt = 0; kt < 4; ++kt) {
+      uint32_t ak[MU][4];
+#pragma unroll
+      for (int m = 0; m < MU; ++m) ldsm4t(ak[m], sm.k + (kt * 16 + nt_row) * P + d0 + 16 * m + nt_col);
+#pragma unroll
+      for (int n2 = 0; n2 < 2; ++n2) {
+        uint32_t wh[4], wl[4];
+        const int at = (kt * 16 + tr_row) * PC + wc + n2 * 16 + tr_col;
+        ldsm4t(wh, sm.w[0] + at);
+        ldsm4t(wl, sm.w[1] + at);
+#pragma unroll
+        for (int m = 0; m < MU; ++m) {
+          mma16816(S[m][2 * n2], ak[m], wh[0], wh[1]);
+          mma16816(S[m][2 * n2 + 1], ak[m], wh[2], wh[3]);
+          mma16816(S[m][2 * n2], ak[m], wl[0], wl[1]);
+          mma16816(S[m][2 * n2 + 1], ak[m], wl[2], wl[3]);
+        }
+      }
+    }
+    if constexpr (OUT) publish();
+    if (more) {
+      __syncthreads();  // keys, values and factors have been read
+      stage_kx(c + 1);
+      cp_commit();
+    }
+  }
+  if (!OUT || seg == nseg - 1) {
+    float* dst = OUT ? p.state + (long long)bh * plane : mine;
+#pragma unroll
+    for (int m = 0; m < MU; ++m)
+#pragma unroll
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int d = d0 + 16 * m + rl + (e >> 1) * 8, cc = wc + 8 * n + pair + (e & 1);
+          if (d < p.Dk && cc < ncol) dst[(long long)d * p.Dv + c0 + cc] = S[m][n][e];
+        }
+  }
+}
+
+// seg_state: own contribution of every segment -> state before every segment. grid (ceil(plane / 256), B H)
+__global__ void ssd_scan_kernel(const ScanParams sp, float* seg_state, int seg_chunks, int nseg) {
+  __shared__ float dec[64];
+  const RecurrentArgs& p = sp.a;
+  const long long plane = (long long)p.Dk * p.Dv, bh = blockIdx.y;
+  const float* fac = sp.fac + bh * sp.nchunks * FACTORS * CL;
+  if (threadIdx.x < nseg) {
+    float s = 0.f;
+    for (int c = threadIdx.x * seg_chunks; c < min(((int)threadIdx.x + 1) * seg_chunks, sp.nchunks); ++c) s += fac[(long long)c * FACTORS * CL + CL - 1];
+    dec[threadIdx.x] = exp_neg(s);
+  }
+  __syncthreads();
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= plane) return;
+  float run = p.state[bh * plane + i];
+  for (int g = 0; g < nseg; ++g) {
+    float* at = seg_state + ((long long)g * p.B * p.H + bh) * plane + i;
+    const float own = *at;
+    *at = run;
+    run = dec[g] * run + own;
+  }
+}
+
+// Segments so that about two blocks per SM walk; none where the heads alone fill the machine.
+int ssd_segments(const RecurrentArgs& a) {
+  const int blocks = a.B * a.H * ((a.Dv + SC - 1) / SC), n = (a.T + CL - 1) / CL;
+  int s = (2 * 148) / blocks;
+  s = s > n / 4 ? n / 4 : s;
+  s = s > 64 ? 64 : s;
+  return s < 2 ? 1 : s;
+}
+
 template <int KIND, int DK>
-void run_scan(const ScanParams& sp, cudaStream_t s) {
+void run_scores(const ScanParams& sp, cudaStream_t s) {
   const RecurrentArgs& a = sp.a;
   auto kern = chunk_scores_kernel<KIND, DK>;
   constexpr int smem = 2 * CL * (DK + 8) * 2 + (KIND == RK_DELTA ? 2 * CL * 65 * 4 : 0);
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   kern<<<a.B * (KIND == RK_DELTA ? a.H : a.KG) * sp.nchunks, 128, smem, s>>>(sp);
   check_launch("chunk_scores");
-  if (KIND == RK_MAMBA2) {
-    const long long n = (long long)a.B * a.H * sp.nchunks;
-    chunk_factors_kernel<<<(unsigned)((n + 3) / 4), 128, 0, s>>>(sp);
-    check_launch("chunk_factors");
+}
+
+template <int DK>
+void run_delta(const ScanParams& sp, cudaStream_t s) {
+  const RecurrentArgs& a = sp.a;
+  run_scores<RK_DELTA, DK>(sp, s);
+  auto walk = delta_walk_kernel<DK>;
+  constexpr int smem = (int)sizeof(WalkSmem<DK>);
+  cudaFuncSetAttribute(walk, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  walk<<<a.B * a.H * ((a.Dv + WCOLS - 1) / WCOLS), 32 * WW, smem, s>>>(sp);
+  check_launch("delta_walk");
+}
+
+template <int DK>
+void run_ssd(const ScanParams& sp, float* seg_state, cudaStream_t s) {
+  const RecurrentArgs& a = sp.a;
+  run_scores<RK_MAMBA2, DK>(sp, s);
+  const long long n = (long long)a.B * a.H * sp.nchunks;
+  chunk_factors_kernel<<<(unsigned)((n + 3) / 4), 128, 0, s>>>(sp);
+  check_launch("chunk_factors");
+  const int want = ssd_segments(a), per = (sp.nchunks + want - 1) / want, nseg = (sp.nchunks + per - 1) / per;
+  const dim3 grid(a.B * a.H * ((a.Dv + SC - 1) / SC), nseg);
+  if (nseg > 1) {
+    auto own = ssd_kernel<DK, false>;
+    constexpr int smem = (int)sizeof(SsdSmem<DK, false>);
+    cudaFuncSetAttribute(own, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    own<<<grid, 32 * SW, smem, s>>>(sp, seg_state, per, nseg);
+    check_launch("ssd_states");
+    ssd_scan_kernel<<<dim3((unsigned)(((long long)a.Dk * a.Dv + 255) / 256), a.B * a.H), 256, 0, s>>>(sp, seg_state, per, nseg);
+    check_launch("ssd_scan");
   }
-  auto walk = chunk_walk_kernel<KIND, DK>;
-  constexpr int wsm = (int)sizeof(WalkSmem<KIND, DK>);
-  cudaFuncSetAttribute(walk, cudaFuncAttributeMaxDynamicSharedMemorySize, wsm);
-  walk<<<a.B * a.H * ((a.Dv + WCOLS - 1) / WCOLS), 32 * WW, wsm, s>>>(sp);
-  check_launch("chunk_walk");
+  auto out = ssd_kernel<DK, true>;
+  constexpr int smem = (int)sizeof(SsdSmem<DK, true>);
+  cudaFuncSetAttribute(out, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  out<<<grid, 32 * SW, smem, s>>>(sp, seg_state, per, nseg);
+  check_launch("ssd_out");
 }
 
 }  // namespace
@@ -602,7 +859,8 @@ bool chunk_scan_supported(const RecurrentArgs& a) { return !a.f32 && a.Dk <= 128
 
 long long chunk_scan_scratch(const RecurrentArgs& a) {
   const long long n = (a.T + CL - 1) / CL;
-  return (long long)a.B * n * (a.H * FACTORS * CL * 4ll + (a.kind == RK_DELTA ? a.H * 2 * 16384ll : a.KG * 16384ll));
+  const long long chunks = (long long)a.B * n * (a.H * FACTORS * CL * 4ll + (a.kind == RK_DELTA ? a.H * 2 * 16384ll : a.KG * 16384ll));
+  return chunks + (a.kind == RK_DELTA ? 0 : (long long)ssd_segments(a) * a.B * a.H * a.Dk * a.Dv * 4);
 }
 
 void launch_chunk_scan(const RecurrentArgs& a, void* scratch, cudaStream_t s) {
@@ -617,12 +875,13 @@ void launch_chunk_scan(const RecurrentArgs& a, void* scratch, cudaStream_t s) {
   if (a.kind == RK_DELTA) {
     sp.frag1 = sp.frag0 + (long long)a.B * a.H * sp.nchunks * 1024;
     sp.fac = (float*)(sp.frag1 + (long long)a.B * a.H * sp.nchunks * 1024);
-    if (a.Dk <= 64) run_scan<RK_DELTA, 64>(sp, s);
-    else run_scan<RK_DELTA, 128>(sp, s);
+    if (a.Dk <= 64) run_delta<64>(sp, s);
+    else run_delta<128>(sp, s);
   } else {
     sp.fac = (float*)(sp.frag0 + (long long)a.B * a.KG * sp.nchunks * 1024);
-    if (a.Dk <= 64) run_scan<RK_MAMBA2, 64>(sp, s);
-    else run_scan<RK_MAMBA2, 128>(sp, s);
+    float* seg = sp.fac + (long long)a.B * a.H * sp.nchunks * FACTORS * CL;
+    if (a.Dk <= 64) run_ssd<64>(sp, seg, s);
+    else run_ssd<128>(sp, seg, s);
   }
 }
 

@@ -141,10 +141,10 @@ void recurrent(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& 
     return;
   }
   // prompts longer than the scratch budget go in parts: the state carries over
-  constexpr int64_t budget = 768ll << 20;
+  constexpr int64_t budget = 1024ll << 20;
   tb::RecurrentArgs part = r;
-  part.T = 64;
-  const int64_t per = std::max<int64_t>(1, budget / std::max<int64_t>(1, tb::chunk_scan_scratch(part))) * 64;
+  int64_t per = (T + 63) / 64 * 64;
+  while (per > 4096 && (part.T = (int)std::min(per, T), tb::chunk_scan_scratch(part)) > budget) per = (per / 2 + 63) / 64 * 64;
   Tensor scratch;
   for (int64_t t = 0; t < T; t += per) {
     part.T = (int)std::min(per, T - t);

@@ -9,53 +9,120 @@ namespace {
 
 constexpr int GV_WARPS = 8;
 
-__device__ void gemv_segment(const GemvSegment& g, int b, float* dst, float* red) {
-  const float* x = g.x + (long long)b * g.ld;
-  const int tid = threadIdx.x, nt = blockDim.x;
+// Sum over the `nt` threads that work on one input row: a warp or the whole block. One barrier per sum: the warps' partial
+// sums are read by everyone, from alternating halves of `red`.
+__device__ __forceinline__ float row_sum(float v, int nt, float* red, int& phase) {
+  v = warp_sum(v);
+  if (nt == 32) return v;
+  float* r = red + (phase & 1) * GV_WARPS;
+  ++phase;
+  if ((threadIdx.x & 31) == 0) r[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+#pragma unroll
+  for (int i = 0; i < GV_WARPS; ++i) t += r[i];
+  return t;
+}
+template <bool EXACT>
+__device__ __forceinline__ float silu_step(float x) {
+  if constexpr (EXACT) return silu_f(x);
+  else return __fdividef(x, 1.f + __expf(-x));
+}
+
+// One segment of input row b by nt threads (tid among them), vectors of four where the layout allows.
+template <bool EXACT, int V>
+__device__ void segment_row(const GemvSegment& g, int b, float* dst, float* red, int& phase, int tid, int nt) {
+  const float *x = g.x + (long long)b * g.ld, *gt = g.gate + (long long)b * g.ldg;
+  const int part = g.n / g.groups, step = nt * V;
+  auto each = [&](const float* p, int i, float (&f)[V]) {
+    if constexpr (V == 4) {
+      const float4 t = *reinterpret_cast<const float4*>(p + i);
+      f[0] = t.x; f[1] = t.y; f[2] = t.z; f[3] = t.w;
+    } else {
+      f[0] = p[i];
+    }
+  };
+  auto put = [&](int i, const float (&f)[V]) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(dst + i) = make_float4(f[0], f[1], f[2], f[3]);
+    else dst[i] = f[0];
+  };
   if (g.kind == 0) {
-    for (int i = tid; i < g.n; i += nt) dst[i] = x[i] * g.scale;
+#pragma unroll 2
+    for (int i = tid * V; i < g.n; i += step) {
+      float f[V];
+      each(x, i, f);
+#pragma unroll
+      for (int e = 0; e < V; ++e) f[e] *= g.scale;
+      put(i, f);
+    }
   } else if (g.kind == 1) {
     float s = 0.f, mean = 0.f;
-    for (int i = tid; i < g.n; i += nt) {
-      dst[i] = x[i];
-      s += dst[i];
+#pragma unroll 2
+    for (int i = tid * V; i < g.n; i += step) {
+      float f[V];
+      each(x, i, f);
+#pragma unroll
+      for (int e = 0; e < V; ++e) s += f[e];
+      put(i, f);
     }
-    if (g.norm_kind == HN_LAYER) mean = block_sum(s, red) / g.n;
+    if (g.norm_kind == HN_LAYER) mean = row_sum(s, nt, red, phase) / g.n;
     float q = 0.f;
-    for (int i = tid; i < g.n; i += nt) q += (dst[i] - mean) * (dst[i] - mean);
-    const float r = g.scale / sqrtf(block_sum(q, red) / g.n + g.eps);
-    for (int i = tid; i < g.n; i += nt) dst[i] = (dst[i] - mean) * r * g.w[i];
-  } else {
-    const float* gt = g.gate + (long long)b * g.ldg;
-    const int part = g.n / g.groups, warp = tid >> 5, lane = tid & 31;
-    if (part > 512) {  // wide parts: the whole block on one part at a time
-      for (int p = 0; p < g.groups; ++p) {
-        float q = 0.f;
-        for (int i = tid; i < part; i += nt) {
-          const int c = p * part + i;
-          const float z = silu_f(gt[c]), v = x[c];
-          const float in = g.norm_kind == GO_GATE_THEN_NORM ? v * z : v;
-          q += in * in;
-          dst[c] = v * z * g.w[c % g.w_period];
-        }
-        const float r = g.scale / sqrtf(block_sum(q, red) / part + g.eps);
-        for (int i = tid; i < part; i += nt) dst[p * part + i] *= r;
-      }
-      return;
+    for (int i = tid * V; i < g.n; i += step) {
+      float f[V];
+      each(dst, i, f);  // written by this thread
+#pragma unroll
+      for (int e = 0; e < V; ++e) q += (f[e] - mean) * (f[e] - mean);
     }
-    for (int p = warp; p < g.groups; p += nt >> 5) {
+    const float r = g.scale / sqrtf(row_sum(q, nt, red, phase) / g.n + g.eps);
+#pragma unroll 2
+    for (int i = tid * V; i < g.n; i += step) {
+      float f[V], w[V];
+      each(dst, i, f);
+      each(g.w, i, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) f[e] = (f[e] - mean) * r * w[e];
+      put(i, f);
+    }
+  } else {
+    // wide parts: all threads of the row on one part at a time; narrow parts: a warp per part
+    const bool wide = part > 512 || nt == 32;
+    const int lane = threadIdx.x & 31, t0 = wide ? tid : lane, ts = (wide ? nt : 32) * V;
+    for (int p = wide ? 0 : tid >> 5; p < g.groups; p += wide ? 1 : nt >> 5) {
       float q = 0.f;
-      for (int i = lane; i < part; i += 32) {
+#pragma unroll 2
+      for (int i = t0 * V; i < part; i += ts) {
         const int c = p * part + i;
-        const float z = silu_f(gt[c]), v = x[c];
-        const float in = g.norm_kind == GO_GATE_THEN_NORM ? v * z : v;
-        q += in * in;
-        dst[c] = v * z * g.w[c % g.w_period];
+        float f[V], z[V], w[V];
+        each(x, c, f);
+        each(gt, c, z);
+        each(g.w, g.w_period == g.n ? c : i, w);  // one weight per channel, or one part's weights for every part
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          const float a = silu_step<EXACT>(z[e]), in = g.norm_kind == GO_GATE_THEN_NORM ? f[e] * a : f[e];
+          q += in * in;
+          f[e] *= a * w[e];
+        }
+        put(c, f);
       }
-      const float r = g.scale / sqrtf(warp_sum(q) / part + g.eps);
-      for (int i = lane; i < part; i += 32) dst[p * part + i] *= r;
+      const float r = g.scale / sqrtf((wide ? row_sum(q, nt, red, phase) : warp_sum(q)) / part + g.eps);
+      for (int i = t0 * V; i < part; i += ts) {
+        float f[V];
+        each(dst, p * part + i, f);
+#pragma unroll
+        for (int e = 0; e < V; ++e) f[e] *= r;
+        put(p * part + i, f);
+      }
     }
   }
+}
+
+template <bool EXACT>
+__device__ __forceinline__ void gemv_segment(const GemvSegment& g, int b, float* dst, float* red, int& phase, int tid, int nt) {
+  const bool quad = ((g.n | (int)g.ld | (g.n / g.groups) | g.w_period) & 3) == 0 && (g.kind != 2 || (g.ldg & 3) == 0) &&
+                    ((reinterpret_cast<uintptr_t>(g.x) | reinterpret_cast<uintptr_t>(g.w) | reinterpret_cast<uintptr_t>(g.gate) |
+                      reinterpret_cast<uintptr_t>(dst)) & 15) == 0;
+  if (quad) segment_row<EXACT, 4>(g, b, dst, red, phase, tid, nt);
+  else segment_row<EXACT, 1>(g, b, dst, red, phase, tid, nt);
 }
 
 template <class T>
@@ -99,9 +166,9 @@ void launch_chained(void (*kern)(Args, Rest...), int blocks, int threads, size_t
 
 // A warp works on two rows at a time (for the gated epilogue: a gate row and its up row).
 template <class T, int NB>
-__global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const GemvArgs p) {
+__global__ void __launch_bounds__(GV_WARPS * 32, 2) gemv_kernel(const GemvArgs p) {
   extern __shared__ __align__(16) float sx[];  // [NB][KP]
-  __shared__ float red[33];
+  __shared__ float red[2 * GV_WARPS];
   constexpr int VEC = 16 / sizeof(T), STEP = 32 * VEC, PRE = 4;
   const int KP = (p.K + 3) & ~3;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -133,10 +200,13 @@ __global__ void __launch_bounds__(GV_WARPS * 32) gemv_kernel(const GemvArgs p) {
   fetch(pr);
   launch_dependents();
   wait_for_previous();
-  for (int b = 0; b < p.B; ++b) {
+  // one row: the whole block forms it; several rows: a warp each
+  const int nt = p.B == 1 ? GV_WARPS * 32 : 32;
+  int phase = 0;
+  for (int b = p.B == 1 ? 0 : warp; b < p.B; b += GV_WARPS) {
     int off = 0;
     for (int i = 0; i < p.nseg; ++i) {
-      gemv_segment(p.seg[i], b, sx + b * KP + off, red);
+      gemv_segment<sizeof(T) == 4>(p.seg[i], b, sx + b * KP + off, red, phase, p.B == 1 ? (int)threadIdx.x : lane, nt);
       off += p.seg[i].n;
     }
   }
@@ -591,7 +661,7 @@ void launch_gemv(const GemvArgs& a, cudaStream_t s) {
   if (sm > 200 * 1024) throw std::runtime_error("gemv: the input rows do not fit into shared memory");
   const int pairs = a.epilogue == 2 ? a.N : (a.N + 1) / 2;
   int blocks = (pairs + GV_WARPS - 1) / GV_WARPS;
-  const int per_sm = sm > 100 * 1024 ? 1 : sm > 50 * 1024 ? 2 : 4;
+  const int per_sm = sm > 100 * 1024 ? 1 : 2;
   if (blocks > 148 * per_sm) blocks = 148 * per_sm;
   auto go = [&](auto* kern) {
     if (sm > 47 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
