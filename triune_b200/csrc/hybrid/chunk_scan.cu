@@ -605,6 +605,7 @@ __global__ void __launch_bounds__(32 * SW, 2) ssd_kernel(const ScanParams sp, fl
     cp_commit();
   }
   if constexpr (OUT) publish();
+  float decay = 1.f;  // of the whole segment
   const int nt_row = (lane & 7) + ((lane >> 4) << 3), nt_col = ((lane >> 3) & 1) * 8;  // transposed A: stored [k][row]
   const int tr_row = lane & 15, tr_col = (lane >> 4) * 8;                              // A [row][k]; transposed B: stored [k][n]
 
@@ -728,6 +729,7 @@ __global__ void __launch_bounds__(32 * SW, 2) ssd_kernel(const ScanParams sp, fl
     const bool more = c + 1 < last;
     if (more) stage_q(c + 1);
     const float dl = F[3 * CL];
+    decay *= dl;
 #pragma unroll
     for (int m = 0; m < MU; ++m)
 #pragma unroll
@@ -772,30 +774,27 @@ __global__ void __launch_bounds__(32 * SW, 2) ssd_kernel(const ScanParams sp, fl
           const int d = d0 + 16 * m + rl + (e >> 1) * 8, cc = wc + 8 * n + pair + (e & 1);
           if (d < p.Dk && cc < ncol) dst[(long long)d * p.Dv + c0 + cc] = S[m][n][e];
         }
+    if (!OUT && slice == 0 && tid == 0) seg_state[(long long)nseg * p.B * p.H * plane + (long long)seg * p.B * p.H + bh] = decay;
   }
 }
 
-// seg_state: own contribution of every segment -> state before every segment. grid (ceil(plane / 256), B H)
-__global__ void ssd_scan_kernel(const ScanParams sp, float* seg_state, int seg_chunks, int nseg) {
-  __shared__ float dec[64];
+// seg_state: own contribution of every segment but the last -> state before every segment; the segments' decays follow
+// the states. grid (ceil(plane / 256), B H)
+__global__ void ssd_scan_kernel(const ScanParams sp, float* seg_state, int nseg) {
   const RecurrentArgs& p = sp.a;
-  const long long plane = (long long)p.Dk * p.Dv, bh = blockIdx.y;
-  const float* fac = sp.fac + bh * sp.nchunks * FACTORS * CL;
-  if (threadIdx.x < nseg) {
-    float s = 0.f;
-    for (int c = threadIdx.x * seg_chunks; c < min(((int)threadIdx.x + 1) * seg_chunks, sp.nchunks); ++c) s += fac[(long long)c * FACTORS * CL + CL - 1];
-    dec[threadIdx.x] = exp_neg(s);
-  }
-  __syncthreads();
+  const long long plane = (long long)p.Dk * p.Dv, bh = blockIdx.y, heads = (long long)p.B * p.H;
+  const float* dec = seg_state + nseg * heads * plane + bh;
   const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
   if (i >= plane) return;
   float run = p.state[bh * plane + i];
-  for (int g = 0; g < nseg; ++g) {
-    float* at = seg_state + ((long long)g * p.B * p.H + bh) * plane + i;
-    const float own = *at;
-    *at = run;
-    run = dec[g] * run + own;
+  float* at = seg_state + bh * plane + i;
+#pragma unroll 4
+  for (int g = 0; g < nseg - 1; ++g) {
+    const float own = at[g * heads * plane];
+    at[g * heads * plane] = run;
+    run = dec[g * heads] * run + own;
   }
+  at[(nseg - 1) * heads * plane] = run;
 }
 
 // Segments so that about two blocks per SM walk; none where the heads alone fill the machine.
@@ -841,9 +840,9 @@ void run_ssd(const ScanParams& sp, float* seg_state, cudaStream_t s) {
     auto own = ssd_kernel<DK, false>;
     constexpr int smem = (int)sizeof(SsdSmem<DK, false>);
     cudaFuncSetAttribute(own, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    own<<<grid, 32 * SW, smem, s>>>(sp, seg_state, per, nseg);
+    own<<<dim3(grid.x, nseg - 1), 32 * SW, smem, s>>>(sp, seg_state, per, nseg);
     check_launch("ssd_states");
-    ssd_scan_kernel<<<dim3((unsigned)(((long long)a.Dk * a.Dv + 255) / 256), a.B * a.H), 256, 0, s>>>(sp, seg_state, per, nseg);
+    ssd_scan_kernel<<<dim3((unsigned)(((long long)a.Dk * a.Dv + 255) / 256), a.B * a.H), 256, 0, s>>>(sp, seg_state, nseg);
     check_launch("ssd_scan");
   }
   auto out = ssd_kernel<DK, true>;
@@ -860,7 +859,7 @@ bool chunk_scan_supported(const RecurrentArgs& a) { return !a.f32 && a.Dk <= 128
 long long chunk_scan_scratch(const RecurrentArgs& a) {
   const long long n = (a.T + CL - 1) / CL;
   const long long chunks = (long long)a.B * n * (a.H * FACTORS * CL * 4ll + (a.kind == RK_DELTA ? a.H * 2 * 16384ll : a.KG * 16384ll));
-  return chunks + (a.kind == RK_DELTA ? 0 : (long long)ssd_segments(a) * a.B * a.H * a.Dk * a.Dv * 4);
+  return chunks + (a.kind == RK_DELTA ? 0 : (long long)ssd_segments(a) * a.B * a.H * ((long long)a.Dk * a.Dv + 1) * 4);
 }
 
 void launch_chunk_scan(const RecurrentArgs& a, void* scratch, cudaStream_t s) {
