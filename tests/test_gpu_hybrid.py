@@ -135,7 +135,7 @@ def attention_case(seed, T, H, G, D, E, rot, dtype, far=None):
 
 
 @pytest.mark.parametrize("dtype", DT)
-@pytest.mark.parametrize("H,G,D,E,rot", [(4, 2, 16, 24, 8), (3, 1, 20, 10, 20), (8, 2, 128, 64, 64), (2, 2, 64, 128, 0), (6, 2, 64, 32, 32),
+@pytest.mark.parametrize("H,G,D,E,rot", [(4, 2, 16, 24, 8), (3, 1, 20, 10, 20), (8, 2, 128, 64, 64), (2, 2, 64, 128, 0), (6, 3, 64, 40, 48),
                                          (4, 4, 80, 48, 16), (2, 1, 128, 128, 128)])
 def test_attention_prompt_portions_and_far_keys(dtype, H, G, D, E, rot):
     from triune_b200.ops import hybrid as hops

@@ -40,6 +40,13 @@ def status_word(device) -> torch.Tensor:
     return _STATUS[key]
 
 
+def check_status(device) -> None:
+    """Raise if a bounded wait of a kernel on ``device`` has expired (reads the word: waits for the device)."""
+    word = _STATUS.get(torch.device(device))
+    if word is not None and int(word.item()):
+        raise RuntimeError(f"a kernel's bounded wait expired (status {int(word.item())}): its results are not valid")
+
+
 def embed_rows(ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
     """Embedding rows as the fp32 residual stream [tokens, width]."""
     ids = ids.reshape(-1)

@@ -35,6 +35,7 @@ class TraceRunner:
         import torch
 
         from ..inference import advance
+        from ..ops import hybrid as hops
 
         rows = []
         for e in entries:
@@ -47,7 +48,12 @@ class TraceRunner:
                     rows.append(logits[0].float())
         for rid in end:
             self.caches.pop(str(rid), None)
-        return torch.cat(rows).cpu() if rows else None
+        if not rows:
+            return None
+        out = torch.cat(rows).cpu()
+        if self.device.type == "cuda":
+            hops.check_status(self.device)
+        return out
 
 
 def load(folder: str, dtype: str, device: Optional[str] = None):
