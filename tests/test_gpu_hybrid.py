@@ -119,6 +119,32 @@ def test_recurrence_whole_and_in_portions(dtype, kind, H, K, D, E):
         assert float((st[0].double().cpu() - S).abs().max() / S.abs().max()) < 1e-4
 
 
+@pytest.mark.parametrize("kind", ["mamba2", "delta"])
+@pytest.mark.parametrize("B,H,K,D,E", [(1, 2, 1, 128, 64), (2, 3, 3, 96, 72), (1, 4, 2, 64, 48), (3, 2, 2, 72, 40), (1, 40, 1, 128, 128), (1, 6, 2, 20, 10)])
+def test_long_prompts_in_segments(kind, B, H, K, D, E):
+    """The chunk-parallel prompt kernels (segments, chunks, ragged ends) against the token recurrence on the same values in
+    fp32, from a state that is not zero; slow and fast decays side by side."""
+    from triune_b200.ops import hybrid as hops
+
+    for T in (1500, 1024, 129, 65):
+        r = gen(T + D)
+        bf = lambda t: t.to("cuda", torch.bfloat16)
+        q, k, v, a, b = bf(r(B * T, K * D)), bf(r(B * T, K * D)), bf(r(B * T, H * E)), bf(r(B * T, H)), bf(r(B * T, H))
+        A, bias, Dd, S0 = dev(torch.linspace(-6, 2.5, H)), dev(r(H) - 1), dev(r(H)), dev(r(B, H, D, E))
+        outs = []
+        for dtype in (torch.float32, torch.bfloat16):
+            c = lambda t: t.to(dtype)
+            st, out = S0.clone(), torch.empty(B * T, H * E, device="cuda", dtype=dtype)
+            hops.recurrent(c(q), c(k), c(v), c(a), c(b) if kind == "delta" else None, A, bias, Dd if kind == "mamba2" else None, st, out, B,
+                           T, kind, K)
+            outs.append((out.view(B, T, H, E).double(), st.double()))
+        hops.check_status(torch.device("cuda", 0))
+        (want, sw), (got, sg) = outs
+        for h in range(H):
+            assert float((got - want)[:, :, h].abs().max() / want[:, :, h].abs().max()) < 1e-2, (T, h)
+            assert float((sg - sw)[:, h].abs().max() / sw[:, h].abs().max()) < 1e-4, (T, h)
+
+
 def attention_case(seed, T, H, G, D, E, rot, dtype, far=None):
     r = gen(seed)
     pr = r(T, H * D + G * D + G * E)

@@ -21,11 +21,10 @@
 // operand layout of the next, with no trip through TMEM or shared memory in between.
 #include "../common/ptx.cuh"
 #include "hybrid.cuh"
+#include "tc_tiles.cuh"
 
 namespace tb {
 namespace {
-
-constexpr int CL = 64;  // tokens per chunk
 
 __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -44,20 +43,6 @@ __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const void* p) {
                : "r"(smem_u32(p))
                : "memory");
 }
-__device__ __forceinline__ float lo_f(uint32_t x) { return __uint_as_float(x << 16); }
-__device__ __forceinline__ float hi_f(uint32_t x) { return __uint_as_float(x & 0xffff0000u); }
-// (a, b) as two bf16 pairs whose sum is the fp32 pair to 2^-17
-__device__ __forceinline__ void split2(float a, float b, uint32_t& h, uint32_t& l) {
-  h = pack_bf16x2(a, b);
-  l = pack_bf16x2(a - lo_f(h), b - hi_f(h));
-}
-// e^x for x <= 0
-__device__ __forceinline__ float exp_neg(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x * 1.4426950408889634f));
-  return y;
-}
-
 // Rows [t0, t0 + 64) x [0, D) of a bf16 matrix into shared memory [64][pitch]; rows past T and columns past D are zero.
 // `vec`: 16-byte asynchronous copies (D a multiple of 8, aligned rows), otherwise plain stores.
 template <int COLS, int PITCH>
@@ -79,9 +64,6 @@ __device__ __forceinline__ void stage_rows(__nv_bfloat16* dst, const __nv_bfloat
     }
   }
 }
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-__device__ __forceinline__ void cp_wait0() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
-
 // Per-token factors of the walk, [B, H, nchunks][FACTORS][64] fp32 (b is the running log decay of the chunk):
 //   mamba2:  0 b   1 dt   2 dt e^{b_end - b}   3 e^{b_end} in entry 0
 //   delta:   0 beta   1 beta e^b / |k|   2 e^{b_end - b} / |k|   3 e^b Dk^-1/2 / |q|   4 e^{b_end} in entry 0
@@ -95,34 +77,6 @@ struct ScanParams {
   uint4* frag1;   // delta: the same of the inverse
   float* fac;
 };
-
-// Log decay and gate of the 64 tokens of a chunk by one warp: lane i holds tokens 2 i and 2 i + 1. Tokens past T change
-// nothing (no decay, zero gate). gate: dt (mamba2) or beta (delta).
-__device__ __forceinline__ void chunk_scalars(const RecurrentArgs& p, float ra0, float ra1, float rb0, float rb1, float ea, float bias,
-                                              int t0, float* sb, float* sgate) {
-  const int lane = threadIdx.x & 31, t = t0 + 2 * lane;
-  const float d0 = t < p.T ? softplus_f(ra0 + bias) : 0.f, d1 = t + 1 < p.T ? softplus_f(ra1 + bias) : 0.f;
-  float x = -ea * (d0 + d1);
-  const float own = x;
-#pragma unroll
-  for (int o = 1; o < 32; o <<= 1) {
-    const float y = __shfl_up_sync(0xffffffffu, x, o);
-    if (lane >= o) x += y;
-  }
-  const float before = x - own;
-  sb[2 * lane] = before - ea * d0;
-  sb[2 * lane + 1] = x;
-  if (p.kind == RK_DELTA) {
-    sgate[2 * lane] = t < p.T ? sigmoid_f(rb0) : 0.f;
-    sgate[2 * lane + 1] = t + 1 < p.T ? sigmoid_f(rb1) : 0.f;
-  } else {
-    sgate[2 * lane] = d0;
-    sgate[2 * lane + 1] = d1;
-  }
-}
-__device__ __forceinline__ float load_or0(const __nv_bfloat16* p, long long ld, int t, int T) {
-  return t < T ? __bfloat162float(p[(long long)t * ld]) : 0.f;
-}
 
 // ------------------------------------------------------------------------------------------------ scores
 template <int KIND, int DK>
@@ -780,8 +734,7 @@ __global__ void __launch_bounds__(32 * SW, 2) ssd_kernel(const ScanParams sp, fl
 
 // seg_state: own contribution of every segment but the last -> state before every segment; the segments' decays follow
 // the states. grid (ceil(plane / 256), B H)
-__global__ void ssd_scan_kernel(const ScanParams sp, float* seg_state, int nseg) {
-  const RecurrentArgs& p = sp.a;
+__global__ void ssd_scan_kernel(const RecurrentArgs p, float* seg_state, int nseg) {
   const long long plane = (long long)p.Dk * p.Dv, bh = blockIdx.y, heads = (long long)p.B * p.H;
   const float* dec = seg_state + nseg * heads * plane + bh;
   const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
@@ -842,8 +795,7 @@ void run_ssd(const ScanParams& sp, float* seg_state, cudaStream_t s) {
     cudaFuncSetAttribute(own, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     own<<<dim3(grid.x, nseg - 1), 32 * SW, smem, s>>>(sp, seg_state, per, nseg);
     check_launch("ssd_states");
-    ssd_scan_kernel<<<dim3((unsigned)(((long long)a.Dk * a.Dv + 255) / 256), a.B * a.H), 256, 0, s>>>(sp, seg_state, nseg);
-    check_launch("ssd_scan");
+    launch_ssd_scan(a, seg_state, nseg, s);
   }
   auto out = ssd_kernel<DK, true>;
   constexpr int smem = (int)sizeof(SsdSmem<DK, true>);
@@ -853,6 +805,11 @@ void run_ssd(const ScanParams& sp, float* seg_state, cudaStream_t s) {
 }
 
 }  // namespace
+
+void launch_ssd_scan(const RecurrentArgs& a, float* seg_state, int nseg, cudaStream_t s) {
+  ssd_scan_kernel<<<dim3((unsigned)(((long long)a.Dk * a.Dv + 255) / 256), a.B * a.H), 256, 0, s>>>(a, seg_state, nseg);
+  check_launch("ssd_scan");
+}
 
 bool chunk_scan_supported(const RecurrentArgs& a) { return !a.f32 && a.Dk <= 128 && a.T >= 32; }
 

@@ -74,6 +74,12 @@ void launch_recurrent(const RecurrentArgs& a, cudaStream_t s);
 bool chunk_scan_supported(const RecurrentArgs& a);
 long long chunk_scan_scratch(const RecurrentArgs& a);
 void launch_chunk_scan(const RecurrentArgs& a, void* scratch, cudaStream_t s);
+// Mamba-2 prompts on tcgen05 (aligned bf16, key sizes 65 to 128); `status` (or null) receives a KernelStatus.
+bool ssd_tc_supported(const RecurrentArgs& a);
+long long ssd_tc_scratch(const RecurrentArgs& a);
+void launch_ssd_tc(const RecurrentArgs& a, void* scratch, int* status, cudaStream_t s);
+// [nseg, B, H, Dk, Dv] contributions of segments (then [nseg, B, H] decays) -> states before the segments, from a.state
+void launch_ssd_scan(const RecurrentArgs& a, float* seg_state, int nseg, cudaStream_t s);
 
 // ---- softmax attention -----------------------------------------------------------------------------------------
 // Query / key head norm + rotation; appends k and v to the cache [B, G, cap, pitch*] at positions pos .. pos+T-1 and

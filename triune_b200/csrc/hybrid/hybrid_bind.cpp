@@ -132,7 +132,7 @@ void fill_recurrent(tb::RecurrentArgs& r, const Tensor& q, const Tensor& k, cons
 
 void recurrent(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& a, const OptT& b, const Tensor& A_log,
                const Tensor& dt_bias, const OptT& D, Tensor& state, Tensor& out, int64_t B, int64_t T, int64_t KG, int64_t kind,
-               double unit_eps, bool chunked) {
+               double unit_eps, bool chunked, const OptT& status) {
   tb::RecurrentArgs r{};
   fill_recurrent(r, q, k, v, a, b, A_log, dt_bias, D, state, out, B, T, KG, kind, unit_eps);
   c10::cuda::CUDAGuard guard(q.device());
@@ -144,7 +144,13 @@ void recurrent(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& 
   constexpr int64_t budget = 1024ll << 20;
   tb::RecurrentArgs part = r;
   int64_t per = (T + 63) / 64 * 64;
-  while (per > 4096 && (part.T = (int)std::min(per, T), tb::chunk_scan_scratch(part)) > budget) per = (per / 2 + 63) / 64 * 64;
+  auto scratch_of = [](const tb::RecurrentArgs& x) { return tb::ssd_tc_supported(x) ? tb::ssd_tc_scratch(x) : tb::chunk_scan_scratch(x); };
+  while (per > 4096 && (part.T = (int)std::min(per, T), scratch_of(part)) > budget) per = (per / 2 + 127) / 128 * 128;
+  int* st = nullptr;
+  if (status.has_value() && status->defined()) {
+    TORCH_CHECK(status->is_cuda() && status->scalar_type() == at::kInt, "status: CUDA int32 expected");
+    st = status->data_ptr<int>();
+  }
   Tensor scratch;
   for (int64_t t = 0; t < T; t += per) {
     part.T = (int)std::min(per, T - t);
@@ -156,9 +162,10 @@ void recurrent(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& 
       tb::launch_recurrent(part, cur_stream());
       continue;
     }
-    const int64_t need = tb::chunk_scan_scratch(part);
+    const int64_t need = scratch_of(part);
     if (!scratch.defined() || scratch.numel() < need) scratch = torch::empty({need}, q.options().dtype(at::kByte));
-    tb::launch_chunk_scan(part, scratch.data_ptr(), cur_stream());
+    if (tb::ssd_tc_supported(part)) tb::launch_ssd_tc(part, scratch.data_ptr(), st, cur_stream());
+    else tb::launch_chunk_scan(part, scratch.data_ptr(), cur_stream());
   }
 }
 
@@ -367,7 +374,8 @@ void register_hybrid(pybind11::module& m) {
   m.def("hybrid_causal_conv", &causal_conv);
   m.def("hybrid_recurrent", &recurrent, pybind11::arg("q"), pybind11::arg("k"), pybind11::arg("v"), pybind11::arg("a"), pybind11::arg("b"),
         pybind11::arg("A_log"), pybind11::arg("dt_bias"), pybind11::arg("D"), pybind11::arg("state"), pybind11::arg("out"), pybind11::arg("B"),
-        pybind11::arg("T"), pybind11::arg("key_groups"), pybind11::arg("kind"), pybind11::arg("unit_eps"), pybind11::arg("chunked") = true);
+        pybind11::arg("T"), pybind11::arg("key_groups"), pybind11::arg("kind"), pybind11::arg("unit_eps"), pybind11::arg("chunked") = true,
+        pybind11::arg("status") = pybind11::none());
   m.def("hybrid_attn_prep", &attn_prep);
   m.def("hybrid_attn_simple", &attn_simple);
   m.def("hybrid_attention", &attention);

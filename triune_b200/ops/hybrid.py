@@ -129,7 +129,8 @@ def recurrent(q, k, v, a, b, A_log, dt_bias, D, state, out, B: int, T: int, kind
     """Advances ``state`` [B, H, Dk, Dv] over T tokens in place; outputs into ``out``'s first H * Dv columns."""
     if _ext.use_kernels(q, state, out):
         _tick()
-        _ext.serving().hybrid_recurrent(q, k, v, a, b, A_log, dt_bias, D, state, out, B, T, key_groups, KINDS[kind], unit_eps)
+        _ext.serving().hybrid_recurrent(q, k, v, a, b, A_log, dt_bias, D, state, out, B, T, key_groups, KINDS[kind], unit_eps,
+                                       True, status_word(out.device))
     else:
         H, Dk, Dv = state.shape[1:]
         n = B * T
