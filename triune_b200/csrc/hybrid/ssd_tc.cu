@@ -5,11 +5,12 @@
 //   G  = C K^T                                     -> M_ij = G_ij dt_j e^{b_i-b_j} (j <= i), two bf16 numbers each, in TMEM
 //   Y  = e^{b_i} (C S) + M x + D x                  S as two bf16 numbers in shared memory, M as the A operand from TMEM
 //   S <- e^{b_end} S + K^T (w x)                    w x as two bf16 numbers; the sum in fp32 registers
-// A block owns 64 value columns of a head and a segment of the sequence. Its 256 threads are two halves of 128 rows: a
+// A block owns 64 value columns of a head and a segment of the sequence. 256 of its threads are two halves of 128 rows: a
 // thread has row r = its TMEM lane (a token for G, M and Y; a key dimension for the state) and half of the columns, so every
 // pass between the products stays in its registers. Shared-memory tiles are 128 rows of 128 bytes in the 128B-swizzled
-// layout: K and C are K-major operands for G, K is read again as the transposed A operand of the update.
-// TMEM columns: 0 G (128), 128 C S (64), 192 M x (64), 256 K^T (w x) (64), 320 low halves of M (64), 384 high halves (64).
+// layout; a ninth warp issues the MMAs (issuing blocks while the tensor pipe is busy): K and C are K-major operands for G, K is read again as the transposed A operand of the update.
+// TMEM columns: 0 G (128), 128 and 448 C S of alternating chunks (64 each), 192 M x (64), 256 K^T (w x) (64), 320 low halves
+// of M (64), 384 high halves (64).
 #include "../common/ptx.cuh"
 #include "hybrid.cuh"
 #include "tc_tiles.cuh"
@@ -78,17 +79,19 @@ __device__ __forceinline__ void stage_tile(uint8_t* dst, const __nv_bfloat16* sr
 
 template <bool OUT>
 struct SsdTcSmem {  // after alignment to 1024 bytes
-  static constexpr int K = 0, X = K + 2 * 2 * TBOX, WH = X + 2 * TBOX, WL = WH + TBOX, F = WL + TBOX;
-  static constexpr int C = F + 2 * TF * TL * 4, SH = C + (OUT ? 2 * TBOX : 0), SL = SH + (OUT ? TBOX : 0), END = SL + (OUT ? TBOX : 0);
+  static constexpr int NS = OUT ? 2 : 3;  // chunks of keys, values and factors in shared memory
+  static constexpr int K = 0, X = K + NS * 2 * TBOX, WH = X + NS * TBOX, WL = WH + TBOX, F = WL + TBOX;
+  static constexpr int C = (F + NS * TF * TL * 4 + 1023) / 1024 * 1024, SH = C + (OUT ? 2 * TBOX : 0), SL = SH + (OUT ? TBOX : 0), END = SL + (OUT ? TBOX : 0);
   static_assert(F % 1024 == 0 && C % 1024 == 0, "tiles start on 1024 bytes");
 };
 
 template <bool OUT>
-__global__ void __launch_bounds__(TT, 1) ssd_tc_kernel(const SsdTcParams sp) {
+__global__ void __launch_bounds__(TT + 32, 1) ssd_tc_kernel(const SsdTcParams sp) {
   using L = SsdTcSmem<OUT>;
   extern __shared__ uint8_t raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~uintptr_t(1023));
-  __shared__ __align__(8) uint64_t bars[4];  // G, C S, M x, update
+  __shared__ __align__(8) uint64_t bars[4];   // products done: G, C S, M x, update
+  __shared__ __align__(8) uint64_t ready[3];  // operands in place: tiles and state, weighted values, M
   __shared__ uint32_t tmem_slot;
   __shared__ int dead;
   const RecurrentArgs& p = sp.a;
@@ -106,11 +109,12 @@ __global__ void __launch_bounds__(TT, 1) ssd_tc_kernel(const SsdTcParams sp) {
 
   if (tid == 0) {
     for (int i = 0; i < 4; ++i) mbar_init(bars + i, 1);
+    for (int i = 0; i < 3; ++i) mbar_init(ready + i, TT);
     mbar_fence_init();
     dead = 0;
   }
   __syncwarp();
-  if (warp == 0) {
+  if (warp == 8) {
     tmem_alloc(&tmem_slot, 512);
     tmem_relinquish();
   }
@@ -119,7 +123,12 @@ __global__ void __launch_bounds__(TT, 1) ssd_tc_kernel(const SsdTcParams sp) {
   const long long plane = (long long)p.Dk * p.Dv;
   float* mine = sp.nseg > 1 ? sp.seg_state + ((long long)seg * p.B * p.H + bh) * plane : p.state + (long long)bh * plane;
 #pragma unroll
-  for (int i = 0; i < 32; ++i) S[i] = OUT && row < p.Dk && col0 + i < ncol ? mine[(long long)row * p.Dv + c0 + col0 + i] : 0.f;
+  for (int g = 0; g < 4; ++g) {
+    float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (OUT && warp < 8 && row < p.Dk && col0 + 8 * g < ncol) ld8v(mine + (long long)row * p.Dv + c0 + col0 + 8 * g, f);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) S[8 * g + i] = f[i];
+  }
   // 32 fp32 values of this thread's row as two bf16 tiles
   auto put = [&](int hi_at, int lo_at, const float (&v)[32]) {
 #pragma unroll
@@ -135,7 +144,7 @@ __global__ void __launch_bounds__(TT, 1) ssd_tc_kernel(const SsdTcParams sp) {
     }
   };
   auto stage_kx = [&](int c) {
-    const int u = (c - first) & 1;
+    const int u = (c - first) % L::NS;
     stage_tile(smem + L::K + u * 2 * TBOX, K, p.ldk, c * TL, p.T, p.Dk, 2, tid);
     stage_tile(smem + L::X + u * TBOX, V, p.ldv, c * TL, p.T, ncol, 1, tid);
     if (tid < TF * TL / 4)
@@ -146,60 +155,127 @@ __global__ void __launch_bounds__(TT, 1) ssd_tc_kernel(const SsdTcParams sp) {
   auto stage_c = [&](int c) {
     if constexpr (OUT) stage_tile(smem + L::C, Q, p.ldq, c * TL, p.T, p.Dk, 2, tid);
   };
-  if (first < last) {
+  if (first < last && warp < 8) {
     stage_c(first);
     stage_kx(first);
     cp_commit();
+    if constexpr (!OUT) {
+      if (first + 1 < last) stage_kx(first + 1);
+      cp_commit();
+    }
   }
-  if constexpr (OUT) put(L::SH, L::SL, S);
+  if (OUT && warp < 8) put(L::SH, L::SL, S);
   __syncthreads();
   tc_fence_after_sync();
   const uint32_t tmem = tmem_slot, lanes = tmem + ((uint32_t)((warp & 3) * 32) << 16);
   const uint32_t base = smem_u32(smem);
-  auto wait_bar = [&](int i, uint32_t parity) {
-    if (*(volatile int*)&dead == 0 && !mbar_wait(bars + i, parity)) {
+  auto wait_on = [&](uint64_t* bar, uint32_t parity) {
+    if (*(volatile int*)&dead == 0 && !mbar_wait(bar, parity)) {
       dead = 1;
       if (sp.status) *sp.status = ST_TIMEOUT_TMEM;
     }
+  };
+  auto wait_bar = [&](int i, uint32_t parity) {
+    wait_on(bars + i, parity);
     __syncwarp();
     tc_fence_after_sync();
   };
-  float decay = 1.f;
-
-  for (int c = first; c < last; ++c) {
-    const int u = (c - first) & 1, t0 = c * TL;
-    const uint32_t par = u;
-    const float* F = reinterpret_cast<const float*>(smem + L::F) + u * TF * TL;
-    const uint8_t* X = smem + L::X + u * TBOX;
-    cp_wait0();
-    fence_proxy_async_smem();
-    tc_fence_before_sync();
-    __syncthreads();  // this chunk's tiles and the state before it
-    const bool more = c + 1 < last;
-    if (OUT && tid == 0) {
-      tc_fence_after_sync();
-      const uint32_t ca = base + L::C, ka = base + L::K + u * 2 * TBOX;
-      constexpr uint32_t id_g = make_idesc(128, 128, 1, 1, 0, 0), id_s = make_idesc(128, 64, 1, 1, 0, 1);
+  auto rows_sync = [&]() { asm volatile("bar.sync 1, 256;" ::: "memory"); };
+  if (warp == 8) {
+    if (lane == 0) {
+      constexpr uint32_t id_g = make_idesc(128, 128, 1, 1, 0, 0), id_s = make_idesc(128, 64, 1, 1, 0, 1), id_u = make_idesc(128, 64, 1, 1, 1, 1);
+      for (int c = first; c < last; ++c) {
+        const uint32_t u = (c - first) & 1, slot = (c - first) % L::NS, ka = base + L::K + slot * 2 * TBOX, xa = base + L::X + slot * TBOX, ca = base + L::C;
+        wait_on(ready + 0, u);
+        tc_fence_after_sync();
+        if constexpr (OUT) {
 #pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const uint32_t off = (k >> 2) * TBOX + (k & 3) * 32;
-        umma_bf16(tmem, make_smem_desc(ca + off, 16, 1024), make_smem_desc(ka + off, 16, 1024), id_g, k > 0);
-      }
-      umma_commit(bars + 0);
+          for (int k = 0; k < 8; ++k) {
+            const uint32_t off = (k >> 2) * TBOX + (k & 3) * 32;
+            umma_bf16(tmem, make_smem_desc(ca + off, 16, 1024), make_smem_desc(ka + off, 16, 1024), id_g, k > 0);
+          }
+          umma_commit(bars + 0);
+          const uint32_t cs = tmem + (u == 0 ? 128 : 448);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const uint32_t off = (k >> 2) * TBOX + (k & 3) * 32;
-        const uint64_t a = make_smem_desc(ca + off, 16, 1024);
-        umma_bf16(tmem + 128, a, make_smem_desc(base + L::SH + k * 2048, TBOX, 1024), id_s, k > 0);
-        umma_bf16(tmem + 128, a, make_smem_desc(base + L::SL + k * 2048, TBOX, 1024), id_s, 1);
+          for (int k = 0; k < 8; ++k) {
+            const uint64_t a = make_smem_desc(ca + (k >> 2) * TBOX + (k & 3) * 32, 16, 1024);
+            umma_bf16(cs, a, make_smem_desc(base + L::SH + k * 2048, TBOX, 1024), id_s, k > 0);
+            umma_bf16(cs, a, make_smem_desc(base + L::SL + k * 2048, TBOX, 1024), id_s, 1);
+          }
+          umma_commit(bars + 1);
+        }
+        wait_on(ready + 1, u);
+        tc_fence_after_sync();
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          const uint64_t a = make_smem_desc(ka + k * 2048, TBOX, 1024);
+          umma_bf16(tmem + 256, a, make_smem_desc(base + L::WH + k * 2048, TBOX, 1024), id_u, k > 0);
+          umma_bf16(tmem + 256, a, make_smem_desc(base + L::WL + k * 2048, TBOX, 1024), id_u, 1);
+        }
+        umma_commit(bars + 3);
+        if constexpr (OUT) {
+          wait_on(ready + 2, u);
+          tc_fence_after_sync();
+#pragma unroll
+          for (int k = 0; k < 8; ++k) {
+            const uint64_t x = make_smem_desc(xa + k * 2048, TBOX, 1024);
+            umma_bf16_ts(tmem + 192, tmem + 384 + k * 8, x, id_s, k > 0);
+            umma_bf16_ts(tmem + 192, tmem + 320 + k * 8, x, id_s, 1);
+          }
+          umma_commit(bars + 2);
+        }
       }
-      umma_commit(bars + 1);
     }
     __syncwarp();
-    if (more) {  // the other buffers were last read by the update of chunk c - 1, which has been waited for
-      stage_kx(c + 1);
-      if (!OUT) cp_commit();
+  } else {
+  float decay = 1.f;
+
+  // outputs of chunk c: e^{b_i} (C S) + M x + D x
+  auto outputs = [&](int c) {
+    const int u = (c - first) & 1, t = c * TL + row;
+    const uint8_t* X = smem + L::X + u * TBOX;
+    const float e = exp_neg(reinterpret_cast<const float*>(smem + L::F)[u * TF * TL + row]);
+    wait_bar(2, u);
+    uint32_t cs[32], mx[32];
+    tmem_ld_32x32b_x32(lanes + (u == 0 ? 128 : 448) + col0, cs);
+    tmem_ld_32x32b_x32(lanes + 192 + col0, mx);
+    tmem_ld_wait_regs(cs);
+    tmem_ld_wait_regs(mx);
+    if (t < p.T) {
+      __nv_bfloat16* dst = O + (long long)t * p.ldo + col0;
+#pragma unroll
+      for (int g = 0; g < 4; ++g) {
+        const uint4 q = *reinterpret_cast<const uint4*>(X + sw(row, half * 4 + g));
+        const uint32_t xs[4] = {q.x, q.y, q.z, q.w};
+        uint4 y;
+        uint32_t* ys = &y.x;
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int k = 8 * g + 2 * i;
+          ys[i] = pack_bf16x2(e * __uint_as_float(cs[k]) + __uint_as_float(mx[k]) + Dh * lo_f(xs[i]),
+                              e * __uint_as_float(cs[k + 1]) + __uint_as_float(mx[k + 1]) + Dh * hi_f(xs[i]));
+        }
+        if (col0 + 8 * g < ncol) *reinterpret_cast<uint4*>(dst + 8 * g) = y;  // Dv is a multiple of eight
+      }
     }
+  };
+
+  // Order within a chunk: scores and state products are issued first; the previous chunk's outputs are written under them;
+  // the update is issued as soon as the weighted values are there and runs under the decay of the scores; the state is
+  // updated and published under the last product.
+  for (int c = first; c < last; ++c) {
+    const int slot = (c - first) % L::NS;
+    const uint32_t par = (c - first) & 1;
+    const float* F = reinterpret_cast<const float*>(smem + L::F) + slot * TF * TL;
+    const uint8_t* X = smem + L::X + slot * TBOX;
+    if constexpr (OUT) cp_wait0();
+    else asm volatile("cp.async.wait_group 1;" ::: "memory");
+    fence_proxy_async_smem();
+    tc_fence_before_sync();
+    rows_sync();  // this chunk's tiles and the state before it
+    mbar_arrive(ready + 0);
+    const bool more = c + 1 < last;
+    if (OUT && c > first) outputs(c - 1);
     {
       const float w = F[2 * TL + row];
       float v[32];
@@ -210,6 +286,16 @@ __global__ void __launch_bounds__(TT, 1) ssd_tc_kernel(const SsdTcParams sp) {
         v[8 * g + 4] = lo_f(q.z) * w; v[8 * g + 5] = hi_f(q.z) * w; v[8 * g + 6] = lo_f(q.w) * w; v[8 * g + 7] = hi_f(q.w) * w;
       }
       put(L::WH, L::WL, v);
+    }
+    fence_proxy_async_smem();
+    tc_fence_before_sync();
+    rows_sync();  // every thread has read what it needs of chunk c - 1
+    mbar_arrive(ready + 1);
+    if constexpr (OUT) {
+      if (more) stage_kx(c + 1);
+    } else {  // one commit per chunk, empty at the end
+      if (c + 2 < last) stage_kx(c + 2);
+      cp_commit();
     }
     if constexpr (OUT) {
       // decayed scores: blocks of 32 tokens before this warp's rows factor through the block's last token, the block of
@@ -252,64 +338,17 @@ __global__ void __launch_bounds__(TT, 1) ssd_tc_kernel(const SsdTcParams sp) {
         }
         tmem_st_32x32b_x16(lanes + 384 + jb * 16, hi);
         tmem_st_32x32b_x16(lanes + 320 + jb * 16, lo);
+        if (k == 0) {
+          wait_bar(1, par);  // the queries and the published state have been read
+          if (more) {
+            stage_c(c + 1);
+            cp_commit();
+          }
+        }
       }
       tmem_st_wait();
-      wait_bar(1, par);  // the queries and the published state have been read
-    }
-    fence_proxy_async_smem();
-    tc_fence_before_sync();
-    __syncthreads();  // weighted values and M are in place
-    if (tid == 0) {
-      tc_fence_after_sync();
-      constexpr uint32_t id_m = make_idesc(128, 64, 1, 1, 0, 1), id_u = make_idesc(128, 64, 1, 1, 1, 1);
-      const uint32_t xa = base + L::X + u * TBOX, ka = base + L::K + u * 2 * TBOX;
-      if constexpr (OUT) {
-#pragma unroll
-        for (int k = 0; k < 8; ++k) {
-          const uint64_t x = make_smem_desc(xa + k * 2048, TBOX, 1024);
-          umma_bf16_ts(tmem + 192, tmem + 384 + k * 8, x, id_m, k > 0);
-          umma_bf16_ts(tmem + 192, tmem + 320 + k * 8, x, id_m, 1);
-        }
-        umma_commit(bars + 2);
-      }
-#pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const uint64_t a = make_smem_desc(ka + k * 2048, TBOX, 1024);
-        umma_bf16(tmem + 256, a, make_smem_desc(base + L::WH + k * 2048, TBOX, 1024), id_u, k > 0);
-        umma_bf16(tmem + 256, a, make_smem_desc(base + L::WL + k * 2048, TBOX, 1024), id_u, 1);
-      }
-      umma_commit(bars + 3);
-    }
-    __syncwarp();
-    if constexpr (OUT) {
-      if (more) {
-        stage_c(c + 1);
-        cp_commit();
-      }
-      wait_bar(2, par);
-      uint32_t cs[32], mx[32];
-      tmem_ld_32x32b_x32(lanes + 128 + col0, cs);
-      tmem_ld_32x32b_x32(lanes + 192 + col0, mx);
-      tmem_ld_wait_regs(cs);
-      tmem_ld_wait_regs(mx);
-      const float e = exp_neg(F[row]);
-      if (t0 + row < p.T) {
-        __nv_bfloat16* dst = O + (long long)(t0 + row) * p.ldo + col0;
-#pragma unroll
-        for (int g = 0; g < 4; ++g) {
-          const uint4 q = *reinterpret_cast<const uint4*>(X + sw(row, half * 4 + g));
-          const uint32_t xs[4] = {q.x, q.y, q.z, q.w};
-          uint4 y;
-          uint32_t* ys = &y.x;
-#pragma unroll
-          for (int i = 0; i < 4; ++i) {
-            const int k = 8 * g + 2 * i;
-            ys[i] = pack_bf16x2(e * __uint_as_float(cs[k]) + __uint_as_float(mx[k]) + Dh * lo_f(xs[i]),
-                                e * __uint_as_float(cs[k + 1]) + __uint_as_float(mx[k + 1]) + Dh * hi_f(xs[i]));
-          }
-          if (col0 + 8 * g < ncol) *reinterpret_cast<uint4*>(dst + 8 * g) = y;  // Dv is a multiple of eight
-        }
-      }
+      tc_fence_before_sync();
+      mbar_arrive(ready + 2);
     }
     const float dl = F[4 * TL];
     decay *= dl;
@@ -321,24 +360,30 @@ __global__ void __launch_bounds__(TT, 1) ssd_tc_kernel(const SsdTcParams sp) {
     for (int i = 0; i < 32; ++i) S[i] = dl * S[i] + __uint_as_float(kv[i]);
     if constexpr (OUT) put(L::SH, L::SL, S);
   }
+  if (OUT && first < last) outputs(last - 1);
   if (!OUT || seg == sp.nseg - 1) {
     float* dst = OUT ? p.state + (long long)bh * plane : mine;
 #pragma unroll
-    for (int i = 0; i < 32; ++i)
-      if (row < p.Dk && col0 + i < ncol) dst[(long long)row * p.Dv + c0 + col0 + i] = S[i];
+    for (int g = 0; g < 4; ++g) {
+      float f[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) f[i] = S[8 * g + i];
+      if (row < p.Dk && col0 + 8 * g < ncol) st8v(dst + (long long)row * p.Dv + c0 + col0 + 8 * g, f);
+    }
     if (!OUT && slice == 0 && tid == 0) sp.seg_state[(long long)sp.nseg * p.B * p.H * plane + (long long)seg * p.B * p.H + bh] = decay;
+  }
   }
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
-  if (warp == 0) tmem_dealloc(tmem, 512);
+  if (warp == 8) tmem_dealloc(tmem, 512);
 }
 
 }  // namespace
 
 bool ssd_tc_supported(const RecurrentArgs& a) {
   return !a.f32 && a.kind == RK_MAMBA2 && a.T >= 64 && a.Dk > 64 && a.Dk <= 128 && a.Dk % 8 == 0 && a.Dv % 8 == 0 && vec8_ok(a.q, a.ldq, false) &&
-         vec8_ok(a.k, a.ldk, false) && vec8_ok(a.v, a.ldv, false) && vec8_ok(a.out, a.ldo, false);
+         vec8_ok(a.k, a.ldk, false) && vec8_ok(a.v, a.ldv, false) && vec8_ok(a.out, a.ldo, false) && vec8_ok(a.state, 4, true);
 }
 
 // About one block per SM; at least two chunks per segment.
@@ -374,14 +419,14 @@ void launch_ssd_tc(const RecurrentArgs& a, void* scratch, int* status, cudaStrea
   if (sp.nseg > 1) {
     constexpr int smem = SsdTcSmem<false>::END + 1024;
     cudaFuncSetAttribute(ssd_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    ssd_tc_kernel<false><<<dim3(blocks, sp.nseg - 1), TT, smem, s>>>(sp);
+    ssd_tc_kernel<false><<<dim3(blocks, sp.nseg - 1), TT + 32, smem, s>>>(sp);
     check_launch("ssd_tc_states");
     launch_ssd_scan(a, sp.seg_state, sp.nseg, s);
   }
   constexpr int smem = SsdTcSmem<true>::END + 1024;
   static_assert(smem <= 227 * 1024, "shared memory of a block");
   cudaFuncSetAttribute(ssd_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  ssd_tc_kernel<true><<<dim3(blocks, sp.nseg), TT, smem, s>>>(sp);
+  ssd_tc_kernel<true><<<dim3(blocks, sp.nseg), TT + 32, smem, s>>>(sp);
   check_launch("ssd_tc_out");
 }
 
