@@ -741,11 +741,20 @@ __global__ void ssd_scan_kernel(const RecurrentArgs p, float* seg_state, int nse
   if (i >= plane) return;
   float run = p.state[bh * plane + i];
   float* at = seg_state + bh * plane + i;
-#pragma unroll 4
-  for (int g = 0; g < nseg - 1; ++g) {
-    const float own = at[g * heads * plane];
-    at[g * heads * plane] = run;
-    run = dec[g * heads] * run + own;
+  for (int g0 = 0; g0 < nseg - 1; g0 += 8) {  // loads first: they do not wait for one another
+    float own[8], d[8];
+#pragma unroll
+    for (int g = 0; g < 8; ++g)
+      if (g0 + g < nseg - 1) {
+        own[g] = at[(g0 + g) * heads * plane];
+        d[g] = dec[(g0 + g) * heads];
+      }
+#pragma unroll
+    for (int g = 0; g < 8; ++g)
+      if (g0 + g < nseg - 1) {
+        at[(g0 + g) * heads * plane] = run;
+        run = d[g] * run + own[g];
+      }
   }
   at[(nseg - 1) * heads * plane] = run;
 }

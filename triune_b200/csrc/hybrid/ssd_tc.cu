@@ -79,9 +79,9 @@ __device__ __forceinline__ void stage_tile(uint8_t* dst, const __nv_bfloat16* sr
 
 template <bool OUT>
 struct SsdTcSmem {  // after alignment to 1024 bytes
-  static constexpr int NS = OUT ? 2 : 3;  // chunks of keys, values and factors in shared memory
-  static constexpr int K = 0, X = K + NS * 2 * TBOX, WH = X + NS * TBOX, WL = WH + TBOX, F = WL + TBOX;
-  static constexpr int C = (F + NS * TF * TL * 4 + 1023) / 1024 * 1024, SH = C + (OUT ? 2 * TBOX : 0), SL = SH + (OUT ? TBOX : 0), END = SL + (OUT ? TBOX : 0);
+  static constexpr int NK = OUT ? 2 : 3, NX = 3;  // chunks of keys, and of values and factors, in shared memory
+  static constexpr int K = 0, X = K + NK * 2 * TBOX, WH = X + NX * TBOX, WL = WH + TBOX, F = WL + TBOX;
+  static constexpr int C = (F + NX * TF * TL * 4 + 1023) / 1024 * 1024, SH = C + (OUT ? 2 * TBOX : 0), SL = SH + (OUT ? TBOX : 0), END = SL + (OUT ? TBOX : 0);
   static_assert(F % 1024 == 0 && C % 1024 == 0, "tiles start on 1024 bytes");
 };
 
@@ -144,8 +144,8 @@ __global__ void __launch_bounds__(TT + 32, 1) ssd_tc_kernel(const SsdTcParams sp
     }
   };
   auto stage_kx = [&](int c) {
-    const int u = (c - first) % L::NS;
-    stage_tile(smem + L::K + u * 2 * TBOX, K, p.ldk, c * TL, p.T, p.Dk, 2, tid);
+    const int u = (c - first) % L::NX;
+    stage_tile(smem + L::K + (c - first) % L::NK * 2 * TBOX, K, p.ldk, c * TL, p.T, p.Dk, 2, tid);
     stage_tile(smem + L::X + u * TBOX, V, p.ldv, c * TL, p.T, ncol, 1, tid);
     if (tid < TF * TL / 4)
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem + L::F + u * TF * TL * 4 + tid * 16)),
@@ -185,7 +185,7 @@ __global__ void __launch_bounds__(TT + 32, 1) ssd_tc_kernel(const SsdTcParams sp
     if (lane == 0) {
       constexpr uint32_t id_g = make_idesc(128, 128, 1, 1, 0, 0), id_s = make_idesc(128, 64, 1, 1, 0, 1), id_u = make_idesc(128, 64, 1, 1, 1, 1);
       for (int c = first; c < last; ++c) {
-        const uint32_t u = (c - first) & 1, slot = (c - first) % L::NS, ka = base + L::K + slot * 2 * TBOX, xa = base + L::X + slot * TBOX, ca = base + L::C;
+        const uint32_t u = (c - first) & 1, ka = base + L::K + (c - first) % L::NK * 2 * TBOX, xa = base + L::X + (c - first) % L::NX * TBOX, ca = base + L::C;
         wait_on(ready + 0, u);
         tc_fence_after_sync();
         if constexpr (OUT) {
@@ -232,9 +232,9 @@ __global__ void __launch_bounds__(TT + 32, 1) ssd_tc_kernel(const SsdTcParams sp
 
   // outputs of chunk c: e^{b_i} (C S) + M x + D x
   auto outputs = [&](int c) {
-    const int u = (c - first) & 1, t = c * TL + row;
-    const uint8_t* X = smem + L::X + u * TBOX;
-    const float e = exp_neg(reinterpret_cast<const float*>(smem + L::F)[u * TF * TL + row]);
+    const int u = (c - first) & 1, slot = (c - first) % L::NX, t = c * TL + row;
+    const uint8_t* X = smem + L::X + slot * TBOX;
+    const float e = exp_neg(reinterpret_cast<const float*>(smem + L::F)[slot * TF * TL + row]);
     wait_bar(2, u);
     uint32_t cs[32], mx[32];
     tmem_ld_32x32b_x32(lanes + (u == 0 ? 128 : 448) + col0, cs);
@@ -264,7 +264,7 @@ __global__ void __launch_bounds__(TT + 32, 1) ssd_tc_kernel(const SsdTcParams sp
   // the update is issued as soon as the weighted values are there and runs under the decay of the scores; the state is
   // updated and published under the last product.
   for (int c = first; c < last; ++c) {
-    const int slot = (c - first) % L::NS;
+    const int slot = (c - first) % L::NX;
     const uint32_t par = (c - first) & 1;
     const float* F = reinterpret_cast<const float*>(smem + L::F) + slot * TF * TL;
     const uint8_t* X = smem + L::X + slot * TBOX;
@@ -275,6 +275,7 @@ __global__ void __launch_bounds__(TT + 32, 1) ssd_tc_kernel(const SsdTcParams sp
     rows_sync();  // this chunk's tiles and the state before it
     mbar_arrive(ready + 0);
     const bool more = c + 1 < last;
+    if (OUT && more) stage_kx(c + 1);  // its keys' slot is free: every update so far has been waited for
     if (OUT && c > first) outputs(c - 1);
     {
       const float w = F[2 * TL + row];
@@ -291,9 +292,7 @@ __global__ void __launch_bounds__(TT + 32, 1) ssd_tc_kernel(const SsdTcParams sp
     tc_fence_before_sync();
     rows_sync();  // every thread has read what it needs of chunk c - 1
     mbar_arrive(ready + 1);
-    if constexpr (OUT) {
-      if (more) stage_kx(c + 1);
-    } else {  // one commit per chunk, empty at the end
+    if constexpr (!OUT) {  // one commit per chunk, empty at the end
       if (c + 2 < last) stage_kx(c + 2);
       cp_commit();
     }
