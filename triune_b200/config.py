@@ -131,10 +131,13 @@ class ModelConfig:
     use_fp8: bool = False
     use_fp4: bool = False
     tie_embeddings: bool = True
-    # family "hybrid": one entry per layer, {"mixers": [{"kind": "attention" | "mamba2" | "delta", sizes ...}, ...],
-    # "ff": hidden width or None, "act": its activation}; see models/hybrid_mixers.py for the sizes of each kind
+    # family "hybrid": one entry per layer, {"mixers": [{"kind": "attention" | "latent" | "mamba2" | "delta" | "retention",
+    # sizes ...}, ...], "ff": hidden width or None, "act": its activation ("clamped": with "limit" and "alpha"),
+    # "ff_bias": biases on its projections}; see models/hybrid_mixers.py for the sizes of each kind
     layers: Optional[List[Dict[str, Any]]] = None
     norm: str = "rms"  # family "hybrid": "rms" | "layer" (with a weight, without a bias)
+    post_norm: bool = False  # family "hybrid": a norm behind every sublayer too, before its sum with the residual
+    token_side: int = 0  # family "hybrid": width of the token table that every layer reads its own part of (0: none)
     norm_eps: float = EPS
 
     def resolved_expert_hidden(self) -> int:
@@ -153,26 +156,47 @@ class ModelConfig:
         for i, layer in enumerate(self.layers):
             if not layer.get("mixers"):
                 raise ValueError(f"layer {i} has no mixer")
-            if layer.get("act", "silu") not in ("relu", "silu", "gelu_tanh"):
-                raise ValueError(f"layer {i}: unknown activation {layer['act']!r}")
+            act = layer.get("act", "silu")
+            if act not in ("relu", "silu", "gelu_tanh", "clamped"):
+                raise ValueError(f"layer {i}: unknown activation {act!r}")
+            if act == "clamped" and layer.get("ff") and not (layer.get("limit", 0) > 0 and layer.get("alpha", 0) > 0):
+                raise ValueError(f"layer {i}: the clamped activation needs a positive limit and alpha")
             for m in layer["mixers"]:
-                kind = m.get("kind")
-                need = {"attention": ("heads", "kv_heads", "dim", "vdim", "scale"), "delta": ("heads", "kv_heads", "dim", "vdim", "conv"),
-                        "mamba2": ("heads", "vdim", "state", "groups", "conv", "norm_groups")}.get(kind)
-                if need is None:
-                    raise ValueError(f"layer {i}: unknown mixer {kind!r}")
-                for k in need:
-                    if not m.get(k, 0) > 0:
-                        raise ValueError(f"layer {i}: {kind} needs a positive {k!r}")
-                groups = m["groups"] if kind == "mamba2" else m["kv_heads"]
-                if m["heads"] % groups:
-                    raise ValueError(f"layer {i}: heads ({m['heads']}) must be a multiple of {groups}")
-                if kind == "mamba2" and (m["heads"] * m["vdim"]) % m["norm_groups"]:
-                    raise ValueError(f"layer {i}: norm_groups must divide heads * vdim")
-                rot = m.get("rot_dims", 0)
-                if kind == "attention" and (rot % 2 or not 0 <= rot <= m["dim"]):
-                    raise ValueError(f"layer {i}: rot_dims must be even and at most dim")
+                self._validate_mixer(i, m)
         return self
+
+    _MIXER_SIZES = {"attention": ("heads", "kv_heads", "dim", "vdim", "scale"), "delta": ("heads", "kv_heads", "dim", "vdim", "conv"),
+                    "mamba2": ("heads", "vdim", "state", "groups", "conv", "norm_groups"),
+                    "latent": ("heads", "dim", "rot_dims", "vdim", "kv_rank", "scale"), "retention": ("heads", "dim", "vdim")}
+
+    def _validate_mixer(self, i: int, m: Dict[str, Any]) -> None:
+        kind = m.get("kind")
+        if kind not in self._MIXER_SIZES:
+            raise ValueError(f"layer {i}: unknown mixer {kind!r}")
+        for k in self._MIXER_SIZES[kind]:
+            if not m.get(k, 0) > 0:
+                raise ValueError(f"layer {i}: {kind} needs a positive {k!r}")
+        groups = {"mamba2": m.get("groups"), "latent": 1, "retention": 1}.get(kind, m.get("kv_heads"))
+        if m["heads"] % groups:
+            raise ValueError(f"layer {i}: heads ({m['heads']}) must be a multiple of {groups}")
+        if kind == "mamba2" and (m["heads"] * m["vdim"]) % m["norm_groups"]:
+            raise ValueError(f"layer {i}: norm_groups must divide heads * vdim")
+        rot = m.get("rot_dims", 0)
+        if kind in ("attention", "retention") and (rot % 2 or not 0 <= rot <= m["dim"]):
+            raise ValueError(f"layer {i}: rot_dims must be even and at most dim")
+        if kind == "retention" and (len(m.get("decay", ())) != m["heads"] or not all(0 < d <= 1 for d in m["decay"])):
+            raise ValueError(f"layer {i}: retention needs a decay in (0, 1] for every head")
+        if kind == "latent":
+            if rot % 2:
+                raise ValueError(f"layer {i}: rot_dims must be even")
+            src = m.get("kv_from")
+            if src is not None:
+                if not 0 <= src < i:
+                    raise ValueError(f"layer {i}: kv_from must name an earlier layer")
+                o = self.layers[src]["mixers"][0]
+                same = ("kv_rank", "rot_dims", "rot_base", "rot_scaling")
+                if o["kind"] != "latent" or o.get("kv_from") is not None or any(o.get(k) != m.get(k) for k in same):
+                    raise ValueError(f"layer {i}: layer {src} has no latent rows of its own that fit")
 
     def validate(self) -> "ModelConfig":
         if self.family == "hybrid":
@@ -225,12 +249,22 @@ class ModelConfig:
         attn = 4 * d * hd + hd * d
         norms = 2 * d
         if self.family == "hybrid":
-            total = 2 * v * d + d
+            total, side, around = 2 * v * d + d, self.token_side, 2 * d if self.post_norm else d
             for layer in self.layers:
-                total += d + (3 * d * layer["ff"] + d if layer.get("ff") else 0)
+                total += around
+                if layer.get("ff"):
+                    total += 3 * d * layer["ff"] + around + (2 * layer["ff"] + d if layer.get("ff_bias") else 0)
+                if side:
+                    total += v * side + 2 * d * side + d
                 for m in layer["mixers"]:
                     h, e = m["heads"], m["vdim"]
-                    if m["kind"] == "attention":
+                    if m["kind"] == "latent":
+                        r, k = m["rot_dims"], m["kv_rank"]
+                        total += d * h * (m["dim"] + r + e) + k * h * (m["dim"] + e) + (h if m.get("sink", True) else 0)
+                        total += (d * h if m.get("gate", True) else 0) + (d * (k + r) + k if m.get("kv_from") is None else 0)
+                    elif m["kind"] == "retention":
+                        total += d * h * (2 * m["dim"] + 3 * e)
+                    elif m["kind"] == "attention":
                         total += d * (h * m["dim"] + m["kv_heads"] * (m["dim"] + e) + h * e) + 2 * m["dim"] + h
                     elif m["kind"] == "mamba2":
                         u = h * e + 2 * m["groups"] * m["state"]

@@ -1,8 +1,9 @@
 """Model families: multi-exit MoE ``TriuneTransformer``, dense ``UniversalTransformer`` and ``HybridTransformer`` with
-layers that differ (``Famalorn``)."""
+layers that differ (``Bubitar``, ``Famalorn``)."""
 
 from .attention import HybridAttention, SoftmaxAttention, VectorisedGLA
 from .block import DenseFFN, TransformerBlock
+from .bubitar import Bubitar
 from .famalorn import Famalorn
 from .hybrid import HybridTransformer
 from .moe import MoE_FFN, RoutingResult
@@ -12,6 +13,6 @@ from .router import GumbelSoftmaxRouter
 from .transformer import TriuneTransformer
 
 __all__ = [
-    "Famalorn", "HybridTransformer", "HybridAttention", "SoftmaxAttention", "VectorisedGLA", "DenseFFN", "TransformerBlock", "MoE_FFN",
+    "Bubitar", "Famalorn", "HybridTransformer", "HybridAttention", "SoftmaxAttention", "VectorisedGLA", "DenseFFN", "TransformerBlock", "MoE_FFN",
     "RoutingResult", "RMSNorm", "RotaryEmbedding", "GumbelSoftmaxRouter", "TriuneTransformer",
 ]

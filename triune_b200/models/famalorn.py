@@ -6,14 +6,12 @@ A Famalorn is a :class:`HybridTransformer` with layer norms and ReLU-gated feed-
 
 from __future__ import annotations
 
-import json
-from pathlib import Path
-from typing import Any, Dict, Iterator, List, Optional, Tuple
+from typing import Any, Dict, Iterator, Tuple
 
 import torch
 
 from ..config import ModelConfig
-from ..export.safetensors_io import load_file, save_file
+from .folder import FolderModel, Stacked
 from .hybrid import HybridTransformer
 from .hybrid_mixers import AttentionCore, Core, DeltaCore
 from .zoo import register_model
@@ -90,27 +88,9 @@ def _core_views(core: Core, w_in: torch.Tensor, col0: int, w_out: torch.Tensor, 
     yield p + "D", core.D
     # one stored matrix [z | x | B | C | dt] and one stored convolution over [x | B | C]
     parts = [_rows(w_in, col0, core, "z")] + [w_in[u0 + ca[n] : u0 + ca[n] + cw[n]] for n in ("v", "k", "q")]
-    yield p + "in", _Stacked(parts + [_rows(w_in, col0, core, "a")])
-    yield p + "conv", _Stacked([core.conv_w[ca[n] : ca[n] + cw[n]] for n in ("v", "k", "q")])
-    yield p + "conv.b", _Stacked([core.conv_b[ca[n] : ca[n] + cw[n]] for n in ("v", "k", "q")])
-
-
-class _Stacked:
-    """Several row blocks of the model that are one tensor in the file."""
-
-    def __init__(self, parts: List[torch.Tensor]):
-        self.parts = parts
-
-    @property
-    def shape(self):
-        return torch.Size([sum(t.shape[0] for t in self.parts), *self.parts[0].shape[1:]])
-
-    def copy_(self, src: torch.Tensor) -> None:
-        for t, s in zip(self.parts, src.split([t.shape[0] for t in self.parts])):
-            t.copy_(s)
-
-    def detach(self) -> torch.Tensor:
-        return torch.cat([t.detach() for t in self.parts])
+    yield p + "in", Stacked(parts + [_rows(w_in, col0, core, "a")])
+    yield p + "conv", Stacked([core.conv_w[ca[n] : ca[n] + cw[n]] for n in ("v", "k", "q")])
+    yield p + "conv.b", Stacked([core.conv_b[ca[n] : ca[n] + cw[n]] for n in ("v", "k", "q")])
 
 
 def named_views(model: HybridTransformer) -> Dict[str, Any]:
@@ -129,41 +109,8 @@ def named_views(model: HybridTransformer) -> Dict[str, Any]:
 
 
 @register_model("famalorn")
-class Famalorn(HybridTransformer):
+class Famalorn(FolderModel):
     """``Famalorn(config=<dict or path>)`` builds one with zero weights; ``from_pretrained(folder)`` loads one."""
 
-    def __init__(self, config=None, cfg: Optional[ModelConfig] = None):
-        if cfg is None:
-            raw = config if isinstance(config, dict) else json.loads(Path(config).read_text(encoding="utf-8"))
-            cfg = read_config(raw)
-            super().__init__(cfg)
-            self.raw_config = raw
-        else:
-            super().__init__(cfg)
-
-    @classmethod
-    def from_pretrained(cls, folder, device="cpu", dtype: Optional[torch.dtype] = None) -> "Famalorn":
-        from ..utils import place_model
-
-        folder = Path(folder)
-        model = cls(config=folder / "config.json")
-        model.load_named(load_file(str(folder / "model.safetensors")))
-        return place_model(model, device, dtype).eval()
-
-    @torch.no_grad()
-    def load_named(self, tensors: Dict[str, torch.Tensor]) -> None:
-        views = named_views(self)
-        missing, extra = sorted(set(views) - set(tensors)), sorted(set(tensors) - set(views))
-        if missing or extra:
-            raise ValueError(f"tensors do not fit the configuration: missing {missing[:4]}, unknown {extra[:4]}")
-        for n, v in views.items():
-            t = tensors[n]
-            if tuple(t.shape) != tuple(v.shape):
-                raise ValueError(f"{n}: stored {tuple(t.shape)}, the configuration implies {tuple(v.shape)}")
-            v.copy_(t.to(torch.float32) if t.dtype == torch.bfloat16 else t)
-
-    def save_pretrained(self, folder, dtype: torch.dtype = torch.bfloat16) -> None:
-        folder = Path(folder)
-        folder.mkdir(parents=True, exist_ok=True)
-        (folder / "config.json").write_text(json.dumps(self.raw_config, indent=1), encoding="utf-8")
-        save_file({n: v.detach().to(dtype).cpu() for n, v in named_views(self).items()}, str(folder / "model.safetensors"))
+    read_config = staticmethod(read_config)
+    named_views = named_views

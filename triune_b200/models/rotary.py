@@ -2,12 +2,33 @@
 
 from __future__ import annotations
 
-from typing import Optional
+import math
+from typing import Any, Dict, Optional, Tuple
 
 import torch
 import torch.nn as nn
 
 from .. import ops
+
+
+def rotary_frequencies(dims: int, base: float, scaling: Optional[Dict[str, Any]] = None) -> Tuple[torch.Tensor, float]:
+    """Turns per position of the ``dims / 2`` rotated pairs (fp64 radians) and the factor of sine and cosine.
+
+    ``scaling`` is YaRN's (Peng et al., "YaRN: Efficient Context Window Extension of Large Language Models"):
+    ``factor`` stretches a context of ``original`` positions; pairs that turn more than ``fast`` times within it keep their
+    frequency, pairs below ``slow`` turns are divided by ``factor``, a linear ramp lies between."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = float(base) ** (-2.0 * i / max(1, dims))
+    if not scaling or not dims:
+        return f, 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+
+    def pair(turns: float) -> float:  # the (fractional) pair that turns so many times within the original context
+        return dims * math.log(original / (2 * math.pi * turns)) / (2 * math.log(base))
+
+    lo, hi = max(math.floor(pair(float(scaling["fast"]))), 0), min(math.ceil(pair(float(scaling["slow"]))), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 1e-3)).clamp(0, 1)
+    return f / factor * ramp + f * (1 - ramp), 0.1 * math.log(factor) + 1.0
 
 
 class RotaryEmbedding(nn.Module):
