@@ -53,4 +53,22 @@ inline CUtensorMap make_tmap_3d(const void* base, CUtensorMapDataType dt, int el
   return m;
 }
 
+// 4-D tiled bf16 map over a [d3][d2][d1][d0] array (d0 contiguous, 128-byte swizzle) with boxes of 64 x b1 x 1 x 1. Strides
+// in BYTES; elements outside read as zero.
+inline CUtensorMap make_tmap_4d_bf16(const void* base, const uint64_t (&d)[4], const uint64_t (&stride_bytes)[3], uint32_t b1) {
+  if ((reinterpret_cast<uintptr_t>(base) & 15) != 0) throw std::runtime_error("TMA base must be 16-byte aligned");
+  cuuint64_t dims[4] = {d[0], d[1], d[2], d[3]}, strides[3];
+  for (int i = 0; i < 3; ++i) {
+    if ((stride_bytes[i] & 15) != 0) throw std::runtime_error("TMA strides must be multiples of 16 bytes");
+    strides[i] = stride_bytes[i] == 0 ? 16 : stride_bytes[i];  // of a dimension of one: never stepped
+  }
+  cuuint32_t box[4] = {64, b1, 1, 1}, estr[4] = {1, 1, 1, 1};
+  CUtensorMap m;
+  CUresult r = get_encode_fn()(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr,
+                               CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                               CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS) throw std::runtime_error("cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
+  return m;
+}
+
 }  // namespace tb

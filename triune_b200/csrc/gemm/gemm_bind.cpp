@@ -118,8 +118,10 @@ void tc_gemm(const Tensor& a, const Tensor& b, Tensor& c, bool a_mn_major, bool 
 }
 
 // SwiGLU over the fused gate/up weight inside the GEMM: h [M, H] = silu(x Wg^T) * (x Wu^T) with w13 = [Wg ; Wu]
-// ([2H, K]); gu (optional, [M, 2H]) receives both pre-activations for the backward pass. act: 0 silu, 1 relu (forward only).
-void tc_gemm_swiglu(const Tensor& x, const Tensor& w13, Tensor& h, const c10::optional<Tensor>& gu, int64_t act) {
+// ([2H, K]); gu (optional, [M, 2H]) receives both pre-activations for the backward pass. act: 0 silu, 1 relu, 2 clamped
+// (see GemmArgs::glu_act); bias: fp32 [2H] or none (forward only, as the last two activations are).
+void tc_gemm_swiglu(const Tensor& x, const Tensor& w13, Tensor& h, const c10::optional<Tensor>& gu, int64_t act,
+                    const c10::optional<Tensor>& bias, double limit, double alpha) {
   check_bf16_cuda(x, "x");
   check_bf16_cuda(w13, "w13");
   check_bf16_cuda(h, "h");
@@ -133,8 +135,16 @@ void tc_gemm_swiglu(const Tensor& x, const Tensor& w13, Tensor& h, const c10::op
   g.M = (int)M; g.N = (int)H; g.K = (int)K;
   g.lda = x.stride(0); g.ldb = w13.stride(0); g.ldc = h.stride(0);
   g.batch = 1; g.mode = tb::GEMM_DENSE; g.flags = tb::GF_SWIGLU; g.alpha = 1.0f; g.n_split = (int)H;
-  TORCH_CHECK(act == 0 || act == 1, "tc_gemm_swiglu: activation");
+  TORCH_CHECK(act >= 0 && act <= 2 && (act != 2 || limit > 0), "tc_gemm_swiglu: activation");
   g.glu_act = (int)act;
+  g.glu_limit = (float)limit;
+  g.glu_alpha = (float)alpha;
+  if (bias.has_value() && bias->defined()) {
+    TORCH_CHECK(bias->is_cuda() && bias->scalar_type() == at::kFloat && bias->is_contiguous() && bias->numel() == 2 * H &&
+                    (reinterpret_cast<uintptr_t>(bias->data_ptr()) & 15) == 0,
+                "tc_gemm_swiglu: bias [2H] fp32");
+    g.glu_bias = bias->data_ptr<float>();
+  }
   if (gu.has_value() && gu->defined()) {
     check_bf16_cuda(*gu, "gu");
     TORCH_CHECK(gu->dim() == 2 && gu->is_contiguous() && gu->size(0) == M && gu->size(1) == 2 * H, "gu must be [M, 2H] contiguous");
@@ -179,6 +189,7 @@ void register_gemm(pybind11::module& m) {
     tb::tc_gemm_set_debug_buffer(on ? (long long*)t->data_ptr<int64_t>() : nullptr);
   });
   m.def("tc_gemm_pair_launches", []() { return (int64_t)tb::tc_gemm_pair_launch_count(); });
-  m.def("tc_gemm_swiglu", &tc_gemm_swiglu, pybind11::arg("x"), pybind11::arg("w13"), pybind11::arg("h"), pybind11::arg("gu"), pybind11::arg("act") = 0);
+  m.def("tc_gemm_swiglu", &tc_gemm_swiglu, pybind11::arg("x"), pybind11::arg("w13"), pybind11::arg("h"), pybind11::arg("gu"), pybind11::arg("act") = 0,
+        pybind11::arg("bias") = pybind11::none(), pybind11::arg("limit") = 0.0, pybind11::arg("alpha") = 0.0);
   m.def("tc_gemm_dswiglu", &tc_gemm_dswiglu);
 }

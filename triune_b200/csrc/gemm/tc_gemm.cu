@@ -359,6 +359,9 @@ void launch_tc_gemm(const GemmArgs& a, cudaStream_t stream) {
   kp.n_split = a.n_split;
   kp.beta = a.beta;
   kp.glu_act = a.glu_act;
+  kp.glu_limit = a.glu_limit;
+  kp.glu_alpha = a.glu_alpha;
+  kp.glu_bias = a.glu_bias;
   kp.ldc = a.ldc; kp.strideC = a.strideC;
   kp.a_batched = a.strideA != 0; kp.b_batched = a.strideB != 0;
   kp.alpha = a.alpha;

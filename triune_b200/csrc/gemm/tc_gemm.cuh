@@ -53,7 +53,9 @@ struct GemmArgs {
   int* status;                  // optional device status word (see KernelStatus)
   int n_split;                  // GF_SWIGLU / GF_DSWIGLU: FFN hidden width (N); 0 otherwise
   float beta;                   // GF_ADDAUX: weight of aux_in
-  int glu_act;                  // GF_SWIGLU: activation of the gate, 0 silu, 1 relu
+  int glu_act;                  // GF_SWIGLU: activation of the gate, 0 silu, 1 relu, 2 clamped: g sigmoid(alpha g) (u + 1)
+  float glu_limit, glu_alpha;   //   with g at most `limit` and u within +- `limit`
+  const float* glu_bias;        // GF_SWIGLU: [2 N], of the gate, then of the up rows; or null
 };
 
 // Launches on `stream`. Throws std::runtime_error on invalid arguments.

@@ -49,7 +49,9 @@ struct KParams {
   int iters_per_split;  // K iterations (of 64) handled by one split
   int n_split;          // SwiGLU epilogues: column offset of the "up" half (= FFN hidden width)
   float beta;           // EPI_ADDAUX: weight of the added rows
-  int glu_act;          // EPI_SWIGLU: activation of the gate, 0 silu, 1 relu
+  int glu_act;          // EPI_SWIGLU: activation of the gate, 0 silu, 1 relu, 2 clamped
+  float glu_limit, glu_alpha;
+  const float* glu_bias;  // EPI_SWIGLU: [2 n_split] or null
 };
 
 struct Tile {
@@ -417,11 +419,34 @@ __device__ __forceinline__ void epilogue_tile_swiglu(const KParams& p, const Til
 #pragma unroll
       for (int i = 0; i < 32; ++i) rg[i] = ru[i] = 0u;
     }
+    if (p.glu_bias != nullptr) {  // the same for every row: broadcast loads
+      const float4 *bg = reinterpret_cast<const float4*>(p.glu_bias + n0 + c), *bu = reinterpret_cast<const float4*>(p.glu_bias + p.n_split + n0 + c);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        const float4 x = __ldg(bg + i), y = __ldg(bu + i);
+        rg[4 * i] = __float_as_uint(__uint_as_float(rg[4 * i]) + x.x);
+        rg[4 * i + 1] = __float_as_uint(__uint_as_float(rg[4 * i + 1]) + x.y);
+        rg[4 * i + 2] = __float_as_uint(__uint_as_float(rg[4 * i + 2]) + x.z);
+        rg[4 * i + 3] = __float_as_uint(__uint_as_float(rg[4 * i + 3]) + x.w);
+        ru[4 * i] = __float_as_uint(__uint_as_float(ru[4 * i]) + y.x);
+        ru[4 * i + 1] = __float_as_uint(__uint_as_float(ru[4 * i + 1]) + y.y);
+        ru[4 * i + 2] = __float_as_uint(__uint_as_float(ru[4 * i + 2]) + y.z);
+        ru[4 * i + 3] = __float_as_uint(__uint_as_float(ru[4 * i + 3]) + y.w);
+      }
+    }
     uint32_t q[16];
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
-      const float g0 = __uint_as_float(rg[2 * i]), g1 = __uint_as_float(rg[2 * i + 1]);
-      const float u0 = __uint_as_float(ru[2 * i]), u1 = __uint_as_float(ru[2 * i + 1]);
+      float g0 = __uint_as_float(rg[2 * i]), g1 = __uint_as_float(rg[2 * i + 1]);
+      float u0 = __uint_as_float(ru[2 * i]), u1 = __uint_as_float(ru[2 * i + 1]);
+      if (p.glu_act == 2) {
+        g0 = fminf(g0, p.glu_limit);
+        g1 = fminf(g1, p.glu_limit);
+        u0 = fminf(fmaxf(u0, -p.glu_limit), p.glu_limit) + 1.f;
+        u1 = fminf(fmaxf(u1, -p.glu_limit), p.glu_limit) + 1.f;
+        q[i] = pack_bf16x2(g0 * sigmoid_f(p.glu_alpha * g0) * u0, g1 * sigmoid_f(p.glu_alpha * g1) * u1);
+        continue;
+      }
       q[i] = p.glu_act == 0 ? pack_bf16x2(g0 * sigmoid_f(g0) * u0, g1 * sigmoid_f(g1) * u1)
                             : pack_bf16x2(fmaxf(g0, 0.f) * u0, fmaxf(g1, 0.f) * u1);
     }

@@ -411,6 +411,9 @@ bool launch_tc_gemm_pair(const GemmArgs& a, cudaStream_t stream) {
   kp.n_split = a.n_split;
   kp.beta = 0.f;
   kp.glu_act = a.glu_act;
+  kp.glu_limit = a.glu_limit;
+  kp.glu_alpha = a.glu_alpha;
+  kp.glu_bias = a.glu_bias;
   kp.ldc = a.ldc; kp.strideC = a.strideC;
   kp.a_batched = 0; kp.b_batched = 0;
   kp.alpha = a.alpha;

@@ -151,19 +151,24 @@ constexpr int AS_Q = 8, AS_K = 32;
 template <class T>
 __global__ void attn_simple_kernel(const AttnArgs p) {
   extern __shared__ float sm[];
-  const int dp = p.D + 1;
+  const int D = p.D + p.R, dp = D + 1;
   float *sk = sm, *sv = sk + AS_K * dp, *sq = sv + AS_K * p.E;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y, b = blockIdx.z, t = blockIdx.x * AS_Q + warp, g = h / (p.H / p.G);
   const long long p0 = pos_of(p.pos);
   const bool live = t < p.T;
   const long long qpos = p0 + t;
-  const long long kend = min(p0 + min((blockIdx.x + 1) * AS_Q, p.T), (long long)p.cap);  // keys any query of the block sees
-  const T* Q = (const T*)p.q + (((long long)b * p.H + h) * p.T + t) * p.pitch_k;
-  const T *K = (const T*)p.kc + ((long long)b * p.G + g) * p.cap * p.pitch_k, *V = (const T*)p.vc + ((long long)b * p.G + g) * p.cap * p.pitch_v;
-  float* q = sq + warp * p.D;
-  if (live)
+  const long long kend = min(p0 + min((blockIdx.x + 1) * AS_Q, p.T), (long long)p.rows);  // keys any query of the block sees
+  auto at = [&](const AttnOperand& o, long long row, int head) { return (const T*)o.p + b * o.sb + row * o.sr + head * o.sh; };
+  float* q = sq + warp * D;
+  if (live) {
+    const T* Q = at(p.q, t, h);
     for (int d = lane; d < p.D; d += 32) q[d] = ldf(Q + d);
+    if (p.R > 0) {
+      const T* Q2 = at(p.q2, t, h);
+      for (int d = lane; d < p.R; d += 32) q[p.D + d] = ldf(Q2 + d);
+    }
+  }
   float m = p.sink != nullptr ? p.sink[h] : -INFINITY, l = p.sink != nullptr ? 1.f : 0.f;
   float acc[8];  // value dimensions up to 256
 #pragma unroll
@@ -171,14 +176,15 @@ __global__ void attn_simple_kernel(const AttnArgs p) {
   for (long long k0 = 0; k0 < kend; k0 += AS_K) {
     const int n = (int)min((long long)AS_K, kend - k0);
     __syncthreads();
-    for (int i = threadIdx.x; i < n * p.D; i += blockDim.x) sk[(i / p.D) * dp + i % p.D] = ldf(K + (k0 + i / p.D) * p.pitch_k + i % p.D);
-    for (int i = threadIdx.x; i < n * p.E; i += blockDim.x) sv[i] = ldf(V + (k0 + i / p.E) * p.pitch_v + i % p.E);
+    for (int i = threadIdx.x; i < n * p.D; i += blockDim.x) sk[(i / p.D) * dp + i % p.D] = ldf(at(p.k, k0 + i / p.D, g) + i % p.D);
+    for (int i = threadIdx.x; i < n * p.R; i += blockDim.x) sk[(i / p.R) * dp + p.D + i % p.R] = ldf(at(p.k2, k0 + i / p.R, 0) + i % p.R);
+    for (int i = threadIdx.x; i < n * p.E; i += blockDim.x) sv[i] = ldf(at(p.v, k0 + i / p.E, g) + i % p.E);
     __syncthreads();
     if (!live || k0 > qpos) continue;
     float s = -INFINITY;
     if (lane < n && k0 + lane <= qpos) {
       float a = 0.f;
-      for (int d = 0; d < p.D; ++d) a += q[d] * sk[lane * dp + d];
+      for (int d = 0; d < D; ++d) a += q[d] * sk[lane * dp + d];
       s = a * p.scale;
     }
     const float mn = fmaxf(m, warp_max(s));
@@ -196,7 +202,8 @@ __global__ void attn_simple_kernel(const AttnArgs p) {
   }
   if (live) {
     T* o = (T*)p.out + ((long long)b * p.T + t) * p.ldo + h * p.E;
-    const float r = p.out_scale / l;
+    float r = p.out_scale / l;
+    if (p.gate != nullptr) r *= sigmoid_f(ldf((const T*)p.gate + ((long long)b * p.T + t) * p.ldg + h));
 #pragma unroll
     for (int i = 0; i < 8; ++i)
       if (lane + 32 * i < p.E) stf(o + lane + 32 * i, acc[i] * r);
@@ -234,7 +241,7 @@ void launch_attn_prep(const AttnPrepArgs& a, cudaStream_t s) {
 void launch_attn_simple(const AttnArgs& a, cudaStream_t s) {
   if (a.B <= 0 || a.T <= 0) return;
   if (a.E > 256) throw std::runtime_error("attention: value dimensions up to 256");
-  const size_t sm = (size_t)(AS_K * (a.D + 1) + AS_K * a.E + AS_Q * a.D) * 4;
+  const size_t sm = (size_t)(AS_K * (a.D + a.R + 1) + AS_K * a.E + AS_Q * (a.D + a.R)) * 4;
   if (sm > 200 * 1024) throw std::runtime_error("attention: head dimension too large");
   dim3 grid((a.T + AS_Q - 1) / AS_Q, a.H, a.B);
   auto go = [&](auto* kern) {

@@ -10,7 +10,8 @@
 // may be issued right behind the product that reads P_w. The running maximum is lazy: the accumulator is rescaled (by
 // the softmax warps, in TMEM) only when the maximum has grown by more than 2^8, otherwise the old reference stays and
 // the weights are at most 256 times larger, which fp32 sums and bf16 weights carry without loss. The sink starts the
-// row's maximum and sum: it has no key and no value.
+// row's maximum and sum: it has no key and no value. A second part of queries and keys (the turned part of latent
+// attention, one for all heads) is a further box of the same tiles; with three boxes and wide values, values have one stage.
 // TMEM: columns 0-127 S_0, 128-255 S_1, 256-383 O_0, 384-511 O_1.
 #include "../common/ptx.cuh"
 #include "../common/tma_desc.h"
@@ -25,21 +26,30 @@ constexpr float FA_LAZY = 8.f;
 
 struct FaParams {
   const float* sink;
+  const __nv_bfloat16* gate;
+  long long ldg;
   __nv_bfloat16* out;
   long long ldo;
-  int T, H, G, D, E, cap;
+  int T, H, G, D, E, R;
   float scale2;  // scale * log2(e)
   float out_scale;
   Pos pos;
   int* status;
 };
 
-template <int DKB, int EVB>  // 64-wide boxes of the key and value head sizes
+template <int KB, int EVB>
+constexpr int fa_value_stages() {  // what 227 KB hold beside two query tiles and two key stages
+  return 4 * KB + 2 * EVB <= 14 ? 2 : 1;
+}
+
+template <int DKB, int RKB, int EVB>  // 64-wide boxes of the key (first and second part) and value head sizes
 __global__ void __launch_bounds__(FA_THREADS, 1) attn_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                                                                const __grid_constant__ CUtensorMap tmV, const FaParams p) {
+                                                                const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQ2,
+                                                                const __grid_constant__ CUtensorMap tmK2, const FaParams p) {
+  constexpr int KB = DKB + RKB, VS = fa_value_stages<KB, EVB>();
   extern __shared__ uint8_t raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~uintptr_t(1023));
-  uint8_t *sQ = smem, *sK = sQ + 2 * DKB * FA_BOX, *sV = sK + 2 * DKB * FA_BOX;
+  uint8_t *sQ = smem, *sK = sQ + 2 * KB * FA_BOX, *sV = sK + 2 * KB * FA_BOX;
   __shared__ __align__(8) uint64_t bars[13];
   uint64_t *q_full = bars, *k_full = bars + 1, *k_empty = bars + 3, *v_full = bars + 5, *v_empty = bars + 7, *s_full = bars + 9,
            *p_ready = bars + 11;
@@ -47,7 +57,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) attn_tc_kernel(const __grid_con
   __shared__ uint32_t tmem_slot;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int bh = blockIdx.x, h = bh % p.H, b = bh / p.H;
-  const int kvh = b * p.G + h / (p.H / p.G);
+  const int kvh = h / (p.H / p.G);
   const int q0 = (gridDim.y - 1 - blockIdx.y) * 2 * FA_BM;  // the longest rows start first
   const long long p0l = pos_of(p.pos);
   const int p0 = (int)p0l;
@@ -86,38 +96,50 @@ __global__ void __launch_bounds__(FA_THREADS, 1) attn_tc_kernel(const __grid_con
       prefetch_tmap(&tmK);
       prefetch_tmap(&tmV);
       const int tiles = n[1] > 0 ? 2 : 1;
-      mbar_expect_tx(q_full, tiles * DKB * FA_BOX);
-      for (int w = 0; w < tiles; ++w)
-        for (int d = 0; d < DKB; ++d) tma_load_3d(sQ + (w * DKB + d) * FA_BOX, &tmQ, q_full, d * 64, q0 + w * FA_BM, bh);
-      bool ok = true;
-      for (int j = 0; j < nt && ok; ++j) {
+      mbar_expect_tx(q_full, tiles * KB * FA_BOX);
+      for (int w = 0; w < tiles; ++w) {
+        for (int d = 0; d < DKB; ++d) tma_load_4d(sQ + (w * KB + d) * FA_BOX, &tmQ, q_full, d * 64, q0 + w * FA_BM, h, b);
+        for (int d = 0; d < RKB; ++d) tma_load_4d(sQ + (w * KB + DKB + d) * FA_BOX, &tmQ2, q_full, d * 64, q0 + w * FA_BM, h, b);
+      }
+      auto keys = [&](int j) {
         const int s = j & 1;
-        const uint32_t par = ((j >> 1) & 1) ^ 1;
-        if (j >= 2) ok = mbar_wait(k_empty + s, par);
+        if (j >= 2 && !mbar_wait(k_empty + s, ((j >> 1) & 1) ^ 1)) return false;
+        mbar_expect_tx(k_full + s, KB * FA_BOX);
+        for (int d = 0; d < DKB; ++d) tma_load_4d(sK + (s * KB + d) * FA_BOX, &tmK, k_full + s, d * 64, j * FA_BN, kvh, b);
+        for (int d = 0; d < RKB; ++d) tma_load_4d(sK + (s * KB + DKB + d) * FA_BOX, &tmK2, k_full + s, d * 64, j * FA_BN, 0, b);
+        return true;
+      };
+      bool ok = keys(0);
+      for (int j = 0; j < nt && ok; ++j) {
+        if (j + 1 < nt) ok = keys(j + 1);  // ahead of these values: the scores of the next tile are issued before their use ends
         if (!ok) break;
-        mbar_expect_tx(k_full + s, DKB * FA_BOX);
-        for (int d = 0; d < DKB; ++d) tma_load_3d(sK + (s * DKB + d) * FA_BOX, &tmK, k_full + s, d * 64, j * FA_BN, kvh);
-        if (j >= 2) ok = mbar_wait(v_empty + s, par);
+        const int s = j % VS;
+        if (j >= VS) ok = mbar_wait(v_empty + s, ((j / VS) & 1) ^ 1);
         if (!ok) break;
         mbar_expect_tx(v_full + s, EVB * FA_BOX);
-        for (int d = 0; d < EVB; ++d) tma_load_3d(sV + (s * EVB + d) * FA_BOX, &tmV, v_full + s, d * 64, j * FA_BN, kvh);
+        for (int d = 0; d < EVB; ++d) tma_load_4d(sV + (s * EVB + d) * FA_BOX, &tmV, v_full + s, d * 64, j * FA_BN, kvh, b);
       }
       if (!ok && p.status) *p.status = ST_TIMEOUT_EMPTY;
     }
   } else if (warp == 1) {
     if (lane == 0) {
       const uint32_t id_s = make_idesc(128, 128, 1, 1, 0, 0), id_o = make_idesc(128, (p.E + 15) / 16 * 16, 1, 1, 0, 1);
-      const int ks = (p.D + 15) / 16;
+      const int ks = (p.D + 15) / 16, rs = (p.R + 15) / 16;
       auto scores = [&](int w, int j) {
-        const uint32_t qa = smem_u32(sQ + w * DKB * FA_BOX), ka = smem_u32(sK + (j & 1) * DKB * FA_BOX);
+        const uint32_t qa = smem_u32(sQ + w * KB * FA_BOX), ka = smem_u32(sK + (j & 1) * KB * FA_BOX);
         for (int k = 0; k < ks; ++k) {
           const uint32_t off = (k >> 2) * FA_BOX + (k & 3) * 32;
           umma_bf16(tmem + w * 128, make_smem_desc(qa + off, 16, 1024), make_smem_desc(ka + off, 16, 1024), id_s, k > 0);
         }
+        if constexpr (RKB > 0)
+          for (int k = 0; k < rs; ++k) {
+            const uint32_t off = (DKB + (k >> 2)) * FA_BOX + (k & 3) * 32;
+            umma_bf16(tmem + w * 128, make_smem_desc(qa + off, 16, 1024), make_smem_desc(ka + off, 16, 1024), id_s, 1);
+          }
         umma_commit(s_full + w);
       };
       auto values = [&](int w, int j) {
-        const uint32_t va = smem_u32(sV + (j & 1) * EVB * FA_BOX);
+        const uint32_t va = smem_u32(sV + (j % VS) * EVB * FA_BOX);
 #pragma unroll
         for (int k = 0; k < FA_BN / 16; ++k)
           umma_bf16_ts(tmem + 256 + w * 128, tmem + w * 128 + k * 8, make_smem_desc(va + k * 2048, FA_BOX, 1024), id_o, j > 0 || k > 0);
@@ -129,7 +151,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) attn_tc_kernel(const __grid_con
           if (n[w] > 0) scores(w, 0);
         umma_commit(k_empty);
         for (int j = 0; j < nt && ok; ++j) {
-          ok = mbar_wait(v_full + (j & 1), (j >> 1) & 1);
+          ok = mbar_wait(v_full + j % VS, (j / VS) & 1);
           if (ok && j + 1 < nt) ok = mbar_wait(k_full + ((j + 1) & 1), ((j + 1) >> 1) & 1);
           for (int w = 0; w < 2 && ok; ++w) {
             if (j >= n[w]) continue;
@@ -141,7 +163,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1) attn_tc_kernel(const __grid_con
             else scores(w, j + 1);
           }
           if (!ok) break;
-          umma_commit(v_empty + (j & 1));
+          umma_commit(v_empty + j % VS);
           if (j + 1 < nt) umma_commit(k_empty + ((j + 1) & 1));
         }
       }
@@ -255,7 +277,8 @@ __global__ void __launch_bounds__(FA_THREADS, 1) attn_tc_kernel(const __grid_con
       ok = mbar_wait(o_full + w, 0);
       if (ok) {
         tc_fence_after_sync();
-        const float r = p.out_scale / l;
+        float r = p.out_scale / l;
+        if (p.gate != nullptr && t < p.T) r *= sigmoid_f(__bfloat162float(p.gate[((long long)b * p.T + t) * p.ldg + h]));
         __nv_bfloat16* o = p.out + ((long long)b * p.T + t) * p.ldo + (long long)h * p.E;
         const bool vec = (p.E & 7) == 0 && (p.ldo & 7) == 0 && (reinterpret_cast<uintptr_t>(p.out) & 15) == 0;
         for (int c = 0; c < p.E; c += 16) {
@@ -291,34 +314,51 @@ __global__ void __launch_bounds__(FA_THREADS, 1) attn_tc_kernel(const __grid_con
   if (warp == 2) tmem_dealloc(tmem, 512);
 }
 
-template <int DKB, int EVB>
+CUtensorMap operand_map(const AttnOperand& o, int d, int rows, int heads, int batch) {
+  return make_tmap_4d_bf16(o.p, {(uint64_t)d, (uint64_t)rows, (uint64_t)heads, (uint64_t)batch},
+                           {(uint64_t)o.sr * 2, (uint64_t)o.sh * 2, (uint64_t)o.sb * 2}, 128);
+}
+
+template <int DKB, int RKB, int EVB>
 void run(const AttnArgs& a, int* status, cudaStream_t s) {
-  const CUtensorMapDataType bf = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
-  CUtensorMap tq = make_tmap_3d(a.q, bf, 2, a.pitch_k, a.T, (uint64_t)a.B * a.H, a.pitch_k * 2ull, (uint64_t)a.T * a.pitch_k * 2ull, 64, 128);
-  CUtensorMap tk = make_tmap_3d(a.kc, bf, 2, a.pitch_k, a.cap, (uint64_t)a.B * a.G, a.pitch_k * 2ull, (uint64_t)a.cap * a.pitch_k * 2ull, 64, 128);
-  CUtensorMap tv = make_tmap_3d(a.vc, bf, 2, a.pitch_v, a.cap, (uint64_t)a.B * a.G, a.pitch_v * 2ull, (uint64_t)a.cap * a.pitch_v * 2ull, 64, 128);
-  FaParams p{a.sink, (__nv_bfloat16*)a.out, a.ldo, a.T, a.H, a.G, a.D, a.E, a.cap, a.scale * 1.4426950408889634f, a.out_scale, a.pos, status};
-  constexpr int smem = (4 * DKB + 2 * EVB) * FA_BOX + 1024;
-  auto kern = attn_tc_kernel<DKB, EVB>;
+  const CUtensorMap tq = operand_map(a.q, a.D, a.T, a.H, a.B), tk = operand_map(a.k, a.D, a.rows, a.G, a.B), tv = operand_map(a.v, a.E, a.rows, a.G, a.B);
+  const CUtensorMap tq2 = RKB > 0 ? operand_map(a.q2, a.R, a.T, a.H, a.B) : tq, tk2 = RKB > 0 ? operand_map(a.k2, a.R, a.rows, 1, a.B) : tk;
+  FaParams p{a.sink, (const __nv_bfloat16*)a.gate, a.ldg, (__nv_bfloat16*)a.out, a.ldo, a.T, a.H, a.G, a.D, a.E, a.R,
+             a.scale * 1.4426950408889634f, a.out_scale, a.pos, status};
+  constexpr int KB = DKB + RKB;
+  constexpr int smem = (4 * KB + fa_value_stages<KB, EVB>() * EVB) * FA_BOX + 1024;
+  static_assert(smem <= 227 * 1024, "shared memory of a block");
+  auto kern = attn_tc_kernel<DKB, RKB, EVB>;
   cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-  kern<<<dim3(a.B * a.H, (a.T + 2 * FA_BM - 1) / (2 * FA_BM)), FA_THREADS, smem, s>>>(tq, tk, tv, p);
+  kern<<<dim3(a.B * a.H, (a.T + 2 * FA_BM - 1) / (2 * FA_BM)), FA_THREADS, smem, s>>>(tq, tk, tv, tq2, tk2, p);
+}
+
+template <int DKB, int RKB>
+void run_values(const AttnArgs& a, int* status, cudaStream_t s) {
+  if (a.E <= 64) run<DKB, RKB, 1>(a, status, s);
+  else run<DKB, RKB, 2>(a, status, s);
 }
 
 }  // namespace
 
 bool attn_tc_supported(const AttnArgs& a) {
-  return !a.f32 && a.D <= 128 && a.E <= 128 && a.scale > 0.f && a.T > 0 && a.pitch_k % 8 == 0 && a.pitch_v % 8 == 0 &&
-         (reinterpret_cast<uintptr_t>(a.q) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.kc) & 15) == 0 &&
-         (reinterpret_cast<uintptr_t>(a.vc) & 15) == 0;
+  auto fits = [](const AttnOperand& o) {
+    return (reinterpret_cast<uintptr_t>(o.p) & 15) == 0 && o.sr % 8 == 0 && o.sh % 8 == 0 && o.sb % 8 == 0;
+  };
+  return !a.f32 && a.D <= 128 && a.E <= 128 && a.R <= 64 && a.scale > 0.f && a.T > 0 && fits(a.q) && fits(a.k) && fits(a.v) &&
+         (a.R == 0 || (fits(a.q2) && fits(a.k2)));
 }
 
 void launch_attn_tc(const AttnArgs& a, int* status, cudaStream_t s) {
   if (a.B <= 0 || a.T <= 0) return;
   if (!attn_tc_supported(a)) throw std::runtime_error("attn_tc: unsupported shape");
-  if (a.D <= 64 && a.E <= 64) run<1, 1>(a, status, s);
-  else if (a.D <= 64) run<1, 2>(a, status, s);
-  else if (a.E <= 64) run<2, 1>(a, status, s);
-  else run<2, 2>(a, status, s);
+  if (a.R > 0) {
+    if (a.D <= 64) run_values<1, 1>(a, status, s);
+    else run_values<2, 1>(a, status, s);
+  } else {
+    if (a.D <= 64) run_values<1, 0>(a, status, s);
+    else run_values<2, 0>(a, status, s);
+  }
   check_launch("attn_tc");
 }
 

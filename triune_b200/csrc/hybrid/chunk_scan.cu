@@ -820,7 +820,7 @@ void launch_ssd_scan(const RecurrentArgs& a, float* seg_state, int nseg, cudaStr
   check_launch("ssd_scan");
 }
 
-bool chunk_scan_supported(const RecurrentArgs& a) { return !a.f32 && a.Dk <= 128 && a.T >= 32; }
+bool chunk_scan_supported(const RecurrentArgs& a) { return a.kind != RK_RETENTION && !a.f32 && a.Dk <= 128 && a.T >= 32; }
 
 long long chunk_scan_scratch(const RecurrentArgs& a) {
   const long long n = (a.T + CL - 1) / CL;

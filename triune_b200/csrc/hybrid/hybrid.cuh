@@ -1,5 +1,6 @@
 // Kernels of the heterogeneous-layer family: models whose layers mix softmax attention (per-head query / key norm,
-// partial rotation, a sink in the softmax), gated delta rule and Mamba-2 mixers, with a 32-bit residual stream.
+// partial rotation, a sink in the softmax), multi-head latent attention, gated delta rule, Mamba-2 and retention mixers,
+// with a 32-bit residual stream.
 //
 // Every kernel exists for bf16 and for fp32 compute tensors (`f32` flag of the launchers). Sequence rows are laid out
 // [B * T, ld]; `pos` is the position of the first of the T tokens, given by value or, when `pos_ptr` is not null, in
@@ -17,9 +18,9 @@
 namespace tb {
 
 enum HybridNorm : int { HN_LAYER = 0, HN_RMS = 1 };
-enum HybridAct : int { HA_RELU = 0, HA_SILU = 1, HA_GELU_TANH = 2, HA_IDENTITY = 3 };
+enum HybridAct : int { HA_RELU = 0, HA_SILU = 1, HA_GELU_TANH = 2, HA_IDENTITY = 3, HA_CLAMPED = 4 };
 enum GateOrder : int { GO_GATE_THEN_NORM = 0, GO_NORM_THEN_GATE = 1 };
-enum RecurrentKind : int { RK_MAMBA2 = 0, RK_DELTA = 1 };
+enum RecurrentKind : int { RK_MAMBA2 = 0, RK_DELTA = 1, RK_RETENTION = 2 };
 
 struct Pos {
   long long host;
@@ -33,11 +34,36 @@ void launch_embed_rows(const void* table, bool f32, const long long* ids, float*
 // y = norm(x) * w over fp32 rows.
 void launch_norm_rows(const float* x, const float* w, void* y, bool f32, int rows, int W, float eps, int kind,
                       cudaStream_t s);
-// out = act(gate) * up, gate at column 0 and up at column F of gu.
-void launch_glu_rows(const void* gu, long long ld, void* out, long long ldo, bool f32, int rows, int F, int act,
+// x += post(y + bias), then out = pre(x): the residual sum of a sublayer with a norm behind it, and the next sublayer's
+// input, in one pass. bias, out and pre_w may be null: no bias, no output, the sum itself as output.
+struct AddNormArgs {
+  float* x;
+  const void* y;
+  long long ldy;
+  bool y_f32, out_f32;
+  const float *bias, *post_w, *pre_w;
+  void* out;
+  int rows, W, post_kind, pre_kind;
+  float post_eps, pre_eps;
+};
+void launch_add_norm(const AddNormArgs& a, cudaStream_t s);
+// How a gated activation combines gate g and up u (both after their biases): act(g) * u, or for HA_CLAMPED
+// g sigmoid(alpha g) (u + 1) with g at most `limit` and u within +- `limit`.
+struct GluArgs {
+  int act;
+  float limit, alpha;
+  const float* bias;  // [2 F]: of the gate, then of the up projection; or null
+};
+// gate at column 0 and up at column F of gu
+void launch_glu_rows(const void* gu, long long ld, void* out, long long ldo, bool f32, int rows, int F, const GluArgs& glu,
                      cudaStream_t s);
+// out = act(gate) * table[ids[row], col0 ...]
+void launch_side_rows(const void* gate, long long ldg, const void* table, long long ldt, const long long* ids, int V, int col0,
+                      void* out, bool f32, int rows, int dim, int act, cudaStream_t s);
+// [T, 2 n]: cosines, then sines of the turns pos + t times freqs[n], times amplitude
+void launch_rotation_rows(const double* freqs, int n, float amplitude, float* out, int T, Pos pos, cudaStream_t s);
 // Gated norm of a mixer's output y [rows, inner] with gate rows: parts of inner / groups elements are divided by their
-// own root mean square. w has inner entries (w_period = inner) or one part's entries repeated (w_period = part).
+// own root mean square. w has inner entries (w_period = inner), one part's entries repeated (w_period = part), or is null.
 void launch_gated_norm(const void* y, long long ldy, const void* gate, long long ldg, const float* w, int w_period,
                        void* out, long long ldo, bool f32, int rows, int inner, int groups, float eps, int order,
                        float scale, cudaStream_t s);
@@ -53,6 +79,7 @@ void launch_causal_conv(const void* u, long long ldu, const float* w, const floa
 //   delta:   k, q unit vectors (q also times Dk^-1/2), g = exp(-exp(A_log) softplus(a + dt_bias)), beta = sigmoid(b)
 //            u = beta (v - g S^T k)
 //   mamba2:  dt = softplus(a + dt_bias), g = exp(-exp(A_log) dt), u = dt v
+//   retention: q and k turned by the rows of `rot` (dimension i with i + rot_dims / 2), k times Dk^-1/2, g = decay[h], u = v
 //   S <- g S + k u^T,  out = S^T q (+ D v)      (S: Dk x Dv fp32 per head)
 struct RecurrentArgs {
   const void *q, *k, *v;             // [B*T, ld*]: head groups of Dk (q, k: KG groups), heads of Dv (v)
@@ -68,6 +95,9 @@ struct RecurrentArgs {
   int kind;
   float unit_eps;                    // under the root of the unit norm (delta)
   bool f32;
+  const float* rot;                  // retention: [T, rot_dims] cosines and sines of the tokens
+  int rot_dims;
+  const double* decay;               // retention: [H]
 };
 void launch_recurrent(const RecurrentArgs& a, cudaStream_t s);
 // Chunk-parallel form for prompts (bf16, Dk <= 128); scratch of chunk_scan_scratch(a) bytes, 16-byte aligned.
@@ -99,36 +129,98 @@ struct AttnPrepArgs {
 };
 void launch_attn_prep(const AttnPrepArgs& a, cudaStream_t s);
 
+// Element (batch, row, head, d) of an operand is at batch * sb + row * sr + head * sh + d. A key row may have a second part
+// (R > 0) that all heads of a sequence share; queries then have it behind their first part, at q2.
+struct AttnOperand {
+  const void* p;
+  long long sr, sh, sb;
+};
 struct AttnArgs {
-  const void *q, *kc, *vc;  // as written by attn_prep
+  AttnOperand q, k, v, q2, k2;
   const float* sink;        // [H] or null
+  const void* gate;         // [B*T, ldg], one column per head: outputs are multiplied by its sigmoid; or null
+  long long ldg;
   void* out;                // [B*T, ldo], heads of E
   long long ldo;
-  int B, T, H, G, D, E, cap, pitch_k, pitch_v;
+  int B, T, H, G, D, E, R, rows;  // rows: key rows per sequence that may be read
   float scale, out_scale;
   Pos pos;
   bool f32;
 };
 void launch_attn_simple(const AttnArgs& a, cudaStream_t s);
-// tcgen05 kernel: bf16, heads up to 128, positive scale. `status` (or null) receives a KernelStatus if a wait expires.
+// tcgen05 kernel: bf16, heads up to 128 (plus a second part up to 64), positive scale. `status` (or null) receives a KernelStatus if a wait expires.
 bool attn_tc_supported(const AttnArgs& a);
 void launch_attn_tc(const AttnArgs& a, int* status, cudaStream_t s);
 
+// ---- latent attention --------------------------------------------------------------------------------------------
+// Prompts: turns the second part of every query head in place and, where the layer has latents of its own (col_c >= 0),
+// appends their normed form and the turned key part to the cache [B, cap, rank_p + Rp].
+struct LatentPrepArgs {
+  void* proj;  // [B*T, ld]
+  long long ld;
+  int col_q, H, Dp, Rp;  // heads of [Dp | Rp]
+  int col_c;
+  const float* norm_w;   // [rank]
+  float eps;
+  void* cache;
+  int cap, rank, rank_p, R;
+  const float* rot;      // [T, R]: cosines, sines
+  int B, T;
+  Pos pos;
+  bool f32;
+};
+void launch_latent_prep(const LatentPrepArgs& a, cudaStream_t s);
+
+// One token per sequence in the latent space, three launches: (1) qa = [W_uk^T q | turned q part] per head, and the append
+// of the new row; (2) attention of qa over the cached rows in split ranges; (3) combination of the splits, value expansion,
+// gate.
+struct LatentStepArgs {
+  const float* proj;  // [B, ld]
+  long long ld;
+  int col_q, col_g, col_c;  // col_g, col_c: -1 where there is none
+  int H, D, Dp, R, Rp, E, Ep, rank, rank_p;
+  const float* norm_w;
+  float eps;
+  void* cache;        // [B, cap, rank_p + Rp]
+  const void* up;     // [H, Dp + Ep, rank_p]
+  bool f32;           // cache and up
+  int cap;
+  const double* freqs;  // [R / 2]
+  float amplitude;
+  const float* sink;
+  float* qa;          // [B, H, rank_p + Rp]
+  float* part;        // [B, H, splits, step_part_stride(rank_p)]
+  int splits;
+  float* out;         // [B, ldo], heads of E
+  long long ldo;
+  float scale, out_scale;
+  int B;
+  Pos pos;
+};
+int latent_step_splits(int B, int H);
+void launch_latent_step(const LatentStepArgs& a, cudaStream_t s);
+
 // ---- decoding (one token per sequence, B <= 8) ------------------------------------------------------------------
 // y[b, n] (+)= sum_k W[n, k] in[b, k] with the input formed in the kernel's prologue from one or two segments:
-// plain fp32 rows, norm(x) * w, or the gated norm of a mixer output. Everything but W is fp32.
+// plain fp32 rows, norm(x) * w, the gated norm of a mixer output, or norm(x + post(y + bias)) (which also leaves the sum in
+// x_out for the kernels behind it). Everything but W is fp32.
 struct GemvSegment {
   const float* x;     // [B, ld]
   long long ld;
   int n;              // entries of this segment
-  int kind;           // 0 plain, 1 norm over the n entries, 2 gated norm
-  int norm_kind;      // kind 1: HN_*; kind 2: GO_*
-  const float* w;     // norm weight
+  int kind;           // 0 plain, 1 norm over the n entries, 2 gated norm, 3 norm of a sum
+  int norm_kind;      // kinds 1, 3: HN_*; kind 2: GO_*
+  const float* w;     // norm weight; null: kind 2 has none, kind 3 is the sum itself
   int w_period;
   const float* gate;  // kind 2: [B, ldg]
   long long ldg;
   int groups;
   float eps, scale;
+  const float *y, *y_bias, *post_w;  // kind 3: [B, ldy], [n] or null, [n]
+  long long ldy;
+  int post_kind;
+  float post_eps;
+  float* x_out;       // kind 3: [B, n] or null
 };
 struct GemvArgs {
   GemvSegment seg[2];
@@ -139,8 +231,12 @@ struct GemvArgs {
   float* y;       // [B, ldy]
   long long ldy;
   int B, N, K;    // K = sum of the segments' entries
-  int epilogue;   // 0 store, 1 add, 2 act(row n) * row n + N (W has 2 N rows)
-  int act;
+  int epilogue;   // 0 store, 1 add, 2 gated activation of rows n and n + N (W has 2 N rows), 3 act(row n) * table entry
+  GluArgs glu;    // act of 2 and 3; bias of 0, 1 ([N]) and 2 ([2 N])
+  const void* table;     // epilogue 3: [V, ldt] in W's type, row ids[b], column col0 + n
+  long long ldt;
+  const long long* ids;  // [B]
+  int V, col0;
 };
 void launch_gemv(const GemvArgs& a, cudaStream_t s);
 
@@ -160,6 +256,10 @@ struct StepRecurrent {
   long long ldo;
   int H, KG, Dk, Dv, kind;
   float unit_eps;
+  int col_q, col_k, col_v;         // retention: columns of proj (no convolution)
+  const double *decay, *freqs;     // retention: [H], [rot_dims / 2]
+  int rot_dims;
+  float amplitude;
 };
 struct StepAttention {
   const float* proj;
@@ -242,6 +342,11 @@ __device__ __forceinline__ float act_f(float x, int act) {
   if (act == HA_SILU) return silu_f(x);
   if (act == HA_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
   return x;
+}
+__device__ __forceinline__ float glu_f(float g, float u, int act, float limit, float alpha) {
+  if (act != HA_CLAMPED) return act_f(g, act) * u;
+  g = fminf(g, limit);
+  return g / (1.f + expf(-alpha * g)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
 }
 // sine and cosine of pos * f radians; the turn count is removed in double so that far positions lose nothing
 __device__ __forceinline__ void rotation(long long pos, double f, float* s, float* c) {

@@ -41,6 +41,12 @@ tb::Pos pos_of(int64_t host, const OptT& dev) {
   return p;
 }
 
+int* status_of(const OptT& status) {
+  if (!status.has_value() || !status->defined()) return nullptr;
+  TORCH_CHECK(status->is_cuda() && status->scalar_type() == at::kInt && status->numel() >= 1, "status: CUDA int32 expected");
+  return status->data_ptr<int>();
+}
+
 Tensor embed_rows(const Tensor& table, const Tensor& ids) {
   TORCH_CHECK(table.is_contiguous(), "table must be contiguous");
   const bool f32 = rows_of(table, 0, 0, "table");
@@ -61,25 +67,81 @@ Tensor norm_rows(const Tensor& x, const Tensor& w, double eps, int64_t kind, boo
   return y;
 }
 
-Tensor glu_rows(const Tensor& gu, int64_t F, int64_t act) {
+tb::GluArgs glu_args(int64_t act, const OptT& bias, int64_t n, double limit, double alpha) {
+  TORCH_CHECK(act != tb::HA_CLAMPED || limit > 0, "the clamped activation needs a positive limit");
+  return tb::GluArgs{(int)act, (float)limit, (float)alpha, f32o(bias, n, "bias")};
+}
+
+Tensor glu_rows(const Tensor& gu, int64_t F, int64_t act, const OptT& bias, double limit, double alpha) {
   const bool f32 = rows_of(gu, 0, 2 * F, "gate_up");
   c10::cuda::CUDAGuard guard(gu.device());
   Tensor out = torch::empty({gu.size(0), F}, gu.options());
-  tb::launch_glu_rows(gu.data_ptr(), gu.stride(0), out.data_ptr(), F, f32, (int)gu.size(0), (int)F, (int)act, cur_stream());
+  tb::launch_glu_rows(gu.data_ptr(), gu.stride(0), out.data_ptr(), F, f32, (int)gu.size(0), (int)F, glu_args(act, bias, 2 * F, limit, alpha),
+                      cur_stream());
   return out;
 }
 
-void gated_norm(const Tensor& y, const Tensor& gate, const Tensor& w, Tensor& out, int64_t inner, int64_t groups, double eps,
+const long long* ids_of(const Tensor& ids, int64_t n) {
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kLong && ids.is_contiguous() && ids.numel() >= n, "ids: contiguous CUDA int64 expected");
+  return reinterpret_cast<const long long*>(ids.data_ptr<int64_t>());
+}
+
+Tensor side_rows(const Tensor& gate, const Tensor& table, const Tensor& ids, int64_t col0, int64_t act) {
+  const int64_t rows = gate.size(0), dim = gate.size(1);
+  const bool f32 = rows_of(gate, rows, dim, "gate");
+  TORCH_CHECK(rows_of(table, 0, col0 + dim, "table") == f32, "side_rows: one dtype expected");
+  c10::cuda::CUDAGuard guard(gate.device());
+  Tensor out = torch::empty({rows, dim}, gate.options());
+  tb::launch_side_rows(gate.data_ptr(), gate.stride(0), table.data_ptr(), table.stride(0), ids_of(ids, rows), (int)table.size(0), (int)col0,
+                       out.data_ptr(), f32, (int)rows, (int)dim, (int)act, cur_stream());
+  return out;
+}
+
+void add_norm(Tensor& x, const Tensor& y, const OptT& bias, const Tensor& post_w, double post_eps, int64_t post_kind, const OptT& out,
+              const OptT& pre_w, double pre_eps, int64_t pre_kind) {
+  TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.scalar_type() == at::kFloat && x.is_contiguous(), "x: contiguous CUDA fp32 rows expected");
+  const int64_t rows = x.size(0), W = x.size(1);
+  tb::AddNormArgs a{};
+  a.x = x.data_ptr<float>();
+  a.y_f32 = rows_of(y, rows, W, "y");
+  a.y = y.data_ptr(); a.ldy = y.stride(0);
+  a.bias = f32o(bias, W, "bias");
+  a.post_w = f32v(post_w, W, "post_w");
+  a.pre_w = f32o(pre_w, W, "pre_w");
+  a.out_f32 = true;
+  if (out.has_value() && out->defined()) {
+    a.out_f32 = rows_of(*out, rows, W, "out");
+    TORCH_CHECK(out->is_contiguous(), "out: contiguous rows expected");
+    a.out = out->data_ptr();
+  }
+  a.rows = (int)rows; a.W = (int)W;
+  a.post_kind = (int)post_kind; a.pre_kind = (int)pre_kind;
+  a.post_eps = (float)post_eps; a.pre_eps = (float)pre_eps;
+  c10::cuda::CUDAGuard guard(x.device());
+  tb::launch_add_norm(a, cur_stream());
+}
+
+Tensor rotation_rows(const Tensor& freqs, double amplitude, int64_t T, int64_t pos, const OptT& pos_dev) {
+  const int64_t n = freqs.numel();
+  c10::cuda::CUDAGuard guard(freqs.device());
+  Tensor out = torch::empty({T, 2 * n}, freqs.options().dtype(at::kFloat));
+  tb::launch_rotation_rows(f64v(freqs, n, "freqs"), (int)n, (float)amplitude, out.data_ptr<float>(), (int)T, pos_of(pos, pos_dev), cur_stream());
+  return out;
+}
+
+void gated_norm(const Tensor& y, const Tensor& gate, const OptT& w, Tensor& out, int64_t inner, int64_t groups, double eps,
                 int64_t order, double scale) {
   const int64_t rows = y.size(0);
   const bool f32 = rows_of(y, rows, inner, "y");
   TORCH_CHECK(rows_of(gate, rows, inner, "gate") == f32 && rows_of(out, rows, inner, "out") == f32, "gated_norm: one dtype expected");
   TORCH_CHECK(groups > 0 && inner % groups == 0, "gated_norm: parts must divide the width");
   const int64_t part = inner / groups;
-  TORCH_CHECK(w.numel() == inner || w.numel() == part, "gated_norm: one weight per channel or per position of a part");
+  const bool weighted = w.has_value() && w->defined();
+  TORCH_CHECK(!weighted || w->numel() == inner || w->numel() == part, "gated_norm: one weight per channel or per position of a part");
   c10::cuda::CUDAGuard guard(y.device());
-  tb::launch_gated_norm(y.data_ptr(), y.stride(0), gate.data_ptr(), gate.stride(0), f32v(w, w.numel(), "w"), (int)w.numel(), out.data_ptr(),
-                        out.stride(0), f32, (int)rows, (int)inner, (int)groups, (float)eps, (int)order, (float)scale, cur_stream());
+  tb::launch_gated_norm(y.data_ptr(), y.stride(0), gate.data_ptr(), gate.stride(0), f32o(w, 0, "w"), weighted ? (int)w->numel() : (int)part,
+                        out.data_ptr(), out.stride(0), f32, (int)rows, (int)inner, (int)groups, (float)eps, (int)order, (float)scale,
+                        cur_stream());
 }
 
 Tensor causal_conv(const Tensor& u, const Tensor& w, const OptT& bias, const Tensor& ring_in, Tensor& ring_out, int64_t B, int64_t T,
@@ -146,11 +208,7 @@ void recurrent(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& 
   int64_t per = (T + 63) / 64 * 64;
   auto scratch_of = [](const tb::RecurrentArgs& x) { return tb::ssd_tc_supported(x) ? tb::ssd_tc_scratch(x) : tb::chunk_scan_scratch(x); };
   while (per > 4096 && (part.T = (int)std::min(per, T), scratch_of(part)) > budget) per = (per / 2 + 127) / 128 * 128;
-  int* st = nullptr;
-  if (status.has_value() && status->defined()) {
-    TORCH_CHECK(status->is_cuda() && status->scalar_type() == at::kInt, "status: CUDA int32 expected");
-    st = status->data_ptr<int>();
-  }
+  int* st = status_of(status);
   Tensor scratch;
   for (int64_t t = 0; t < T; t += per) {
     part.T = (int)std::min(per, T - t);
@@ -167,6 +225,31 @@ void recurrent(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& 
     if (tb::ssd_tc_supported(part)) tb::launch_ssd_tc(part, scratch.data_ptr(), st, cur_stream());
     else tb::launch_chunk_scan(part, scratch.data_ptr(), cur_stream());
   }
+}
+
+// q, k, v: column views of row matrices; rot [T, 2 n]; state [B, H, Dk, Dv] fp32 in place
+void retention(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& rot, const Tensor& decay, Tensor& state, Tensor& out, int64_t B,
+               int64_t T, bool chunked, const OptT& status) {
+  TORCH_CHECK(state.dim() == 4 && state.is_cuda() && state.scalar_type() == at::kFloat && state.is_contiguous() && state.size(0) == B,
+              "state: contiguous CUDA fp32 [B, H, Dk, Dv] expected");
+  const int64_t H = state.size(1), Dk = state.size(2), Dv = state.size(3), rows = B * T;
+  tb::RecurrentArgs r{};
+  r.f32 = rows_of(q, rows, H * Dk, "q");
+  TORCH_CHECK(rows_of(k, rows, H * Dk, "k") == r.f32 && rows_of(v, rows, H * Dv, "v") == r.f32 && rows_of(out, rows, H * Dv, "out") == r.f32,
+              "retention: one dtype expected");
+  TORCH_CHECK(rot.dim() == 2 && rot.size(0) == T && rot.size(1) <= Dk && rot.size(1) % 2 == 0, "retention: rotation rows");
+  r.q = q.data_ptr(); r.k = k.data_ptr(); r.v = v.data_ptr();
+  r.ldq = q.stride(0); r.ldk = k.stride(0); r.ldv = v.stride(0);
+  r.state = state.data_ptr<float>();
+  r.out = out.data_ptr(); r.ldo = out.stride(0);
+  r.B = (int)B; r.T = (int)T; r.H = r.KG = (int)H; r.Dk = (int)Dk; r.Dv = (int)Dv;
+  r.rows = T;
+  r.kind = tb::RK_RETENTION;
+  r.rot = f32v(rot, T * rot.size(1), "rotation rows");
+  r.rot_dims = (int)rot.size(1);
+  r.decay = f64v(decay, H, "decay");
+  c10::cuda::CUDAGuard guard(q.device());
+  tb::launch_recurrent(r, cur_stream());
 }
 
 bool cache_of(const Tensor& c, int64_t B, int64_t G, int64_t d, const char* n) {
@@ -214,10 +297,11 @@ tb::AttnArgs attn_args(const Tensor& q, const Tensor& kc, const Tensor& vc, cons
               "attention: shapes or dtypes differ");
   TORCH_CHECK(rows_of(out, (int64_t)a.B * a.T, (int64_t)a.H * E, "out") == a.f32, "attention: one dtype expected");
   if (!(pos_dev.has_value() && pos_dev->defined())) TORCH_CHECK(pos + a.T <= kc.size(2), "attention: the cache is too small");
-  a.q = q.data_ptr(); a.kc = kc.data_ptr(); a.vc = vc.data_ptr();
+  auto operand = [](const Tensor& t) { return tb::AttnOperand{t.data_ptr(), t.stride(2), t.stride(1), t.stride(0)}; };
+  a.q = operand(q); a.k = operand(kc); a.v = operand(vc);
   a.sink = f32o(sink, a.H, "sink");
   a.out = out.data_ptr(); a.ldo = out.stride(0);
-  a.cap = (int)kc.size(2); a.pitch_k = (int)kc.size(3); a.pitch_v = (int)vc.size(3);
+  a.rows = (int)kc.size(2);
   a.scale = (float)scale; a.out_scale = (float)out_scale;
   a.pos = pos_of(pos, pos_dev);
   return a;
@@ -235,17 +319,120 @@ void attention(const Tensor& q, const Tensor& kc, const Tensor& vc, const OptT& 
                double out_scale, int64_t pos, const OptT& pos_dev, const OptT& status) {
   tb::AttnArgs a = attn_args(q, kc, vc, sink, out, D, E, scale, out_scale, pos, pos_dev);
   c10::cuda::CUDAGuard guard(q.device());
-  int* st = nullptr;
-  if (status.has_value() && status->defined()) {
-    TORCH_CHECK(status->is_cuda() && status->scalar_type() == at::kInt, "status: CUDA int32 expected");
-    st = status->data_ptr<int>();
-  }
+  int* st = status_of(status);
   if (tb::attn_tc_supported(a)) tb::launch_attn_tc(a, st, cur_stream());
   else tb::launch_attn_simple(a, cur_stream());
 }
 
+// Query heads of [Dp | Rp] columns of proj, cache [B, 1, capacity, rank_p + Rp]
+void check_latent(const Tensor& proj, int64_t rows, int64_t col_q, int64_t H, int64_t Dp, int64_t Rp, int64_t col_c, const OptT& norm_w,
+                  const Tensor& cache, int64_t B, int64_t rank, int64_t rank_p, int64_t R) {
+  rows_of(proj, rows, std::max(col_q + H * (Dp + Rp), col_c + rank_p + Rp), "proj");
+  cache_of(cache, B, 1, rank_p + Rp, "latent cache");
+  TORCH_CHECK(cache.size(3) == rank_p + Rp && rank > 0 && rank <= rank_p && R >= 0 && R <= Rp && R % 2 == 0 && Dp % 8 == 0 && Rp % 8 == 0 &&
+                  rank_p % 8 == 0 && col_q >= 0,
+              "latent attention: shapes");
+  if (col_c >= 0) TORCH_CHECK(norm_w.has_value() && norm_w->defined(), "latent attention: own latents need their norm");
+}
+
+void latent_prep(Tensor& proj, int64_t col_q, int64_t H, int64_t Dp, int64_t Rp, int64_t col_c, const OptT& norm_w, double eps, Tensor& cache,
+                 int64_t rank, int64_t rank_p, int64_t R, const Tensor& rot, int64_t B, int64_t T, int64_t pos, const OptT& pos_dev) {
+  check_latent(proj, B * T, col_q, H, Dp, Rp, col_c, norm_w, cache, B, rank, rank_p, R);
+  tb::LatentPrepArgs a{};
+  a.f32 = proj.scalar_type() == at::kFloat;
+  TORCH_CHECK((cache.scalar_type() == at::kFloat) == a.f32, "latent_prep: one dtype expected");
+  TORCH_CHECK(rot.dim() == 2 && rot.size(0) == T && rot.size(1) == R, "latent_prep: rotation rows");
+  if (!(pos_dev.has_value() && pos_dev->defined())) TORCH_CHECK(pos + T <= cache.size(2), "latent_prep: the cache is too small");
+  a.proj = proj.data_ptr(); a.ld = proj.stride(0);
+  a.col_q = (int)col_q; a.H = (int)H; a.Dp = (int)Dp; a.Rp = (int)Rp; a.col_c = (int)col_c;
+  a.norm_w = f32o(norm_w, rank, "norm_w");
+  a.eps = (float)eps;
+  a.cache = cache.data_ptr(); a.cap = (int)cache.size(2);
+  a.rank = (int)rank; a.rank_p = (int)rank_p; a.R = (int)R;
+  a.rot = f32v(rot, T * R, "rotation rows");
+  a.B = (int)B; a.T = (int)T;
+  a.pos = pos_of(pos, pos_dev);
+  c10::cuda::CUDAGuard guard(proj.device());
+  tb::launch_latent_prep(a, cur_stream());
+}
+
+// Heads g0 .. g0 + Hn - 1 of a layer, whose keys and values are expanded in kv [B, n, Hn (Dp + Ep)].
+void latent_attention(const Tensor& proj, int64_t col_q, int64_t col_g, const Tensor& cache, const Tensor& kv, const OptT& sink, Tensor& out,
+                      int64_t g0, int64_t Hn, int64_t B, int64_t T, int64_t Dp, int64_t Rp, int64_t rank_p, int64_t D, int64_t R, int64_t E,
+                      double scale, double out_scale, int64_t pos, const OptT& pos_dev, const OptT& status) {
+  const int64_t Ep = (E + 7) / 8 * 8;
+  check_latent(proj, B * T, col_q, g0 + Hn, Dp, Rp, -1, c10::nullopt, cache, B, rank_p, rank_p, R);
+  TORCH_CHECK(kv.is_cuda() && kv.dim() == 3 && kv.size(0) == B && kv.is_contiguous() && kv.size(2) == Hn * (Dp + Ep) && D <= Dp,
+              "latent_attention: expanded keys and values [B, n, heads * (key + value)] expected");
+  TORCH_CHECK(kv.scalar_type() == proj.scalar_type() && cache.scalar_type() == proj.scalar_type() && out.scalar_type() == proj.scalar_type(),
+              "latent_attention: one dtype expected");
+  const int64_t n = kv.size(1), size = kv.element_size();
+  TORCH_CHECK(n <= cache.size(2), "latent_attention: more keys than cached rows");
+  const bool on_device = pos_dev.has_value() && pos_dev->defined();
+  TORCH_CHECK(on_device ? n == cache.size(2) : pos + T <= n, "latent_attention: ", n, " keys for ", T, " tokens after ", pos);
+  rows_of(out, B * T, (g0 + Hn) * E, "out");
+  TORCH_CHECK(col_g < 0 || col_g + g0 + Hn <= proj.size(1), "latent_attention: gate columns");
+  auto at = [&](const Tensor& t, int64_t off) { return static_cast<char*>(t.data_ptr()) + off * size; };
+  const int64_t ld = proj.stride(0), head = Dp + Rp;
+  tb::AttnArgs a{};
+  a.q = {at(proj, col_q + g0 * head), ld, head, T * ld};
+  a.q2 = {at(proj, col_q + g0 * head + Dp), ld, head, T * ld};
+  a.k = {kv.data_ptr(), kv.stride(1), Dp + Ep, kv.stride(0)};
+  a.v = {at(kv, Dp), kv.stride(1), Dp + Ep, kv.stride(0)};
+  a.k2 = {at(cache, rank_p), cache.stride(2), 0, cache.stride(0)};
+  a.sink = f32o(sink, g0 + Hn, "sink");
+  if (a.sink != nullptr) a.sink += g0;
+  if (col_g >= 0) a.gate = at(proj, col_g + g0);
+  a.ldg = ld;
+  a.out = at(out, g0 * E); a.ldo = out.stride(0);
+  a.B = (int)B; a.T = (int)T; a.H = a.G = (int)Hn; a.D = (int)D; a.E = (int)E; a.R = (int)R;
+  a.rows = (int)n;
+  a.scale = (float)scale; a.out_scale = (float)out_scale;
+  a.pos = pos_of(pos, pos_dev);
+  a.f32 = proj.scalar_type() == at::kFloat;
+  c10::cuda::CUDAGuard guard(proj.device());
+  if (tb::attn_tc_supported(a)) tb::launch_attn_tc(a, status_of(status), cur_stream());
+  else tb::launch_attn_simple(a, cur_stream());
+}
+
+void latent_step(const Tensor& proj, int64_t col_q, int64_t col_g, int64_t col_c, const OptT& norm_w, double eps, Tensor& cache, const Tensor& up,
+                 const Tensor& freqs, double amplitude, const OptT& sink, Tensor& qa, Tensor& part, Tensor& out, int64_t rank, int64_t D,
+                 int64_t R, int64_t E, double scale, double out_scale, int64_t pos, const OptT& pos_dev) {
+  const int64_t B = proj.size(0), Dp = (D + 7) / 8 * 8, Ep = (E + 7) / 8 * 8, Rp = (R + 7) / 8 * 8;
+  TORCH_CHECK(up.is_cuda() && up.dim() == 3 && up.is_contiguous() && up.size(1) == Dp + Ep, "latent_step: expansion [H, key + value, latent] expected");
+  const int64_t H = up.size(0), rank_p = up.size(2);
+  TORCH_CHECK(rows_of(proj, B, 0, "proj"), "latent_step: fp32 projection rows expected");
+  check_latent(proj, B, col_q, H, Dp, Rp, col_c, norm_w, cache, B, rank, rank_p, R);
+  TORCH_CHECK(cache.scalar_type() == up.scalar_type() && 2 * freqs.numel() == R && (col_g < 0 || col_g + H <= proj.size(1)), "latent_step: shapes");
+  if (!(pos_dev.has_value() && pos_dev->defined())) TORCH_CHECK(pos < cache.size(2), "latent_step: the cache is full");
+  tb::LatentStepArgs a{};
+  a.proj = proj.data_ptr<float>(); a.ld = proj.stride(0);
+  a.col_q = (int)col_q; a.col_g = (int)col_g; a.col_c = (int)col_c;
+  a.H = (int)H; a.D = (int)D; a.Dp = (int)Dp; a.R = (int)R; a.Rp = (int)Rp; a.E = (int)E; a.Ep = (int)Ep; a.rank = (int)rank; a.rank_p = (int)rank_p;
+  a.norm_w = f32o(norm_w, rank, "norm_w");
+  a.eps = (float)eps;
+  a.cache = cache.data_ptr(); a.up = up.data_ptr();
+  a.f32 = up.scalar_type() == at::kFloat;
+  a.cap = (int)cache.size(2);
+  a.freqs = f64v(freqs, R / 2, "freqs");
+  a.amplitude = (float)amplitude;
+  a.sink = f32o(sink, H, "sink");
+  a.qa = const_cast<float*>(f32v(qa, B * H * (rank_p + Rp), "qa"));
+  TORCH_CHECK(part.dim() == 4 && part.size(0) == B && part.size(1) == H && part.size(2) >= 1 && part.size(2) <= 128, "latent_step: split results");
+  a.splits = (int)part.size(2);
+  a.part = const_cast<float*>(f32v(part, B * H * a.splits * tb::step_part_stride((int)rank_p), "part"));
+  TORCH_CHECK(rows_of(out, B, H * E, "out"), "latent_step: fp32 output expected");
+  a.out = out.data_ptr<float>(); a.ldo = out.stride(0);
+  a.scale = (float)scale; a.out_scale = (float)out_scale;
+  a.B = (int)B;
+  a.pos = pos_of(pos, pos_dev);
+  c10::cuda::CUDAGuard guard(proj.device());
+  tb::launch_latent_step(a, cur_stream());
+}
+
 // segments: dicts with x [B, n], kind, and what the kind needs
-void gemv(const std::vector<py::dict>& segs, const Tensor& W, Tensor& y, int64_t epilogue, int64_t act) {
+void gemv(const std::vector<py::dict>& segs, const Tensor& W, Tensor& y, int64_t epilogue, int64_t act, const OptT& bias, double limit,
+          double alpha, const OptT& table, const OptT& ids, int64_t col0) {
   TORCH_CHECK(segs.size() >= 1 && segs.size() <= 2, "gemv: one or two input segments");
   tb::GemvArgs g{};
   g.nseg = (int)segs.size();
@@ -263,20 +450,41 @@ void gemv(const std::vector<py::dict>& segs, const Tensor& W, Tensor& y, int64_t
     s.scale = d.contains("scale") ? d["scale"].cast<float>() : 1.f;
     s.groups = 1; s.w_period = s.n;
     if (s.kind != 0) {
-      Tensor w = d["w"].cast<Tensor>();
       s.norm_kind = d["norm"].cast<int>();
       s.eps = d["eps"].cast<float>();
+      const bool weighted = !d["w"].is_none();
+      TORCH_CHECK(weighted || s.kind != 1, "gemv: norm weight");
+      if (weighted) {
+        Tensor w = d["w"].cast<Tensor>();
+        s.w = f32v(w, w.numel(), "w");
+        s.w_period = (int)w.numel();
+      }
       if (s.kind == 2) {
         s.groups = d["groups"].cast<int>();
-        TORCH_CHECK(s.groups > 0 && s.n % s.groups == 0 && (w.numel() == s.n || w.numel() == s.n / s.groups), "gemv: gated norm parts");
+        TORCH_CHECK(s.groups > 0 && s.n % s.groups == 0, "gemv: gated norm parts");
+        if (!weighted) s.w_period = s.n / s.groups;
+        TORCH_CHECK(s.w_period == s.n || s.w_period == s.n / s.groups, "gemv: gated norm weight");
         Tensor gate = d["gate"].cast<Tensor>();
         TORCH_CHECK(rows_of(gate, g.B, s.n, "gate"), "gemv: fp32 gate rows expected");
         s.gate = gate.data_ptr<float>(); s.ldg = gate.stride(0);
       } else {
-        TORCH_CHECK(w.numel() == s.n, "gemv: norm weight");
+        TORCH_CHECK(s.w_period == s.n, "gemv: norm weight");
       }
-      s.w = f32v(w, w.numel(), "w");
-      s.w_period = (int)w.numel();
+      if (s.kind == 3) {
+        TORCH_CHECK(i == 0 && segs.size() == 1, "gemv: a sum is the only segment");
+        Tensor add = d["y"].cast<Tensor>();
+        TORCH_CHECK(rows_of(add, g.B, s.n, "y"), "gemv: fp32 rows to add expected");
+        s.y = add.data_ptr<float>(); s.ldy = add.stride(0);
+        if (!d["bias"].is_none()) s.y_bias = f32v(d["bias"].cast<Tensor>(), s.n, "bias");
+        s.post_w = f32v(d["post_w"].cast<Tensor>(), s.n, "post_w");
+        s.post_kind = d["post_norm"].cast<int>();
+        s.post_eps = d["post_eps"].cast<float>();
+        if (!d["x_out"].is_none()) {
+          Tensor xo = d["x_out"].cast<Tensor>();
+          s.x_out = const_cast<float*>(f32v(xo, (int64_t)g.B * s.n, "x_out"));
+          TORCH_CHECK(s.x_out != s.x, "gemv: the sum goes to rows of its own");
+        }
+      }
     }
     g.K += s.n;
   }
@@ -284,20 +492,45 @@ void gemv(const std::vector<py::dict>& segs, const Tensor& W, Tensor& y, int64_t
   TORCH_CHECK(W.size(1) == g.K, "gemv: W has ", W.size(1), " columns, the input ", g.K);
   g.W = W.data_ptr(); g.ldw = W.stride(0);
   g.y = y.data_ptr<float>(); g.ldy = y.stride(0);
-  g.epilogue = (int)epilogue; g.act = (int)act;
+  g.epilogue = (int)epilogue;
+  g.glu = glu_args(act, bias, epilogue == 2 ? 2 * g.N : g.N, limit, alpha);
+  if (epilogue == 3) {
+    TORCH_CHECK(table.has_value() && ids.has_value(), "gemv: the side epilogue needs a table and token ids");
+    TORCH_CHECK(rows_of(*table, 0, col0 + g.N, "table") == g.f32 && col0 >= 0, "gemv: the table has W's dtype");
+    g.table = table->data_ptr(); g.ldt = table->stride(0);
+    g.ids = ids_of(*ids, g.B);
+    g.V = (int)table->size(0); g.col0 = (int)col0;
+  }
   c10::cuda::CUDAGuard guard(W.device());
   tb::launch_gemv(g, cur_stream());
 }
 
 tb::StepRecurrent step_recurrent(const py::dict& d, const Tensor& proj, int64_t B) {
   tb::StepRecurrent r{};
-  Tensor state = d["state"].cast<Tensor>(), ring = d["ring"].cast<Tensor>(), cw = d["conv_w"].cast<Tensor>(), out = d["out"].cast<Tensor>();
+  Tensor state = d["state"].cast<Tensor>(), out = d["out"].cast<Tensor>();
   TORCH_CHECK(state.dim() == 4 && state.size(0) == B, "step: state");
   r.H = (int)state.size(1); r.Dk = (int)state.size(2); r.Dv = (int)state.size(3);
-  r.KG = d["key_groups"].cast<int>();
   r.kind = d["kind"].cast<int>();
-  r.C = (int)cw.size(0); r.taps = (int)cw.size(1);
   r.proj = proj.data_ptr<float>(); r.ld = proj.stride(0);
+  r.state = const_cast<float*>(f32v(state, 0, "state"));
+  TORCH_CHECK(rows_of(out, B, (int64_t)r.H * r.Dv, "out"), "step: fp32 output expected");
+  r.out = out.data_ptr<float>(); r.ldo = out.stride(0);
+  if (r.kind == tb::RK_RETENTION) {
+    r.KG = r.H;
+    r.col_q = d["col_q"].cast<int>(); r.col_k = d["col_k"].cast<int>(); r.col_v = d["col_v"].cast<int>();
+    TORCH_CHECK(r.col_q + r.H * r.Dk <= proj.size(1) && r.col_k + r.H * r.Dk <= proj.size(1) && r.col_v + r.H * r.Dv <= proj.size(1),
+                "step: columns outside the projection");
+    Tensor freqs = d["freqs"].cast<Tensor>();
+    r.rot_dims = (int)(2 * freqs.numel());
+    TORCH_CHECK(r.rot_dims <= r.Dk, "step: rotated dimensions");
+    r.freqs = f64v(freqs, 0, "freqs");
+    r.decay = f64v(d["decay"].cast<Tensor>(), r.H, "decay");
+    r.amplitude = d["amplitude"].cast<float>();
+    return r;
+  }
+  Tensor ring = d["ring"].cast<Tensor>(), cw = d["conv_w"].cast<Tensor>();
+  r.KG = d["key_groups"].cast<int>();
+  r.C = (int)cw.size(0); r.taps = (int)cw.size(1);
   r.col_u = d["col_u"].cast<int>(); r.col_a = d["col_a"].cast<int>(); r.col_b = d["col_b"].cast<int>();
   r.off_q = d["off_q"].cast<int>(); r.off_k = d["off_k"].cast<int>(); r.off_v = d["off_v"].cast<int>();
   TORCH_CHECK(r.KG > 0 && r.H % r.KG == 0 && r.off_q + r.KG * r.Dk <= r.C && r.off_k + r.KG * r.Dk <= r.C && r.off_v + r.H * r.Dv <= r.C &&
@@ -309,9 +542,6 @@ tb::StepRecurrent step_recurrent(const py::dict& d, const Tensor& proj, int64_t 
   r.A_log = f32v(d["A_log"].cast<Tensor>(), r.H, "A_log");
   r.dt_bias = f32v(d["dt_bias"].cast<Tensor>(), r.H, "dt_bias");
   if (r.kind == tb::RK_MAMBA2) r.D = f32v(d["D"].cast<Tensor>(), r.H, "D");
-  r.state = const_cast<float*>(f32v(state, 0, "state"));
-  TORCH_CHECK(rows_of(out, B, (int64_t)r.H * r.Dv, "out"), "step: fp32 output expected");
-  r.out = out.data_ptr<float>(); r.ldo = out.stride(0);
   r.unit_eps = d["unit_eps"].cast<float>();
   return r;
 }
@@ -370,6 +600,14 @@ void register_hybrid(pybind11::module& m) {
   m.def("hybrid_embed_rows", &embed_rows);
   m.def("hybrid_norm_rows", &norm_rows);
   m.def("hybrid_glu_rows", &glu_rows);
+  m.def("hybrid_side_rows", &side_rows);
+  m.def("hybrid_add_norm", &add_norm);
+  m.def("hybrid_rotation_rows", &rotation_rows);
+  m.def("hybrid_retention", &retention);
+  m.def("hybrid_latent_prep", &latent_prep);
+  m.def("hybrid_latent_attention", &latent_attention);
+  m.def("hybrid_latent_step", &latent_step);
+  m.def("hybrid_latent_step_splits", &tb::latent_step_splits);
   m.def("hybrid_gated_norm", &gated_norm);
   m.def("hybrid_causal_conv", &causal_conv);
   m.def("hybrid_recurrent", &recurrent, pybind11::arg("q"), pybind11::arg("k"), pybind11::arg("v"), pybind11::arg("a"), pybind11::arg("b"),

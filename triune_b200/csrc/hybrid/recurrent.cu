@@ -1,11 +1,11 @@
-// Token recurrence of the matrix-state mixers (Mamba-2 and gated delta rule), exact in fp32, any number of tokens.
+// Token recurrence of the matrix-state mixers (Mamba-2, gated delta rule and retention), exact in fp32, any number of tokens.
 //
 // The columns of a head's Dk x Dv state are independent given the head's keys, queries and scalars, so a head is cut
 // into slices of 16 columns and every slice is a block of four warps. A warp owns four columns; eight lanes share a
 // column and each keeps Dk / 8 of its rows in registers. Both contractions of a token act on the state BEFORE it:
 //   S_new = g S + k u^T   =>   S_new^T q = g S^T q + (k . q) u
 // so a token costs one pass over the registers and one 8-lane reduction. Tokens are staged 16 at a time: a warp loads
-// a token's key and query, makes them unit vectors where the rule asks for it, and leaves fp32 rows, k . q and the
+// a token's key and query, makes them unit vectors or turns them where the rule asks for it, and leaves fp32 rows, k . q and the
 // scalars (g, beta or dt) in shared memory.
 #include "hybrid.cuh"
 
@@ -35,10 +35,13 @@ __global__ void __launch_bounds__(RB_WARPS * 32) recurrent_kernel(const Recurren
   }
   const T *Q = (const T*)p.q + (long long)b * p.rows * p.ldq + kh * p.Dk, *K = (const T*)p.k + (long long)b * p.rows * p.ldk + kh * p.Dk;
   const T* V = (const T*)p.v + (long long)b * p.rows * p.ldv + h * p.Dv;
-  const T* A = (const T*)p.a + (long long)b * p.rows * p.lda + h;
+  const bool turn = p.kind == RK_RETENTION;
+  const T* A = turn ? nullptr : (const T*)p.a + (long long)b * p.rows * p.lda + h;
   const T* Bt = p.kind == RK_DELTA ? (const T*)p.b + (long long)b * p.rows * p.ldb + h : nullptr;
   T* O = (T*)p.out + (long long)b * p.rows * p.ldo + h * p.Dv;
-  const float ea = expf(p.A_log[h]), bias = p.dt_bias[h], Dh = p.kind == RK_MAMBA2 ? p.D[h] : 0.f;
+  const float ea = turn ? 0.f : expf(p.A_log[h]), bias = turn ? 0.f : p.dt_bias[h], Dh = p.kind == RK_MAMBA2 ? p.D[h] : 0.f;
+  const float fixed = turn ? (float)p.decay[h] : 0.f, ks = turn ? 1.f / sqrtf((float)p.Dk) : 1.f;
+  const int half = p.rot_dims / 2;
   const float qs = p.kind == RK_DELTA ? 1.f / sqrtf((float)p.Dk) : 1.f;
 
   for (int t0 = 0; t0 < p.T; t0 += RB_TOK) {
@@ -48,7 +51,14 @@ __global__ void __launch_bounds__(RB_WARPS * 32) recurrent_kernel(const Recurren
       const long long t = t0 + i;
       float kk = 0.f, qq = 0.f, kq = 0.f;
       for (int d = lane; d < DK; d += 32) {
-        const float kv = d < p.Dk ? ldf(K + t * p.ldk + d) : 0.f, qv = d < p.Dk ? ldf(Q + t * p.ldq + d) : 0.f;
+        float kv = d < p.Dk ? ldf(K + t * p.ldk + d) : 0.f, qv = d < p.Dk ? ldf(Q + t * p.ldq + d) : 0.f;
+        if (turn && d < p.rot_dims) {
+          const int i = d < half ? d : d - half, o = d < half ? d + half : d - half;
+          const float c = p.rot[t * p.rot_dims + i], s = d < half ? -p.rot[t * p.rot_dims + half + i] : p.rot[t * p.rot_dims + half + i];
+          kv = kv * c + ldf(K + t * p.ldk + o) * s;
+          qv = qv * c + ldf(Q + t * p.ldq + o) * s;
+        }
+        kv *= ks;
         sk[i][d] = kv;
         sq[i][d] = qv;
         kk += kv * kv;
@@ -66,8 +76,8 @@ __global__ void __launch_bounds__(RB_WARPS * 32) recurrent_kernel(const Recurren
       }
       if (lane < RB_COLS) sv[i][lane] = slice * RB_COLS + lane < p.Dv ? ldf(V + t * p.ldv + slice * RB_COLS + lane) : 0.f;
       if (lane == 0) {
-        const float dt = softplus_f(ldf(A + t * p.lda) + bias);
-        sg[i] = expf(-ea * dt);
+        const float dt = turn ? 1.f : softplus_f(ldf(A + t * p.lda) + bias);
+        sg[i] = turn ? fixed : expf(-ea * dt);
         sb[i] = p.kind == RK_DELTA ? sigmoid_f(ldf(Bt + t * p.ldb)) : dt;
         skq[i] = kq;
       }

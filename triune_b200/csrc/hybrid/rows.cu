@@ -113,13 +113,158 @@ __global__ void __launch_bounds__(128) norm_warp_kernel(const float* __restrict_
   }
 }
 
+// L lanes per row (a warp, or a block of 128), the row's sum in registers: NV float4 per lane.
+template <class Y, class T, int L, int NV>
+__global__ void __launch_bounds__(128) add_norm_vec_kernel(const AddNormArgs p) {
+  __shared__ float red[33];
+  const long long row = (long long)blockIdx.x * (128 / L) + threadIdx.x / L;
+  if (row >= p.rows) return;  // whole warps (L = 32), never part of a block (L = 128)
+  const int l = threadIdx.x % L;
+  float* xr = p.x + row * p.W;
+  const Y* yr = (const Y*)p.y + row * p.ldy;
+  auto sum = [&](float v) { return L == 32 ? warp_sum(v) : block_sum(v, red); };
+  float4 v[NV], x[NV];
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * L + l) * 4;
+    v[i] = x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < p.W) {
+      x[i] = *reinterpret_cast<const float4*>(xr + c);
+      if constexpr (sizeof(Y) == 4) {
+        v[i] = *reinterpret_cast<const float4*>(yr + c);
+      } else {
+        const uint2 u = *reinterpret_cast<const uint2*>(yr + c);
+        v[i] = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                           __uint_as_float(u.y & 0xffff0000u));
+      }
+      if (p.bias != nullptr) {
+        const float4 b = *reinterpret_cast<const float4*>(p.bias + c);
+        v[i] = make_float4(v[i].x + b.x, v[i].y + b.y, v[i].z + b.z, v[i].w + b.w);
+      }
+      s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    }
+  }
+  // v: norm of itself, times w; entries past W stay out of the sums
+  auto normed = [&](int kind, float total, const float* w, float eps) {
+    const float mean = kind == HN_LAYER ? sum(total) / p.W : 0.f;
+    float q = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if ((i * L + l) * 4 < p.W) {
+        v[i] = make_float4(v[i].x - mean, v[i].y - mean, v[i].z - mean, v[i].w - mean);
+        q += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+      }
+    const float r = 1.f / sqrtf(sum(q) / p.W + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * L + l) * 4;
+      if (c < p.W) {
+        const float4 g = *reinterpret_cast<const float4*>(w + c);
+        v[i] = make_float4(v[i].x * r * g.x, v[i].y * r * g.y, v[i].z * r * g.z, v[i].w * r * g.w);
+      }
+    }
+  };
+  normed(p.post_kind, s, p.post_w, p.post_eps);
+  s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * L + l) * 4;
+    if (c < p.W) {
+      v[i] = make_float4(x[i].x + v[i].x, x[i].y + v[i].y, x[i].z + v[i].z, x[i].w + v[i].w);
+      *reinterpret_cast<float4*>(xr + c) = v[i];
+      s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    }
+  }
+  if (p.out == nullptr) return;
+  if (p.pre_w != nullptr) normed(p.pre_kind, s, p.pre_w, p.pre_eps);
+  T* orow = (T*)p.out + row * p.W;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * L + l) * 4;
+    if (c < p.W) {
+      if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(orow + c) = v[i];
+      } else {
+        __nv_bfloat162 p0 = __floats2bfloat162_rn(v[i].x, v[i].y), p1 = __floats2bfloat162_rn(v[i].z, v[i].w);
+        uint2 u;
+        u.x = *reinterpret_cast<uint32_t*>(&p0);
+        u.y = *reinterpret_cast<uint32_t*>(&p1);
+        *reinterpret_cast<uint2*>(orow + c) = u;
+      }
+    }
+  }
+}
+
+// any width: a block per row, the row in shared memory (every thread re-reads only what it wrote)
+template <class Y, class T>
+__global__ void __launch_bounds__(256) add_norm_kernel(const AddNormArgs p) {
+  extern __shared__ float sx[];
+  __shared__ float red[33];
+  const long long row = blockIdx.x;
+  float* xr = p.x + row * p.W;
+  const Y* yr = (const Y*)p.y + row * p.ldy;
+  auto stats = [&](int kind, float total, float eps, float* mean) {
+    *mean = kind == HN_LAYER ? block_sum(total, red) / p.W : 0.f;
+    float q = 0.f;
+    for (int i = threadIdx.x; i < p.W; i += blockDim.x) q += (sx[i] - *mean) * (sx[i] - *mean);
+    return 1.f / sqrtf(block_sum(q, red) / p.W + eps);
+  };
+  float s = 0.f, mean;
+  for (int i = threadIdx.x; i < p.W; i += blockDim.x) {
+    sx[i] = ldf(yr + i) + (p.bias != nullptr ? p.bias[i] : 0.f);
+    s += sx[i];
+  }
+  float r = stats(p.post_kind, s, p.post_eps, &mean);
+  s = 0.f;
+  for (int i = threadIdx.x; i < p.W; i += blockDim.x) {
+    sx[i] = xr[i] + (sx[i] - mean) * r * p.post_w[i];
+    xr[i] = sx[i];
+    s += sx[i];
+  }
+  if (p.out == nullptr) return;
+  T* orow = (T*)p.out + row * p.W;
+  if (p.pre_w == nullptr) {
+    for (int i = threadIdx.x; i < p.W; i += blockDim.x) stf(orow + i, sx[i]);
+    return;
+  }
+  r = stats(p.pre_kind, s, p.pre_eps, &mean);
+  for (int i = threadIdx.x; i < p.W; i += blockDim.x) stf(orow + i, (sx[i] - mean) * r * p.pre_w[i]);
+}
+
 template <class T>
 __global__ void glu_rows_kernel(const T* __restrict__ gu, long long ld, T* __restrict__ out, long long ldo, int F,
-                                long long n, int act) {
+                                long long n, const GluArgs glu) {
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
     const long long row = i / F, c = i % F;
-    stf(out + row * ldo + c, act_f(ldf(gu + row * ld + c), act) * ldf(gu + row * ld + F + c));
+    float g = ldf(gu + row * ld + c), u = ldf(gu + row * ld + F + c);
+    if (glu.bias != nullptr) {
+      g += glu.bias[c];
+      u += glu.bias[F + c];
+    }
+    stf(out + row * ldo + c, glu_f(g, u, glu.act, glu.limit, glu.alpha));
   }
+}
+
+template <class T>
+__global__ void side_rows_kernel(const T* __restrict__ gate, long long ldg, const T* __restrict__ table, long long ldt,
+                                 const long long* __restrict__ ids, int V, int col0, T* __restrict__ out, int dim, long long n, int act) {
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+    const long long row = i / dim, c = i % dim, id = ids[row];
+    const float e = id >= 0 && id < V ? ldf(table + id * ldt + col0 + c) : 0.f;
+    stf(out + i, act_f(ldf(gate + row * ldg + c), act) * e);
+  }
+}
+
+__global__ void rotation_rows_kernel(const double* __restrict__ freqs, int n, float amplitude, float* __restrict__ out, long long total,
+                                     const Pos pos) {
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total) return;
+  const long long t = i / n, c = i % n;
+  float s, co;
+  rotation(pos_of(pos) + t, freqs[c], &s, &co);
+  out[t * 2 * n + c] = co * amplitude;
+  out[t * 2 * n + n + c] = s * amplitude;
 }
 
 // Gated norm of parts that are a multiple of eight wide: L lanes per part (L = 8, 16, 32 lanes of a warp, or L = 128, a
@@ -136,7 +281,7 @@ __global__ void __launch_bounds__(128) gated_norm_vec_kernel(const T* __restrict
   const long long row = id / groups;
   const int c0 = (int)(id % groups) * part;
   const T *yr = y + row * ldy + c0, *gr = gate + row * ldg + c0;
-  const float* wr = w + c0 % w_period;
+  const float* wr = w == nullptr ? nullptr : w + c0 % w_period;
   float v[NV][8], q = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
@@ -169,8 +314,8 @@ __global__ void __launch_bounds__(128) gated_norm_vec_kernel(const T* __restrict
   for (int i = 0; i < NV; ++i) {
     const int c = (i * L + l) * 8;
     if (on && c < part) {
-      float g[8];
-      ld8v(wr + c, g);
+      float g[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
+      if (wr != nullptr) ld8v(wr + c, g);
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[i][j] *= r * g[j];
       st8v(out + row * ldo + c0 + c, v[i]);
@@ -189,7 +334,7 @@ __global__ void gated_norm_kernel(const T* __restrict__ y, long long ldy, const 
   const long long row = id / groups;
   const int c0 = (int)(id % groups) * part;
   const T *yr = y + row * ldy + c0, *gr = gate + row * ldg + c0;
-  const float* wr = w + c0 % w_period;
+  const float* wr = w == nullptr ? nullptr : w + c0 % w_period;
   T* orow = out + row * ldo + c0;
   float q = 0.f;
   for (int i = lane; i < part; i += 32) {
@@ -200,7 +345,7 @@ __global__ void gated_norm_kernel(const T* __restrict__ y, long long ldy, const 
   const float r = scale / sqrtf(warp_sum(q) / part + eps);
   for (int i = lane; i < part; i += 32) {
     const float v = ldf(yr + i) * silu_f(ldf(gr + i));
-    stf(orow + i, v * r * wr[i]);
+    stf(orow + i, v * r * (wr != nullptr ? wr[i] : 1.f));
   }
 }
 
@@ -247,13 +392,68 @@ void launch_norm_rows(const float* x, const float* w, void* y, bool f32, int row
   check_launch("norm_rows");
 }
 
-void launch_glu_rows(const void* gu, long long ld, void* out, long long ldo, bool f32, int rows, int F, int act,
+void launch_add_norm(const AddNormArgs& a, cudaStream_t s) {
+  if (a.rows <= 0) return;
+  auto go = [&](auto* y, auto* out) {
+    using Y = std::remove_pointer_t<decltype(y)>;
+    using T = std::remove_pointer_t<decltype(out)>;
+    auto vec = [&](auto lanes, auto nv) {
+      constexpr int L = decltype(lanes)::value;
+      add_norm_vec_kernel<Y, T, L, decltype(nv)::value><<<(a.rows + 128 / L - 1) / (128 / L), 128, 0, s>>>(a);
+    };
+    using std::integral_constant;
+    const auto quad = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) & (4 * bytes - 1)) == 0; };
+    if (a.W % 4 == 0 && a.ldy % 4 == 0 && a.W <= 8192 && quad(a.x, 4) && quad(a.y, sizeof(Y)) && quad(a.bias, 4) && quad(a.post_w, 4) &&
+        quad(a.pre_w, 4) && quad(a.out, sizeof(T))) {
+      if (a.W <= 512) vec(integral_constant<int, 32>(), integral_constant<int, 4>());
+      else if (a.W <= 1024) vec(integral_constant<int, 32>(), integral_constant<int, 8>());
+      else if (a.W <= 2048) vec(integral_constant<int, 128>(), integral_constant<int, 4>());
+      else if (a.W <= 4096) vec(integral_constant<int, 128>(), integral_constant<int, 8>());
+      else vec(integral_constant<int, 128>(), integral_constant<int, 16>());
+      return;
+    }
+    const size_t sm = (size_t)a.W * 4;
+    if (sm > 160 * 1024) throw std::runtime_error("add_norm: rows of at most 40960 elements");
+    auto kern = add_norm_kernel<Y, T>;
+    if (sm > 47 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
+    kern<<<a.rows, 256, sm, s>>>(a);
+  };
+  if (a.y_f32) {
+    if (a.out_f32) go((float*)nullptr, (float*)nullptr);
+    else go((float*)nullptr, (__nv_bfloat16*)nullptr);
+  } else {
+    if (a.out_f32) go((__nv_bfloat16*)nullptr, (float*)nullptr);
+    else go((__nv_bfloat16*)nullptr, (__nv_bfloat16*)nullptr);
+  }
+  check_launch("add_norm");
+}
+
+void launch_side_rows(const void* gate, long long ldg, const void* table, long long ldt, const long long* ids, int V, int col0,
+                      void* out, bool f32, int rows, int dim, int act, cudaStream_t s) {
+  const long long n = (long long)rows * dim;
+  if (n <= 0) return;
+  const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+  if (f32) side_rows_kernel<<<blocks, 256, 0, s>>>((const float*)gate, ldg, (const float*)table, ldt, ids, V, col0, (float*)out, dim, n, act);
+  else
+    side_rows_kernel<<<blocks, 256, 0, s>>>((const __nv_bfloat16*)gate, ldg, (const __nv_bfloat16*)table, ldt, ids, V, col0, (__nv_bfloat16*)out,
+                                            dim, n, act);
+  check_launch("side_rows");
+}
+
+void launch_rotation_rows(const double* freqs, int n, float amplitude, float* out, int T, Pos pos, cudaStream_t s) {
+  const long long total = (long long)T * n;
+  if (total <= 0) return;
+  rotation_rows_kernel<<<(unsigned)((total + 255) / 256), 256, 0, s>>>(freqs, n, amplitude, out, total, pos);
+  check_launch("rotation_rows");
+}
+
+void launch_glu_rows(const void* gu, long long ld, void* out, long long ldo, bool f32, int rows, int F, const GluArgs& glu,
                      cudaStream_t s) {
   const long long n = (long long)rows * F;
   if (n <= 0) return;
   const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
-  if (f32) glu_rows_kernel<<<blocks, 256, 0, s>>>((const float*)gu, ld, (float*)out, ldo, F, n, act);
-  else glu_rows_kernel<<<blocks, 256, 0, s>>>((const __nv_bfloat16*)gu, ld, (__nv_bfloat16*)out, ldo, F, n, act);
+  if (f32) glu_rows_kernel<<<blocks, 256, 0, s>>>((const float*)gu, ld, (float*)out, ldo, F, n, glu);
+  else glu_rows_kernel<<<blocks, 256, 0, s>>>((const __nv_bfloat16*)gu, ld, (__nv_bfloat16*)out, ldo, F, n, glu);
   check_launch("glu_rows");
 }
 
@@ -264,7 +464,7 @@ void launch_gated_norm(const void* y, long long ldy, const void* gate, long long
   const long long parts = (long long)rows * groups;
   const int part = inner / groups;
   if (part % 8 == 0 && part <= 8192 && vec8_ok(y, ldy, f32) && vec8_ok(gate, ldg, f32) && vec8_ok(out, ldo, f32) &&
-      vec8_ok(w, 4, true) && w_period % 8 == 0) {
+      vec8_ok(w, 4, true) && (w == nullptr || w_period % 8 == 0)) {
     auto vec = [&](auto* yy, auto lanes, auto nv) {
       using T = std::remove_const_t<std::remove_pointer_t<decltype(yy)>>;
       constexpr int L = decltype(lanes)::value, NV = decltype(nv)::value;

@@ -3,6 +3,7 @@
 // whose epilogue adds into the residual or applies the gated activation, and one launch for the mixer itself.
 #include "../common/ptx.cuh"
 #include "hybrid.cuh"
+#include "step_common.cuh"
 
 namespace tb {
 namespace {
@@ -46,6 +47,29 @@ __device__ void segment_row(const GemvSegment& g, int b, float* dst, float* red,
     if constexpr (V == 4) *reinterpret_cast<float4*>(dst + i) = make_float4(f[0], f[1], f[2], f[3]);
     else dst[i] = f[0];
   };
+  // norm of the row in dst (its sum is s when that is needed), times weight and scale, in place
+  auto norm_row = [&](int kind, float s, const float* wt, float eps, float scale, auto&& use) {
+    const float mean = kind == HN_LAYER ? row_sum(s, nt, red, phase) / g.n : 0.f;
+    float q = 0.f;
+    for (int i = tid * V; i < g.n; i += step) {
+      float f[V];
+      each(dst, i, f);  // written by this thread
+#pragma unroll
+      for (int e = 0; e < V; ++e) q += (f[e] - mean) * (f[e] - mean);
+    }
+    const float r = scale / sqrtf(row_sum(q, nt, red, phase) / g.n + eps);
+#pragma unroll 2
+    for (int i = tid * V; i < g.n; i += step) {
+      float f[V], w[V];
+      each(dst, i, f);
+      each(wt, i, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) f[e] = (f[e] - mean) * r * w[e];
+      use(i, f);
+      put(i, f);
+    }
+  };
+  const auto nothing = [](int, float (&)[V]) {};
   if (g.kind == 0) {
 #pragma unroll 2
     for (int i = tid * V; i < g.n; i += step) {
@@ -56,7 +80,7 @@ __device__ void segment_row(const GemvSegment& g, int b, float* dst, float* red,
       put(i, f);
     }
   } else if (g.kind == 1) {
-    float s = 0.f, mean = 0.f;
+    float s = 0.f;
 #pragma unroll 2
     for (int i = tid * V; i < g.n; i += step) {
       float f[V];
@@ -65,24 +89,36 @@ __device__ void segment_row(const GemvSegment& g, int b, float* dst, float* red,
       for (int e = 0; e < V; ++e) s += f[e];
       put(i, f);
     }
-    if (g.norm_kind == HN_LAYER) mean = row_sum(s, nt, red, phase) / g.n;
-    float q = 0.f;
-    for (int i = tid * V; i < g.n; i += step) {
-      float f[V];
-      each(dst, i, f);  // written by this thread
-#pragma unroll
-      for (int e = 0; e < V; ++e) q += (f[e] - mean) * (f[e] - mean);
-    }
-    const float r = g.scale / sqrtf(row_sum(q, nt, red, phase) / g.n + g.eps);
+    norm_row(g.norm_kind, s, g.w, g.eps, g.scale, nothing);
+  } else if (g.kind == 3) {
+    const float* y = g.y + (long long)b * g.ldy;
+    float s = 0.f, total = 0.f;
 #pragma unroll 2
     for (int i = tid * V; i < g.n; i += step) {
-      float f[V], w[V];
-      each(dst, i, f);
-      each(g.w, i, w);
+      float f[V], a[V];
+      each(y, i, f);
+      if (g.y_bias != nullptr) {
+        each(g.y_bias, i, a);
 #pragma unroll
-      for (int e = 0; e < V; ++e) f[e] = (f[e] - mean) * r * w[e];
+        for (int e = 0; e < V; ++e) f[e] += a[e];
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) s += f[e];
       put(i, f);
     }
+    // every block forms the sum for itself; the first one leaves it for the kernels behind
+    float* keep = blockIdx.x == 0 && g.x_out != nullptr ? g.x_out + (long long)b * g.n : nullptr;
+    norm_row(g.post_kind, s, g.post_w, g.post_eps, 1.f, [&](int i, float (&f)[V]) {
+      float a[V];
+      each(x, i, a);
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        f[e] += a[e];
+        total += f[e];
+        if (keep != nullptr) keep[i + e] = f[e];
+      }
+    });
+    if (g.w != nullptr) norm_row(g.norm_kind, total, g.w, g.eps, g.scale, nothing);
   } else {
     // wide parts: all threads of the row on one part at a time; narrow parts: a warp per part
     const bool wide = part > 512 || nt == 32;
@@ -95,7 +131,12 @@ __device__ void segment_row(const GemvSegment& g, int b, float* dst, float* red,
         float f[V], z[V], w[V];
         each(x, c, f);
         each(gt, c, z);
-        each(g.w, g.w_period == g.n ? c : i, w);  // one weight per channel, or one part's weights for every part
+        if (g.w != nullptr) {
+          each(g.w, g.w_period == g.n ? c : i, w);  // one weight per channel, or one part's weights for every part
+        } else {
+#pragma unroll
+          for (int e = 0; e < V; ++e) w[e] = 1.f;
+        }
 #pragma unroll
         for (int e = 0; e < V; ++e) {
           const float a = silu_step<EXACT>(z[e]), in = g.norm_kind == GO_GATE_THEN_NORM ? f[e] * a : f[e];
@@ -118,50 +159,12 @@ __device__ void segment_row(const GemvSegment& g, int b, float* dst, float* red,
 
 template <bool EXACT>
 __device__ __forceinline__ void gemv_segment(const GemvSegment& g, int b, float* dst, float* red, int& phase, int tid, int nt) {
-  const bool quad = ((g.n | (int)g.ld | (g.n / g.groups) | g.w_period) & 3) == 0 && (g.kind != 2 || (g.ldg & 3) == 0) &&
+  const bool quad = ((g.n | (int)g.ld | (g.n / g.groups) | g.w_period) & 3) == 0 && (g.kind != 2 || (g.ldg & 3) == 0) && (g.kind != 3 || (g.ldy & 3) == 0) &&
                     ((reinterpret_cast<uintptr_t>(g.x) | reinterpret_cast<uintptr_t>(g.w) | reinterpret_cast<uintptr_t>(g.gate) |
+                      reinterpret_cast<uintptr_t>(g.y) | reinterpret_cast<uintptr_t>(g.y_bias) | reinterpret_cast<uintptr_t>(g.post_w) |
                       reinterpret_cast<uintptr_t>(dst)) & 15) == 0;
   if (quad) segment_row<EXACT, 4>(g, b, dst, red, phase, tid, nt);
   else segment_row<EXACT, 1>(g, b, dst, red, phase, tid, nt);
-}
-
-template <class T>
-__device__ __forceinline__ void unpack_vec(const uint4& u, float (&f)[16 / sizeof(T)]) {
-  if constexpr (sizeof(T) == 4) {
-    f[0] = __uint_as_float(u.x); f[1] = __uint_as_float(u.y); f[2] = __uint_as_float(u.z); f[3] = __uint_as_float(u.w);
-  } else {
-    const uint32_t a[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      f[2 * i] = __uint_as_float(a[i] << 16);
-      f[2 * i + 1] = __uint_as_float(a[i] & 0xffff0000u);
-    }
-  }
-}
-
-template <class T>
-__device__ __forceinline__ void load_vec(const T* p, float (&f)[16 / sizeof(T)]) {
-  unpack_vec<T>(*reinterpret_cast<const uint4*>(p), f);
-}
-
-// Programmatic dependent launch: the step's kernels follow one another closely, so each lets its successor start at once
-// and itself waits for its predecessor's results before it touches anything but weights.
-__device__ __forceinline__ void launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
-__device__ __forceinline__ void wait_for_previous() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
-
-template <class Args, class... Rest>
-void launch_chained(void (*kern)(Args, Rest...), int blocks, int threads, size_t smem, cudaStream_t s, const Args& a, Rest... rest) {
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(blocks);
-  cfg.blockDim = dim3(threads);
-  cfg.dynamicSmemBytes = smem;
-  cfg.stream = s;
-  cudaLaunchAttribute at[1];
-  at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  at[0].val.programmaticStreamSerializationAllowed = 1;
-  cfg.attrs = at;
-  cfg.numAttrs = 1;
-  cudaLaunchKernelEx(&cfg, kern, a, rest...);
 }
 
 // A warp works on two rows at a time (for the gated epilogue: a gate row and its up row).
@@ -269,13 +272,22 @@ __global__ void __launch_bounds__(GV_WARPS * 32, 2) gemv_kernel(const GemvArgs p
       const float s0 = warp_sum(a0[b]), s1 = warp_sum(a1[b]);
       if (lane == 0) {
         float* y = p.y + (long long)b * p.ldy;
-        if (glu) y[r0] = act_f(s0, p.act) * s1;
-        else if (p.epilogue == 1) {
-          y[r0] += s0;
-          if (two) y[r1] += s1;
+        const float* bias = p.glu.bias;
+        const float b0 = bias != nullptr ? bias[r0] : 0.f, b1 = bias != nullptr && (glu || two) ? bias[glu ? r0 + p.N : r1] : 0.f;
+        if (glu) {
+          y[r0] = glu_f(s0 + b0, s1 + b1, p.glu.act, p.glu.limit, p.glu.alpha);
+        } else if (p.epilogue == 1) {
+          y[r0] += s0 + b0;
+          if (two) y[r1] += s1 + b1;
+        } else if (p.epilogue == 3) {
+          const long long id = p.ids[b];
+          const bool ok = id >= 0 && id < p.V;
+          const T* e = (const T*)p.table + (ok ? id * p.ldt + p.col0 : 0);
+          y[r0] = ok ? act_f(s0, p.glu.act) * ldf(e + r0) : 0.f;
+          if (two) y[r1] = ok ? act_f(s1, p.glu.act) * ldf(e + r1) : 0.f;
         } else {
-          y[r0] = s0;
-          if (two) y[r1] = s1;
+          y[r0] = s0 + b0;
+          if (two) y[r1] = s1 + b1;
         }
       }
     }
@@ -301,6 +313,18 @@ __device__ float conv_step(const StepRecurrent& p, int b, int c, long long pos, 
   return silu_f(acc);
 }
 
+// Channel d of a head's query or key as retention has it: turned with the channel half of the rotated dimensions away.
+__device__ __forceinline__ float turned(const StepRecurrent& p, const float* head, int d, long long pos) {
+  const float v = head[d];
+  if (d >= p.rot_dims) return v;
+  const int half = p.rot_dims / 2, i = d < half ? d : d - half;
+  float s, c;
+  rotation(pos, p.freqs[i], &s, &c);
+  s *= p.amplitude;
+  c *= p.amplitude;
+  return d < half ? v * c - head[d + half] * s : v * c + head[d - half] * s;
+}
+
 __device__ void recurrent_step(const StepRecurrent& p, int block, long long pos, float* sm) {
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, sub = lane & 7;
   const int slices = (p.Dv + ST_COLS - 1) / ST_COLS;
@@ -309,10 +333,16 @@ __device__ void recurrent_step(const StepRecurrent& p, int block, long long pos,
   const int DP = (p.Dk + 31) & ~31;
   float *sk = sm, *sq = sk + DP, *sv = sq + DP, *red = sv + ST_COLS;
   const bool owner = slice == 0 && h % rep == 0;
+  const bool plain = p.kind == RK_RETENTION;
+  const float* pr = p.proj + (long long)b * p.ld;
+  const float ks = plain ? 1.f / sqrtf((float)p.Dk) : 1.f;
   float kk = 0.f, qq = 0.f, kq = 0.f;
   for (int d = tid; d < DP; d += ST_THREADS) {
-    const float kv = d < p.Dk ? conv_step(p, b, p.off_k + kh * p.Dk + d, pos, owner) : 0.f;
-    const float qv = d < p.Dk ? conv_step(p, b, p.off_q + kh * p.Dk + d, pos, owner) : 0.f;
+    float kv = 0.f, qv = 0.f;
+    if (d < p.Dk) {
+      kv = plain ? turned(p, pr + p.col_k + kh * p.Dk, d, pos) * ks : conv_step(p, b, p.off_k + kh * p.Dk + d, pos, owner);
+      qv = plain ? turned(p, pr + p.col_q + kh * p.Dk, d, pos) : conv_step(p, b, p.off_q + kh * p.Dk + d, pos, owner);
+    }
     sk[d] = kv;
     sq[d] = qv;
     kk += kv * kv;
@@ -321,7 +351,7 @@ __device__ void recurrent_step(const StepRecurrent& p, int block, long long pos,
   }
   if (tid < ST_COLS) {
     const int c = slice * ST_COLS + tid;
-    sv[tid] = c < p.Dv ? conv_step(p, b, p.off_v + h * p.Dv + c, pos, true) : 0.f;
+    sv[tid] = c >= p.Dv ? 0.f : plain ? pr[p.col_v + h * p.Dv + c] : conv_step(p, b, p.off_v + h * p.Dv + c, pos, true);
   }
   kq = block_sum(kq, red);
   float rk = 1.f, rq = 1.f;
@@ -329,9 +359,8 @@ __device__ void recurrent_step(const StepRecurrent& p, int block, long long pos,
     rk = 1.f / sqrtf(block_sum(kk, red) + p.unit_eps);
     rq = 1.f / (sqrtf(block_sum(qq, red) + p.unit_eps) * sqrtf((float)p.Dk));
   }
-  const float* pr = p.proj + (long long)b * p.ld;
-  const float dt = softplus_f(pr[p.col_a + h] + p.dt_bias[h]);
-  const float g = expf(-expf(p.A_log[h]) * dt);
+  const float dt = plain ? 1.f : softplus_f(pr[p.col_a + h] + p.dt_bias[h]);
+  const float g = plain ? (float)p.decay[h] : expf(-expf(p.A_log[h]) * dt);
   const int cl = warp * 4 + (lane >> 3), col = slice * ST_COLS + cl;
   const bool live = col < p.Dv;
   float* st = p.state + (long long)bh * p.Dk * p.Dv;
@@ -389,9 +418,6 @@ __device__ void head_row(const float* src, const float* w, float eps, int D, int
   }
   for (int d = D + lane; d < padded; d += 32) dst[d] = 0.f;
 }
-
-// Floats of one partial result: maximum, sum, two of padding, the values padded to whole quads.
-__host__ __device__ constexpr int part_stride(int E) { return ((E + 3) & ~3) + 4; }
 
 // Keys of split `s` of `splits` over n keys: whole multiples of 32, at least 64 keys per split.
 __device__ __forceinline__ void split_range(int n, int splits, int s, int* k0, int* k1) {
