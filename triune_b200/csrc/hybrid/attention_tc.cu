@@ -101,41 +101,41 @@ __global__ void __launch_bounds__(FA_THREADS, 1) attn_tc_kernel(const __grid_con
         for (int d = 0; d < DKB; ++d) tma_load_4d(sQ + (w * KB + d) * FA_BOX, &tmQ, q_full, d * 64, q0 + w * FA_BM, h, b);
         for (int d = 0; d < RKB; ++d) tma_load_4d(sQ + (w * KB + DKB + d) * FA_BOX, &tmQ2, q_full, d * 64, q0 + w * FA_BM, h, b);
       }
-      auto keys = [&](int j) {
-        const int s = j & 1;
-        if (j >= 2 && !mbar_wait(k_empty + s, ((j >> 1) & 1) ^ 1)) return false;
-        mbar_expect_tx(k_full + s, KB * FA_BOX);
-        for (int d = 0; d < DKB; ++d) tma_load_4d(sK + (s * KB + d) * FA_BOX, &tmK, k_full + s, d * 64, j * FA_BN, kvh, b);
-        for (int d = 0; d < RKB; ++d) tma_load_4d(sK + (s * KB + DKB + d) * FA_BOX, &tmK2, k_full + s, d * 64, j * FA_BN, 0, b);
-        return true;
-      };
-      bool ok = keys(0);
-      for (int j = 0; j < nt && ok; ++j) {
-        if (j + 1 < nt) ok = keys(j + 1);  // ahead of these values: the scores of the next tile are issued before their use ends
-        if (!ok) break;
-        const int s = j % VS;
-        if (j >= VS) ok = mbar_wait(v_empty + s, ((j / VS) & 1) ^ 1);
-        if (!ok) break;
-        mbar_expect_tx(v_full + s, EVB * FA_BOX);
-        for (int d = 0; d < EVB; ++d) tma_load_4d(sV + (s * EVB + d) * FA_BOX, &tmV, v_full + s, d * 64, j * FA_BN, kvh, b);
+      bool ok = true;
+      // keys run one tile ahead of values: the scores of the next tile are issued before the use of these values ends
+      for (int j = 0; j <= nt && ok; ++j) {
+        if (j < nt) {
+          const int s = j & 1;
+          if (j >= 2) ok = mbar_wait(k_empty + s, ((j >> 1) & 1) ^ 1);
+          if (!ok) break;
+          mbar_expect_tx(k_full + s, KB * FA_BOX);
+          for (int d = 0; d < DKB; ++d) tma_load_4d(sK + (s * KB + d) * FA_BOX, &tmK, k_full + s, d * 64, j * FA_BN, kvh, b);
+          for (int d = 0; d < RKB; ++d) tma_load_4d(sK + (s * KB + DKB + d) * FA_BOX, &tmK2, k_full + s, d * 64, j * FA_BN, 0, b);
+        }
+        if (j > 0) {
+          const int i = j - 1, s = i % VS;
+          if (i >= VS) ok = mbar_wait(v_empty + s, ((i / VS) & 1) ^ 1);
+          if (!ok) break;
+          mbar_expect_tx(v_full + s, EVB * FA_BOX);
+          for (int d = 0; d < EVB; ++d) tma_load_4d(sV + (s * EVB + d) * FA_BOX, &tmV, v_full + s, d * 64, i * FA_BN, kvh, b);
+        }
       }
       if (!ok && p.status) *p.status = ST_TIMEOUT_EMPTY;
     }
   } else if (warp == 1) {
     if (lane == 0) {
       const uint32_t id_s = make_idesc(128, 128, 1, 1, 0, 0), id_o = make_idesc(128, (p.E + 15) / 16 * 16, 1, 1, 0, 1);
-      const int ks = (p.D + 15) / 16, rs = (p.R + 15) / 16;
+      const int ks = (p.D + 15) / 16, rs = RKB > 0 ? (p.R + 15) / 16 : 0;
       auto scores = [&](int w, int j) {
         const uint32_t qa = smem_u32(sQ + w * KB * FA_BOX), ka = smem_u32(sK + (j & 1) * KB * FA_BOX);
         for (int k = 0; k < ks; ++k) {
           const uint32_t off = (k >> 2) * FA_BOX + (k & 3) * 32;
           umma_bf16(tmem + w * 128, make_smem_desc(qa + off, 16, 1024), make_smem_desc(ka + off, 16, 1024), id_s, k > 0);
         }
-        if constexpr (RKB > 0)
-          for (int k = 0; k < rs; ++k) {
-            const uint32_t off = (DKB + (k >> 2)) * FA_BOX + (k & 3) * 32;
-            umma_bf16(tmem + w * 128, make_smem_desc(qa + off, 16, 1024), make_smem_desc(ka + off, 16, 1024), id_s, 1);
-          }
+        for (int k = 0; k < rs; ++k) {
+          const uint32_t off = (DKB + (k >> 2)) * FA_BOX + (k & 3) * 32;
+          umma_bf16(tmem + w * 128, make_smem_desc(qa + off, 16, 1024), make_smem_desc(ka + off, 16, 1024), id_s, 1);
+        }
         umma_commit(s_full + w);
       };
       auto values = [&](int w, int j) {
