@@ -55,21 +55,28 @@ def latent_rows(h, W, c, eps):
     return lat, rotate_halves(z[:, None, r:], torch.arange(h.shape[0]), {**c["rot"], "dims": c["rot_dim"]})[:, 0]
 
 
+def latent_core(q, qr, lat, krot, uk, uv, gate, sink, scale):
+    """q [T, H, D], qr [T, H, R] turned, lat [T, rank], krot [T, R] turned, uk [H, D, rank], uv [H, E, rank], gate [T, H] or
+    None, sink [H] or None -> [T, H, E]"""
+    T, H, _ = q.shape
+    out = torch.zeros(T, H, uv.shape[1], dtype=q.dtype)
+    for n in range(H):
+        k, v = lat @ uk[n].T, lat @ uv[n].T
+        for t in range(T):
+            s = (k[: t + 1] @ q[t, n] + krot[: t + 1] @ qr[t, n]) * scale
+            m = s.max() if sink is None else torch.maximum(s.max(), sink[n])
+            p = torch.exp(s - m)
+            total = p.sum() if sink is None else p.sum() + torch.exp(sink[n] - m)
+            out[t, n] = (p @ v[: t + 1]) / total * (1 if gate is None else gate[t, n])
+    return out
+
+
 def latent_attention(h, W, c, lat, krot):
     T = h.shape[0]
     H, D, R, E, rank = c["heads"], c["dim"], c["rot_dim"], c["vdim"], c["kv_rank"]
     q = (h @ W["q"].T).view(T, H, D + R)
     qr = rotate_halves(q[..., D:], torch.arange(T), {**c["rot"], "dims": R})
-    gate = sigmoid(h @ W["g"].T)
-    out = torch.zeros(T, H, E, dtype=h.dtype)
-    for n in range(H):
-        k = lat @ W["uk"].view(H, D, rank)[n].T
-        v = lat @ W["uv"].view(H, E, rank)[n].T
-        for t in range(T):
-            s = (k[: t + 1] @ q[t, n, :D] + krot[: t + 1] @ qr[t, n]) * c["scale"]
-            m = torch.maximum(s.max(), W["sink"][n])
-            p = torch.exp(s - m)
-            out[t, n] = gate[t, n] * (p @ v[: t + 1]) / (p.sum() + torch.exp(W["sink"][n] - m))
+    out = latent_core(q[..., :D], qr, lat, krot, W["uk"].view(H, D, rank), W["uv"].view(H, E, rank), sigmoid(h @ W["g"].T), W["sink"], c["scale"])
     return out.reshape(T, H * E) @ W["o"].T
 
 
@@ -129,3 +136,51 @@ def forward(cfg, W, tokens, dtype=torch.float64, want_layers=False):
         layers.append(x)
     logits = rms_norm(x, W["final.norm"], eps) @ W["head"].T
     return (logits, torch.stack(layers)) if want_layers else logits
+
+
+def make_config(layers, vocab=70, width=40, eps=1e-5, side=6):
+    return {"architecture": "Bubitar", "layers": layers, "norm": {"eps": eps}, "token_side": {"dim": side}, "vocab": vocab, "width": width}
+
+
+def make_weights(cfg, seed=0, dtype=torch.bfloat16):
+    """Random weights of the shapes ``cfg`` implies, rounded to ``dtype``."""
+    g = torch.Generator().manual_seed(seed)
+    W, d, dim = {}, cfg["width"], cfg["token_side"]["dim"]
+
+    def lin(name, o, i, gain=1.0):
+        W[name] = torch.randn(o, i, generator=g) * gain / math.sqrt(i)
+
+    def vec(name, n, lo, hi):
+        W[name] = lo + (hi - lo) * torch.rand(n, generator=g)
+
+    lin("embed", cfg["vocab"], d, math.sqrt(d))
+    lin("side.embed", cfg["vocab"], dim * len(cfg["layers"]), math.sqrt(dim * len(cfg["layers"])))
+    for i, s in enumerate(cfg["layers"]):
+        p, c, m = f"l{i}.", s["mixer"], f"l{i}.mix."
+        H, D, E = c["heads"], c["dim"], c["vdim"]
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if s["mlp"] is not None else ()):
+            vec(p + n, d, 0.5, 1.5)
+        lin(m + "o", d, H * E)
+        if s["type"] == "retention":
+            for n, rows in (("q", H * D), ("k", H * D), ("v", H * E), ("g", H * E)):
+                lin(m + n, rows, d)
+        else:
+            lin(m + "q", H * (D + c["rot_dim"]), d, 1.5)
+            if c.get("kv_from") is None:
+                lin(m + "dkv", c["kv_rank"] + c["rot_dim"], d, 1.5)
+                vec(m + "dkv.norm", c["kv_rank"], 0.6, 1.6)
+            lin(m + "uk", H * D, c["kv_rank"], 1.5)
+            lin(m + "uv", H * E, c["kv_rank"])
+            vec(m + "sink", H, -1.0, 2.0)
+            lin(m + "g", H, d)
+        if s["mlp"] is not None:
+            F = s["mlp"]["ff"]
+            for n, rows, cols in (("gate", F, d), ("up", F, d), ("down", d, F)):
+                lin(p + "mlp." + n, rows, cols, 1.5)
+                vec(f"{p}mlp.{n}.b", rows, -0.5, 0.5)
+        lin(p + "side.gate", dim, d)
+        lin(p + "side.proj", d, dim)
+        vec(p + "side.norm", d, 0.3, 1.0)
+    vec("final.norm", d, 0.5, 1.5)
+    lin("head", cfg["vocab"], d)
+    return {k: v.to(dtype) for k, v in W.items()}

@@ -54,10 +54,10 @@ CONFIGS = {
 
 
 def build(cfg, W, device="cpu", dtype=torch.float32):
-    from triune_b200.models import Famalorn
+    from triune_b200.models.zoo import MODEL_REGISTRY
     from triune_b200.utils import place_model
 
-    m = Famalorn(config=cfg)
+    m = MODEL_REGISTRY[cfg["architecture"].lower()](config=cfg)
     m.load_named(W)
     return place_model(m, device, dtype).eval()
 
