@@ -491,6 +491,8 @@ def main():
                          "(the faster one is reported)")
     ap.add_argument("--workload", default="train", choices=["train", "hybrid"],
                     help="train: the headline benchmark; hybrid: serving of heterogeneous-layer models, one JSON line per measurement")
+    ap.add_argument("--hybrid-design", default="famalorn", choices=["famalorn", "bubitar"],
+                    help="design of the hybrid workload: famalorn (beside the dense family) or bubitar (beside famalorn)")
     ap.add_argument("--hybrid-size", default="1b,3b", help="comma-separated layer sizes of the hybrid workload (1b, 3b)")
     ap.add_argument("--hybrid-seq", type=int, default=8192, help="prompt length of the hybrid workload")
     ap.add_argument("--hybrid-parts", default="model,kernels")
@@ -504,7 +506,7 @@ def main():
 
         sampler = ClockSampler(0)
         sampler.start()
-        run_hybrid(args.hybrid_size.split(","), args.hybrid_seq, args.hybrid_parts)
+        run_hybrid(args.hybrid_size.split(","), args.hybrid_seq, args.hybrid_parts, design=args.hybrid_design)
         print(json.dumps({"workload": "hybrid", "clocks": sampler.stop()}), flush=True)
         return
     if args.impl == "reference":
