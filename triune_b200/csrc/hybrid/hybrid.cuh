@@ -108,6 +108,10 @@ void launch_chunk_scan(const RecurrentArgs& a, void* scratch, cudaStream_t s);
 bool ssd_tc_supported(const RecurrentArgs& a);
 long long ssd_tc_scratch(const RecurrentArgs& a);
 void launch_ssd_tc(const RecurrentArgs& a, void* scratch, int* status, cudaStream_t s);
+// Retention prompts on tcgen05 (aligned bf16, key sizes up to 128), every chunk of 128 tokens on its own.
+bool retention_tc_supported(const RecurrentArgs& a);
+long long retention_tc_scratch(const RecurrentArgs& a);
+void launch_retention_tc(const RecurrentArgs& a, void* scratch, int* status, cudaStream_t s);
 // [nseg, B, H, Dk, Dv] contributions of segments (then [nseg, B, H] decays) -> states before the segments, from a.state
 void launch_ssd_scan(const RecurrentArgs& a, float* seg_state, int nseg, cudaStream_t s);
 

@@ -249,7 +249,30 @@ void retention(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& 
   r.rot_dims = (int)rot.size(1);
   r.decay = f64v(decay, H, "decay");
   c10::cuda::CUDAGuard guard(q.device());
-  tb::launch_recurrent(r, cur_stream());
+  if (!chunked || !tb::retention_tc_supported(r)) {
+    tb::launch_recurrent(r, cur_stream());
+    return;
+  }
+  // prompts longer than the scratch budget go in parts: the state carries over
+  constexpr int64_t budget = 1024ll << 20;
+  tb::RecurrentArgs part = r;
+  int64_t per = (T + 127) / 128 * 128;
+  while (per > 2048 && (part.T = (int)std::min(per, T), tb::retention_tc_scratch(part)) > budget) per = (per / 2 + 127) / 128 * 128;
+  Tensor scratch;
+  for (int64_t t = 0; t < T; t += per) {
+    part.T = (int)std::min(per, T - t);
+    auto at = [&](const void* p, int64_t ld) { return static_cast<const char*>(p) + t * ld * 2; };
+    part.q = at(r.q, r.ldq); part.k = at(r.k, r.ldk); part.v = at(r.v, r.ldv);
+    part.out = const_cast<char*>(at(r.out, r.ldo));
+    part.rot = r.rot + t * r.rot_dims;
+    if (!tb::retention_tc_supported(part)) {  // a short rest
+      tb::launch_recurrent(part, cur_stream());
+      continue;
+    }
+    const int64_t need = tb::retention_tc_scratch(part);
+    if (!scratch.defined() || scratch.numel() < need) scratch = torch::empty({need}, q.options().dtype(at::kByte));
+    tb::launch_retention_tc(part, scratch.data_ptr(), status_of(status), cur_stream());
+  }
 }
 
 bool cache_of(const Tensor& c, int64_t B, int64_t G, int64_t d, const char* n) {

@@ -58,9 +58,6 @@ __global__ void __launch_bounds__(128) ssd_tc_factors_kernel(const SsdTcParams s
   }
 }
 
-// 16-byte piece `ch` (of 8) of row r of a swizzled tile
-__device__ __forceinline__ uint32_t sw(int r, int ch) { return (uint32_t)(r * 128 + ((ch ^ (r & 7)) << 4)); }
-
 // Rows t0 .. t0 + 127 and `boxes` tiles of 64 columns into swizzled tiles; rows past T and columns past D become zero.
 __device__ __forceinline__ void stage_tile(uint8_t* dst, const __nv_bfloat16* src, long long ld, int t0, int T, int D, int boxes, int tid) {
   const int ch = tid & 7, r0 = tid >> 3;

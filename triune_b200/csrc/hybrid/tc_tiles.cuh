@@ -35,6 +35,9 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
+// 16-byte piece `ch` (of 8) of row r of a swizzled tile
+__device__ __forceinline__ uint32_t sw(int r, int ch) { return (uint32_t)(r * 128 + ((ch ^ (r & 7)) << 4)); }
+
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void cp_wait0() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 
