@@ -69,7 +69,15 @@ __global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(const LatentSt
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[33];
   const int tid = threadIdx.x, unit = blockIdx.x, b = unit / (slices * p.H + 1), w = unit % (slices * p.H + 1);
-  const int pitch = p.rank_p + p.Rp;
+  const int pitch = p.rank_p + p.Rp, h = w / slices, c0 = (w % slices) * LQ_COLS;
+  const int tx = tid % TX, gr = tid / TX, col = c0 + tx * VEC;
+  const bool work = h < p.H && col < p.rank_p;  // rank_p is a multiple of eight
+  const T* up = (const T*)p.up + (long long)h * (p.Dp + p.Ep) * p.rank_p + col;
+  constexpr int PRE = 4;  // weights fetched before the wait: they do not depend on the previous kernel
+  uint4 pre[PRE];
+#pragma unroll
+  for (int i = 0; i < PRE; ++i)
+    if (work && gr + i * GR < p.D) pre[i] = *reinterpret_cast<const uint4*>(up + (long long)(gr + i * GR) * p.rank_p);
   launch_dependents();
   wait_for_previous();
   const long long pos = pos_of(p.pos);
@@ -85,7 +93,6 @@ __global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(const LatentSt
     for (int i = tid; i < p.Rp; i += LQ_THREADS) stf(dst + p.rank_p + i, i < p.R ? turn_part(p, z + p.rank_p, i, pos) : 0.f);
     return;
   }
-  const int h = w / slices, c0 = (w % slices) * LQ_COLS;
   const float* q = pr + p.col_q + h * (p.Dp + p.Rp);
   float* qa = p.qa + ((long long)b * p.H + h) * pitch;
   float *sq = sm, *acc = sm + p.Dp;
@@ -93,19 +100,21 @@ __global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(const LatentSt
   if (c0 == 0)
     for (int i = tid; i < p.Rp; i += LQ_THREADS) qa[p.rank_p + i] = i < p.R ? turn_part(p, q + p.Dp, i, pos) : 0.f;
   __syncthreads();
-  const int tx = tid % TX, gr = tid / TX, col = c0 + tx * VEC;
   float a[VEC];
 #pragma unroll
   for (int i = 0; i < VEC; ++i) a[i] = 0.f;
-  if (col < p.rank_p) {  // rank_p is a multiple of eight
-    const T* up = (const T*)p.up + (long long)h * (p.Dp + p.Ep) * p.rank_p + col;
-#pragma unroll 4
-    for (int d = gr; d < p.D; d += GR) {
+  if (work) {
+    auto take = [&](const uint4& u, int d) {
       float f[VEC];
-      load_vec(up + (long long)d * p.rank_p, f);
+      unpack_vec<T>(u, f);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) a[i] += f[i] * sq[d];
-    }
+    };
+#pragma unroll
+    for (int i = 0; i < PRE; ++i)
+      if (gr + i * GR < p.D) take(pre[i], gr + i * GR);
+#pragma unroll 4
+    for (int d = gr + PRE * GR; d < p.D; d += GR) take(*reinterpret_cast<const uint4*>(up + (long long)d * p.rank_p), d);
   }
 #pragma unroll
   for (int i = 0; i < VEC; ++i) acc[gr * LQ_COLS + tx * VEC + i] = a[i];
@@ -127,7 +136,7 @@ __device__ __forceinline__ void latent_range(long long n, int splits, int s, int
   *k1 = min((int)n, *k0 + per);
 }
 
-// Any sizes, fp32 arithmetic: blocks (split, head, sequence); a warp per key for the scores, a thread per column for the sums.
+// Any sizes and fp32 caches, fp32 arithmetic: blocks (split, head, sequence); a warp per key for the scores, a thread per column for the sums.
 template <class T>
 __global__ void __launch_bounds__(LS_THREADS) latent_step_kernel(const LatentStepArgs p) {
   constexpr int VEC = 16 / sizeof(T), NC = 2048 / LS_THREADS;
@@ -201,6 +210,183 @@ __global__ void __launch_bounds__(LS_THREADS) latent_step_kernel(const LatentSte
   }
 }
 
+// bf16 caches on the tensor cores, up to 16 heads at a time: blocks (split, group of 16 heads, sequence). Queries are fp32
+// and enter as two bf16 numbers, cached rows are exact operands, softmax weights enter as two bf16 numbers again. A warp has
+// eight keys of a tile of 64 for the scores, and NG times 16 columns of the latent for the sums; the accumulators stay in
+// registers while two tiles of rows alternate in shared memory.
+constexpr int LM_THREADS = 256, LM_KEYS = 64, LM_PITCH = 640;
+
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ld_matrix(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p))
+               : "memory");
+}
+__device__ __forceinline__ void ld_matrix_t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
+               : "r"(smem_u32(p))
+               : "memory");
+}
+__host__ __device__ constexpr int lm_row(int pitch) { return (pitch + 31) / 32 * 32 + 8; }  // shared-memory row, no bank conflicts
+constexpr int LM_PROW = LM_KEYS + 8;
+inline size_t lm_smem(int pitch) {
+  return (size_t)(2 * 16 + 2 * LM_KEYS) * lm_row(pitch) * 2 + 16 * LM_KEYS * 4 + 2 * 16 * LM_PROW * 2 + 3 * 16 * 4;
+}
+
+template <int NG>
+__global__ void __launch_bounds__(LM_THREADS) latent_step_mma_kernel(const LatentStepArgs p) {
+  using bf16 = __nv_bfloat16;
+  extern __shared__ __align__(16) uint8_t lm_raw[];
+  const int pitch = p.rank_p + p.Rp, row = lm_row(pitch), groups = (p.H + 15) / 16;
+  bf16 *qh = reinterpret_cast<bf16*>(lm_raw), *ql = qh + 16 * row, *keys = ql + 16 * row;
+  float* ss = reinterpret_cast<float*>(keys + 2 * LM_KEYS * row);
+  bf16 *ph = reinterpret_cast<bf16*>(ss + 16 * LM_KEYS), *pl = ph + 16 * LM_PROW;
+  float *sm_m = reinterpret_cast<float*>(pl + 16 * LM_PROW), *sm_l = sm_m + 16, *sm_c = sm_l + 16;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int split = blockIdx.x % p.splits, u = blockIdx.x / p.splits, grp = u % groups, b = u / groups, h0 = grp * 16, nh = min(16, p.H - h0);
+  launch_dependents();
+  wait_for_previous();
+  const long long pos = pos_of(p.pos);
+  int k0 = 0, k1 = 0;
+  if (pos >= 0 && pos < p.cap) latent_range(pos + 1, p.splits, split, &k0, &k1);
+  const bf16* C = (const bf16*)p.cache + (long long)b * p.cap * pitch;
+  const int pieces = pitch / 8, wide = (row - 8) / 8;  // 16-byte pieces of a cached row, and with the zeros behind it
+  auto stage = [&](int buf, int kb) {
+    bf16* dst = keys + buf * LM_KEYS * row;
+    for (int i = tid; i < LM_KEYS * wide; i += LM_THREADS) {
+      const int r = i / wide, c = i % wide;
+      const bool on = kb + r < k1 && c < pieces;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * row + c * 8)),
+                   "l"(on ? C + (long long)(kb + r) * pitch + c * 8 : C), "r"(on ? 16 : 0)
+                   : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (k0 < k1) stage(0, k0);
+  const float* qa = p.qa + ((long long)b * p.H + h0) * pitch;
+  for (int i = tid; i < 16 * (row - 8) / 2; i += LM_THREADS) {
+    const int r = i / ((row - 8) / 2), c = (i % ((row - 8) / 2)) * 2;
+    const bool on = r < nh && c < pitch;
+    const float x = on ? qa[r * pitch + c] : 0.f, y = on ? qa[r * pitch + c + 1] : 0.f;
+    const uint32_t hi = pack_bf16x2(x, y);
+    *reinterpret_cast<uint32_t*>(qh + r * row + c) = hi;
+    *reinterpret_cast<uint32_t*>(ql + r * row + c) = pack_bf16x2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
+  }
+  if (tid < 16) {
+    sm_m[tid] = -INFINITY;
+    sm_l[tid] = 0.f;
+  }
+  float acc[NG][8];
+#pragma unroll
+  for (int g = 0; g < NG; ++g)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[g][e] = 0.f;
+  const int a_off = (lane & 15) * row + (lane >> 4) * 8;
+  for (int kb = k0, buf = 0; kb < k1; kb += LM_KEYS, buf ^= 1) {
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    if (kb + LM_KEYS < k1) stage(buf ^ 1, kb + LM_KEYS);
+    const bf16* kt = keys + buf * LM_KEYS * row;
+    float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
+    const bf16* kr = kt + (warp * 8 + (lane & 7)) * row + (lane >> 3) * 8;
+#pragma unroll 4
+    for (int d = 0; d < row - 8; d += 32) {
+      uint32_t kv[4], a0[4], a1[4], l0[4], l1[4];
+      ld_matrix(kv, kr + d);
+      ld_matrix(a0, qh + a_off + d);
+      ld_matrix(a1, qh + a_off + d + 16);
+      ld_matrix(l0, ql + a_off + d);
+      ld_matrix(l1, ql + a_off + d + 16);
+      mma_bf16(s, a0, kv[0], kv[1]);
+      mma_bf16(s2, l0, kv[0], kv[1]);
+      mma_bf16(s, a1, kv[2], kv[3]);
+      mma_bf16(s2, l1, kv[2], kv[3]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int key = warp * 8 + 2 * (lane & 3) + (e & 1), hh = (lane >> 2) + (e >> 1) * 8;
+      ss[hh * LM_KEYS + key] = kb + key < k1 ? (s[e] + s2[e]) * p.scale : -INFINITY;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int hh = warp * 2 + i;
+      const float x0 = ss[hh * LM_KEYS + 2 * lane], x1 = ss[hh * LM_KEYS + 2 * lane + 1];
+      const float mo = sm_m[hh], mn = fmaxf(mo, warp_max(fmaxf(x0, x1)));  // every tile has a key: finite
+      const float e0 = expf(x0 - mn), e1 = expf(x1 - mn), l = warp_sum(e0 + e1);
+      const uint32_t hi = pack_bf16x2(e0, e1);
+      *reinterpret_cast<uint32_t*>(ph + hh * LM_PROW + 2 * lane) = hi;
+      *reinterpret_cast<uint32_t*>(pl + hh * LM_PROW + 2 * lane) =
+          pack_bf16x2(e0 - __uint_as_float(hi << 16), e1 - __uint_as_float(hi & 0xffff0000u));
+      __syncwarp();
+      if (lane == 0) {
+        const float c = expf(mo - mn);
+        sm_c[hh] = c;
+        sm_l[hh] = sm_l[hh] * c + l;
+        sm_m[hh] = mn;
+      }
+    }
+    __syncthreads();
+    const float c0 = sm_c[lane >> 2], c1 = sm_c[(lane >> 2) + 8];
+    uint32_t wh[4][4], wl[4][4];
+#pragma unroll
+    for (int t = 0; t < 4; ++t) {
+      ld_matrix(wh[t], ph + (lane & 15) * LM_PROW + t * 16 + (lane >> 4) * 8);
+      ld_matrix(wl[t], pl + (lane & 15) * LM_PROW + t * 16 + (lane >> 4) * 8);
+    }
+#pragma unroll
+    for (int g = 0; g < NG; ++g) {
+      const int col = (warp + 8 * g) * 16;
+      if (col < p.rank_p) {
+        float lo[4], hi[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          lo[e] = acc[g][e] * (e < 2 ? c0 : c1);
+          hi[e] = acc[g][4 + e] * (e < 2 ? c0 : c1);
+        }
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+          uint32_t v[4];
+          ld_matrix_t(v, kt + (t * 16 + (lane & 15)) * row + col + (lane >> 4) * 8);
+          mma_bf16(lo, wh[t], v[0], v[1]);
+          mma_bf16(hi, wh[t], v[2], v[3]);
+          mma_bf16(lo, wl[t], v[0], v[1]);
+          mma_bf16(hi, wl[t], v[2], v[3]);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          acc[g][e] = lo[e];
+          acc[g][4 + e] = hi[e];
+        }
+      }
+    }
+  }
+  __syncthreads();
+  const int ES = part_stride(p.rank_p);
+  auto part_of = [&](int hh) { return p.part + (((long long)b * p.H + h0 + hh) * p.splits + split) * ES; };
+  if (tid < nh) {
+    float* o = part_of(tid);
+    o[0] = sm_m[tid];
+    o[1] = sm_l[tid];
+  }
+  if (k0 >= k1) return;  // the combination does not read the values of empty splits
+#pragma unroll
+  for (int g = 0; g < NG; ++g) {
+    const int col = (warp + 8 * g) * 16 + 2 * (lane & 3);
+#pragma unroll
+    for (int e = 0; e < 8; e += 2) {
+      const int hh = (lane >> 2) + ((e >> 1) & 1) * 8, c = col + (e >> 2) * 8;
+      if (hh < nh && c < p.rank_p) *reinterpret_cast<float2*>(part_of(hh) + 4 + c) = make_float2(acc[g][e], acc[g][e + 1]);
+    }
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ step: values
 constexpr int LV_THREADS = 256, LV_ROWS = 32;
 
@@ -213,6 +399,16 @@ __global__ void __launch_bounds__(LV_THREADS) latent_value_kernel(const LatentSt
   const int slice = blockIdx.x % slices, bh = blockIdx.x / slices, h = bh % p.H, b = bh / p.H;
   const int ES = part_stride(p.rank_p);
   float *sa = sm, *sc = sm + p.rank_p;
+  constexpr int ROWS = LV_ROWS / (LV_THREADS / 32), PRE = 2;  // rows per warp; pieces of a row fetched before the wait
+  const T* up = (const T*)p.up + ((long long)h * (p.Dp + p.Ep) + p.Dp) * p.rank_p;
+  uint4 pre[ROWS][PRE];
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+    const int r = slice * LV_ROWS + warp + i * (LV_THREADS / 32);
+#pragma unroll
+    for (int j = 0; j < PRE; ++j)
+      if (r < p.E && (j * 32 + lane) * VEC < p.rank_p) pre[i][j] = *reinterpret_cast<const uint4*>(up + (long long)r * p.rank_p + (j * 32 + lane) * VEC);
+  }
   launch_dependents();
   wait_for_previous();
   const float* part = p.part + (long long)bh * p.splits * ES;
@@ -251,16 +447,21 @@ __global__ void __launch_bounds__(LV_THREADS) latent_value_kernel(const LatentSt
     *reinterpret_cast<float4*>(sa + i) = t;
   }
   __syncthreads();
-  const T* up = (const T*)p.up + ((long long)h * (p.Dp + p.Ep) + p.Dp) * p.rank_p;
-  for (int r = slice * LV_ROWS + warp; r < min(p.E, (slice + 1) * LV_ROWS); r += LV_THREADS / 32) {
-    const T* wr = up + (long long)r * p.rank_p;
-    float s = 0.f;
-    for (int d = lane * VEC; d < p.rank_p; d += 32 * VEC) {
-      float f[VEC];
-      load_vec(wr + d, f);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) s += f[i] * sa[d + i];
-    }
+  for (int i = 0; i < ROWS; ++i) {
+    const int r = slice * LV_ROWS + warp + i * (LV_THREADS / 32);
+    if (r >= p.E) break;
+    float s = 0.f;
+    auto take = [&](const uint4& u, int d) {
+      float f[VEC];
+      unpack_vec<T>(u, f);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) s += f[e] * sa[d + e];
+    };
+#pragma unroll
+    for (int j = 0; j < PRE; ++j)
+      if ((j * 32 + lane) * VEC < p.rank_p) take(pre[i][j], (j * 32 + lane) * VEC);
+    for (int d = (PRE * 32 + lane) * VEC; d < p.rank_p; d += 32 * VEC) take(*reinterpret_cast<const uint4*>(up + (long long)r * p.rank_p + d), d);
     s = warp_sum(s);
     if (lane == 0) p.out[(long long)b * p.ldo + h * p.E + r] = s;
   }
@@ -290,7 +491,20 @@ void launch_latent_step(const LatentStepArgs& a, cudaStream_t s) {
     constexpr int VEC = 16 / sizeof(T), GR = LQ_THREADS / (LQ_COLS / VEC);
     const int slices = (a.rank_p + LQ_COLS - 1) / LQ_COLS, vs = (a.E + LV_ROWS - 1) / LV_ROWS;
     launch_chained(latent_query_kernel<T>, a.B * (slices * a.H + 1), LQ_THREADS, (size_t)(a.Dp + GR * LQ_COLS) * 4, s, a, slices);
-    launch_chained(latent_step_kernel<T>, a.B * a.H * a.splits, LS_THREADS, (size_t)(a.rank_p + a.Rp + LS_KEYS) * 4, s, a);
+    if (sizeof(T) == 2 && a.rank_p + a.Rp <= LM_PITCH) {
+      const int blocks = a.B * ((a.H + 15) / 16) * a.splits, groups = (a.rank_p + 127) / 128;  // 128 columns per round of the warps
+      const size_t sm = lm_smem(a.rank_p + a.Rp);
+      auto run = [&](auto* kern) {
+        cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
+        launch_chained(kern, blocks, LM_THREADS, sm, s, a);
+      };
+      if (groups <= 1) run(latent_step_mma_kernel<1>);
+      else if (groups <= 2) run(latent_step_mma_kernel<2>);
+      else if (groups <= 4) run(latent_step_mma_kernel<4>);
+      else run(latent_step_mma_kernel<5>);
+    } else {
+      launch_chained(latent_step_kernel<T>, a.B * a.H * a.splits, LS_THREADS, (size_t)(a.rank_p + a.Rp + LS_KEYS) * 4, s, a);
+    }
     launch_chained(latent_value_kernel<T>, a.B * a.H * vs, LV_THREADS, (size_t)(a.rank_p + a.splits) * 4, s, a, vs);
   };
   if (a.f32) go(float{});
