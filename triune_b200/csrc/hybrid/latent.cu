@@ -17,26 +17,62 @@ constexpr int LP_THREADS = 128;
 
 // block: one token of one sequence
 template <class T>
-__global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(const LatentPrepArgs p) {
+__global__ void __launch_bounds__(LP_THREADS) latent_prep_kernel(const LatentPrepArgs p, bool vec) {
   __shared__ float red[33];
   const int t = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, half = p.R / 2;
   T* pr = (T*)p.proj + ((long long)b * p.T + t) * p.ld;
   const float *cs = p.rot + (long long)t * p.R, *sn = cs + half;
-  for (int i = tid; i < p.H * half; i += LP_THREADS) {
-    const int h = i / half, d = i % half;
-    T* q = pr + p.col_q + h * (p.Dp + p.Rp) + p.Dp;
-    const float u = ldf(q + d), v = ldf(q + half + d), c = cs[d], s = sn[d];
-    stf(q + d, u * c - v * s);
-    stf(q + half + d, v * c + u * s);
+  if (vec) {  // halves in pieces of eight
+    const int n = half / 8;
+    for (int i = tid; i < p.H * n; i += LP_THREADS) {
+      const int h = i / n, d = (i % n) * 8;
+      T* q = pr + p.col_q + h * (p.Dp + p.Rp) + p.Dp;
+      float u[8], v[8], c[8], s[8], a[8], o[8];
+      ld8v(q + d, u);
+      ld8v(q + half + d, v);
+      ld8v(cs + d, c);
+      ld8v(sn + d, s);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        a[e] = u[e] * c[e] - v[e] * s[e];
+        o[e] = v[e] * c[e] + u[e] * s[e];
+      }
+      st8v(q + d, a);
+      st8v(q + half + d, o);
+    }
+  } else {
+    for (int i = tid; i < p.H * half; i += LP_THREADS) {
+      const int h = i / half, d = i % half;
+      T* q = pr + p.col_q + h * (p.Dp + p.Rp) + p.Dp;
+      const float u = ldf(q + d), v = ldf(q + half + d), c = cs[d], s = sn[d];
+      stf(q + d, u * c - v * s);
+      stf(q + half + d, v * c + u * s);
+    }
   }
   const long long pos = pos_of(p.pos) + t;
   if (p.col_c < 0 || pos < 0 || pos >= p.cap) return;  // the host reserves before every call
   const T* z = pr + p.col_c;
   T* dst = (T*)p.cache + ((long long)b * p.cap + pos) * (p.rank_p + p.Rp);
   float ss = 0.f;
-  for (int i = tid; i < p.rank; i += LP_THREADS) ss += ldf(z + i) * ldf(z + i);
-  const float r = 1.f / sqrtf(block_sum(ss, red) / p.rank + p.eps);
-  for (int i = tid; i < p.rank_p; i += LP_THREADS) stf(dst + i, i < p.rank ? ldf(z + i) * r * p.norm_w[i] : 0.f);
+  if (vec && p.rank % 8 == 0 && p.rank <= LP_THREADS * 8) {
+    float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    const bool on = tid * 8 < p.rank;
+    if (on) ld8v(z + tid * 8, f);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += f[e] * f[e];
+    const float r = 1.f / sqrtf(block_sum(ss, red) / p.rank + p.eps);
+    if (on) {
+      float w[8];
+      ld8v(p.norm_w + tid * 8, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] *= r * w[e];
+      st8v(dst + tid * 8, f);
+    }
+  } else {
+    for (int i = tid; i < p.rank; i += LP_THREADS) ss += ldf(z + i) * ldf(z + i);
+    const float r = 1.f / sqrtf(block_sum(ss, red) / p.rank + p.eps);
+    for (int i = tid; i < p.rank_p; i += LP_THREADS) stf(dst + i, i < p.rank ? ldf(z + i) * r * p.norm_w[i] : 0.f);
+  }
   for (int i = tid; i < p.Rp; i += LP_THREADS) {
     float v = 0.f;
     if (i < p.R) {
@@ -270,13 +306,21 @@ __global__ void __launch_bounds__(LM_THREADS) latent_step_mma_kernel(const Laten
   };
   if (k0 < k1) stage(0, k0);
   const float* qa = p.qa + ((long long)b * p.H + h0) * pitch;
-  for (int i = tid; i < 16 * (row - 8) / 2; i += LM_THREADS) {
-    const int r = i / ((row - 8) / 2), c = (i % ((row - 8) / 2)) * 2;
-    const bool on = r < nh && c < pitch;
-    const float x = on ? qa[r * pitch + c] : 0.f, y = on ? qa[r * pitch + c + 1] : 0.f;
-    const uint32_t hi = pack_bf16x2(x, y);
-    *reinterpret_cast<uint32_t*>(qh + r * row + c) = hi;
-    *reinterpret_cast<uint32_t*>(ql + r * row + c) = pack_bf16x2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {  // a warp has two heads, a lane four neighbouring entries
+    const int r = warp * 2 + i;
+#pragma unroll
+    for (int j = 0; j < LM_PITCH / 128; ++j) {
+      const int c = (j * 32 + lane) * 4;
+      if (c < row - 8) {
+        const float4 x = r < nh && c < pitch ? *reinterpret_cast<const float4*>(qa + (long long)r * pitch + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        const uint32_t a = pack_bf16x2(x.x, x.y), d = pack_bf16x2(x.z, x.w);
+        *reinterpret_cast<uint2*>(qh + r * row + c) = make_uint2(a, d);
+        *reinterpret_cast<uint2*>(ql + r * row + c) =
+            make_uint2(pack_bf16x2(x.x - __uint_as_float(a << 16), x.y - __uint_as_float(a & 0xffff0000u)),
+                       pack_bf16x2(x.z - __uint_as_float(d << 16), x.w - __uint_as_float(d & 0xffff0000u)));
+      }
+    }
   }
   if (tid < 16) {
     sm_m[tid] = -INFINITY;
@@ -388,7 +432,7 @@ __global__ void __launch_bounds__(LM_THREADS) latent_step_mma_kernel(const Laten
 }
 
 // ------------------------------------------------------------------------------------------------ step: values
-constexpr int LV_THREADS = 256, LV_ROWS = 32;
+constexpr int LV_THREADS = 512, LV_ROWS = 32;
 
 // blocks (32 rows of a head's value expansion, head, sequence): combines the head's splits, then a warp per row
 template <class T>
@@ -436,15 +480,25 @@ __global__ void __launch_bounds__(LV_THREADS) latent_value_kernel(const LatentSt
     for (int s = lane; s < active; s += 32) sc[s] *= r;
   }
   __syncthreads();
-  for (int i = tid * 4; i < p.rank_p; i += LV_THREADS * 4) {
+  // threads of a group have the quads of a latent, the groups share the splits
+  const int quads = p.rank_p / 4, groups = max(1, LV_THREADS / quads);
+  float* red = sc + (p.splits + 3) / 4 * 4;
+  for (int i = tid; i < quads * groups; i += LV_THREADS) {
+    const int qd = i % quads, g = i / quads;
     float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-    for (int s = 0; s < active; ++s) {
+#pragma unroll 16
+    for (int s = g; s < active; s += groups) {
       const float c = sc[s];
-      const float4 v = *reinterpret_cast<const float4*>(part + (long long)s * ES + 4 + i);
+      const float4 v = *reinterpret_cast<const float4*>(part + (long long)s * ES + 4 + qd * 4);
       t.x += c * v.x; t.y += c * v.y; t.z += c * v.z; t.w += c * v.w;
     }
-    *reinterpret_cast<float4*>(sa + i) = t;
+    *reinterpret_cast<float4*>(red + i * 4) = t;
+  }
+  __syncthreads();
+  for (int i = tid; i < p.rank_p; i += LV_THREADS) {
+    float t = 0.f;
+    for (int g = 0; g < groups; ++g) t += red[g * p.rank_p + i];
+    sa[i] = t;
   }
   __syncthreads();
 #pragma unroll
@@ -472,8 +526,11 @@ __global__ void __launch_bounds__(LV_THREADS) latent_value_kernel(const LatentSt
 void launch_latent_prep(const LatentPrepArgs& a, cudaStream_t s) {
   if (a.B <= 0 || a.T <= 0) return;
   const dim3 grid(a.T, a.B);
-  if (a.f32) latent_prep_kernel<float><<<grid, LP_THREADS, 0, s>>>(a);
-  else latent_prep_kernel<__nv_bfloat16><<<grid, LP_THREADS, 0, s>>>(a);
+  // heads and cached rows are multiples of eight wide; the matrix itself may start anywhere
+  const bool vec = a.R % 16 == 0 && a.col_q % 8 == 0 && (a.col_c < 0 || a.col_c % 8 == 0) && vec8_ok(a.proj, a.ld, a.f32) &&
+                   vec8_ok(a.cache, 8, a.f32) && vec8_ok(a.rot, 4, true) && vec8_ok(a.norm_w, 4, true);
+  if (a.f32) latent_prep_kernel<float><<<grid, LP_THREADS, 0, s>>>(a, vec);
+  else latent_prep_kernel<__nv_bfloat16><<<grid, LP_THREADS, 0, s>>>(a, vec);
   check_launch("latent_prep");
 }
 
@@ -505,7 +562,7 @@ void launch_latent_step(const LatentStepArgs& a, cudaStream_t s) {
     } else {
       launch_chained(latent_step_kernel<T>, a.B * a.H * a.splits, LS_THREADS, (size_t)(a.rank_p + a.Rp + LS_KEYS) * 4, s, a);
     }
-    launch_chained(latent_value_kernel<T>, a.B * a.H * vs, LV_THREADS, (size_t)(a.rank_p + a.splits) * 4, s, a, vs);
+    launch_chained(latent_value_kernel<T>, a.B * a.H * vs, LV_THREADS, (size_t)(a.rank_p + (a.splits + 3) / 4 * 4 + (a.rank_p > LV_THREADS * 4 ? a.rank_p : LV_THREADS * 4)) * 4, s, a, vs);
   };
   if (a.f32) go(float{});
   else go(__nv_bfloat16{});

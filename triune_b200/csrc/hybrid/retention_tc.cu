@@ -43,43 +43,66 @@ __device__ __forceinline__ void put8(uint8_t* hi, uint8_t* lo, uint32_t at, cons
   *reinterpret_cast<uint4*>(lo + at) = l;
 }
 
-// Rows t0 .. t0 + 127 of a head's queries or keys, turned, times `scale` and the row's weight, into `boxes` swizzled tiles of
-// 64 columns; rows past T and columns past D become zero. Dimensions come in pieces of eight: pieces below half the rotated
-// dimensions together with the piece half of them away.
-__device__ __forceinline__ void stage_turned(uint8_t* hi, uint8_t* lo, const __nv_bfloat16* src, long long ld, const float* rot,
-                                             int rot_dims, int t0, int T, int D, int boxes, float scale, const float* weight, int tid) {
+// One of the operands that stage_turned writes: a head's rows, the tiles of their high and low halves, their factor and the
+// rows' weights (or null).
+struct Turned {
+  const __nv_bfloat16* src;
+  long long ld;
+  uint8_t *hi, *lo;
+  float scale;
+  const float* weight;
+};
+
+// Rows t0 .. t0 + 127 of N operands, turned, times factor and weight, into `boxes` swizzled tiles of 64 columns each; rows past
+// T and columns past D become zero. Dimensions come in pieces of eight: pieces below half the rotated dimensions together
+// with the piece half of them away. The loads of AHEAD items of a thread are in flight before the first is used.
+template <int N>
+__device__ __forceinline__ void stage_turned(const Turned (&ops)[N], const float* rot, int rot_dims, int t0, int T, int D, int boxes, int tid) {
+  constexpr int AHEAD = 4;
   const int hg = rot_dims / 16, items = boxes * 8 - hg, half = rot_dims / 2;
-  for (int it = tid; it < RT * items; it += RTH) {
-    const int r = it / items, x = it % items, t = t0 + r;
-    const bool on = t < T;
-    const __nv_bfloat16* row = src + (long long)t * ld;
-    const float w = on ? (weight != nullptr ? scale * weight[r] : scale) : 0.f;
-    if (x < hg) {
-      float u[8], v[8], c[8], s[8];
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  for (int i0 = tid; i0 < RT * items; i0 += AHEAD * RTH) {
+    uint4 u[AHEAD][N], v[AHEAD][N];
+    float4 cs[AHEAD][4];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) u[i] = v[i] = c[i] = s[i] = 0.f;
-      if (on) {
-        ld8v(row + x * 8, u);
-        ld8v(row + half + x * 8, v);
-        ld8v(rot + (long long)t * rot_dims + x * 8, c);
-        ld8v(rot + (long long)t * rot_dims + half + x * 8, s);
+    for (int a = 0; a < AHEAD; ++a) {
+      const int it = i0 + a * RTH, r = it / items, x = it % items, t = t0 + r;
+      const bool on = it < RT * items && t < T, pair = x < hg;
+#pragma unroll
+      for (int n = 0; n < N; ++n) {
+        const __nv_bfloat16* row = ops[n].src + (long long)t * ops[n].ld;
+        u[a][n] = on && (pair ? x : x + hg) * 8 < D ? *reinterpret_cast<const uint4*>(row + (pair ? x : x + hg) * 8) : zero;
+        v[a][n] = on && pair ? *reinterpret_cast<const uint4*>(row + half + x * 8) : zero;
       }
-      float a[8], b[8];
-#pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        a[i] = (u[i] * c[i] - v[i] * s[i]) * w;
-        b[i] = (v[i] * c[i] + u[i] * s[i]) * w;
+      if (on && pair) {
+        const float4 *c = reinterpret_cast<const float4*>(rot + (long long)t * rot_dims + x * 8),
+                     *s = reinterpret_cast<const float4*>(rot + (long long)t * rot_dims + half + x * 8);
+        cs[a][0] = __ldg(c); cs[a][1] = __ldg(c + 1); cs[a][2] = __ldg(s); cs[a][3] = __ldg(s + 1);
+      } else {
+        cs[a][0] = cs[a][1] = make_float4(1.f, 1.f, 1.f, 1.f);
+        cs[a][2] = cs[a][3] = make_float4(0.f, 0.f, 0.f, 0.f);
       }
-      const int g = x + hg;
-      put8(hi + (x >> 3) * RBOX, lo + (x >> 3) * RBOX, sw(r, x & 7), a);
-      put8(hi + (g >> 3) * RBOX, lo + (g >> 3) * RBOX, sw(r, g & 7), b);
-    } else {
-      const int g = x + hg;
-      float u[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-      if (on && g * 8 < D) ld8v(row + g * 8, u);
+    }
 #pragma unroll
-      for (int i = 0; i < 8; ++i) u[i] *= w;
-      put8(hi + (g >> 3) * RBOX, lo + (g >> 3) * RBOX, sw(r, g & 7), u);
+    for (int a = 0; a < AHEAD; ++a) {
+      const int it = i0 + a * RTH, r = it / items, x = it % items, g = x + hg;
+      if (it >= RT * items) break;
+      const float c[8] = {cs[a][0].x, cs[a][0].y, cs[a][0].z, cs[a][0].w, cs[a][1].x, cs[a][1].y, cs[a][1].z, cs[a][1].w};
+      const float s[8] = {cs[a][2].x, cs[a][2].y, cs[a][2].z, cs[a][2].w, cs[a][3].x, cs[a][3].y, cs[a][3].z, cs[a][3].w};
+#pragma unroll
+      for (int n = 0; n < N; ++n) {
+        const float w = ops[n].weight != nullptr ? ops[n].scale * ops[n].weight[r] : ops[n].scale;
+        const uint32_t ua[4] = {u[a][n].x, u[a][n].y, u[a][n].z, u[a][n].w}, va[4] = {v[a][n].x, v[a][n].y, v[a][n].z, v[a][n].w};
+        float p[8], q[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const float x0 = (i & 1) ? hi_f(ua[i / 2]) : lo_f(ua[i / 2]), x1 = (i & 1) ? hi_f(va[i / 2]) : lo_f(va[i / 2]);
+          p[i] = (x0 * c[i] - x1 * s[i]) * w;
+          q[i] = (x1 * c[i] + x0 * s[i]) * w;
+        }
+        if (x < hg) put8(ops[n].hi + (x >> 3) * RBOX, ops[n].lo + (x >> 3) * RBOX, sw(r, x & 7), p);
+        put8(ops[n].hi + (g >> 3) * RBOX, ops[n].lo + (g >> 3) * RBOX, sw(r, g & 7), x < hg ? q : p);
+      }
     }
   }
 }
@@ -129,7 +152,8 @@ __global__ void __launch_bounds__(RTH, 2) retention_states_kernel(const __grid_c
   if (tid < RT) weight[tid] = tid < n ? exp2f(lg * (n - 1 - tid)) : 0.f;
   __syncthreads();
   const __nv_bfloat16* K = (const __nv_bfloat16*)p.k + (long long)at.b * p.rows * p.ldk + at.h * p.Dk;
-  stage_turned(smem, smem + 2 * RBOX, K, p.ldk, p.rot, p.rot_dims, at.t0, p.T, p.Dk, 2, 1.f / sqrtf((float)p.Dk), weight, tid);
+  const Turned keys[1] = {{K, p.ldk, smem, smem + 2 * RBOX, 1.f / sqrtf((float)p.Dk), weight}};
+  stage_turned(keys, p.rot, p.rot_dims, at.t0, p.T, p.Dk, 2, tid);
   fence_proxy_async_smem();
   tc_fence_before_sync();
   __syncthreads();
@@ -257,8 +281,8 @@ __global__ void __launch_bounds__(RTH, 1) retention_out_kernel(const __grid_cons
   if (tid <= RT) power[tid] = exp2f(lg * tid);
   const __nv_bfloat16 *Q = (const __nv_bfloat16*)p.q + (long long)at.b * p.rows * p.ldq + at.h * p.Dk,
                       *K = (const __nv_bfloat16*)p.k + (long long)at.b * p.rows * p.ldk + at.h * p.Dk;
-  stage_turned(smem + L::QH, smem + L::QL, Q, p.ldq, p.rot, p.rot_dims, at.t0, p.T, p.Dk, DKB, 1.f, nullptr, tid);
-  stage_turned(smem + L::KH, smem + L::KL, K, p.ldk, p.rot, p.rot_dims, at.t0, p.T, p.Dk, DKB, 1.f / sqrtf((float)p.Dk), nullptr, tid);
+  const Turned both[2] = {{Q, p.ldq, smem + L::QH, smem + L::QL, 1.f, nullptr}, {K, p.ldk, smem + L::KH, smem + L::KL, 1.f / sqrtf((float)p.Dk), nullptr}};
+  stage_turned(both, p.rot, p.rot_dims, at.t0, p.T, p.Dk, DKB, tid);
   fence_proxy_async_smem();
   tc_fence_before_sync();
   __syncthreads();

@@ -256,6 +256,22 @@ __global__ void side_rows_kernel(const T* __restrict__ gate, long long ldg, cons
   }
 }
 
+// dim, columns and pitches multiples of eight
+template <class T>
+__global__ void side_rows_vec_kernel(const T* __restrict__ gate, long long ldg, const T* __restrict__ table, long long ldt,
+                                     const long long* __restrict__ ids, int V, int col0, T* __restrict__ out, int pieces, int n, int act) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const long long row = i / pieces, id = ids[row];
+  const int c = (i % pieces) * 8;
+  float g[8], e[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  ld8v(gate + row * ldg + c, g);
+  if (id >= 0 && id < V) ld8v(table + id * ldt + col0 + c, e);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) g[j] = act_f(g[j], act) * e[j];
+  st8v(out + (long long)i * 8, g);
+}
+
 __global__ void rotation_rows_kernel(const double* __restrict__ freqs, int n, float amplitude, float* __restrict__ out, long long total,
                                      const Pos pos) {
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -432,6 +448,17 @@ void launch_side_rows(const void* gate, long long ldg, const void* table, long l
                       void* out, bool f32, int rows, int dim, int act, cudaStream_t s) {
   const long long n = (long long)rows * dim;
   if (n <= 0) return;
+  if (dim % 8 == 0 && col0 % 8 == 0 && n / 8 < (1ll << 31) && vec8_ok(gate, ldg, f32) && vec8_ok(table, ldt, f32) && vec8_ok(out, dim, f32)) {
+    const int pieces = (int)(n / 8);
+    auto go = [&](auto* o) {
+      using T = std::remove_pointer_t<decltype(o)>;
+      side_rows_vec_kernel<T><<<(pieces + 255) / 256, 256, 0, s>>>((const T*)gate, ldg, (const T*)table, ldt, ids, V, col0, o, dim / 8, pieces, act);
+    };
+    if (f32) go((float*)out);
+    else go((__nv_bfloat16*)out);
+    check_launch("side_rows");
+    return;
+  }
   const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
   if (f32) side_rows_kernel<<<blocks, 256, 0, s>>>((const float*)gate, ldg, (const float*)table, ldt, ids, V, col0, (float*)out, dim, n, act);
   else
