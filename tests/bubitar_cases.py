@@ -33,19 +33,19 @@ CONFIGS = {
     "odd": oracle.make_config([
         with_mlp(retention(3, 20, 10, [0.25, 0.875, 0.999], 12, 5e5), 30, 0.9),
         with_mlp(latent(3, 10, 6, 14, 20, 0.35, 1e3, {"factor": 2.5, "original": 40, "fast": 4.0, "slow": 0.5}), 18, 1.5),
-        with_mlp(retention(1, 6, 5, [0.96875])),
+        with_mlp(retention(1, 6, 5, [0.95])),
         with_mlp(latent(5, 7, 6, 9, 20, 0.3, 1e3, {"factor": 2.5, "original": 40, "fast": 4.0, "slow": 0.5}, kv_from=1), 21, 0.8),
     ], vocab=51, width=36, eps=1e-4, side=5),
     # heads of serving size
     "wide": oracle.make_config([
-        with_mlp(retention(2, 128, 128, [0.96875, 0.998046875]), 128, 1.3),
-        with_mlp(latent(4, 128, 64, 128, 256, 0.07, 1e5, {"factor": 4.0, "original": 128, "fast": 32.0, "slow": 1.0}), 64, 2.0),
-        with_mlp(retention(3, 64, 192, [0.9375, 0.99, 0.9990234375], 32)),
+        with_mlp(retention(2, 128, 128, [0.95, 0.9975]), 128, 1.3),
+        with_mlp(latent(4, 128, 64, 128, 256, 0.07, 1e5, {"factor": 6.0, "original": 128, "fast": 24.0, "slow": 1.0}), 64, 2.0),
+        with_mlp(retention(3, 64, 192, [0.9375, 0.99, 0.999], 32)),
         with_mlp(latent(20, 64, 32, 64, 256, 0.1)),
     ], vocab=128, width=96, side=16),
     # one head of everything, no rotation in the retention
     "single": oracle.make_config([
         with_mlp(latent(1, 32, 16, 32, 64, 0.14), 64),
-        with_mlp(retention(1, 32, 32, [0.984375], 0), 32),
+        with_mlp(retention(1, 32, 32, [0.985], 0), 32),
     ], vocab=64, width=64, side=8),
 }

@@ -216,6 +216,7 @@ def bubitar_kernels(size: str, T: int, iters: int) -> None:
             y = torch.empty(T, mix.out_weight.shape[1], device=dev, dtype=bf)
             N, K, at = mix.in_weight.shape[0], mix.out_weight.shape[1], c.inputs.at
             if i == 0:
+                t(name, "shortest launch (one embedding row)", lambda: hops.embed_rows(p.ids[:1], m.embed), 6 * W)
                 t(name, "norm behind + sum + next norm", lambda: hops.add_norm(x, ys, None, layer.norm1b.args, layer.norm2.args, bf), 12 * T * W)
             t(name, f"{label}: input GEMM", lambda: hops.linear(h, mix.in_weight), 2 * (T * W + N * W + T * N), 2 * T * N * W)
             if i == 0:

@@ -331,10 +331,7 @@ void launch_tc_gemm(const GemmArgs& a, cudaStream_t stream) {
     if (dswiglu && a.aux_in == nullptr) throw std::runtime_error("tc_gemm: gate/up rows missing");
   }
 
-  // Tall products of few columns: wide tiles would leave half of the machine without work
-  const bool few = a.mode == GEMM_DENSE && a.batch <= 1 && !(a.flags & (GF_ACCUMULATE | GF_SWIGLU | GF_DSWIGLU)) && a.N > 64 && a.N <= 512 &&
-                   (long long)((a.M + BM - 1) / BM) * ((a.N + 255) / 256) * 2 <= sm_count();
-  if (!few) {
+  {
     static const bool pairs = [] {
       const char* e = std::getenv("TRIUNE_GEMM_PAIR");  // "0" keeps every product on the one-CTA kernel
       return !(e && e[0] == '0');
@@ -344,7 +341,6 @@ void launch_tc_gemm(const GemmArgs& a, cudaStream_t stream) {
 
   // widest tile that divides N: the tensor core is most efficient at N = 256, then 192 (e.g. N = 384), then 128
   int BN = (a.N >= 256 && a.N % 256 == 0) ? 256 : ((a.N >= 192 && a.N % 192 == 0) ? 192 : (a.N > 64 ? 128 : 64));
-  if (few) BN = 128;
   {
     static const int forced = [] {
       const char* e = std::getenv("TRIUNE_GEMM_BN");  // experiments only: force the tile width

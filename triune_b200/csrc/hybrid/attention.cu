@@ -147,8 +147,8 @@ __global__ void __launch_bounds__(AP_WARPS * 32) attn_prep_vec_kernel(const Attn
 
 constexpr int AS_Q = 8, AS_K = 32;
 
-// block: AS_Q consecutive queries of one head, a warp each; keys and values in tiles of 32
-template <class T>
+// block: AS_Q consecutive queries of one head, a warp each; keys and values in tiles of 32; value sizes up to 32 NE
+template <class T, int NE>
 __global__ void attn_simple_kernel(const AttnArgs p) {
   extern __shared__ float sm[];
   const int D = p.D + p.R, dp = D + 1;
@@ -170,9 +170,9 @@ __global__ void attn_simple_kernel(const AttnArgs p) {
     }
   }
   float m = p.sink != nullptr ? p.sink[h] : -INFINITY, l = p.sink != nullptr ? 1.f : 0.f;
-  float acc[8];  // value dimensions up to 256
+  float acc[NE];
 #pragma unroll
-  for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+  for (int i = 0; i < NE; ++i) acc[i] = 0.f;
   for (long long k0 = 0; k0 < kend; k0 += AS_K) {
     const int n = (int)min((long long)AS_K, kend - k0);
     __syncthreads();
@@ -192,11 +192,11 @@ __global__ void attn_simple_kernel(const AttnArgs p) {
     l = l * corr + warp_sum(e);
     m = mn;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) acc[i] *= corr;
+    for (int i = 0; i < NE; ++i) acc[i] *= corr;
     for (int j = 0; j < n; ++j) {
       const float w = __shfl_sync(0xffffffffu, e, j);
 #pragma unroll
-      for (int i = 0; i < 8; ++i)
+      for (int i = 0; i < NE; ++i)
         if (lane + 32 * i < p.E) acc[i] += w * sv[j * p.E + lane + 32 * i];
     }
   }
@@ -205,7 +205,7 @@ __global__ void attn_simple_kernel(const AttnArgs p) {
     float r = p.out_scale / l;
     if (p.gate != nullptr) r *= sigmoid_f(ldf((const T*)p.gate + ((long long)b * p.T + t) * p.ldg + h));
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < NE; ++i)
       if (lane + 32 * i < p.E) stf(o + lane + 32 * i, acc[i] * r);
   }
 }
@@ -240,7 +240,7 @@ void launch_attn_prep(const AttnPrepArgs& a, cudaStream_t s) {
 
 void launch_attn_simple(const AttnArgs& a, cudaStream_t s) {
   if (a.B <= 0 || a.T <= 0) return;
-  if (a.E > 256) throw std::runtime_error("attention: value dimensions up to 256");
+  if (a.E > 512) throw std::runtime_error("attention: value dimensions up to 512");
   const size_t sm = (size_t)(AS_K * (a.D + a.R + 1) + AS_K * a.E + AS_Q * (a.D + a.R)) * 4;
   if (sm > 200 * 1024) throw std::runtime_error("attention: head dimension too large");
   dim3 grid((a.T + AS_Q - 1) / AS_Q, a.H, a.B);
@@ -248,8 +248,13 @@ void launch_attn_simple(const AttnArgs& a, cudaStream_t s) {
     if (sm > 47 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);
     kern<<<grid, AS_Q * 32, sm, s>>>(a);
   };
-  if (a.f32) go(attn_simple_kernel<float>);
-  else go(attn_simple_kernel<__nv_bfloat16>);
+  if (a.E <= 256) {
+    if (a.f32) go(attn_simple_kernel<float, 8>);
+    else go(attn_simple_kernel<__nv_bfloat16, 8>);
+  } else {
+    if (a.f32) go(attn_simple_kernel<float, 16>);
+    else go(attn_simple_kernel<__nv_bfloat16, 16>);
+  }
   check_launch("attn_simple");
 }
 

@@ -152,12 +152,20 @@ __global__ void __launch_bounds__(LQ_THREADS) latent_query_kernel(const LatentSt
 #pragma unroll 4
     for (int d = gr + PRE * GR; d < p.D; d += GR) take(*reinterpret_cast<const uint4*>(up + (long long)d * p.rank_p), d);
   }
+  // key rows of a warp's lanes, then of the warps
 #pragma unroll
-  for (int i = 0; i < VEC; ++i) acc[gr * LQ_COLS + tx * VEC + i] = a[i];
+  for (int o = TX; o < 32; o <<= 1)
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) a[i] += __shfl_xor_sync(0xffffffffu, a[i], o);
+  if ((tid & 31) < TX) {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc[(tid >> 5) * LQ_COLS + tx * VEC + i] = a[i];
+  }
   __syncthreads();
   if (tid < LQ_COLS && c0 + tid < p.rank_p) {
     float s = 0.f;
-    for (int g = 0; g < GR; ++g) s += acc[g * LQ_COLS + tid];
+#pragma unroll
+    for (int g = 0; g < LQ_THREADS / 32; ++g) s += acc[g * LQ_COLS + tid];
     qa[c0 + tid] = s;
   }
 }
@@ -248,9 +256,9 @@ __global__ void __launch_bounds__(LS_THREADS) latent_step_kernel(const LatentSte
 
 // bf16 caches on the tensor cores, up to 16 heads at a time: blocks (split, group of 16 heads, sequence). Queries are fp32
 // and enter as two bf16 numbers, cached rows are exact operands, softmax weights enter as two bf16 numbers again. A warp has
-// eight keys of a tile of 64 for the scores, and NG times 16 columns of the latent for the sums; the accumulators stay in
-// registers while two tiles of rows alternate in shared memory.
-constexpr int LM_THREADS = 256, LM_KEYS = 64, LM_PITCH = 640;
+// the query entries of every eighth step of 32 in registers and forms its part of the scores of a tile of 64 keys; for the
+// sums it has NG times 16 columns of the latent. Accumulators stay in registers, two tiles of rows alternate in shared memory.
+constexpr int LM_THREADS = 256, LM_KEYS = 64, LM_PITCH = 640, LM_STEPS = (LM_PITCH / 32 + 7) / 8;
 
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -271,8 +279,10 @@ __device__ __forceinline__ void ld_matrix_t(uint32_t (&r)[4], const void* p) {
 }
 __host__ __device__ constexpr int lm_row(int pitch) { return (pitch + 31) / 32 * 32 + 8; }  // shared-memory row, no bank conflicts
 constexpr int LM_PROW = LM_KEYS + 8;
+constexpr int LM_PARTS = 8 * 16 * LM_KEYS * 4;  // bytes of the warps' parts of the scores, in the place of the queries
+__host__ __device__ constexpr int lm_queries(int pitch) { return 2 * 16 * lm_row(pitch) * 2 > LM_PARTS ? 2 * 16 * lm_row(pitch) * 2 : LM_PARTS; }
 inline size_t lm_smem(int pitch) {
-  return (size_t)(2 * 16 + 2 * LM_KEYS) * lm_row(pitch) * 2 + 16 * LM_KEYS * 4 + 2 * 16 * LM_PROW * 2 + 3 * 16 * 4;
+  return (size_t)lm_queries(pitch) + 2 * LM_KEYS * lm_row(pitch) * 2 + 2 * 16 * LM_PROW * 2 + 3 * 16 * 4;
 }
 
 template <int NG>
@@ -280,14 +290,12 @@ __global__ void __launch_bounds__(LM_THREADS) latent_step_mma_kernel(const Laten
   using bf16 = __nv_bfloat16;
   extern __shared__ __align__(16) uint8_t lm_raw[];
   const int pitch = p.rank_p + p.Rp, row = lm_row(pitch), groups = (p.H + 15) / 16;
-  bf16 *qh = reinterpret_cast<bf16*>(lm_raw), *ql = qh + 16 * row, *keys = ql + 16 * row;
-  float* ss = reinterpret_cast<float*>(keys + 2 * LM_KEYS * row);
-  bf16 *ph = reinterpret_cast<bf16*>(ss + 16 * LM_KEYS), *pl = ph + 16 * LM_PROW;
+  bf16 *qh = reinterpret_cast<bf16*>(lm_raw), *ql = qh + 16 * row, *keys = reinterpret_cast<bf16*>(lm_raw + lm_queries(pitch));
+  float* ss = reinterpret_cast<float*>(lm_raw);  // [warp][head][key], once the queries are in registers
+  bf16 *ph = keys + 2 * LM_KEYS * row, *pl = ph + 16 * LM_PROW;
   float *sm_m = reinterpret_cast<float*>(pl + 16 * LM_PROW), *sm_l = sm_m + 16, *sm_c = sm_l + 16;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int split = blockIdx.x % p.splits, u = blockIdx.x / p.splits, grp = u % groups, b = u / groups, h0 = grp * 16, nh = min(16, p.H - h0);
-  launch_dependents();
-  wait_for_previous();
   const long long pos = pos_of(p.pos);
   int k0 = 0, k1 = 0;
   if (pos >= 0 && pos < p.cap) latent_range(pos + 1, p.splits, split, &k0, &k1);
@@ -295,16 +303,29 @@ __global__ void __launch_bounds__(LM_THREADS) latent_step_mma_kernel(const Laten
   const int pieces = pitch / 8, wide = (row - 8) / 8;  // 16-byte pieces of a cached row, and with the zeros behind it
   auto stage = [&](int buf, int kb) {
     bf16* dst = keys + buf * LM_KEYS * row;
-    for (int i = tid; i < LM_KEYS * wide; i += LM_THREADS) {
-      const int r = i / wide, c = i % wide;
-      const bool on = kb + r < k1 && c < pieces;
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * row + c * 8)),
-                   "l"(on ? C + (long long)(kb + r) * pitch + c * 8 : C), "r"(on ? 16 : 0)
-                   : "memory");
+#pragma unroll
+    for (int i = 0; i < LM_KEYS / 8; ++i) {
+      const int r = warp + 8 * i;
+      const bf16* src = C + (long long)(kb + r) * pitch;
+#pragma unroll
+      for (int j = 0; j < (LM_PITCH / 8 + 31) / 32; ++j) {
+        const int c = j * 32 + lane;
+        const bool on = kb + r < k1 && c < pieces;
+        if (c < wide)
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * row + c * 8)), "l"(on ? src + c * 8 : C),
+                       "r"(on ? 16 : 0)
+                       : "memory");
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  if (k0 < k1) stage(0, k0);
+  // Rows of earlier positions were complete before this step's first kernel started (the embedding rows, launched without
+  // overlap): they are fetched ahead of the wait. Only the position's own row comes from the kernel before this one.
+  const bool ahead = k0 < k1 && min(k0 + LM_KEYS, k1) <= pos;
+  if (ahead) stage(0, k0);
+  launch_dependents();
+  wait_for_previous();
+  if (k0 < k1 && !ahead) stage(0, k0);
   const float* qa = p.qa + ((long long)b * p.H + h0) * pitch;
 #pragma unroll
   for (int i = 0; i < 2; ++i) {  // a warp has two heads, a lane four neighbouring entries
@@ -331,37 +352,60 @@ __global__ void __launch_bounds__(LM_THREADS) latent_step_mma_kernel(const Laten
   for (int g = 0; g < NG; ++g)
 #pragma unroll
     for (int e = 0; e < 8; ++e) acc[g][e] = 0.f;
-  const int a_off = (lane & 15) * row + (lane >> 4) * 8;
+  __syncthreads();
+  // a warp's steps beyond the row have zero queries on the first columns, which keeps the products free of branches
+  uint32_t ah[LM_STEPS][2][4], al[LM_STEPS][2][4];
+  int at[LM_STEPS];
+#pragma unroll
+  for (int i = 0; i < LM_STEPS; ++i) {
+    const bool on = (warp + 8 * i) * 32 < row - 8;
+    at[i] = on ? (warp + 8 * i) * 32 : 0;
+    const int off = (lane & 15) * row + (lane >> 4) * 8 + at[i];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      ld_matrix(ah[i][j], qh + off + 16 * j);
+      ld_matrix(al[i][j], ql + off + 16 * j);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        ah[i][j][e] = on ? ah[i][j][e] : 0u;
+        al[i][j][e] = on ? al[i][j][e] : 0u;
+      }
+    }
+  }
   for (int kb = k0, buf = 0; kb < k1; kb += LM_KEYS, buf ^= 1) {
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     if (kb + LM_KEYS < k1) stage(buf ^ 1, kb + LM_KEYS);
     const bf16* kt = keys + buf * LM_KEYS * row;
-    float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
-    const bf16* kr = kt + (warp * 8 + (lane & 7)) * row + (lane >> 3) * 8;
-#pragma unroll 4
-    for (int d = 0; d < row - 8; d += 32) {
-      uint32_t kv[4], a0[4], a1[4], l0[4], l1[4];
-      ld_matrix(kv, kr + d);
-      ld_matrix(a0, qh + a_off + d);
-      ld_matrix(a1, qh + a_off + d + 16);
-      ld_matrix(l0, ql + a_off + d);
-      ld_matrix(l1, ql + a_off + d + 16);
-      mma_bf16(s, a0, kv[0], kv[1]);
-      mma_bf16(s2, l0, kv[0], kv[1]);
-      mma_bf16(s, a1, kv[2], kv[3]);
-      mma_bf16(s2, l1, kv[2], kv[3]);
-    }
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int key = warp * 8 + 2 * (lane & 3) + (e & 1), hh = (lane >> 2) + (e >> 1) * 8;
-      ss[hh * LM_KEYS + key] = kb + key < k1 ? (s[e] + s2[e]) * p.scale : -INFINITY;
+    for (int t = 0; t < LM_KEYS / 8; ++t) {
+      float s[4] = {0.f, 0.f, 0.f, 0.f}, s2[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int i = 0; i < LM_STEPS; ++i) {
+        uint32_t kv[4];
+        ld_matrix(kv, kt + (t * 8 + (lane & 7)) * row + (lane >> 3) * 8 + at[i]);
+        mma_bf16(s, ah[i][0], kv[0], kv[1]);
+        mma_bf16(s2, al[i][0], kv[0], kv[1]);
+        mma_bf16(s, ah[i][1], kv[2], kv[3]);
+        mma_bf16(s2, al[i][1], kv[2], kv[3]);
+      }
+      float* o = ss + (warp * 16 + (lane >> 2)) * LM_KEYS + t * 8 + 2 * (lane & 3);
+      *reinterpret_cast<float2*>(o) = make_float2(s[0] + s2[0], s[1] + s2[1]);
+      *reinterpret_cast<float2*>(o + 8 * LM_KEYS) = make_float2(s[2] + s2[2], s[3] + s2[3]);
     }
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int hh = warp * 2 + i;
-      const float x0 = ss[hh * LM_KEYS + 2 * lane], x1 = ss[hh * LM_KEYS + 2 * lane + 1];
+      float x0 = 0.f, x1 = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) {
+        const float2 v = *reinterpret_cast<const float2*>(ss + (w * 16 + hh) * LM_KEYS + 2 * lane);
+        x0 += v.x;
+        x1 += v.y;
+      }
+      x0 = kb + 2 * lane < k1 ? x0 * p.scale : -INFINITY;
+      x1 = kb + 2 * lane + 1 < k1 ? x1 * p.scale : -INFINITY;
       const float mo = sm_m[hh], mn = fmaxf(mo, warp_max(fmaxf(x0, x1)));  // every tile has a key: finite
       const float e0 = expf(x0 - mn), e1 = expf(x1 - mn), l = warp_sum(e0 + e1);
       const uint32_t hi = pack_bf16x2(e0, e1);
@@ -386,28 +430,27 @@ __global__ void __launch_bounds__(LM_THREADS) latent_step_mma_kernel(const Laten
     }
 #pragma unroll
     for (int g = 0; g < NG; ++g) {
-      const int col = (warp + 8 * g) * 16;
-      if (col < p.rank_p) {
-        float lo[4], hi[4];
+      // groups beyond the latent repeat the first columns; they are not stored
+      const int col = (warp + 8 * g) * 16 < p.rank_p ? (warp + 8 * g) * 16 : 0;
+      float lo[4], hi[4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          lo[e] = acc[g][e] * (e < 2 ? c0 : c1);
-          hi[e] = acc[g][4 + e] * (e < 2 ? c0 : c1);
-        }
+      for (int e = 0; e < 4; ++e) {
+        lo[e] = acc[g][e] * (e < 2 ? c0 : c1);
+        hi[e] = acc[g][4 + e] * (e < 2 ? c0 : c1);
+      }
 #pragma unroll
-        for (int t = 0; t < 4; ++t) {
-          uint32_t v[4];
-          ld_matrix_t(v, kt + (t * 16 + (lane & 15)) * row + col + (lane >> 4) * 8);
-          mma_bf16(lo, wh[t], v[0], v[1]);
-          mma_bf16(hi, wh[t], v[2], v[3]);
-          mma_bf16(lo, wl[t], v[0], v[1]);
-          mma_bf16(hi, wl[t], v[2], v[3]);
-        }
+      for (int t = 0; t < 4; ++t) {
+        uint32_t v[4];
+        ld_matrix_t(v, kt + (t * 16 + (lane & 15)) * row + col + (lane >> 4) * 8);
+        mma_bf16(lo, wh[t], v[0], v[1]);
+        mma_bf16(hi, wh[t], v[2], v[3]);
+        mma_bf16(lo, wl[t], v[0], v[1]);
+        mma_bf16(hi, wl[t], v[2], v[3]);
+      }
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          acc[g][e] = lo[e];
-          acc[g][4 + e] = hi[e];
-        }
+      for (int e = 0; e < 4; ++e) {
+        acc[g][e] = lo[e];
+        acc[g][4 + e] = hi[e];
       }
     }
   }
@@ -545,9 +588,8 @@ void launch_latent_step(const LatentStepArgs& a, cudaStream_t s) {
   if (a.rank_p > 2048 || a.rank_p % 8 != 0 || a.Rp % 8 != 0) throw std::runtime_error("latent_step: latents of up to 2048 entries, padded to eight");
   auto go = [&](auto tag) {
     using T = decltype(tag);
-    constexpr int VEC = 16 / sizeof(T), GR = LQ_THREADS / (LQ_COLS / VEC);
     const int slices = (a.rank_p + LQ_COLS - 1) / LQ_COLS, vs = (a.E + LV_ROWS - 1) / LV_ROWS;
-    launch_chained(latent_query_kernel<T>, a.B * (slices * a.H + 1), LQ_THREADS, (size_t)(a.Dp + GR * LQ_COLS) * 4, s, a, slices);
+    launch_chained(latent_query_kernel<T>, a.B * (slices * a.H + 1), LQ_THREADS, (size_t)(a.Dp + LQ_THREADS / 32 * LQ_COLS) * 4, s, a, slices);
     if (sizeof(T) == 2 && a.rank_p + a.Rp <= LM_PITCH) {
       const int blocks = a.B * ((a.H + 15) / 16) * a.splits, groups = (a.rank_p + 127) / 128;  // 128 columns per round of the warps
       const size_t sm = lm_smem(a.rank_p + a.Rp);

@@ -10,8 +10,8 @@
 // operands take three MMAs). Accumulators and the carried state are fp32.
 //
 // A block owns 128 value columns of a head and chunk. Shared-memory tiles are rows of 128 bytes in the 128B-swizzled layout:
-// queries and keys are written by the threads that turn and split them, values and states come by TMA. 256 threads are
-// two halves of 128 rows: a thread has the row of its TMEM lane and half of the columns.
+// queries and keys are written by the threads that turn and split them, values and states come by TMA. 512 threads are
+// four times 128 rows: a thread has the row of its TMEM lane and a quarter of the columns.
 // TMEM columns of the outputs kernel: 0 scores (128), 128 decayed scores as bf16 pairs, high (64) and low (64) halves,
 // 256 queries times state (128), 384 decayed scores times values (128).
 #include "../common/ptx.cuh"
@@ -22,7 +22,7 @@
 namespace tb {
 namespace {
 
-constexpr int RT = 128, RTH = 256, RBOX = 128 * 128, RCOLS = 128;  // tokens, threads, bytes of a 128 x 64 tile, value columns
+constexpr int RT = 128, RTH = 512, RBOX = 128 * 128, RCOLS = 128;  // tokens, threads, bytes of a 128 x 64 tile, value columns
 
 struct RetParams {
   RecurrentArgs a;
@@ -58,7 +58,7 @@ struct Turned {
 // with the piece half of them away. The loads of AHEAD items of a thread are in flight before the first is used.
 template <int N>
 __device__ __forceinline__ void stage_turned(const Turned (&ops)[N], const float* rot, int rot_dims, int t0, int T, int D, int boxes, int tid) {
-  constexpr int AHEAD = 4;
+  constexpr int AHEAD = 2;
   const int hg = rot_dims / 16, items = boxes * 8 - hg, half = rot_dims / 2;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
   for (int i0 = tid; i0 < RT * items; i0 += AHEAD * RTH) {
@@ -181,22 +181,19 @@ __global__ void __launch_bounds__(RTH, 2) retention_states_kernel(const __grid_c
   __syncwarp();
   tc_fence_after_sync();
   if (ok) {
-    const int row = (warp & 3) * 32 + lane, col0 = (warp >> 2) * 64;
+    const int row = (warp & 3) * 32 + lane, col0 = (warp >> 2) * 32;
     const uint32_t t = tmem + ((uint32_t)((warp & 3) * 32) << 16);
     float* dst = sp.own + (((long long)at.bh * sp.nchunks + at.c) * p.Dk + row) * p.Dv + at.c0 + col0;
+    uint32_t v[32];
+    tmem_ld_32x32b_x32(t + col0, v);
+    tmem_ld_wait_regs(v);
+    if (row < p.Dk) {
 #pragma unroll
-    for (int g = 0; g < 2; ++g) {
-      uint32_t v[32];
-      tmem_ld_32x32b_x32(t + col0 + 32 * g, v);
-      tmem_ld_wait_regs(v);
-      if (row < p.Dk) {
+      for (int i = 0; i < 4; ++i) {
+        float f[8];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          float f[8];
-#pragma unroll
-          for (int j = 0; j < 8; ++j) f[j] = __uint_as_float(v[8 * i + j]);
-          if (col0 + 32 * g + 8 * i < at.ncol) st8v(dst + 32 * g + 8 * i, f);
-        }
+        for (int j = 0; j < 8; ++j) f[j] = __uint_as_float(v[8 * i + j]);
+        if (col0 + 8 * i < at.ncol) st8v(dst + 8 * i, f);
       }
     }
   }
@@ -314,23 +311,21 @@ __global__ void __launch_bounds__(RTH, 1) retention_out_kernel(const __grid_cons
     }
   }
   __syncwarp();
-  const int row = (warp & 3) * 32 + lane, half = warp >> 2;
+  const int row = (warp & 3) * 32 + lane, col0 = (warp >> 2) * 32;
   const uint32_t lanes = tmem + ((uint32_t)((warp & 3) * 32) << 16);
   bool ok = mbar_wait(&scored, 0);
   if (!ok && sp.status) *sp.status = ST_TIMEOUT_TMEM;
   __syncwarp();
   tc_fence_after_sync();
-#pragma unroll
-  for (int g = 0; g < 2; ++g) {  // decayed scores of 32 columns at a time; columns past the row's token are zero
-    const int j0 = half * 64 + g * 32;
+  {  // decayed scores of 32 columns; columns past the row's token are zero
     uint32_t hi[16], lo[16];
-    if (j0 <= (warp & 3) * 32 + 31) {  // some row of this warp sees them
+    if (col0 <= (warp & 3) * 32 + 31) {  // some row of this warp sees them
       uint32_t s[32];
-      tmem_ld_32x32b_x32(lanes + j0, s);
+      tmem_ld_32x32b_x32(lanes + col0, s);
       tmem_ld_wait_regs(s);
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
-        const int n = row - j0 - 2 * i;
+        const int n = row - col0 - 2 * i;
         const float a = n >= 0 ? __uint_as_float(s[2 * i]) * power[n] : 0.f, b = n >= 1 ? __uint_as_float(s[2 * i + 1]) * power[n - 1] : 0.f;
         split2(a, b, hi[i], lo[i]);
       }
@@ -338,8 +333,8 @@ __global__ void __launch_bounds__(RTH, 1) retention_out_kernel(const __grid_cons
 #pragma unroll
       for (int i = 0; i < 16; ++i) hi[i] = lo[i] = 0u;
     }
-    tmem_st_32x32b_x16(lanes + 128 + j0 / 2, hi);
-    tmem_st_32x32b_x16(lanes + 192 + j0 / 2, lo);
+    tmem_st_32x32b_x16(lanes + 128 + col0 / 2, hi);
+    tmem_st_32x32b_x16(lanes + 192 + col0 / 2, lo);
   }
   tmem_st_wait();
   tc_fence_before_sync();
@@ -366,22 +361,19 @@ __global__ void __launch_bounds__(RTH, 1) retention_out_kernel(const __grid_cons
   tc_fence_after_sync();
   const int t = at.t0 + row;
   const float e = power[row + 1];
-  __nv_bfloat16* O = (__nv_bfloat16*)p.out + ((long long)at.b * p.rows + t) * p.ldo + at.h * p.Dv + at.c0 + half * 64;
+  __nv_bfloat16* O = (__nv_bfloat16*)p.out + ((long long)at.b * p.rows + t) * p.ldo + at.h * p.Dv + at.c0 + col0;
+  uint32_t a[32], b[32];
+  tmem_ld_32x32b_x32(lanes + 256 + col0, a);
+  tmem_ld_32x32b_x32(lanes + 384 + col0, b);
+  tmem_ld_wait_regs(a);
+  tmem_ld_wait_regs(b);
+  if (ok && t < p.T) {
 #pragma unroll
-  for (int g = 0; g < 2; ++g) {
-    uint32_t a[32], b[32];
-    tmem_ld_32x32b_x32(lanes + 256 + half * 64 + 32 * g, a);
-    tmem_ld_32x32b_x32(lanes + 384 + half * 64 + 32 * g, b);
-    tmem_ld_wait_regs(a);
-    tmem_ld_wait_regs(b);
-    if (ok && t < p.T) {
+    for (int i = 0; i < 4; ++i) {
+      float f[8];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        float f[8];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) f[j] = e * __uint_as_float(a[8 * i + j]) + __uint_as_float(b[8 * i + j]);
-        if (half * 64 + 32 * g + 8 * i < at.ncol) st8v(O + 32 * g + 8 * i, f);  // Dv is a multiple of eight
-      }
+      for (int j = 0; j < 8; ++j) f[j] = e * __uint_as_float(a[8 * i + j]) + __uint_as_float(b[8 * i + j]);
+      if (col0 + 8 * i < at.ncol) st8v(O + 8 * i, f);  // Dv is a multiple of eight
     }
   }
   tc_fence_before_sync();

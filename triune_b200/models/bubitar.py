@@ -7,7 +7,7 @@ part. This module maps its configuration to a :class:`ModelConfig` and its tenso
 
 from __future__ import annotations
 
-from typing import Any, Dict, Iterator, Tuple
+from typing import Any, Dict, Iterator, Optional, Tuple
 
 import torch
 
@@ -20,14 +20,15 @@ from .zoo import register_model
 FF_ALPHA = 1.702  # slope of the feed-forward's sigmoid
 
 
-def _rotation(rot: Dict[str, Any], dims: int) -> Dict[str, Any]:
-    return {"rot_dims": dims, "rot_base": rot["base"], "rot_scaling": rot.get("scaling")}
+def _rotation(rot: Optional[Dict[str, Any]], dims: Optional[int] = None) -> Dict[str, Any]:
+    rot = rot or {"dims": 0, "base": 1.0}
+    return {"rot_dims": rot["dims"] if dims is None else dims, "rot_base": rot["base"], "rot_scaling": rot.get("scaling")}
 
 
 def layer_spec(entry: Dict[str, Any]) -> Dict[str, Any]:
     m, mlp = entry["mixer"], entry.get("mlp")
     if entry["type"] == "retention":
-        mixer = {"kind": "retention", **{k: m[k] for k in ("heads", "dim", "vdim", "decay")}, **_rotation(m["rot"], m["rot"]["dims"])}
+        mixer = {"kind": "retention", **{k: m[k] for k in ("heads", "dim", "vdim", "decay")}, **_rotation(m.get("rot"))}
     elif entry["type"] == "latent_attention":
         mixer = {"kind": "latent", **{k: m[k] for k in ("heads", "dim", "vdim", "kv_rank", "scale")}, **_rotation(m["rot"], m["rot_dim"]),
                  "kv_from": m.get("kv_from")}
