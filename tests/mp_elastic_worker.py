@@ -27,8 +27,8 @@ def main():
         # and a rank only ever leaves between two steps with its own work drained
         torch.cuda.set_device(ident)
         dev = torch.device("cuda", ident)
-    group = ElasticGroup("127.0.0.1", port, ident, world, backend="nccl" if on_gpu else "gloo", hb_interval=0.1, hb_timeout=1.0,
-                         pg_timeout=20.0 if on_gpu else 4.0, device_id=dev if on_gpu else None, strict_steps=strict)
+    group = ElasticGroup("127.0.0.1", port, ident, world, backend="nccl" if on_gpu else "gloo", hb_interval=0.1, hb_timeout=3.0,
+                         pg_timeout=20.0 if on_gpu else 8.0, device_id=dev if on_gpu else None, strict_steps=strict)
     torch.manual_seed(0)
     w = torch.zeros(4, dtype=torch.float64, device=dev)
     target = torch.tensor([1.0, -2.0, 0.5, 3.0], dtype=torch.float64, device=dev)

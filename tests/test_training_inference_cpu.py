@@ -614,7 +614,7 @@ def test_elastic_data_parallel_survives_a_lost_rank(tmp_path, victim, mode, stri
     from triune_b200.parallel.elastic import connect_store
     from triune_b200.desktop import find_free_port
 
-    port = find_free_port(29800, attempts=100)
+    port = find_free_port(20000 + os.getpid() % 4000, attempts=100)  # test processes do not meet
     store = connect_store("127.0.0.1", port, is_master=True)  # noqa: F841  (kept alive for the workers)
     env = dict(os.environ, OMP_NUM_THREADS="1", EL_PORT=str(port), EL_WORLD="3", EL_VICTIM=str(victim), EL_DIE_AT="5",
                EL_MODE=mode, EL_CKPT=str(tmp_path / "ck.pt"), EL_STEPS="8", EL_STRICT=strict)  # strict: meet on the store before every step
@@ -651,7 +651,7 @@ def test_elastic_training_command_survives_a_killed_rank(tmp_path):
     from triune_b200.desktop import find_free_port
     from triune_b200.parallel.elastic import connect_store
 
-    port = find_free_port(29900, attempts=100)
+    port = find_free_port(24200 + os.getpid() % 4000, attempts=100)
     store = connect_store("127.0.0.1", port, is_master=True)  # noqa: F841
     ck = tmp_path / "ck"
     tiny = json.dumps(dict(vocab_size=256, hidden_dim=64, num_layers=5, num_heads=2, head_dim=32, num_experts=4, reflex_exit_layer=2,
